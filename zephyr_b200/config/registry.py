@@ -19,6 +19,7 @@ from .errors import ConfigError
 from .fekotar import FekotarConfig
 from .gefovik import GefovikConfig
 from .legelix import LegelixConfig
+from .legilix import LegilixConfig
 from .qwen3 import Qwen3Config
 from .rizovik import RizovikConfig
 from .spec import ModelSpec
@@ -113,3 +114,4 @@ register_architecture(LegelixConfig.model_type, LegelixConfig.architecture, Lege
 register_architecture(GefovikConfig.model_type, GefovikConfig.architecture, GefovikConfig)
 register_architecture(FekotarConfig.model_type, FekotarConfig.architecture, FekotarConfig)
 register_architecture(RizovikConfig.model_type, RizovikConfig.architecture, RizovikConfig)
+register_architecture(LegilixConfig.model_type, LegilixConfig.architecture, LegilixConfig)

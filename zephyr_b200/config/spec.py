@@ -25,6 +25,7 @@ class NormSpec:
     eps: float
     weight: str        # full tensor name of the scale
     bias: str | None = None    # full tensor name of the shift, for norms that have one
+    groups: int = 1    # equal consecutive parts of the row with a statistic of their own, for norms that have it
 
 
 @dataclass(frozen=True)

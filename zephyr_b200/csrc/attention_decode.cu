@@ -67,6 +67,8 @@ struct DecodeArgs {
   float softcap_log2;            // > 0: scores are softcap * tanh(scale * s / softcap); this is softcap * log2(e)
   float scale_over_cap;          // scale / softcap
   int keys_only;                 // a page holds keys alone, [nkv][page_size][hd], and they are the values too
+  const float* bias_r1;          // null, or [nh] each: r1_h ln(1 + r2_h d) is taken off head h's scaled score of the
+  const float* bias_r2;          // key d positions back
   int* status;
   // Position encoding inside this kernel (`qkv` null: off; q then holds finished queries and the
   // cache the newest keys and values).  With it, q is not read: a request's new token lies raw in
@@ -662,6 +664,17 @@ paged_decode_kernel(const DecodeArgs a) {
     float o[HD / 8][4];
 #pragma unroll
     for (int n = 0; n < HD / 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.0f;
+    // The distance bias of this lane's two heads (in powers of two: r1 ln(x) log2(e) = r1 log2(x)).
+    const bool distant = a.bias_r1 != nullptr;
+    float r1[2] = {0.0f, 0.0f}, r2[2] = {0.0f, 0.0f};
+    if (distant) {
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int head = it.kvh * g + min(quad_row + 8 * h, g - 1);
+        r1[h] = a.bias_r1[head];
+        r2[h] = a.bias_r2[head];
+      }
+    }
 
     for (int j = warp; j < it.n_tiles; j += DEC_CONSUMERS) {
       const int seq = tile_base + j, slot = seq % R, filling = seq / R;
@@ -710,8 +723,10 @@ paged_decode_kernel(const DecodeArgs a) {
         for (int c = 0; c < 4; ++c) {
           const int pos = key0 + nt * 8 + quad_col + (c & 1);
           const bool valid = pos >= it.begin && pos < it.end;
-          const float scaled = a.softcap_log2 > 0.0f ? a.softcap_log2 * tanhf(s[nt][c] * a.scale_over_cap)
-                                                     : s[nt][c] * a.scale_log2;
+          float scaled = a.softcap_log2 > 0.0f ? a.softcap_log2 * tanhf(s[nt][c] * a.scale_over_cap)
+                                               : s[nt][c] * a.scale_log2;
+          if (distant)
+            scaled = fmaf(-r1[c >> 1], __log2f(fmaf(r2[c >> 1], static_cast<float>(it.ctx_total - 1 - pos), 1.0f)), scaled);
           s[nt][c] = valid ? scaled : -INFINITY;
           tile_max[c >> 1] = fmaxf(tile_max[c >> 1], s[nt][c]);
         }
@@ -995,8 +1010,9 @@ static int paged_decode_entry(void* out, const void* q, const void* kv_cache, co
                               const int* row_q_start, const int* row_ctx, int nh, int nkv, int hd, int window,
                               float scale, int split_size, int max_splits, float* scratch, int* counters, int* status,
                               const DecodeFusion* fusion, void* stream, int chunk = 0, const float* sinks = nullptr,
-                              float softcap = 0.0f, int keys_only = 0) {
-  if (n_rows < 0 || max_splits <= 0 || split_size < 0 || split_size % DEC_TILE != 0 || page_size <= 0 || window < 0 ||
+                              float softcap = 0.0f, int keys_only = 0, const float* bias_r1 = nullptr,
+                              const float* bias_r2 = nullptr) {
+  if ((bias_r1 == nullptr) != (bias_r2 == nullptr) || n_rows < 0 || max_splits <= 0 || split_size < 0 || split_size % DEC_TILE != 0 || page_size <= 0 || window < 0 ||
       chunk < 0 || counters == nullptr || softcap < 0.0f || (keys_only && fusion != nullptr))
     return ERR_BAD_ARGUMENT;
   if (!zb_paged_decode_supported(nh, nkv, hd, DTYPE_BF16) || (page_size & (page_size - 1)) != 0) return ERR_UNSUPPORTED;
@@ -1045,6 +1061,7 @@ static int paged_decode_entry(void* out, const void* q, const void* kv_cache, co
   a.softcap_log2 = softcap * 1.4426950408889634f;
   a.scale_over_cap = softcap > 0.0f ? scale / softcap : 0.0f;
   a.keys_only = keys_only;
+  a.bias_r1 = bias_r1; a.bias_r2 = bias_r2;
   a.status = status;
   auto s = static_cast<cudaStream_t>(stream);
   switch (hd) {
@@ -1065,17 +1082,17 @@ ZB_API int zb_paged_decode(void* out, const void* q, const void* kv_cache, const
                             status, nullptr, stream);
 }
 
-// The same with a chunked mask, sinks, a smooth bound on the scores and a cache of keys that are the values
-// too, as in the general kernel (attention_simt.cu).
+// The same with a chunked mask, sinks, a smooth bound on the scores, a cache of keys that are the values
+// too and a bias on the distance, as in the general kernel (attention_simt.cu).
 ZB_API int zb_paged_decode_masked(void* out, const void* q, const void* kv_cache, const int* block_table,
                                   int max_blocks, int page_size, int num_pages, int num_rows, const int* rows,
                                   int n_rows, const int* row_q_start, const int* row_ctx, int nh, int nkv, int hd,
                                   int window, int chunk, float scale, float softcap, int keys_only,
-                                  const float* sinks, int split_size, int max_splits, float* scratch, int* counters,
-                                  int* status, void* stream) {
+                                  const float* sinks, const float* bias_r1, const float* bias_r2, int split_size,
+                                  int max_splits, float* scratch, int* counters, int* status, void* stream) {
   return paged_decode_entry(out, q, kv_cache, block_table, max_blocks, page_size, num_pages, num_rows, rows, n_rows,
                             row_q_start, row_ctx, nh, nkv, hd, window, scale, split_size, max_splits, scratch, counters,
-                            status, nullptr, stream, chunk, sinks, softcap, keys_only);
+                            status, nullptr, stream, chunk, sinks, softcap, keys_only, bias_r1, bias_r2);
 }
 
 // The same with the new tokens' position encoding inside the kernel: `qkv` [T, qkv_stride] holds each

@@ -1,0 +1,540 @@
+// Paged causal attention with ALL heads of a tile of tokens in one CTA, bfloat16 on tensor cores, for layers
+// whose heads depend on one another between the scores and the softmax, and for keys and values of any two
+// widths:
+//
+//   s_h(i, j) = scale q_h(i) . k_c(h)(j)              c(h) = h / (heads / kv_heads)
+//   s_h <- sum_g M[h, g] s_g                          `score_mix` [nh, nh], or nothing
+//   s_h <- s_h - r1_h ln(1 + r2_h (i - j))            `bias_r1`, `bias_r2` [nh], or nothing
+//   softmax over the keys in sight (a window that may keep the first `keep_first` tokens), then the values
+//
+// The scores are float32 from the product to the softmax, the mixing included.
+//
+// One CTA = 8 or 16 consecutive new tokens of one request (or ONE decoded token), eight warps of 1, 2 or 4
+// heads each.  The products put keys on the 16-row side of m16n8k16 and tokens on its 8-column side
+// (S^T = K Q^T, O^T = V^T P^T), so a warp keeps its heads' queries and outputs in registers whatever the count
+// of tokens, and heads that share a key/value head share its fragments.  A tile of 32 (or 16) keys, with the
+// keys and values of every key/value head, goes through three phases:
+//   scores    each warp forms its heads' raw scores and leaves them in shared memory, [head][token][key];
+//   mixing    a thread owns one or two (token, key) pairs: it reads the raw scores of all heads, forms the
+//             mixed ones, takes off the bias, applies the mask and writes them back in place;
+//   values    each warp reads its heads' scores as the second product's operand: online softmax in float32 in
+//             base 2, probabilities rounded to bfloat16.
+// The next tile's keys are fetched (16-byte asynchronous copies, straight from the pages) while this tile is
+// mixed and weighed, its values while the next scores are formed.
+//
+// A decoded token's keys may be cut into `splits` runs of tiles, one CTA each; a second small kernel merges
+// their partial results in the order of the context.  Math and masking as in attention_simt.cu.
+#include "common.cuh"
+#include "mma.cuh"
+
+namespace zb {
+
+constexpr int AH_WARPS = 8;
+constexpr int AH_THREADS = AH_WARPS * 32;
+constexpr size_t AH_SMEM_LIMIT = 227 * 1024;
+
+struct HeadsAttentionArgs {
+  const __nv_bfloat16* q;        // [T, nh * kd]
+  __nv_bfloat16* out;            // [T, nh * vd]
+  const __nv_bfloat16* kv_cache; // [num_pages]{[nkv][page_size][kd], [nkv][page_size][vd]}
+  const int* block_table;        // [R, max_blocks]
+  const int* tile_row;           // [n_tiles]
+  const int* tile_q0;            // [n_tiles]
+  const int* row_q_start;        // [R]
+  const int* row_q_len;          // [R]
+  const int* row_ctx;            // [R]
+  int max_blocks, page_size, page_shift, num_pages, num_rows;      // page_shift: -1 where page_size is no power of two
+  int nh, nkv, kd, vd, window, keep_first;
+  float scale_log2;              // scale * log2(e)
+  const float* score_mix;        // null, or [nh, nh]
+  const float* bias_r1;          // null, or [nh] each
+  const float* bias_r2;
+  int splits;                    // > 1: every tile is one token, and its keys' tiles are shared by this many CTAs
+  float* part_o;                 // [n_tiles, splits, nh, vd]
+  float* part_ml;                // [n_tiles, splits, nh, 2]
+  int* status;
+};
+
+__host__ __device__ constexpr int ah_padded(int dim) { return (dim + 15) / 16 * 16 + 8; }      // a row in shared memory
+
+// HPW heads a warp, NT columns of 8 tokens, DM: keys and values of up to 16 DM values, BK keys a tile.
+template <int HPW, int NT, int DM, int BK>
+__global__ void __launch_bounds__(AH_THREADS, 1) heads_attention_kernel(const HeadsAttentionArgs a) {
+  constexpr int HM = AH_WARPS * HPW, NTOK = 8 * NT, SST = BK + 8, MT = BK / 16;
+  constexpr int KPT = NTOK * BK >= 2 * AH_THREADS ? 2 : 1;             // keys a thread mixes at a time
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  const int kst = ah_padded(a.kd), vst = ah_padded(a.vd);
+  __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smem_raw);                     // [nkv][BK][kst]
+  __nv_bfloat16* v_s = k_s + a.nkv * BK * kst;                                         // [nkv][BK][vst]
+  float* mix_s = reinterpret_cast<float*>(v_s + a.nkv * BK * vst);                     // [HM][HM], times scale and log2(e)
+  float* s_s = mix_s + HM * HM;                                                        // [nh][NTOK][SST]
+  __shared__ int2 where_s[2][BK];                    // a tile's keys: (page, position), page 0: not in sight of anyone
+
+  // The host lists the tiles by the number of keys they see, fewest first: the longest work starts first.
+  const int tile = gridDim.y - 1 - blockIdx.y, split = blockIdx.x;
+  const int row = a.tile_row[tile], q0 = a.tile_q0[tile];
+  if (row < 0 || row >= a.num_rows) {
+    if (threadIdx.x == 0) report(a.status, STATUS_ROW_OUT_OF_RANGE, row, tile);
+    return;
+  }
+  const int g = a.nh / a.nkv;
+  const int q_len = a.row_q_len[row], ctx = a.row_ctx[row], tok0 = a.row_q_start[row] + q0;
+  const int n_tok = min(a.splits > 1 ? 1 : NTOK, q_len - q0);
+  if (n_tok <= 0) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int quad_row = lane >> 2, quad = lane & 3;
+  const int* table = a.block_table + static_cast<size_t>(row) * a.max_blocks;
+  const int ks_n = (a.kd + 15) / 16, vm_n = (a.vd + 15) / 16;
+
+  // Keys any query of this tile may see: the kept first tokens below every window, and [lo, hi).
+  const int hi = ctx + q0 + n_tok;
+  const int lo = a.window > 0 ? max(0, ctx + q0 - a.window + 1) : 0;
+  const int kept = a.window > 0 ? min(a.keep_first, lo) : 0;
+  const int first_tile = lo / BK * BK;
+  const int kept_tiles = (kept + BK - 1) / BK;
+  const int all_tiles = kept_tiles + (hi - first_tile + BK - 1) / BK;
+  const int t_begin = static_cast<int>(static_cast<long long>(all_tiles) * split / a.splits);
+  const int t_end = static_cast<int>(static_cast<long long>(all_tiles) * (split + 1) / a.splits);
+  auto tile_start = [&](int t) { return t < kept_tiles ? t * BK : first_tile + (t - kept_tiles) * BK; };
+
+  auto plan = [&](int t, int buffer) {               // by the first BK threads
+    if (threadIdx.x >= BK) return;
+    const int pos = tile_start(t) + static_cast<int>(threadIdx.x);
+    int page = 0;
+    if (t < kept_tiles ? pos < kept : (pos >= lo && pos < hi)) {
+      const int block = a.page_shift >= 0 ? pos >> a.page_shift : pos / a.page_size;
+      page = block < a.max_blocks ? table[block] : -1;
+      if (page <= 0 || page >= a.num_pages) {
+        report(a.status, STATUS_PAGE_OUT_OF_RANGE, page, tok0);
+        page = 0;
+      }
+    }
+    where_s[buffer][threadIdx.x] = make_int2(page, pos);
+  };
+  const long long page_elems = static_cast<long long>(a.nkv) * a.page_size * (a.kd + a.vd);
+  // The planned tile's rows of every key/value head; zeros for keys that nobody sees.
+  auto load_rows = [&](__nv_bfloat16* dst, int stride, int dim, long long part, int buffer) {
+    if (dim % 8 == 0) {
+      const int chunks = dim / 8;
+      const int lanes = chunks <= 4 ? 4 : (chunks <= 8 ? 8 : (chunks <= 16 ? 16 : 32)), rows = 32 / lanes;      // a row
+      for (int r = warp * rows + lane / lanes; r < a.nkv * BK; r += AH_WARPS * rows) {
+        const int kvh = r / BK, key = r % BK;
+        const int2 w = where_s[buffer][key];
+        const int in_page = a.page_shift >= 0 ? w.y & (a.page_size - 1) : w.y % a.page_size;
+        const int swizzle = kv_swizzle(w.y, chunks);
+        const __nv_bfloat16* src = a.kv_cache;
+        if (w.x > 0) src += w.x * page_elems + part + (static_cast<long long>(kvh) * a.page_size + in_page) * dim;
+        for (int c = lane & (lanes - 1); c < chunks; c += lanes)
+          cp_async_16(dst + r * stride + c * 8, w.x > 0 ? src + ((c ^ swizzle) << 3) : src, w.x > 0);
+      }
+    } else {                                           // rows stored as they are, on any boundary
+      for (int r = warp; r < a.nkv * BK; r += AH_WARPS) {
+        const int kvh = r / BK, key = r % BK;
+        const int2 w = where_s[buffer][key];
+        const long long from = w.x * page_elems + part + (static_cast<long long>(kvh) * a.page_size + w.y % a.page_size) * dim;
+        for (int i = lane; i < dim; i += 32)
+          dst[r * stride + i] = w.x > 0 ? a.kv_cache[from + i] : __float2bfloat16_rn(0.0f);
+      }
+    }
+  };
+  const long long value_part = static_cast<long long>(a.nkv) * a.page_size * a.kd;
+  auto load_keys = [&](int buffer) { load_rows(k_s, kst, a.kd, 0, buffer); };
+  auto load_values = [&](int buffer) { load_rows(v_s, vst, a.vd, value_part, buffer); };
+
+  if (t_begin < t_end) plan(t_begin, 0);
+  // The columns that pad a row to whole steps of 16 stay zero for good.
+  for (int e = threadIdx.x; e < a.nkv * BK * (kst + vst) / 8; e += AH_THREADS)
+    reinterpret_cast<uint4*>(k_s)[e] = make_uint4(0, 0, 0, 0);
+  if (a.score_mix != nullptr)
+    for (int e = threadIdx.x; e < HM * HM; e += AH_THREADS) {
+      const int h = e / HM, o = e - h * HM;
+      mix_s[e] = h < a.nh && o < a.nh ? a.score_mix[h * a.nh + o] * a.scale_log2 : 0.0f;
+    }
+  __syncthreads();
+  if (t_begin < t_end) load_keys(0);
+  cp_async_commit();
+  if (t_begin < t_end) load_values(0);
+  cp_async_commit();
+
+  // This warp's heads; their queries as the B operand (k = dims, n = tokens).
+  const int head0 = warp * HPW;
+  unsigned qf[HPW][NT][DM][2];
+#pragma unroll
+  for (int i = 0; i < HPW; ++i) {
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) {
+      const int tok = nt * 8 + quad_row, head = head0 + i;
+      const bool ok = tok < n_tok && head < a.nh;
+      const __nv_bfloat16* src = a.q + (static_cast<size_t>(tok0 + (ok ? tok : 0)) * a.nh + (ok ? head : 0)) * a.kd;
+      const bool pairs = a.kd % 2 == 0;
+#pragma unroll
+      for (int ks = 0; ks < DM; ++ks) {
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int d = ks * 16 + half * 8 + 2 * quad;
+          unsigned word = 0;
+          if (ok && d < a.kd) {
+            if (pairs) {
+              word = *reinterpret_cast<const unsigned*>(src + d);
+            } else {
+              const __nv_bfloat162 two(src[d], d + 1 < a.kd ? src[d + 1] : __float2bfloat16_rn(0.0f));
+              word = *reinterpret_cast<const unsigned*>(&two);
+            }
+          }
+          qf[i][nt][ks][half] = word;
+        }
+      }
+    }
+  }
+  float m_run[HPW][NT], l_run[HPW][NT];              // of token quad_row of each column
+  float o[HPW][NT][DM][4];
+#pragma unroll
+  for (int i = 0; i < HPW; ++i)
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) {
+      m_run[i][nt] = -INFINITY;
+      l_run[i][nt] = 0.0f;
+#pragma unroll
+      for (int m = 0; m < DM; ++m) o[i][nt][m][0] = o[i][nt][m][1] = o[i][nt][m][2] = o[i][nt][m][3] = 0.0f;
+    }
+
+  cp_async_wait<1>();
+  __syncthreads();                                   // the first tile's keys have landed
+  for (int t = t_begin; t < t_end; ++t) {
+    const int buffer = (t - t_begin) & 1;
+    const bool more = t + 1 < t_end;
+    if (more) plan(t + 1, buffer ^ 1);
+    // ------------------------------------------------------------------------------------ raw scores
+    if (head0 < a.nh) {
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt) {
+        float acc[HPW][NT][4];
+#pragma unroll
+        for (int i = 0; i < HPW; ++i)
+#pragma unroll
+          for (int nt = 0; nt < NT; ++nt) acc[i][nt][0] = acc[i][nt][1] = acc[i][nt][2] = acc[i][nt][3] = 0.0f;
+#pragma unroll
+        for (int ks = 0; ks < DM; ++ks) {
+          if (ks >= ks_n) break;
+          unsigned ka[4];
+          int held = -1;
+#pragma unroll
+          for (int i = 0; i < HPW; ++i) {
+            if (head0 + i >= a.nh) break;
+            const int kvh = (head0 + i) / g;
+            if (kvh != held)
+              ldmatrix_x4(ka, k_s + (kvh * BK + mt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * kst + ks * 16 + (lane >> 4) * 8);
+            held = kvh;
+#pragma unroll
+            for (int nt = 0; nt < NT; ++nt) mma_bf16_16816(acc[i][nt], ka, qf[i][nt][ks][0], qf[i][nt][ks][1]);
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < HPW; ++i) {
+          if (head0 + i >= a.nh) break;
+#pragma unroll
+          for (int nt = 0; nt < NT; ++nt) {
+            float* dst = s_s + ((head0 + i) * NTOK + nt * 8 + 2 * quad) * SST + mt * 16 + quad_row;
+            dst[0] = acc[i][nt][0];
+            dst[SST] = acc[i][nt][1];
+            dst[8] = acc[i][nt][2];
+            dst[SST + 8] = acc[i][nt][3];
+          }
+        }
+      }
+    }
+    __syncthreads();                                 // every head's raw scores are there, the keys are read
+    if (more) load_keys(buffer ^ 1);
+    cp_async_commit();
+    // --------------------------------------------------------------------- mixing, bias, mask, in place
+    {
+      const int e = threadIdx.x * KPT, tok = e / BK, key = e % BK;
+      if (tok < n_tok) {
+        const int k0 = tile_start(t), qp = ctx + q0 + tok;
+        bool valid[KPT];
+        float distance[KPT];
+#pragma unroll
+        for (int u = 0; u < KPT; ++u) {
+          const int pos = k0 + key + u;
+          valid[u] = t < kept_tiles ? pos < kept
+                                    : pos <= qp && pos >= lo && (a.window == 0 || pos > qp - a.window || pos < a.keep_first);
+          distance[u] = static_cast<float>(qp - pos);
+        }
+        float* at = s_s + tok * SST + key;
+        auto finish = [&](int h, float (&v)[KPT]) {
+#pragma unroll
+          for (int u = 0; u < KPT; ++u) {
+            if (a.bias_r1 != nullptr) v[u] = fmaf(-a.bias_r1[h], __log2f(fmaf(a.bias_r2[h], distance[u], 1.0f)), v[u]);
+            at[h * NTOK * SST + u] = valid[u] ? v[u] : -INFINITY;
+          }
+        };
+        if (a.score_mix != nullptr) {
+          float s[HM][KPT];
+#pragma unroll
+          for (int h = 0; h < HM; ++h)
+#pragma unroll
+            for (int u = 0; u < KPT; ++u) s[h][u] = h < a.nh ? at[h * NTOK * SST + u] : 0.0f;
+          for (int h = 0; h < a.nh; ++h) {
+            float v[KPT];
+#pragma unroll
+            for (int u = 0; u < KPT; ++u) v[u] = 0.0f;
+#pragma unroll
+            for (int o4 = 0; o4 < HM / 4; ++o4) {
+              const float4 m = *reinterpret_cast<const float4*>(mix_s + h * HM + 4 * o4);
+#pragma unroll
+              for (int u = 0; u < KPT; ++u) {
+                v[u] = fmaf(m.x, s[4 * o4][u], v[u]);
+                v[u] = fmaf(m.y, s[4 * o4 + 1][u], v[u]);
+                v[u] = fmaf(m.z, s[4 * o4 + 2][u], v[u]);
+                v[u] = fmaf(m.w, s[4 * o4 + 3][u], v[u]);
+              }
+            }
+            finish(h, v);
+          }
+        } else {
+          for (int h = 0; h < a.nh; ++h) {
+            float v[KPT];
+#pragma unroll
+            for (int u = 0; u < KPT; ++u) v[u] = at[h * NTOK * SST + u] * a.scale_log2;
+            finish(h, v);
+          }
+        }
+      }
+    }
+    cp_async_wait<1>();
+    __syncthreads();                                 // the scores are final, this tile's values have landed
+    // ------------------------------------------------------------------------------ softmax and values
+    if (head0 < a.nh) {
+      unsigned pb[HPW][NT][MT][2];
+#pragma unroll
+      for (int i = 0; i < HPW; ++i) {
+        if (head0 + i >= a.nh) break;
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt) {
+          const float* src = s_s + ((head0 + i) * NTOK + nt * 8 + quad_row) * SST + 2 * quad;
+          float2 v[BK / 8];
+          float top = -INFINITY;
+#pragma unroll
+          for (int j = 0; j < BK / 8; ++j) {
+            v[j] = *reinterpret_cast<const float2*>(src + 8 * j);
+            top = fmaxf(top, fmaxf(v[j].x, v[j].y));
+          }
+          top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 1));
+          top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 2));
+          const float new_m = fmaxf(m_run[i][nt], top);
+          const float m_use = new_m == -INFINITY ? 0.0f : new_m;      // a token that has seen no key yet
+          const float corr = exp2f(m_run[i][nt] - m_use);
+          m_run[i][nt] = new_m;
+          float sum = 0.0f;
+#pragma unroll
+          for (int j = 0; j < BK / 8; ++j) {
+            v[j].x = exp2f(v[j].x - m_use);
+            v[j].y = exp2f(v[j].y - m_use);
+            sum += v[j].x + v[j].y;
+          }
+          sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+          sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+          l_run[i][nt] = l_run[i][nt] * corr + sum;
+#pragma unroll
+          for (int ks = 0; ks < MT; ++ks) {
+            pb[i][nt][ks][0] = pack_bf16(v[2 * ks].x, v[2 * ks].y);
+            pb[i][nt][ks][1] = pack_bf16(v[2 * ks + 1].x, v[2 * ks + 1].y);
+          }
+          if (!__all_sync(0xffffffffu, corr == 1.0f)) {               // tokens 2 quad and 2 quad + 1 own this lane's columns
+            const float c0 = __shfl_sync(0xffffffffu, corr, 8 * quad), c1 = __shfl_sync(0xffffffffu, corr, 8 * quad + 4);
+#pragma unroll
+            for (int m = 0; m < DM; ++m) {
+              o[i][nt][m][0] *= c0; o[i][nt][m][1] *= c1; o[i][nt][m][2] *= c0; o[i][nt][m][3] *= c1;
+            }
+          }
+        }
+      }
+#pragma unroll
+      for (int m = 0; m < DM; ++m) {
+        if (m >= vm_n) break;
+#pragma unroll
+        for (int ks = 0; ks < MT; ++ks) {
+          unsigned va[4];
+          int held = -1;
+#pragma unroll
+          for (int i = 0; i < HPW; ++i) {
+            if (head0 + i >= a.nh) break;
+            const int kvh = (head0 + i) / g;
+            if (kvh != held)
+              ldmatrix_x4_trans(va, v_s + (kvh * BK + ks * 16 + (lane >> 4) * 8 + (lane & 7)) * vst + m * 16 + ((lane >> 3) & 1) * 8);
+            held = kvh;
+#pragma unroll
+            for (int nt = 0; nt < NT; ++nt) mma_bf16_16816(o[i][nt][m], va, pb[i][nt][ks][0], pb[i][nt][ks][1]);
+          }
+        }
+      }
+    }
+    cp_async_wait<0>();
+    __syncthreads();                                 // the next keys have landed; scores and values are read
+    if (more) load_values(buffer ^ 1);
+    cp_async_commit();
+  }
+  cp_async_wait<0>();
+
+#pragma unroll
+  for (int i = 0; i < HPW; ++i) {
+    const int head = head0 + i;
+    if (head >= a.nh) break;
+    if (a.splits > 1) {                              // one token: column 0 of the first tokens' column
+      const size_t slot = (static_cast<size_t>(tile) * a.splits + split) * a.nh + head;
+      if (lane == 0) {
+        a.part_ml[2 * slot] = m_run[i][0];
+        a.part_ml[2 * slot + 1] = l_run[i][0];
+      }
+      if (quad == 0) {
+#pragma unroll
+        for (int m = 0; m < DM; ++m) {
+          const int d = m * 16 + quad_row;
+          if (d < a.vd) a.part_o[slot * a.vd + d] = o[i][0][m][0];
+          if (d + 8 < a.vd) a.part_o[slot * a.vd + d + 8] = o[i][0][m][2];
+        }
+      }
+      continue;
+    }
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) {
+      const float l0 = __shfl_sync(0xffffffffu, l_run[i][nt], 8 * quad), l1 = __shfl_sync(0xffffffffu, l_run[i][nt], 8 * quad + 4);
+      const float inv[2] = {l0 > 0.0f ? 1.0f / l0 : 0.0f, l1 > 0.0f ? 1.0f / l1 : 0.0f};
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const int tok = nt * 8 + 2 * quad + u;
+        if (tok >= n_tok) continue;
+        __nv_bfloat16* dst = a.out + (static_cast<size_t>(tok0 + tok) * a.nh + head) * a.vd;
+#pragma unroll
+        for (int m = 0; m < DM; ++m) {
+          const int d = m * 16 + quad_row;
+          if (d < a.vd) dst[d] = __float2bfloat16_rn(o[i][nt][m][u] * inv[u]);
+          if (d + 8 < a.vd) dst[d + 8] = __float2bfloat16_rn(o[i][nt][m][2 + u] * inv[u]);
+        }
+      }
+    }
+  }
+}
+
+// The splits' partial results of one token and head, in the order of the context.
+__global__ void __launch_bounds__(128) heads_merge_kernel(const HeadsAttentionArgs a) {
+  const int tile = blockIdx.x, head = blockIdx.y;
+  const int row = a.tile_row[tile];
+  if (row < 0 || row >= a.num_rows || a.row_q_len[row] - a.tile_q0[tile] <= 0) return;       // (reported by the other kernel)
+  const size_t slot0 = static_cast<size_t>(tile) * a.splits * a.nh + head;
+  float top = -INFINITY;
+  for (int s = 0; s < a.splits; ++s) top = fmaxf(top, a.part_ml[2 * (slot0 + static_cast<size_t>(s) * a.nh)]);
+  float l = 0.0f;
+  for (int s = 0; s < a.splits; ++s) {
+    const size_t slot = slot0 + static_cast<size_t>(s) * a.nh;
+    const float m = a.part_ml[2 * slot];
+    if (m > -INFINITY) l = fmaf(a.part_ml[2 * slot + 1], exp2f(m - top), l);
+  }
+  const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+  const size_t token = a.row_q_start[row] + a.tile_q0[tile];
+  for (int d = threadIdx.x; d < a.vd; d += blockDim.x) {
+    float v = 0.0f;
+    for (int s = 0; s < a.splits; ++s) {
+      const size_t slot = slot0 + static_cast<size_t>(s) * a.nh;
+      const float m = a.part_ml[2 * slot];
+      if (m > -INFINITY) v = fmaf(a.part_o[slot * a.vd + d], exp2f(m - top), v);
+    }
+    a.out[(token * a.nh + head) * a.vd + d] = __float2bfloat16_rn(v * inv);
+  }
+}
+
+struct HeadsShape {
+  int hpw, nt, dm, bk;
+  size_t smem;
+};
+
+// How the kernel runs this layer (hpw 0: it does not take it); `single`: for tiles of one token.
+HeadsShape heads_shape(int nh, int nkv, int kd, int vd, bool single) {
+  HeadsShape shape{0, 0, 0, 0, 0};
+  if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || kd <= 0 || vd <= 0) return shape;
+  const int widest = (kd > vd ? kd : vd);
+  const int dm = widest <= 64 ? 4 : (widest <= 128 ? 8 : (widest <= 256 ? 16 : 0));
+  const int hpw = nh <= 8 ? 1 : (nh <= 16 ? 2 : (nh <= 32 ? 4 : 0));
+  if (dm == 0 || hpw == 0 || (dm == 16 && hpw == 4)) return shape;
+  const int nt = single || hpw == 4 || (dm == 16 && hpw == 2) ? 1 : 2;
+  for (int bk = 32; bk >= 16; bk -= 16) {
+    const size_t smem = static_cast<size_t>(nkv) * bk * (ah_padded(kd) + ah_padded(vd)) * sizeof(__nv_bfloat16) +
+                        (static_cast<size_t>(64) * hpw * hpw + static_cast<size_t>(nh) * 8 * nt * (bk + 8)) * sizeof(float);
+    if (smem + 1024 <= AH_SMEM_LIMIT) {
+      shape = HeadsShape{hpw, nt, dm, bk, smem};
+      return shape;
+    }
+  }
+  return shape;
+}
+
+template <int HPW, int NT, int DM, int BK>
+int heads_launch(const HeadsAttentionArgs& a, int n_tiles, size_t smem, cudaStream_t stream) {
+  auto kernel = heads_attention_kernel<HPW, NT, DM, BK>;
+  if (cuda_failed(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)))) return ERR_CUDA;
+  kernel<<<dim3(a.splits, n_tiles), AH_THREADS, smem, stream>>>(a);
+  return launch_result();
+}
+
+}  // namespace zb
+
+using namespace zb;
+
+// New tokens of one request that a tile covers for rows with several of them (0: the shape is not taken).
+ZB_API int zb_heads_attention_tile_tokens(int nh, int nkv, int kd, int vd, int dtype) {
+  if (dtype != DTYPE_BF16) return 0;
+  if (heads_shape(nh, nkv, kd, vd, true).hpw == 0) return 0;
+  return 8 * heads_shape(nh, nkv, kd, vd, false).nt;
+}
+
+// Keys of a tile of a decoded token: its keys can be cut into at most ceil(keys / this) splits that all have work.
+ZB_API int zb_heads_attention_tile_keys(int nh, int nkv, int kd, int vd) { return heads_shape(nh, nkv, kd, vd, true).bk; }
+
+// Attention of the tiles' tokens over their requests' pages; writes those tokens' rows of `out` [T, nh * vd].
+// `single`: every tile is one token, whose keys `splits` CTAs share; with splits > 1 `scratch` holds
+// n_tiles * splits * nh * (vd + 2) floats (contents irrelevant).
+ZB_API int zb_heads_attention(void* out, const void* q, const void* kv_cache, const int* block_table, int max_blocks,
+                              int page_size, int num_pages, int num_rows, const int* tile_row, const int* tile_q0,
+                              int n_tiles, const int* row_q_start, const int* row_q_len, const int* row_ctx, int nh,
+                              int nkv, int kd, int vd, int window, int keep_first, float scale, const float* score_mix,
+                              const float* bias_r1, const float* bias_r2, int single, int splits, float* scratch,
+                              int* status, void* stream) {
+  if (n_tiles < 0 || page_size <= 0 || window < 0 || keep_first < 0 || splits <= 0 || (splits > 1 && (!single || scratch == nullptr)) ||
+      (bias_r1 == nullptr) != (bias_r2 == nullptr) || reinterpret_cast<uintptr_t>(q) % 4 != 0 ||
+      reinterpret_cast<uintptr_t>(kv_cache) % 16 != 0)
+    return ERR_BAD_ARGUMENT;
+  const HeadsShape shape = heads_shape(nh, nkv, kd, vd, single != 0);
+  if (shape.hpw == 0) return ERR_UNSUPPORTED;
+  if (n_tiles == 0) return OK;
+  if (n_tiles > 65535) return ERR_UNSUPPORTED;
+  HeadsAttentionArgs a;
+  a.q = static_cast<const __nv_bfloat16*>(q);
+  a.out = static_cast<__nv_bfloat16*>(out);
+  a.kv_cache = static_cast<const __nv_bfloat16*>(kv_cache);
+  a.block_table = block_table; a.tile_row = tile_row; a.tile_q0 = tile_q0;
+  a.row_q_start = row_q_start; a.row_q_len = row_q_len; a.row_ctx = row_ctx;
+  a.max_blocks = max_blocks; a.page_size = page_size; a.num_pages = num_pages; a.num_rows = num_rows;
+  a.page_shift = -1;
+  for (int shift = 0; shift < 31; ++shift)
+    if (page_size == (1 << shift)) a.page_shift = shift;
+  a.nh = nh; a.nkv = nkv; a.kd = kd; a.vd = vd; a.window = window; a.keep_first = window > 0 ? keep_first : 0;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  a.score_mix = score_mix; a.bias_r1 = bias_r1; a.bias_r2 = bias_r2;
+  a.splits = splits;
+  a.part_o = scratch;
+  a.part_ml = scratch != nullptr ? scratch + static_cast<size_t>(n_tiles) * splits * nh * vd : nullptr;
+  a.status = status;
+  auto s = static_cast<cudaStream_t>(stream);
+  int rc = ERR_UNSUPPORTED;
+#define ZB_AH(HPW, NT, DM, BK) \
+  if (shape.hpw == HPW && shape.nt == NT && shape.dm == DM && shape.bk == BK) rc = heads_launch<HPW, NT, DM, BK>(a, n_tiles, shape.smem, s);
+#define ZB_AH_BK(HPW, NT, DM) ZB_AH(HPW, NT, DM, 32) ZB_AH(HPW, NT, DM, 16)
+  ZB_AH_BK(1, 1, 4) ZB_AH_BK(1, 2, 4) ZB_AH_BK(2, 1, 4) ZB_AH_BK(2, 2, 4) ZB_AH_BK(4, 1, 4)
+  ZB_AH_BK(1, 1, 8) ZB_AH_BK(1, 2, 8) ZB_AH_BK(2, 1, 8) ZB_AH_BK(2, 2, 8) ZB_AH_BK(4, 1, 8)
+  ZB_AH_BK(1, 1, 16) ZB_AH_BK(1, 2, 16) ZB_AH_BK(2, 1, 16)
+#undef ZB_AH_BK
+#undef ZB_AH
+  if (rc != OK || splits == 1) return rc;
+  heads_merge_kernel<<<dim3(n_tiles, nh), 128, 0, s>>>(a);
+  return launch_result();
+}

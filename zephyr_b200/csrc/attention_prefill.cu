@@ -25,6 +25,9 @@
 // and values stream once for the whole group and the products fill the tensor cores' rows with heads; the
 // grid's x counts key/value heads (times value heads with `cross_values`).
 //
+// `bias_r1`, `bias_r2` (one float32 per query head each): r1_h ln(1 + r2_h d) is taken off head h's scaled score
+// of the key d positions back.
+//
 // Head sizes: every multiple of 32 up to 256 (a query tile's outputs stay in registers: 16 float32
 // values a thread for every 32 of the head).  A tile may hold a single token (one warp works, the
 // others help to fetch): latent attention serves decoded tokens this way where the split-context
@@ -64,6 +67,8 @@ struct PrefillArgs {
   int pool_max_blocks, pool_num_pages;
   int cross_values;              // grid x = nh * nkv: head + nh * value head
   int out_f32;
+  const float* bias_r1;          // null, or [nh]
+  const float* bias_r2;
   int* status;
 };
 
@@ -178,6 +183,24 @@ paged_prefill_kernel(const PrefillArgs a) {
   const int warp_seen = a.pool > 0 ? (warp_last_pos - a.window + 1) / a.pool : 0;
   const int warp_seen_first = a.pool > 0 ? (warp_pos0 - a.window + 1) / a.pool : 0;      // what the warp's first row sees
 
+  // The distance bias of this lane's two rows (in powers of two: r1 ln(x) log2(e) = r1 log2(x)).
+  const bool distant = a.bias_r1 != nullptr;
+  float r1[2] = {0.0f, 0.0f}, r2[2] = {0.0f, 0.0f};
+  if (distant) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int row_head = DEC ? head + min(quad_row + 8 * h, g - 1) : head;
+      r1[h] = a.bias_r1[row_head];
+      r2[h] = a.bias_r2[row_head];
+    }
+  }
+  // A raw score of this lane's row h whose key lies at `pos`, scaled, bounded and biased.
+  auto finished = [&](float raw, int h, int pos) {
+    float v = a.softcap_log2 > 0.0f ? a.softcap_log2 * tanhf(raw * a.scale_over_cap) : raw * a.scale_log2;
+    if (distant) v = fmaf(-r1[h], __log2f(fmaf(r2[h], static_cast<float>(qpos[h] - pos), 1.0f)), v);
+    return v;
+  };
+
   unsigned qa[HD / 16][4];
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};
   float o[HD / 8][4];
@@ -229,9 +252,10 @@ paged_prefill_kernel(const PrefillArgs a) {
     if (whole_tile) {
 #pragma unroll
       for (int i = 0; i < NTS; ++i) {
+        const int nt = DEC ? warp : i;
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
-          s[i][c] = a.softcap_log2 > 0.0f ? a.softcap_log2 * tanhf(s[i][c] * a.scale_over_cap) : s[i][c] * a.scale_log2;
+          s[i][c] = finished(s[i][c], c >> 1, k0 + nt * 8 + quad_col + (c & 1));
           tile_max[c >> 1] = fmaxf(tile_max[c >> 1], s[i][c]);
         }
       }
@@ -248,9 +272,8 @@ paged_prefill_kernel(const PrefillArgs a) {
                                       : pos <= qp && pos >= lo &&
                                             (a.window == 0 || pos > qp - a.window || pos < a.keep_first) &&
                                             pos >= chunk_start[c >> 1];
-          const float scaled = a.softcap_log2 > 0.0f ? a.softcap_log2 * tanhf(s[i][c] * a.scale_over_cap)
-                                                     : s[i][c] * a.scale_log2;
-          s[i][c] = valid ? scaled : -INFINITY;
+          const float score = finished(s[i][c], c >> 1, pos);
+          s[i][c] = valid ? score : -INFINITY;
           tile_max[c >> 1] = fmaxf(tile_max[c >> 1], s[i][c]);
         }
       }
@@ -416,9 +439,10 @@ ZB_API int zb_paged_prefill_windowed(void* out, const void* q, const void* kv_ca
                                      const int* row_ctx, int nh, int nkv, int hd, int window, int chunk, float scale,
                                      float softcap, int keys_only, const float* sinks, int keep_first, int pool,
                                      const void* pool_cache, const int* pool_table, int pool_max_blocks,
-                                     int pool_num_pages, int cross_values, int out_f32, int by_group, int* status,
-                                     void* stream) {
-  if (n_tiles < 0 || page_size <= 0 || window < 0 || chunk < 0 || softcap < 0.0f || keep_first < 0 || pool < 0 ||
+                                     int pool_num_pages, int cross_values, int out_f32, int by_group,
+                                     const float* bias_r1, const float* bias_r2, int* status, void* stream) {
+  if ((bias_r1 == nullptr) != (bias_r2 == nullptr) || (bias_r1 != nullptr && pool > 0) ||
+      n_tiles < 0 || page_size <= 0 || window < 0 || chunk < 0 || softcap < 0.0f || keep_first < 0 || pool < 0 ||
       (pool > 0 && (window <= 0 || pool_cache == nullptr || pool_table == nullptr || pool_max_blocks <= 0 || keys_only)) ||
       (cross_values && keys_only) || nh * (cross_values ? nkv : 1) > 65535 || (by_group && nh / (nkv > 0 ? nkv : 1) > 16))
     return ERR_BAD_ARGUMENT;
@@ -444,6 +468,7 @@ ZB_API int zb_paged_prefill_windowed(void* out, const void* q, const void* kv_ca
   a.pool_cache = static_cast<const __nv_bfloat16*>(pool_cache);
   a.pool_table = pool_table; a.pool_max_blocks = pool_max_blocks; a.pool_num_pages = pool_num_pages;
   a.cross_values = cross_values; a.out_f32 = out_f32;
+  a.bias_r1 = bias_r1; a.bias_r2 = bias_r2;
   a.status = status;
   auto s = static_cast<cudaStream_t>(stream);
   switch (hd) {
@@ -465,7 +490,8 @@ ZB_API int zb_paged_prefill_masked(void* out, const void* q, const void* kv_cach
                                    float softcap, int keys_only, const float* sinks, int* status, void* stream) {
   return zb_paged_prefill_windowed(out, q, kv_cache, block_table, max_blocks, page_size, num_pages, num_rows, tile_row,
                                    tile_q0, n_tiles, row_q_start, row_q_len, row_ctx, nh, nkv, hd, window, chunk, scale,
-                                   softcap, keys_only, sinks, 0, 0, nullptr, nullptr, 0, 0, 0, 0, 0, status, stream);
+                                   softcap, keys_only, sinks, 0, 0, nullptr, nullptr, 0, 0, 0, 0, 0, nullptr, nullptr, status,
+                                   stream);
 }
 
 ZB_API int zb_paged_prefill(void* out, const void* q, const void* kv_cache, const int* block_table, int max_blocks,

@@ -76,6 +76,8 @@ struct PrefillTcArgs {
   float scale_over_cap;          // scale / softcap
   int keys_only;                 // a page holds keys alone, [nkv][page_size][hd], and they are the values too
   const float* sinks;            // null, or [nh]: exp(sinks[h]) joins the softmax's denominator of head h
+  const float* bias_r1;          // null, or [nh] each: r1_h ln(1 + r2_h d) is taken off head h's scaled score of the
+  const float* bias_r2;          // key d positions back
   int* status;
   int* trace;                    // null, or 4 ints per tile of the first CTA (the longest work of the launch): the global
                                  // timer (ns, low 32 bits) when S of the tile was issued, when its softmax began (S
@@ -101,6 +103,12 @@ __device__ __forceinline__ float exp2_approx(float x) {
   return y;
 }
 
+__device__ __forceinline__ float log2_approx(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+  return y;
+}
+
 // tanh from the special-function unit's exp2 and reciprocal, 1 - 2 / (e^(2x) + 1): absolute error about 1e-7 over
 // the whole line (the unit's own tanh is good to 2^-11 only, which would move a score capped at 30 by 0.02).
 __device__ __forceinline__ float tanh_from_exp2(float x) {
@@ -112,11 +120,15 @@ __device__ __forceinline__ float tanh_from_exp2(float x) {
 // One half (64 columns) of a row of S (this thread's TMEM lane) -> probabilities exp2(s * scale + neg_shift)
 // as 32 words of two bfloat16 each, their sum, and the largest raw score.  MASKED: column i counts only if
 // after < i <= last and i >= first (positions relative to the tile's first key).
-// CAPPED: the exponent is cap_log2 * tanh(raw * scale) + neg_shift, `scale` then being scale / softcap.
-template <bool MASKED, bool CAPPED>
+// MODE CAPPED: the exponent is cap_log2 * tanh(raw * scale) + neg_shift, `scale` then being scale / softcap.
+// MODE BIASED: the exponent is raw * scale - r1 log2(1 + r2 d) + neg_shift, d = last - i being how far the key of
+// column i lies behind the query (`last` is given with and without a mask); the largest score is then the
+// largest of the biased ones, scaled.
+constexpr int TC_PLAIN = 0, TC_CAPPED = 1, TC_BIASED = 2;
+template <bool MASKED, int MODE>
 __device__ __forceinline__ void softmax_pass(unsigned tmem_row, unsigned (&words)[TC_BN / 4], int half, float scale, float neg_shift,
                                              int last, int first, int after, float& raw_max, float& row_sum,
-                                             float cap_log2 = 0.0f) {
+                                             float cap_log2 = 0.0f, float r1 = 0.0f, float r2 = 0.0f) {
   // Four running maxima and sums side by side: with one warp per scheduler a single chain of 128
   // dependent additions would cost its full latency 128 times.
   float max4[4] = {raw_max, -INFINITY, -INFINITY, -INFINITY}, sum4[4] = {row_sum, 0.0f, 0.0f, 0.0f};
@@ -131,11 +143,14 @@ __device__ __forceinline__ void softmax_pass(unsigned tmem_row, unsigned (&words
       float p[2];
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const float raw = __uint_as_float(v[i + e]);
+        float raw = __uint_as_float(v[i + e]);
         const int column = c4 * 32 + i + e;
+        if (MODE == TC_BIASED)
+          raw = fmaf(raw, scale, -r1 * log2_approx(fmaf(r2, static_cast<float>(last - column), 1.0f)));
         const bool ok = !MASKED || (column <= last && column >= first && column > after);
         if (ok) max4[(i >> 1) & 3] = fmaxf(max4[(i >> 1) & 3], raw);
-        const float exponent = CAPPED ? fmaf(cap_log2, tanh_from_exp2(raw * scale), neg_shift) : fmaf(raw, scale, neg_shift);
+        const float exponent = MODE == TC_CAPPED ? fmaf(cap_log2, tanh_from_exp2(raw * scale), neg_shift)
+                               : MODE == TC_BIASED ? raw + neg_shift : fmaf(raw, scale, neg_shift);
         p[e] = ok ? exp2_approx(exponent) : 0.0f;
         sum4[(i >> 1) & 3] += p[e];
       }
@@ -429,7 +444,8 @@ paged_prefill_tc_kernel(const __grid_constant__ PrefillTcArgs a) {
     const unsigned tmem_o = tmem_base + lane_base + 2 * TC_BN;
     const int qp = ctx + q0 + r;
     float m_used = -INFINITY, l_run = 0.0f;
-    const bool capped = a.softcap_log2 > 0.0f;
+    const bool capped = a.softcap_log2 > 0.0f, biased = a.bias_r1 != nullptr;
+    const float r1 = biased ? a.bias_r1[head] : 0.0f, r2 = biased ? a.bias_r2[head] : 0.0f;
     bool failed = false;
     for (int j = 0; j < n_tiles; ++j) {
       const int k0 = first_tile + j * TC_BN;
@@ -456,14 +472,21 @@ paged_prefill_tc_kernel(const __grid_constant__ PrefillTcArgs a) {
         const int after = a.window > 0 ? qp - a.window - k0 : -(1 << 30);
         if (capped) {
           if (open_tile)
-            softmax_pass<false, true>(tmem_s, words, half, a.scale_over_cap, neg_shift, 0, 0, 0, raw_max, row_sum, a.softcap_log2);
+            softmax_pass<false, TC_CAPPED>(tmem_s, words, half, a.scale_over_cap, neg_shift, 0, 0, 0, raw_max, row_sum, a.softcap_log2);
           else
-            softmax_pass<true, true>(tmem_s, words, half, a.scale_over_cap, neg_shift, qp - k0, lo - k0, after, raw_max, row_sum,
-                                     a.softcap_log2);
+            softmax_pass<true, TC_CAPPED>(tmem_s, words, half, a.scale_over_cap, neg_shift, qp - k0, lo - k0, after, raw_max,
+                                          row_sum, a.softcap_log2);
+        } else if (biased) {
+          if (open_tile)
+            softmax_pass<false, TC_BIASED>(tmem_s, words, half, a.scale_log2, neg_shift, qp - k0, 0, 0, raw_max, row_sum, 0.0f,
+                                           r1, r2);
+          else
+            softmax_pass<true, TC_BIASED>(tmem_s, words, half, a.scale_log2, neg_shift, qp - k0, lo - k0, after, raw_max, row_sum,
+                                          0.0f, r1, r2);
         } else if (open_tile) {
-          softmax_pass<false, false>(tmem_s, words, half, a.scale_log2, neg_shift, 0, 0, 0, raw_max, row_sum);
+          softmax_pass<false, TC_PLAIN>(tmem_s, words, half, a.scale_log2, neg_shift, 0, 0, 0, raw_max, row_sum);
         } else {
-          softmax_pass<true, false>(tmem_s, words, half, a.scale_log2, neg_shift, qp - k0, lo - k0, after, raw_max, row_sum);
+          softmax_pass<true, TC_PLAIN>(tmem_s, words, half, a.scale_log2, neg_shift, qp - k0, lo - k0, after, raw_max, row_sum);
         }
         if (attempt == 0) {
           // The row's largest score is the larger of its halves'.
@@ -473,7 +496,8 @@ paged_prefill_tc_kernel(const __grid_constant__ PrefillTcArgs a) {
           raw_max = fmaxf(raw_max, half_note[j & 1][half ^ 1][r]);
         }
         // The scale is positive and the bound grows with its argument: the largest raw score gives the largest exponent.
-        const float row_max = capped ? a.softcap_log2 * tanh_from_exp2(raw_max * a.scale_over_cap) : raw_max * a.scale_log2;
+        const float row_max = capped ? a.softcap_log2 * tanh_from_exp2(raw_max * a.scale_over_cap)
+                              : biased ? raw_max : raw_max * a.scale_log2;
         const bool grow = attempt == 0 && (row_max > m_used + TC_RESCALE_THRESHOLD || (m_used == -INFINITY && row_max > -INFINITY));
         if (!__any_sync(0xffffffffu, grow)) {
           l_run += row_sum;
@@ -622,13 +646,15 @@ ZB_API int zb_paged_prefill_tc_supported(int nh, int nkv, int hd, int dtype, int
 // Attention of the tiles' tokens (tiles of 128 new tokens of one request) over their requests'
 // pages; writes those tokens' rows of `out`.  Arguments as zb_paged_prefill_masked without the chunked mask:
 // `softcap` > 0 bounds the scaled scores by softcap * tanh(. / softcap); `keys_only`: a page holds keys alone
-// and they are the values too; `sinks` (null, or one float32 per query head) join the softmax's denominator.
+// and they are the values too; `sinks` (null, or one float32 per query head) join the softmax's denominator;
+// `bias_r1`, `bias_r2` (null, or one float32 per query head each; not with a softcap) bias the distances.
 ZB_API int zb_paged_prefill_tc_masked(void* out, const void* q, const void* kv_cache, const int* block_table,
                                       int max_blocks, int page_size, int num_pages, int num_rows, const int* tile_row,
                                       const int* tile_q0, int n_tiles, const int* row_q_start, const int* row_q_len,
                                       const int* row_ctx, int nh, int nkv, int hd, int window, float scale, float softcap,
-                                      int keys_only, const float* sinks, int* status, void* stream) {
-  if (n_tiles < 0 || page_size <= 0 || window < 0 || softcap < 0.0f) return ERR_BAD_ARGUMENT;
+                                      int keys_only, const float* sinks, const float* bias_r1, const float* bias_r2,
+                                      int* status, void* stream) {
+  if ((bias_r1 == nullptr) != (bias_r2 == nullptr) || (bias_r1 != nullptr && softcap > 0.0f) || n_tiles < 0 || page_size <= 0 || window < 0 || softcap < 0.0f) return ERR_BAD_ARGUMENT;
   if (!zb_paged_prefill_tc_supported(nh, nkv, hd, DTYPE_BF16, page_size)) return ERR_UNSUPPORTED;
   if (reinterpret_cast<uintptr_t>(q) % 16 != 0 || reinterpret_cast<uintptr_t>(out) % 16 != 0 ||
       reinterpret_cast<uintptr_t>(kv_cache) % 16 != 0)
@@ -654,6 +680,7 @@ ZB_API int zb_paged_prefill_tc_masked(void* out, const void* q, const void* kv_c
   a.scale_over_cap = softcap > 0.0f ? scale / softcap : 0.0f;
   a.keys_only = keys_only;
   a.sinks = sinks;
+  a.bias_r1 = bias_r1; a.bias_r2 = bias_r2;
   a.status = status;
   a.trace = prefill_tc_trace();
   const size_t smem = 2 * TC_STAGES * TC_TILE_BYTES;
@@ -669,5 +696,5 @@ ZB_API int zb_paged_prefill_tc(void* out, const void* q, const void* kv_cache, c
                                int nkv, int hd, int window, float scale, int* status, void* stream) {
   return zb_paged_prefill_tc_masked(out, q, kv_cache, block_table, max_blocks, page_size, num_pages, num_rows, tile_row,
                                     tile_q0, n_tiles, row_q_start, row_q_len, row_ctx, nh, nkv, hd, window, scale, 0.0f, 0,
-                                    nullptr, status, stream);
+                                    nullptr, nullptr, nullptr, status, stream);
 }

@@ -30,6 +30,14 @@
 // only its own: the result is [T, nh, nkv, vd] (a mixing of the heads' weights behind the softmax is a
 // linear map of these).  `out_f32`: the result is written as float32 whatever the cache's type.
 //
+// `bias_r1`, `bias_r2` (one float32 per query head each): r1_h ln(1 + r2_h d) is taken off head h's score of the
+// key d positions back.
+//
+// `score_mix` [nh, nh] mixes the heads' scores ahead of the softmax: s_h <- sum_g M[h, g] s_g.  The scores being
+// linear in the queries, head h's mixed score of position j is the product of ONE wider query with all key
+// heads of j side by side, sum_c q'_hc . k_c(j) with q'_hc = sum over the heads g that read key head c of
+// M[h, g] q_g; so a tile walks the key heads, with the mixed queries of each in float32.
+//
 // One CTA serves one tile: a run of consecutive new tokens of one request, one key/value head,
 // and a chunk of that head's query heads.  The (token, head) pairs of the tile are dealt to the
 // warps; key/value tiles of 32 positions are staged in shared memory once and used by all pairs.
@@ -64,6 +72,9 @@ struct AttentionArgs {
   int pool_max_blocks, pool_num_pages;
   int cross_values;          // grid y = nkv * nkv: (key head, value head) pairs; out [T, nh, nkv, vd]
   int out_f32;
+  const float* bias_r1;      // null, or [nh] each
+  const float* bias_r2;
+  const float* score_mix;    // null, or [nh, nh]
   const float* sinks;        // null, or [nh]: exp(sinks[h]) joins the denominator of head h's softmax
   const float* head_slopes;  // null, or [nh]: query head h adds head_slopes[h] * (key position - query position) to its scores
   int* status;
@@ -141,7 +152,8 @@ paged_attention_simt_kernel(const AttentionArgs a) {
   const T* q = static_cast<const T*>(a.q);
   const T* cache = static_cast<const T*>(a.kv_cache);
 
-  // Queries of all pairs, as float32.
+  // Queries of all pairs, as float32; with mixed scores the mixed queries of one key head (below).
+  if (a.score_mix == nullptr)
   for (int e = threadIdx.x; e < n_pairs * kd; e += blockDim.x) {
     const int p = e / kd, d = e - p * kd;
     const int qi = p / n_heads, hj = p - qi * n_heads;
@@ -181,8 +193,37 @@ paged_attention_simt_kernel(const AttentionArgs a) {
       __syncthreads();     // the previous tile is no longer read (and q_s is complete on the first pass)
       // Positions outside [run_lo, run_hi) hold zeros: a page that was given back, or one that another
       // request used before, is never read.
-      stage_rows<T>(k_s, kstride, source, table, max_blocks, num_pages, a, row, kvh, k0, run_lo, run_hi, kd,
-                    page_elems, 0, tok0);
+      float mixed[ATT_PAIRS_PER_WARP];
+#pragma unroll
+      for (int i = 0; i < ATT_PAIRS_PER_WARP; ++i) mixed[i] = 0.0f;
+      if (a.score_mix != nullptr) {
+        for (int c = 0; c < a.nkv; ++c) {
+          if (c > 0) __syncthreads();                      // the previous key head's tile and queries are read
+          for (int e = threadIdx.x; e < n_pairs * kd; e += blockDim.x) {
+            const int p = e / kd, d = e - p * kd;
+            const int qi = p / n_heads, hj = p - qi * n_heads;
+            const float* m_row = a.score_mix + static_cast<size_t>(kvh * g + chunk * a.heads_per_chunk + hj) * a.nh + c * g;
+            const T* q_row = q + (static_cast<size_t>(tok0 + qi) * a.nh + c * g) * kd + d;
+            float sum = 0.0f;
+            for (int j = 0; j < g; ++j) sum = fmaf(m_row[j], to_float(q_row[static_cast<size_t>(j) * kd]), sum);
+            q_s[p * kd + d] = sum;
+          }
+          stage_rows<T>(k_s, kstride, source, table, max_blocks, num_pages, a, row, c, k0, run_lo, run_hi, kd,
+                        page_elems, 0, tok0);
+          __syncthreads();
+#pragma unroll
+          for (int i = 0; i < ATT_PAIRS_PER_WARP; ++i) {
+            const int p = warp + i * ATT_WARPS;
+            if (p >= n_pairs) continue;
+            const float* qp = q_s + p * kd;
+            const T* kr = k_s + lane * kstride;
+            for (int d = 0; d < kd; ++d) mixed[i] = fmaf(qp[d], to_float(kr[d]), mixed[i]);
+          }
+        }
+      } else {
+        stage_rows<T>(k_s, kstride, source, table, max_blocks, num_pages, a, row, kvh, k0, run_lo, run_hi, kd,
+                      page_elems, 0, tok0);
+      }
       if (!a.shared_kv)
         stage_rows<T>(v_s, vd, source, table, max_blocks, num_pages, a, row, vh, k0, run_lo, run_hi, vd, page_elems,
                       value_part, tok0);
@@ -209,16 +250,22 @@ paged_attention_simt_kernel(const AttentionArgs a) {
           if (k0 > qpos || (k0 + ATT_TILE <= first && k0 >= a.keep_first)) continue;  // no key of this tile is visible
           valid = kp >= lo && kp <= qpos && (kp >= first || kp < a.keep_first);
         }
-        float s = 0.0f;
-        const float* qp = q_s + p * kd;
-        const T* kr = k_s + lane * kstride;
-        for (int d = 0; d + 1 < kd; d += 2) {
-          s = fmaf(qp[d], to_float(kr[d]), s);
-          s = fmaf(qp[d + 1], to_float(kr[d + 1]), s);
+        float s = mixed[i];
+        if (a.score_mix == nullptr) {
+          const float* qp = q_s + p * kd;
+          const T* kr = k_s + lane * kstride;
+          for (int d = 0; d + 1 < kd; d += 2) {
+            s = fmaf(qp[d], to_float(kr[d]), s);
+            s = fmaf(qp[d + 1], to_float(kr[d + 1]), s);
+          }
+          if (kd & 1) s = fmaf(qp[kd - 1], to_float(kr[kd - 1]), s);
         }
-        if (kd & 1) s = fmaf(qp[kd - 1], to_float(kr[kd - 1]), s);
         s *= a.scale;
         if (a.softcap > 0.0f) s = a.softcap * tanhf(s / a.softcap);
+        if (a.bias_r1 != nullptr && valid) {
+          const int head = kvh * g + chunk * a.heads_per_chunk + (p - p / n_heads * n_heads);
+          s -= a.bias_r1[head] * logf(fmaf(a.bias_r2[head], static_cast<float>(qpos - kp), 1.0f));
+        }
         s = valid ? (run == 2 ? fmaf(slope, static_cast<float>(kp - qpos), s) : s) : -INFINITY;
         const float tile_m = warp_max(s);
         if (tile_m == -INFINITY) continue;                 // (a tile of the window that this query has passed)
@@ -322,9 +369,10 @@ ZB_API int zb_paged_attention_simt(void* out, const void* q, const void* kv_cach
                                    int window, int chunk, float scale, float softcap, int shared_kv,
                                    const float* head_slopes, const float* sinks, int keep_first, int pool,
                                    const void* pool_cache, const int* pool_table, int pool_max_blocks,
-                                   int pool_num_pages, int cross_values, int out_f32, int dtype, int* status,
-                                   void* stream) {
-  if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || kd <= 0 || vd <= 0 || page_size <= 0 || n_tiles < 0 || window < 0 ||
+                                   int pool_num_pages, int cross_values, int out_f32, const float* bias_r1,
+                                   const float* bias_r2, const float* score_mix, int dtype, int* status, void* stream) {
+  if ((bias_r1 == nullptr) != (bias_r2 == nullptr) || (score_mix != nullptr && shared_kv) || ((bias_r1 != nullptr || score_mix != nullptr) && pool > 0) ||
+      nh <= 0 || nkv <= 0 || nh % nkv != 0 || kd <= 0 || vd <= 0 || page_size <= 0 || n_tiles < 0 || window < 0 ||
       chunk < 0 || softcap < 0.0f || (shared_kv && kd != vd) || keep_first < 0 || pool < 0 ||
       (pool > 0 && (window <= 0 || pool_cache == nullptr || pool_table == nullptr || pool_max_blocks <= 0)) ||
       (cross_values && shared_kv))
@@ -345,6 +393,7 @@ ZB_API int zb_paged_attention_simt(void* out, const void* q, const void* kv_cach
   a.keep_first = keep_first; a.pool = pool; a.pool_cache = pool_cache; a.pool_table = pool_table;
   a.pool_max_blocks = pool_max_blocks; a.pool_num_pages = pool_num_pages; a.cross_values = cross_values;
   a.out_f32 = out_f32;
+  a.bias_r1 = bias_r1; a.bias_r2 = bias_r2; a.score_mix = score_mix;
   a.status = status;
   auto s = static_cast<cudaStream_t>(stream);
   return dtype == DTYPE_F32 ? attention_simt_dispatch<float>(a, n_tiles, head_chunks, s)

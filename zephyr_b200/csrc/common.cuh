@@ -60,13 +60,16 @@ constexpr int GATE_SILU = 0;
 constexpr int GATE_RELU = 1;
 constexpr int GATE_BOUNDED = 2;
 
+// `row_scale`: null, or one float32 per row of the product; both sums of a row are multiplied by its value
+// first, which is what scaling the row that goes into the product does: act(s G) * (s U).
 struct GateForm {
   int kind;
   const float* bias;
   float limit, alpha, shift;
+  const float* row_scale;
 };
 
-inline GateForm plain_gate(int kind) { return GateForm{kind, nullptr, 0.0f, 1.0f, 0.0f}; }
+inline GateForm plain_gate(int kind) { return GateForm{kind, nullptr, 0.0f, 1.0f, 0.0f, nullptr}; }
 
 // The bounded gate from sums that already carry their biases.
 template <bool FAST>
@@ -82,6 +85,21 @@ __device__ __forceinline__ float bounded_gate(float g, float u, const GateForm& 
     s = 1.0f / (1.0f + expf(-f.alpha * g));
   }
   return g * s * (u + f.shift);
+}
+
+// What an ungated feed-forward's product may do to its sums: the tanh form of GELU,
+// 0.5 z (1 + tanh(u)) with u = sqrt(2 / pi) (z + 0.044715 z^3), as z / (1 + e^(-2u)).
+__device__ __forceinline__ float gelu_tanh(float z) {
+  const float u = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
+  return z / (1.0f + expf(-2.0f * u));
+}
+// The same with the special-function unit's exp2 and reciprocal (about 2^-21, far inside a bfloat16 rounding).
+__device__ __forceinline__ float gelu_tanh_fast(float z) {
+  const float u = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(e) : "f"(-2.8853900817779268f * u));
+  asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(r) : "f"(1.0f + e));
+  return z * r;
 }
 
 __device__ __forceinline__ float warp_sum(float v) {

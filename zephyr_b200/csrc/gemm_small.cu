@@ -34,6 +34,7 @@ struct SmallGemmArgs {
   int M, N, K;
   long long ldx, ldw, ldy;
   GateForm gate;      // with the gated epilogue: what becomes of a gate sum and its up sum
+  int gelu;           // without it: 1 takes the sums through the tanh form of GELU
 };
 
 __device__ __forceinline__ uint4 load16_or_zero(const __nv_bfloat16* p, bool ok) {
@@ -145,7 +146,8 @@ gemm_small_kernel(const SmallGemmArgs a) {
 #pragma unroll
           for (int w = 0; w < GS_WARPS; ++w) sum += parts[c][w * PER_WARP + e];
         const int token = mt * 8 + tok;
-        if (token < a.M && n0 + r < a.N) store_out<TOut>(y + static_cast<size_t>(token) * a.ldy + n0 + r, sum);
+        if (token < a.M && n0 + r < a.N)
+          store_out<TOut>(y + static_cast<size_t>(token) * a.ldy + n0 + r, a.gelu ? gelu_tanh(sum) : sum);
       }
     }
   }
@@ -204,7 +206,8 @@ ZB_API int zb_gemm_small_ksplit(int N, int K) {
 // x: [M, K] bfloat16 rows ldx apart (ldx, ldw multiples of 8, pointers 16-byte aligned);
 // out_dtype: bfloat16 or float32.
 static int small_gemm(void* y, const void* x, const void* w, int M, int N, int K, long long ldx, long long ldw,
-                      long long ldy, int out_dtype, bool gated, const GateForm& gate, void* stream) {
+                      long long ldy, int out_dtype, bool gated, const GateForm& gate, void* stream,
+                      int gelu = 0) {
   if (!zb_gemm_small_supported(M, N, K)) return ERR_UNSUPPORTED;
   if (ldx < K || ldw < K || ldx % 8 != 0 || ldw % 8 != 0 || reinterpret_cast<uintptr_t>(x) % 16 != 0 ||
       reinterpret_cast<uintptr_t>(w) % 16 != 0 || (gated && N % 16 != 0))
@@ -215,6 +218,7 @@ static int small_gemm(void* y, const void* x, const void* w, int M, int N, int K
   a.w = static_cast<const __nv_bfloat16*>(w);
   a.M = M; a.N = N; a.K = K; a.ldx = ldx; a.ldw = ldw; a.ldy = ldy;
   a.gate = gate;
+  a.gelu = gelu;
   const int ksplit = zb_gemm_small_ksplit(N, K);
   auto s = static_cast<cudaStream_t>(stream);
   if (gated)
@@ -230,12 +234,18 @@ ZB_API int zb_gemm_small(void* y, const void* x, const void* w, int M, int N, in
                     plain_gate(swiglu == 2 ? GATE_RELU : GATE_SILU), stream);
 }
 
+// y = gelu_tanh(x w^T).
+ZB_API int zb_gemm_small_gelu(void* y, const void* x, const void* w, int M, int N, int K, long long ldx, long long ldw,
+                              long long ldy, int out_dtype, void* stream) {
+  return small_gemm(y, x, w, M, N, K, ldx, ldw, ldy, out_dtype, false, plain_gate(GATE_SILU), stream, 1);
+}
+
 // The gated form with the bounded gate: y[:, 8j + r] from the sums of w's rows 16j + r (gate) and 16j + 8 + r
 // (up), their biases (bias: float32 [N] in w's row order, or null), the bounds and the shifted product.
 ZB_API int zb_gemm_small_bounded(void* y, const void* x, const void* w, const float* bias, float limit, float alpha,
                                  float shift, int M, int N, int K, long long ldx, long long ldw, long long ldy,
                                  int out_dtype, void* stream) {
   if (!(limit > 0.0f)) return ERR_BAD_ARGUMENT;
-  return small_gemm(y, x, w, M, N, K, ldx, ldw, ldy, out_dtype, true, GateForm{GATE_BOUNDED, bias, limit, alpha, shift},
+  return small_gemm(y, x, w, M, N, K, ldx, ldw, ldy, out_dtype, true, GateForm{GATE_BOUNDED, bias, limit, alpha, shift, nullptr},
                     stream);
 }

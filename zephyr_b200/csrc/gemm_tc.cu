@@ -1,6 +1,6 @@
 // y = x w^T for a prompt's many rows on the fifth-generation tensor cores (tcgen05.mma, accumulators
 // in tensor memory, operands by TMA), with what follows the product done where the sums are read
-// out: nothing, or silu(gate) * up for a packed gate/up weight whose rows alternate in blocks of 8.
+// out: nothing, an activation, or silu(gate) * up for a packed gate/up weight whose rows alternate in blocks of 8.
 //
 // x [M, K] and w [N, K] are bfloat16 with K contiguous.  The kernel is persistent: one CTA per SM
 // takes output tiles of 128 rows x BN columns (BN = 256 or 128) in turn, the tiles that share
@@ -38,6 +38,7 @@ constexpr int GT_THREADS = 192;
 constexpr int GT_WAIT_LIMIT = 1 << 18;
 constexpr int GT_PAIR = 2;                 // as block_n: tiles of 256 x 256 on pairs of SMs
 constexpr int GT_EPI_PLAIN = 0;
+constexpr int GT_EPI_GELU = 4;             // the sums through the tanh form of GELU
 constexpr int GT_EPI_RELU_GATE = 3;        // the interface's code for the gated epilogue with max(gate, 0) in SiLU's place
 constexpr int GT_EPI_SWIGLU = 1;           // columns 16 j .. 16 j + 7 are gates, 16 j + 8 .. 16 j + 15 their ups
 constexpr int GT_EPI_FLOAT = 2;            // the sums as they are, float32 (logits)
@@ -115,6 +116,8 @@ __device__ __forceinline__ void write_out_rows(const CUtensorMap& y_map, unsigne
   constexpr int READS = EPI == GT_EPI_SWIGLU ? 4 : EPI == GT_EPI_FLOAT ? 1 : 2;
   constexpr int PIECES = 8 / READS;                                  // 16-byte pieces a read leaves
   constexpr int GROUP_COLUMNS = EPI == GT_EPI_FLOAT ? 32 : 64;       // output columns of a group
+  // (rows of a grouped product are whole tiles, so every row has its scale)
+  const float scale = EPI == GT_EPI_SWIGLU && form.row_scale != nullptr ? __ldg(form.row_scale + row0 + lane) : 1.0f;
 #pragma unroll 1
   for (int group = 0; group < BN / (32 * READS); ++group) {
     const int out_col = (EPI == GT_EPI_SWIGLU ? n0 / 2 : n0) + group * GROUP_COLUMNS;
@@ -156,8 +159,10 @@ __device__ __forceinline__ void write_out_rows(const CUtensorMap& y_map, unsigne
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
               if (EPI == GT_EPI_SWIGLU) {
-                const float gate = __uint_as_float(v[16 * j + i]), up = __uint_as_float(v[16 * j + 8 + i]);
+                const float gate = __uint_as_float(v[16 * j + i]) * scale, up = __uint_as_float(v[16 * j + 8 + i]) * scale;
                 o[i] = (form.kind == GATE_RELU ? fmaxf(gate, 0.0f) : silu_fast(gate)) * up;
+              } else if (EPI == GT_EPI_GELU) {
+                o[i] = gelu_tanh_fast(__uint_as_float(v[8 * j + i]));
               } else {
                 o[i] = __uint_as_float(v[8 * j + i]);
               }
@@ -575,12 +580,12 @@ ZB_API int zb_gemm_tc_supported(int M, int N, int K, long long ldx, int ldy, int
   if (M <= 0 || N <= 0 || K <= 0 || K % 8 != 0 || ldx % 8 != 0 || ldx < K || (epilogue != GT_EPI_FLOAT && ldy % 8 != 0)) return 0;
   if (epilogue == GT_EPI_SWIGLU) return N % 16 == 0 && ldy >= N / 2;
   if (epilogue == GT_EPI_FLOAT) return ldy % 4 == 0 && ldy >= N;          // ldy counts float32 elements then
-  return epilogue == GT_EPI_PLAIN && ldy >= N;
+  return (epilogue == GT_EPI_PLAIN || epilogue == GT_EPI_GELU) && ldy >= N;
 }
 
 // y = epilogue(x w^T), x and w bfloat16.  epilogue 0: y [M, N] bfloat16; 2: the same in float32;
 // 1: y [M, N / 2] = silu(gate) * up for w's rows in
-// blocks of 8 gate rows and their 8 up rows; 3: the same with max(gate, 0) * up.  block_n is 256 or 128, or 2 for tiles of 256 x 256 on pairs of
+// blocks of 8 gate rows and their 8 up rows; 3: the same with max(gate, 0) * up; 4: y [M, N] bfloat16 = gelu_tanh of the sums.  block_n is 256 or 128, or 2 for tiles of 256 x 256 on pairs of
 // SMs (0: chosen from the sizes).
 static int gemm_tc_run(void* y, const void* x, const void* w, int M, int N, int K, long long ldx, int ldy, int epilogue,
                        const GateForm& gate, int block_n, int* status, void* stream) {
@@ -611,7 +616,10 @@ static int gemm_tc_run(void* y, const void* x, const void* w, int M, int N, int 
   const cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (block_n == GT_PAIR)
     return epilogue == GT_EPI_SWIGLU ? gemm_tc_pair_launch<GT_EPI_SWIGLU>(a, w, sms, s)
-           : epilogue == GT_EPI_FLOAT ? gemm_tc_pair_launch<GT_EPI_FLOAT>(a, w, sms, s) : gemm_tc_pair_launch<GT_EPI_PLAIN>(a, w, sms, s);
+           : epilogue == GT_EPI_FLOAT ? gemm_tc_pair_launch<GT_EPI_FLOAT>(a, w, sms, s)
+           : epilogue == GT_EPI_GELU ? gemm_tc_pair_launch<GT_EPI_GELU>(a, w, sms, s) : gemm_tc_pair_launch<GT_EPI_PLAIN>(a, w, sms, s);
+  if (epilogue == GT_EPI_GELU)
+    return block_n == 256 ? gemm_tc_launch<256, GT_EPI_GELU>(a, w, sms, s) : gemm_tc_launch<128, GT_EPI_GELU>(a, w, sms, s);
   if (epilogue == GT_EPI_FLOAT)
     return block_n == 256 ? gemm_tc_launch<256, GT_EPI_FLOAT>(a, w, sms, s) : gemm_tc_launch<128, GT_EPI_FLOAT>(a, w, sms, s);
   if (epilogue == GT_EPI_SWIGLU)
@@ -633,17 +641,19 @@ ZB_API int zb_gemm_tc_bounded(void* y, const void* x, const void* w, const float
                               float shift, int M, int N, int K, long long ldx, int ldy, int block_n, int* status,
                               void* stream) {
   if (!(limit > 0.0f) || reinterpret_cast<uintptr_t>(bias) % 16 != 0) return ERR_BAD_ARGUMENT;
-  return gemm_tc_run(y, x, w, M, N, K, ldx, ldy, GT_EPI_SWIGLU, GateForm{GATE_BOUNDED, bias, limit, alpha, shift}, block_n,
+  return gemm_tc_run(y, x, w, M, N, K, ldx, ldy, GT_EPI_SWIGLU, GateForm{GATE_BOUNDED, bias, limit, alpha, shift, nullptr}, block_n,
                      status, stream);
 }
 
 // The same over several matrices stacked in w ([groups * N, K]): x [tiles_m * 128, K] is cut into tiles of
 // 128 rows, and tile i multiplies with matrix tile_group[i] (a device array; a negative entry leaves the
 // tile out, its rows of y unwritten).  Rows sorted by expert and padded to whole tiles make a routed
-// feed-forward's products one launch.  Tiles of one SM; epilogues as zb_gemm_tc.
+// feed-forward's products one launch.  Tiles of one SM; epilogues as zb_gemm_tc (not 4).  `row_scale`: null, or one
+// float32 per row of x that goes on both sums of the gated epilogue.
 ZB_API int zb_gemm_tc_grouped(void* y, const void* x, const void* w, const int* tile_group, int tiles_m, int groups,
-                              int N, int K, long long ldx, int ldy, int epilogue, int* status, void* stream) {
-  if (tiles_m <= 0 || groups <= 0 || tile_group == nullptr) return ERR_BAD_ARGUMENT;
+                              int N, int K, long long ldx, int ldy, int epilogue, const float* row_scale, int* status,
+                              void* stream) {
+  if (tiles_m <= 0 || groups <= 0 || tile_group == nullptr || epilogue == GT_EPI_GELU) return ERR_BAD_ARGUMENT;
   const int M = tiles_m * GT_BM;
   if (!zb_gemm_tc_supported(M, N, K, ldx, ldy, epilogue)) return ERR_UNSUPPORTED;
   const int relu_gate = epilogue == GT_EPI_RELU_GATE;
@@ -658,6 +668,7 @@ ZB_API int zb_gemm_tc_grouped(void* y, const void* x, const void* w, const int* 
   GemmTcArgs a;
   a.M = M; a.N = N; a.K = K;
   a.gate = plain_gate(relu_gate ? GATE_RELU : GATE_SILU);
+  a.gate.row_scale = row_scale;
   a.tile_group = tile_group;
   a.groups = groups;
   a.status = status;

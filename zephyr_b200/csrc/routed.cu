@@ -18,6 +18,10 @@
 //             was routed to its expert; float32 on CUDA cores, bfloat16 on the tensor cores
 //   combine   out[t] = sum_j weight[t, j] * (expert output of slot (t, j), or x[t] for an identity
 //             expert), in float32 and in the order of j, rounded once.
+//
+// The weights may go on the experts' inputs instead: out = sum of expert_e(s_e x).  The gate and up sums of a
+// slot are then multiplied by its weight, unrounded, ahead of the activation, and the outputs are added up as
+// they are.
 #include "tile_product.cuh"
 #include "tile_product_mma.cuh"
 
@@ -262,8 +266,11 @@ align_padded_kernel(int* tile_group, int* slots, int* place_of_slot, const int* 
 }
 
 // out[place, :] = x[slots[place] / top, :], zeros where the place pads an expert's run.  16-byte pieces.
-__global__ void gather_places_kernel(uint4* out, const uint4* x, long long x_stride16, const int* slots, int pieces, int top) {
+// With `place_scale` also the slot's weight for each place (zero for a pad).
+__global__ void gather_places_kernel(uint4* out, const uint4* x, long long x_stride16, const int* slots, int pieces, int top,
+                                     float* place_scale, const float* weights) {
   const int place = blockIdx.x, slot = slots[place];
+  if (place_scale != nullptr && threadIdx.x == 0) place_scale[place] = slot >= 0 ? weights[slot] : 0.0f;
   const uint4* src = slot >= 0 ? x + static_cast<long long>(slot / top) * x_stride16 : nullptr;
   for (int i = threadIdx.x; i < pieces; i += blockDim.x)
     out[static_cast<size_t>(place) * pieces + i] = src != nullptr ? src[i] : make_uint4(0, 0, 0, 0);
@@ -279,6 +286,7 @@ struct ExpertProductArgs {
   const int* slots;
   long long x_stride;
   int N, K, top, act;
+  const float* weights;    // null, or per slot what both sums of the gate/up product are multiplied by
   int interleaved;         // gate/up: w0 is [experts, 2 N, K], blocks of 8 gate rows each followed by its 8 up rows
 };
 
@@ -297,6 +305,14 @@ __device__ __forceinline__ void gate_up_rows(const ExpertProductArgs& a, int exp
 
 __device__ __forceinline__ float expert_act(float g, int act) {
   return act == 1 ? fmaxf(g, 0.0f) : g / (1.0f + expf(-g));
+}
+
+// What a gate sum and its up sum become.  Without weights on the inputs both are rounded to the model's type
+// before the activation, as separate products would leave them.
+template <typename T>
+__device__ __forceinline__ float gated_value(float gate, float up, float scale, const ExpertProductArgs& a) {
+  if (a.weights != nullptr) return expert_act(scale * gate, a.act) * (scale * up);
+  return expert_act(to_float(from_float<T>(gate)), a.act) * to_float(from_float<T>(up));
 }
 
 // hidden[place, n] = act(gate_e x_t) * (up_e x_t) for the tile's places; x_t is gathered by slot / top.
@@ -323,12 +339,11 @@ __global__ void __launch_bounds__(TP_THREADS) expert_gate_up_kernel(const Expert
     const int r = 2 * ty + m;
     if (r >= rows) continue;
     T* dst = static_cast<T*>(a.out) + static_cast<size_t>(place0 + r) * a.N;
+    const float scale = a.weights != nullptr ? a.weights[a.slots[place0 + r]] : 1.0f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx + 16 * j;
-      // The gate is rounded to the model's type before its activation, as a separate product would leave it.
-      if (n < a.N) dst[n] = from_float<T>(expert_act(to_float(from_float<T>(acc[m][0][j])), a.act) *
-                                          to_float(from_float<T>(acc[m][1][j])));
+      if (n < a.N) dst[n] = from_float<T>(gated_value<T>(acc[m][0][j], acc[m][1][j], scale, a));
     }
   }
 }
@@ -381,6 +396,10 @@ __global__ void __launch_bounds__(TM_THREADS) expert_gate_up_mma_kernel(const Ex
   gate_up_rows(a, expert, n0, gate, up);
   float acc[2][4][4];
   tile_product_mma<true, T>(sm, gate, up, a.N - n0, a.K, vectors != 0, vectors != 0, acc, a.interleaved != 0);
+  float scale[4];
+#pragma unroll
+  for (int c = 0; c < 4; ++c)
+    scale[c] = a.weights != nullptr && tm_row(c) < rows ? a.weights[a.slots[place0 + tm_row(c)]] : 1.0f;
 #pragma unroll
   for (int nt = 0; nt < 4; ++nt)
 #pragma unroll
@@ -388,7 +407,7 @@ __global__ void __launch_bounds__(TM_THREADS) expert_gate_up_mma_kernel(const Ex
       const int r = tm_row(c), n = n0 + tm_col(nt, c);
       if (r < rows && n < a.N)
         static_cast<T*>(a.out)[static_cast<size_t>(place0 + r) * a.N + n] =
-            from_float<T>(expert_act(to_float(from_float<T>(acc[0][nt][c])), a.act) * to_float(from_float<T>(acc[1][nt][c])));
+            from_float<T>(gated_value<T>(acc[0][nt][c], acc[1][nt][c], scale[c], a));
     }
 }
 
@@ -426,7 +445,7 @@ __global__ void combine_kernel(T* out, const Y* y, long long y_stride, const T* 
     float sum = 0.0f;
     for (int j = 0; j < top; ++j) {
       const int slot = t * top + j, place = place_of_slot[slot];
-      const float w = weights[slot];
+      const float w = weights != nullptr ? weights[slot] : 1.0f;
       // An expert's output takes the model's type before it is weighted, as a layer of its own would leave it.
       const float v = place >= 0 ? to_float(from_float<T>(to_float(y[static_cast<size_t>(place) * y_stride + i])))
                                  : to_float(x[t * x_stride + i]);
@@ -446,7 +465,7 @@ __global__ void combine_pieces_kernel(uint4* out, const uint4* y, long long y_st
   __shared__ float weight_s[COMBINE_MAX_TOP];
   if (threadIdx.x < top) {
     place_s[threadIdx.x] = place_of_slot[t * top + threadIdx.x];
-    weight_s[threadIdx.x] = weights[t * top + threadIdx.x];
+    weight_s[threadIdx.x] = weights != nullptr ? weights[t * top + threadIdx.x] : 1.0f;
   }
   __syncthreads();
   for (int i = threadIdx.x; i < pieces; i += blockDim.x) {
@@ -522,16 +541,18 @@ ZB_API int zb_route_align(int* plan, int* slots, int* place_of_slot, const int* 
 }
 
 // `down` = 0: hidden = act(gate x) * (up x), N = ff, K = width; 1: y = down hidden, N = width, K = ff.
+// `input_weights` (gate/up only; null: none): one float32 per slot that goes on both sums ahead of the activation.
 // Without w1 the gate/up product reads w0 as [experts, 2 N, K] in blocks of 8 gate rows and their 8 up rows.
 ZB_API int zb_expert_product(void* out, const void* x, long long x_stride, const void* w0, const void* w1,
-                             const int* plan, const int* slots, int max_tiles, int N, int K, int top, int act,
-                             int down, int dtype, void* stream) {
-  if (max_tiles < 0 || N <= 0 || K <= 0 || top <= 0 || (act != 0 && act != 1)) return ERR_BAD_ARGUMENT;
+                             const int* plan, const int* slots, const float* input_weights, int max_tiles, int N,
+                             int K, int top, int act, int down, int dtype, void* stream) {
+  if ((down && input_weights != nullptr) || max_tiles < 0 || N <= 0 || K <= 0 || top <= 0 || (act != 0 && act != 1)) return ERR_BAD_ARGUMENT;
   if (!down && w1 == nullptr && N % 8 != 0) return ERR_BAD_ARGUMENT;
   if (max_tiles == 0) return OK;
   ExpertProductArgs a;
   a.out = out; a.x = x; a.w0 = w0; a.w1 = w1; a.plan = plan; a.slots = slots; a.x_stride = x_stride;
   a.N = N; a.K = K; a.top = top; a.act = act;
+  a.weights = input_weights;
   a.interleaved = !down && w1 == nullptr;
   const dim3 grid(max_tiles, (N + TP_BN - 1) / TP_BN);       // both tile forms are 64 outputs wide
   static_assert(TP_BN == TM_BN, "one grid for both forms");
@@ -561,17 +582,17 @@ ZB_API int zb_route_align_padded(int* tile_group, int* slots, int* place_of_slot
 
 // out [places, width] = the tokens' rows in the order of `slots` (bfloat16; width a multiple of 8, 16-byte aligned rows).
 ZB_API int zb_gather_places(void* out, const void* x, long long x_stride, const int* slots, int places, int width,
-                            int top, void* stream) {
-  if (places < 0 || width <= 0 || width % 8 != 0 || x_stride % 8 != 0 || top <= 0 ||
+                            int top, float* place_scale, const float* weights, void* stream) {
+  if ((place_scale != nullptr && weights == nullptr) || places < 0 || width <= 0 || width % 8 != 0 || x_stride % 8 != 0 || top <= 0 ||
       reinterpret_cast<uintptr_t>(out) % 16 != 0 || reinterpret_cast<uintptr_t>(x) % 16 != 0)
     return ERR_BAD_ARGUMENT;
   if (places == 0) return OK;
   gather_places_kernel<<<places, 128, 0, static_cast<cudaStream_t>(stream)>>>(
-      static_cast<uint4*>(out), static_cast<const uint4*>(x), x_stride / 8, slots, width / 8, top);
+      static_cast<uint4*>(out), static_cast<const uint4*>(x), x_stride / 8, slots, width / 8, top, place_scale, weights);
   return launch_result();
 }
 
-// `y_dtype`: float32 sums, or the model's type (what the grouped tcgen05 product writes).
+// `weights` null: the outputs are added up as they are.  `y_dtype`: float32 sums, or the model's type (what the grouped tcgen05 product writes).
 ZB_API int zb_route_combine(void* out, const void* y, long long y_stride, int y_dtype, const void* x, long long x_stride,
                             const int* ids, const float* weights, const int* place_of_slot, int tokens, int width, int top,
                             int dtype, void* stream) {

@@ -7,10 +7,13 @@
 //                           second small kernel refreshes with the step's last token.
 //   sum + RMS norm          x += (a + b) in float32 (either summand may be absent), then
 //                           y = x / sqrt(mean(x^2) + eps) * w in the model's type; also the plain norm of
-//                           float32 rows that are a slice of wider rows.
+//                           float32 rows that are a slice of wider rows; and the norm in groups, where each
+//                           of several equal consecutive parts of a row has a mean square of its own.
 //   clamped gate            g = min(G + b_g, limit), u = clamp(U + b_u, -limit, limit),
 //                           y = g * sigmoid(alpha * g) * (u + shift), from a float32 or bfloat16 product.
 //   scale                   y *= s on float32 rows (a multiplier on logits).
+//   activation              y = gelu(x), element by element (an ungated feed-forward whose product has no
+//                           epilogue for it).
 #include "common.cuh"
 
 #include <algorithm>
@@ -102,8 +105,9 @@ __global__ void store_last_token_kernel(int* last_token, const int* ids, const i
 }
 
 // ------------------------------------------------------------------------------------ sum + RMS norm
-// One CTA a row.  The row is summed into the stream first (and kept in registers where it fits), then
-// normed.  PER: elements a thread keeps; rows longer than PER * threads re-read the stream.
+// One CTA a row, or a group of a row (the grid's y counts the groups of H values; a norm without groups has
+// one).  The values are summed into the stream first (and kept in registers where they fit), then normed.
+// PER: elements a thread keeps; rows longer than PER * threads re-read the stream.
 constexpr int SN_THREADS = 256;
 constexpr int SN_PER = 16;
 
@@ -112,16 +116,17 @@ __global__ void __launch_bounds__(SN_THREADS)
 sum_rms_norm_kernel(OUT* out, long long out_stride, float* x, long long x_stride, const A* a, const B* b,
                     const float* bias, const void* w, int w_dtype, float eps, int H) {
   __shared__ float scratch[33];
-  const long long r = blockIdx.x;
-  float* xr = x + r * x_stride;
-  const A* ar = a != nullptr ? a + r * H : nullptr;
-  const B* br = b != nullptr ? b + r * H : nullptr;
+  const long long r = blockIdx.x, summand_stride = static_cast<long long>(H) * gridDim.y;
+  const int g0 = blockIdx.y * H;             // where this group begins in its row
+  float* xr = x + r * x_stride + g0;
+  const A* ar = a != nullptr ? a + r * summand_stride + g0 : nullptr;
+  const B* br = b != nullptr ? b + r * summand_stride + g0 : nullptr;
   const bool sums = ar != nullptr || br != nullptr;
   auto summed = [&](int i) {
     float v = xr[i];
     if (sums) {
       float s = (ar != nullptr ? to_float(ar[i]) : 0.0f) + (br != nullptr ? to_float(br[i]) : 0.0f);
-      if (bias != nullptr) s += bias[i];
+      if (bias != nullptr) s += bias[g0 + i];
       v += s;
       xr[i] = v;
     }
@@ -141,14 +146,14 @@ sum_rms_norm_kernel(OUT* out, long long out_stride, float* x, long long x_stride
   }
   if (out == nullptr) return;
   const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(H) + eps);
-  OUT* o = out + r * out_stride;
+  OUT* o = out + r * out_stride + g0;
 #pragma unroll
   for (int k = 0; k < SN_PER; ++k) {
     const int i = threadIdx.x + k * SN_THREADS;
-    if (i < H) o[i] = from_float<OUT>(keep[k] * inv * load_scale(w, w_dtype, i));
+    if (i < H) o[i] = from_float<OUT>(keep[k] * inv * load_scale(w, w_dtype, g0 + i));
   }
   for (int i = threadIdx.x + SN_PER * SN_THREADS; i < H; i += SN_THREADS)
-    o[i] = from_float<OUT>(xr[i] * inv * load_scale(w, w_dtype, i));
+    o[i] = from_float<OUT>(xr[i] * inv * load_scale(w, w_dtype, g0 + i));
 }
 
 // The same with four values a thread and step: H a multiple of 4, every row and base aligned for that.
@@ -157,10 +162,11 @@ __global__ void __launch_bounds__(SN_THREADS)
 sum_rms_norm_vec_kernel(OUT* out, long long out_stride, float* x, long long x_stride, const A* a, const B* b,
                         const float* bias, const void* w, int w_dtype, float eps, int H) {
   __shared__ float scratch[33];
-  const long long r = blockIdx.x;
-  float* xr = x + r * x_stride;
-  const A* ar = a != nullptr ? a + r * H : nullptr;
-  const B* br = b != nullptr ? b + r * H : nullptr;
+  const long long r = blockIdx.x, summand_stride = static_cast<long long>(H) * gridDim.y;
+  const int g0 = blockIdx.y * H;             // where this group begins in its row
+  float* xr = x + r * x_stride + g0;
+  const A* ar = a != nullptr ? a + r * summand_stride + g0 : nullptr;
+  const B* br = b != nullptr ? b + r * summand_stride + g0 : nullptr;
   const bool sums = ar != nullptr || br != nullptr;
   auto summed = [&](int i) {
     float4 v = load4(xr + i);
@@ -169,7 +175,7 @@ sum_rms_norm_vec_kernel(OUT* out, long long out_stride, float* x, long long x_st
       const float4 q = br != nullptr ? load4(br + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
       float4 s = make_float4(p.x + q.x, p.y + q.y, p.z + q.z, p.w + q.w);
       if (bias != nullptr) {
-        const float4 c = load4(bias + i);
+        const float4 c = load4(bias + g0 + i);
         s.x += c.x; s.y += c.y; s.z += c.z; s.w += c.w;
       }
       v.x += s.x; v.y += s.y; v.z += s.z; v.w += s.w;
@@ -178,8 +184,8 @@ sum_rms_norm_vec_kernel(OUT* out, long long out_stride, float* x, long long x_st
     return v;
   };
   auto scaled = [&](float4 v, float inv, int i) {
-    const float4 s = w_dtype == DTYPE_F32 ? load4(static_cast<const float*>(w) + i)
-                                          : load4(static_cast<const __nv_bfloat16*>(w) + i);
+    const float4 s = w_dtype == DTYPE_F32 ? load4(static_cast<const float*>(w) + g0 + i)
+                                          : load4(static_cast<const __nv_bfloat16*>(w) + g0 + i);
     return make_float4(v.x * inv * s.x, v.y * inv * s.y, v.z * inv * s.z, v.w * inv * s.w);
   };
   constexpr int PER = SN_PER / 4;
@@ -197,7 +203,7 @@ sum_rms_norm_vec_kernel(OUT* out, long long out_stride, float* x, long long x_st
   }
   if (out == nullptr) return;
   const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(H) + eps);
-  OUT* o = out + r * out_stride;
+  OUT* o = out + r * out_stride + g0;
 #pragma unroll
   for (int k = 0; k < PER; ++k) {
     const int i = 4 * (threadIdx.x + k * SN_THREADS);
@@ -217,7 +223,7 @@ clamped_gate_vec_kernel(OUT* out, const IN* gu, const float* bias, int T, int I,
   constexpr int PIECE = 16 / sizeof(IN);
   // A CTA walks rows, a thread pieces of its row: no division, and a row's pieces are neighbours.
   const int per_row = I / PIECE;
-  const GateForm form{GATE_BOUNDED, bias, limit, alpha, shift};
+  const GateForm form{GATE_BOUNDED, bias, limit, alpha, shift, nullptr};
   for (long long t = blockIdx.x; t < T; t += gridDim.x)
   for (int j = threadIdx.x; j < per_row; j += blockDim.x) {
     const int o0 = PIECE * j;
@@ -276,6 +282,23 @@ __global__ void scale_rows_kernel(float* y, long long total, float scale) {
     y[at] *= scale;
 }
 
+template <typename IN, typename OUT>
+__global__ void __launch_bounds__(256) gelu_rows_kernel(OUT* out, const IN* x, long long total) {
+  for (long long at = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; at < total;
+       at += static_cast<long long>(gridDim.x) * blockDim.x)
+    out[at] = from_float<OUT>(gelu_tanh(to_float(x[at])));
+}
+
+// The same four values at a time.
+template <typename IN, typename OUT>
+__global__ void __launch_bounds__(256) gelu_rows_vec_kernel(OUT* out, const IN* x, long long total4) {
+  for (long long at = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; at < total4;
+       at += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const float4 v = load4(x + 4 * at);
+    store4(out + 4 * at, make_float4(gelu_tanh(v.x), gelu_tanh(v.y), gelu_tanh(v.z), gelu_tanh(v.w)));
+  }
+}
+
 inline int grid_for(long long total, int threads) {
   return static_cast<int>(std::min<long long>((total + threads - 1) / threads, 148LL * 16));
 }
@@ -324,11 +347,12 @@ ZB_API int zb_store_last_token(int* last_token, const int* ids, const int* row_q
 
 // x [rows, H] float32 (rows x_stride apart) += (a + b + bias), a and b contiguous [rows, H] of their own types
 // or null, bias float32 [H] (a shift of one of the summands, added to every row; only beside a summand) or
-// null; then, unless out is null, out [rows, H] (rows out_stride apart) = rmsnorm(x) * w.
+// null; then, unless out is null, out [rows, H] (rows out_stride apart) = rmsnorm(x) * w, each of `groups` equal
+// consecutive parts of a row divided by its own root mean square.
 ZB_API int zb_sum_rms_norm(void* out, long long out_stride, int out_dtype, float* x, long long x_stride, const void* a,
                            int a_dtype, const void* b, int b_dtype, const float* bias, const void* w, int w_dtype,
-                           float eps, int rows, int H, void* stream) {
-  if (rows < 0 || H <= 0 || x_stride < H || (out != nullptr && (out_stride < H || w == nullptr)) ||
+                           float eps, int rows, int H, int groups, void* stream) {
+  if (groups <= 0 || groups > 65535 || rows < 0 || H <= 0 || H % groups != 0 || x_stride < H || (out != nullptr && (out_stride < H || w == nullptr)) ||
       (bias != nullptr && a == nullptr && b == nullptr))
     return ERR_BAD_ARGUMENT;
   if (rows == 0) return OK;
@@ -337,16 +361,18 @@ ZB_API int zb_sum_rms_norm(void* out, long long out_stride, int out_dtype, float
   const int a_bytes = a_dtype == DTYPE_F32 ? 16 : 8, b_bytes = b_dtype == DTYPE_F32 ? 16 : 8;
   const int o_bytes = out_dtype == DTYPE_F32 ? 16 : 8, w_bytes = w_dtype == DTYPE_F32 ? 16 : 8;
   auto fits = [](const void* p, int bytes) { return reinterpret_cast<uintptr_t>(p) % bytes == 0; };
-  const bool vectors = H % 4 == 0 && x_stride % 4 == 0 && out_stride % 4 == 0 && fits(x, 16) && fits(a, a_bytes) &&
+  const int part = H / groups;
+  const dim3 grid(rows, groups);
+  const bool vectors = part % 4 == 0 && x_stride % 4 == 0 && out_stride % 4 == 0 && fits(x, 16) && fits(a, a_bytes) &&
                        fits(b, b_bytes) && fits(out, o_bytes) && fits(w, w_bytes) && fits(bias, 16);
 #define ZB_SN(A_, B_, OUT_)                                                                                          \
   {                                                                                                                  \
     if (vectors)                                                                                                     \
-      sum_rms_norm_vec_kernel<A_, B_, OUT_><<<rows, SN_THREADS, 0, s>>>((OUT_*)out, out_stride, x, x_stride,         \
-                                                                         (const A_*)a, (const B_*)b, bias, w, w_dtype, eps, H); \
+      sum_rms_norm_vec_kernel<A_, B_, OUT_><<<grid, SN_THREADS, 0, s>>>((OUT_*)out, out_stride, x, x_stride,         \
+                                                                         (const A_*)a, (const B_*)b, bias, w, w_dtype, eps, part); \
     else                                                                                                             \
-      sum_rms_norm_kernel<A_, B_, OUT_><<<rows, SN_THREADS, 0, s>>>((OUT_*)out, out_stride, x, x_stride, (const A_*)a, \
-                                                                     (const B_*)b, bias, w, w_dtype, eps, H);        \
+      sum_rms_norm_kernel<A_, B_, OUT_><<<grid, SN_THREADS, 0, s>>>((OUT_*)out, out_stride, x, x_stride, (const A_*)a, \
+                                                                     (const B_*)b, bias, w, w_dtype, eps, part);     \
   }
 #define ZB_SN_OUT(A_, B_)                              \
   {                                                    \
@@ -401,5 +427,25 @@ ZB_API int zb_scale_rows(float* y, long long total, float scale, void* stream) {
   if (total < 0) return ERR_BAD_ARGUMENT;
   if (total == 0) return OK;
   scale_rows_kernel<<<grid_for(total, 256), 256, 0, static_cast<cudaStream_t>(stream)>>>(y, total, scale);
+  return launch_result();
+}
+
+// out [total] = gelu_tanh(x [total]) in float32, rounded once; both contiguous.
+ZB_API int zb_gelu_rows(void* out, int out_dtype, const void* x, int in_dtype, long long total, void* stream) {
+  if (total < 0 || (out_dtype == DTYPE_F32 && in_dtype != DTYPE_F32)) return ERR_BAD_ARGUMENT;
+  if (total == 0) return OK;
+  auto s = static_cast<cudaStream_t>(stream);
+  using bf16 = __nv_bfloat16;
+#define ZB_GELU(IN, OUT)                                                                                       \
+  {                                                                                                            \
+    if (total % 4 == 0 && aligned_for4<IN>(x) && aligned_for4<OUT>(out))                                       \
+      gelu_rows_vec_kernel<IN, OUT><<<grid_for(total / 4, 256), 256, 0, s>>>((OUT*)out, (const IN*)x, total / 4); \
+    else                                                                                                       \
+      gelu_rows_kernel<IN, OUT><<<grid_for(total, 256), 256, 0, s>>>((OUT*)out, (const IN*)x, total);          \
+  }
+  if (out_dtype == DTYPE_F32) ZB_GELU(float, float)
+  else if (in_dtype == DTYPE_F32) ZB_GELU(float, bf16)
+  else ZB_GELU(bf16, bf16)
+#undef ZB_GELU
   return launch_result();
 }

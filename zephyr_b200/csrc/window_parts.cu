@@ -2,7 +2,7 @@
 // pooled blocks, and whose heads' weights are mixed behind the softmax.
 //
 //   qkv_halves   from a fused q/k/v projection (float32 or the model's type) to queries and cache entries:
-//                  an RMS norm of q and of k, either per head with one scale vector shared by the heads,
+//                  optionally a bias on every column; an RMS norm of q and of k, either per head with one scale vector shared by the heads,
 //                  or over ALL heads of the projection at once with a scale per column, or none;
 //                  the rotation of halves on the first `rot_dims` values of every q and k head: value i
 //                  pairs with value i + rot_dims / 2, (u, v) -> (u c - v s, v c + u s), c, s = cos, sin of
@@ -15,7 +15,8 @@
 //                  CTA of the token that completes a block writes it.
 //   head_mix     out[t, h] = sum_g M[h, g] * a[t, g, kv(h)], with a [T, heads, kv_heads, vd] float32 what
 //                  every head's softmax weights make of every key/value head's values.
-//   sigmoid_gate x[t, c] *= 1 / (1 + exp(-gate[t, c])), the gate float32 with strided rows.
+//   sigmoid_gate x[t, c] *= 1 / (1 + exp(-gate[t, c / per])), the gate float32 with strided rows: value by value
+//                  (per = 1), or one gate for every run of `per` values (a head's output).
 #include "common.cuh"
 
 namespace zb {
@@ -31,6 +32,7 @@ struct QkvHalvesArgs {
   void* q_out;               // [T, nh * kd]
   const void* qkv;           // [T, stride]: q heads, k heads, v heads
   long long stride;
+  const float* bias;         // null or [columns]
   int norm_mode;
   const float* q_norm_w;
   const float* k_norm_w;
@@ -58,7 +60,7 @@ __global__ void __launch_bounds__(QH_THREADS) qkv_halves_kernel(const QkvHalvesA
   float* x = qh_smem;                    // [cols]
   float* head_ss = qh_smem + cols;       // [heads]
   const IN* src = static_cast<const IN*>(a.qkv) + static_cast<long long>(t) * a.stride;
-  for (int i = threadIdx.x; i < cols; i += QH_THREADS) x[i] = to_float(src[i]);
+  for (int i = threadIdx.x; i < cols; i += QH_THREADS) x[i] = to_float(src[i]) + (a.bias != nullptr ? a.bias[i] : 0.0f);
   __syncthreads();
   // Every head's sum of squares, by one warp in lane order.
   for (int h = warp; h < heads; h += QH_WARPS) {
@@ -259,10 +261,10 @@ head_mix_kernel(T* out, const float* a, const float* mix, int nh, int nkv, int v
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-sigmoid_gate_kernel(T* x, const float* gate, long long gate_stride, int width) {
+sigmoid_gate_kernel(T* x, const float* gate, long long gate_stride, int width, int per) {
   const long long t = blockIdx.x;
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
-    const float g = 1.0f / (1.0f + expf(-gate[t * gate_stride + c]));
+    const float g = 1.0f / (1.0f + expf(-gate[t * gate_stride + (per == 1 ? c : c / per)]));
     x[t * width + c] = from_float<T>(to_float(x[t * width + c]) * g);
   }
 }
@@ -271,7 +273,7 @@ sigmoid_gate_kernel(T* x, const float* gate, long long gate_stride, int width) {
 
 using namespace zb;
 
-ZB_API int zb_qkv_halves(void* q_out, const void* qkv, long long stride, int norm_mode, const float* q_norm_w,
+ZB_API int zb_qkv_halves(void* q_out, const void* qkv, long long stride, const float* bias, int norm_mode, const float* q_norm_w,
                          const float* k_norm_w, float eps, const float* freqs, int rot_dims, float rot_mult,
                          int value_unit_norm, const int* positions, const int* token_row, void* cache,
                          const int* block_table, int max_blocks, int page_size, int num_pages, int num_rows,
@@ -284,7 +286,7 @@ ZB_API int zb_qkv_halves(void* q_out, const void* qkv, long long stride, int nor
   if (dtype == DTYPE_F32 && in_dtype != DTYPE_F32) return ERR_BAD_ARGUMENT;
   if (tokens == 0) return OK;
   QkvHalvesArgs a;
-  a.q_out = q_out; a.qkv = qkv; a.stride = stride; a.norm_mode = norm_mode; a.q_norm_w = q_norm_w;
+  a.q_out = q_out; a.qkv = qkv; a.stride = stride; a.bias = bias; a.norm_mode = norm_mode; a.q_norm_w = q_norm_w;
   a.k_norm_w = k_norm_w; a.eps = eps; a.freqs = freqs; a.rot_dims = freqs != nullptr ? rot_dims : 0;
   a.rot_mult = rot_mult; a.value_unit_norm = value_unit_norm; a.positions = positions; a.token_row = token_row;
   a.cache = cache; a.block_table = block_table; a.max_blocks = max_blocks; a.page_size = page_size;
@@ -340,12 +342,12 @@ ZB_API int zb_head_mix(void* out, const float* a, const float* mix, int tokens, 
   return launch_result();
 }
 
-ZB_API int zb_sigmoid_gate(void* x, const float* gate, long long gate_stride, int tokens, int width, int dtype,
-                           void* stream) {
-  if (tokens < 0 || width <= 0 || gate_stride < width) return ERR_BAD_ARGUMENT;
+ZB_API int zb_sigmoid_gate(void* x, const float* gate, long long gate_stride, int tokens, int width, int per,
+                           int dtype, void* stream) {
+  if (tokens < 0 || width <= 0 || per <= 0 || width % per != 0 || gate_stride < width / per) return ERR_BAD_ARGUMENT;
   if (tokens == 0) return OK;
   auto s = static_cast<cudaStream_t>(stream);
-  if (dtype == DTYPE_F32) sigmoid_gate_kernel<float><<<tokens, 256, 0, s>>>(static_cast<float*>(x), gate, gate_stride, width);
-  else sigmoid_gate_kernel<__nv_bfloat16><<<tokens, 256, 0, s>>>(static_cast<__nv_bfloat16*>(x), gate, gate_stride, width);
+  if (dtype == DTYPE_F32) sigmoid_gate_kernel<float><<<tokens, 256, 0, s>>>(static_cast<float*>(x), gate, gate_stride, width, per);
+  else sigmoid_gate_kernel<__nv_bfloat16><<<tokens, 256, 0, s>>>(static_cast<__nv_bfloat16*>(x), gate, gate_stride, width, per);
   return launch_result();
 }

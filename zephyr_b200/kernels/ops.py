@@ -66,7 +66,8 @@ _SIGNATURES = {
                           c_void_p],
     "zb_store_last_token": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
     "zb_sum_rms_norm": [c_void_p, c_longlong, c_int, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_int, c_void_p,
-                        c_void_p, c_int, c_float, c_int, c_int, c_void_p],
+                        c_void_p, c_int, c_float, c_int, c_int, c_int, c_void_p],
+    "zb_gelu_rows": [c_void_p, c_int, c_void_p, c_int, c_longlong, c_void_p],
     "zb_clamped_gate": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float,
                         c_void_p],
     "zb_scale_rows": [c_void_p, c_longlong, c_float, c_void_p],
@@ -77,12 +78,12 @@ _SIGNATURES = {
     "zb_expert_tile_rows": [c_int],
     "zb_route": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_void_p],
     "zb_route_align": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
-    "zb_expert_product": [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                          c_int, c_int, c_int, c_int, c_void_p],
+    "zb_expert_product": [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                          c_int, c_int, c_int, c_int, c_int, c_void_p],
     "zb_route_align_padded": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
-    "zb_gather_places": [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_void_p],
+    "zb_gather_places": [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
     "zb_gemm_tc_grouped": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_longlong, c_int, c_int,
-                           c_void_p, c_void_p],
+                           c_void_p, c_void_p, c_void_p],
     "zb_route_combine": [c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int,
                          c_int, c_int, c_int, c_void_p],
     "zb_add_bias": [c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
@@ -97,14 +98,19 @@ _SIGNATURES = {
     "zb_paged_attention_simt": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
                                 c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                 c_int, c_float, c_float, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
-                                c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
-    "zb_qkv_halves": [c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_float,
+                                c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
+    "zb_heads_attention_tile_tokens": [c_int, c_int, c_int, c_int, c_int],
+    "zb_heads_attention_tile_keys": [c_int, c_int, c_int, c_int],
+    "zb_heads_attention": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
+                           c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p,
+                           c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p],
+    "zb_qkv_halves": [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_float,
                       c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                       c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "zb_pool_blocks": [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int,
                        c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "zb_head_mix": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
-    "zb_sigmoid_gate": [c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p],
+    "zb_sigmoid_gate": [c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p],
     "zb_delta_max_channels": [],
     "zb_delta_gates": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p,
                        c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_int,
@@ -140,14 +146,14 @@ _SIGNATURES = {
                         c_void_p, c_void_p],
     "zb_paged_decode_masked": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int,
                                c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p,
-                               c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
+                               c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
     "zb_paged_prefill_masked": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
                                 c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
                                 c_float, c_int, c_void_p, c_void_p, c_void_p],
     "zb_paged_prefill_windowed": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
                                   c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
                                   c_float, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                                  c_int, c_void_p, c_void_p],
+                                  c_int, c_void_p, c_void_p, c_void_p, c_void_p],
     "zb_paged_decode_fused": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p,
                               c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                               c_longlong, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p],
@@ -160,7 +166,7 @@ _SIGNATURES = {
     "zb_paged_prefill_tc_set_trace": [c_void_p],
     "zb_paged_prefill_tc_masked": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
                                    c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_int,
-                                   c_void_p, c_void_p, c_void_p],
+                                   c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
     "zb_paged_prefill_tc": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
                             c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p],
     "zb_gemm_small_supported": [c_int, c_int, c_int],
@@ -173,6 +179,8 @@ _SIGNATURES = {
                            c_int, c_int, c_void_p, c_void_p],
     "zb_gemm_small_bounded": [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_float, c_int, c_int, c_int,
                               c_longlong, c_longlong, c_longlong, c_int, c_void_p],
+    "zb_gemm_small_gelu": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong, c_int,
+                           c_void_p],
     "zb_gemm_nt_simt": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong,
                         c_int, c_int, c_void_p],
     "zb_fused_chain_stage_supported": [c_int, c_int, c_int, c_int, c_int],
@@ -421,6 +429,17 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor | None = None, blocked: bo
     return out
 
 
+def gelu_rows(x: torch.Tensor, out_dtype: torch.dtype | None = None) -> torch.Tensor:
+    """The tanh form of GELU, 0.5 x (1 + tanh(sqrt(2 / pi) (x + 0.044715 x^3))), of a contiguous tensor, in float32
+    with one rounding."""
+    _cuda(x)
+    _require(x.is_contiguous() and x.dtype in DTYPE_CODE, "a contiguous float32 or bfloat16 tensor")
+    out = torch.empty(x.shape, dtype=out_dtype or x.dtype, device=x.device)
+    _check(library().zb_gelu_rows(_ptr(out), DTYPE_CODE[out.dtype], _ptr(x), DTYPE_CODE[x.dtype], x.numel(), _stream()),
+           "gelu_rows")
+    return out
+
+
 # ------------------------------------------------------- layer norm, recurrences and their norms
 def _f32_vector(v: torch.Tensor | None, size: int, what: str) -> None:
     _require(v is None or (v.dtype == torch.float32 and v.is_contiguous() and v.numel() == size),
@@ -528,16 +547,19 @@ def pair_embedding(table: torch.Tensor, pair_table: torch.Tensor, ctx_ids: torch
 
 
 def sum_rms_norm(x: torch.Tensor, a: torch.Tensor | None, b: torch.Tensor | None, w: torch.Tensor | None,
-                 eps: float, out_dtype: torch.dtype | None = None, bias: torch.Tensor | None = None) -> torch.Tensor | None:
+                 eps: float, out_dtype: torch.dtype | None = None, bias: torch.Tensor | None = None,
+                 groups: int = 1) -> torch.Tensor | None:
     """x (float32 [rows, H], unit inner stride, rows may be slices of wider rows) += (a + b + bias) in place,
     where a and b are contiguous [rows, H] summands of either type or None and ``bias`` is a float32 [H] shift
     of one of them (added to every row), or None; then, with a scale ``w``, returns
-    x / sqrt(mean(x^2) + eps) * w in ``out_dtype``.  Statistics and sums are float32."""
+    x / sqrt(mean(x^2) + eps) * w in ``out_dtype``; with ``groups`` > 1 each of that many equal consecutive parts
+    of a row has a mean square of its own.  Statistics and sums are float32."""
     _cuda(x, a, b, w, bias)
     _f32_vector(bias, x.shape[-1], "the shift")
     _require(bias is None or a is not None or b is not None, "a shift comes with a summand")
     _require(x.dim() == 2 and x.dtype == torch.float32 and x.stride(1) == 1, "a float32 stream [rows, H]")
     rows, H = x.shape
+    _require(groups > 0 and H % groups == 0, "groups divide a row evenly")
     for summand in (a, b):
         _require(summand is None or (summand.shape == x.shape and summand.is_contiguous() and summand.dtype in DTYPE_CODE),
                  "summands are contiguous [rows, H]")
@@ -547,7 +569,7 @@ def sum_rms_norm(x: torch.Tensor, a: torch.Tensor | None, b: torch.Tensor | None
     _check(library().zb_sum_rms_norm(_ptr(out), H, DTYPE_CODE[out.dtype] if out is not None else 0, _ptr(x), x.stride(0),
                                      _ptr(a), DTYPE_CODE[a.dtype] if a is not None else 0, _ptr(b),
                                      DTYPE_CODE[b.dtype] if b is not None else 0, _ptr(bias), _ptr(w),
-                                     _scale_code(w, H) if w is not None else 0, float(eps), rows, H, _stream()),
+                                     _scale_code(w, H) if w is not None else 0, float(eps), rows, H, int(groups), _stream()),
            "sum_rms_norm")
     return out
 
@@ -859,6 +881,16 @@ def _cache_geometry(kv_cache: torch.Tensor, nkv: int, kd: int, vd: int, dtype: t
     return kv_cache.shape[0], page_size
 
 
+def _distance_bias(bias: tuple[torch.Tensor, torch.Tensor] | None, nh: int) -> tuple[torch.Tensor | None, torch.Tensor | None]:
+    if bias is None:
+        return None, None
+    _cuda(*bias)
+    for vector in bias:
+        _require(vector.dtype == torch.float32 and vector.is_contiguous() and vector.numel() == nh,
+                 "a distance bias is two float32 values per query head")
+    return bias
+
+
 def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.Tensor, tile_row: torch.Tensor,
                     tile_q0: torch.Tensor, tile_tokens: int, row_q_start: torch.Tensor, row_q_len: torch.Tensor,
                     row_ctx: torch.Tensor, nh: int, nkv: int, hd: int, window: int, scale: float,
@@ -867,7 +899,8 @@ def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.
                     sinks: torch.Tensor | None = None, softcap: float = 0.0, shared_kv: bool = False,
                     keep_first: int = 0, pool: int = 0, pool_cache: torch.Tensor | None = None,
                     pool_table: torch.Tensor | None = None, cross_values: bool = False,
-                    out_dtype: torch.dtype | None = None) -> torch.Tensor:
+                    out_dtype: torch.dtype | None = None, distance_bias: tuple[torch.Tensor, torch.Tensor] | None = None,
+                    score_mix: torch.Tensor | None = None) -> torch.Tensor:
     """The general kernel: causal attention of every new token over its request's pages.
     ``head_slopes`` (float32 [nh]): query head h adds head_slopes[h] * (key position - query position)
     to its scores, a position encoding that is a bias on the scores.  ``value_dim``: the width of the
@@ -880,12 +913,19 @@ def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.
     ``pool_table``: a second store of one entry per block of P positions; a query at position i also sees
     the first floor((i - window + 1) / P) entries, in the same softmax.  ``cross_values``: every query
     head's weights applied to every key/value head's values; the result is [T, nh, nkv, value_dim].
-    ``out_dtype``: float32 for a result that is not rounded to the cache's type."""
+    ``out_dtype``: float32 for a result that is not rounded to the cache's type.  ``distance_bias`` = (r1, r2),
+    float32 [nh] each: r1_h ln(1 + r2_h d) is taken off head h's score of the key d positions back.
+    ``score_mix`` (float32 [nh, nh]): head h's scaled score becomes sum_g score_mix[h, g] times head g's, ahead of
+    the bias, the bound and the softmax."""
     _cuda(q, kv_cache, block_table, tile_row, tile_q0, row_q_start, row_q_len, row_ctx, status, head_slopes, sinks,
           pool_cache, pool_table)
     for per_head in (head_slopes, sinks):
         _require(per_head is None or (per_head.dtype == torch.float32 and per_head.is_contiguous()
                                       and per_head.numel() == nh), "one float32 value per query head")
+    r1, r2 = _distance_bias(distance_bias, nh)
+    _cuda(score_mix)
+    _require(score_mix is None or (score_mix.dtype == torch.float32 and score_mix.is_contiguous()
+                                   and score_mix.shape == (nh, nh)), "score_mix: float32 [heads, heads]")
     _i32(block_table, tile_row, tile_q0, row_q_start, row_q_len, row_ctx)
     vd = hd if value_dim is None else int(value_dim)
     _require(q.dim() == 2 and q.is_contiguous() and q.shape[1] == nh * hd and q.dtype in DTYPE_CODE, "q shape")
@@ -910,7 +950,51 @@ def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.
         _ptr(row_q_len), _ptr(row_ctx), nh, nkv, hd, vd, int(window), int(chunk), float(scale), float(softcap),
         int(shared_kv), _ptr(head_slopes), _ptr(sinks), int(keep_first), int(pool), _ptr(pool_cache),
         _ptr(pool_table), pool_blocks, pool_pages, int(cross_values), int(out_dtype == torch.float32 and q.dtype != torch.float32),
-        DTYPE_CODE[q.dtype], _ptr(status), _stream()), "paged_attention")
+        _ptr(r1), _ptr(r2), _ptr(score_mix), DTYPE_CODE[q.dtype], _ptr(status), _stream()), "paged_attention")
+    return out
+
+
+def heads_attention_tile_tokens(nh: int, nkv: int, kd: int, vd: int, dtype: torch.dtype) -> int:
+    """New tokens of one request per tile of the kernel that keeps all heads of a tile in one CTA; 0 where it
+    does not take the layer (bfloat16, up to 32 heads, widths up to 256; what fits in shared memory)."""
+    return int(library().zb_heads_attention_tile_tokens(nh, nkv, kd, vd, DTYPE_CODE[dtype])) if dtype in DTYPE_CODE else 0
+
+
+def heads_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.Tensor, tile_row: torch.Tensor,
+                    tile_q0: torch.Tensor, row_q_start: torch.Tensor, row_q_len: torch.Tensor, row_ctx: torch.Tensor,
+                    nh: int, nkv: int, kd: int, vd: int, window: int, scale: float, status: torch.Tensor,
+                    out: torch.Tensor, keep_first: int = 0, score_mix: torch.Tensor | None = None,
+                    distance_bias: tuple[torch.Tensor, torch.Tensor] | None = None, single: bool = False,
+                    max_context: int = 0, splits: int | None = None) -> torch.Tensor:
+    """Tensor-core attention with all heads of a tile in one CTA, for layers that mix the heads' scores ahead
+    of the softmax (``score_mix``) and for keys and values of any two widths; ``keep_first``, ``score_mix`` and
+    ``distance_bias`` as in ``paged_attention``.  Tiles hold ``heads_attention_tile_tokens`` tokens, or with
+    ``single`` one token each, whose keys are then shared by ``splits`` CTAs (default: as many as fill the SMs,
+    with ``max_context`` at least the longest context of the rows, the new token included).  Writes the tiles'
+    rows of ``out`` [T, nh * vd]."""
+    _cuda(q, kv_cache, block_table, tile_row, tile_q0, row_q_start, row_q_len, row_ctx, status, out, score_mix)
+    _i32(block_table, tile_row, tile_q0, row_q_start, row_q_len, row_ctx)
+    r1, r2 = _distance_bias(distance_bias, nh)
+    _require(q.dim() == 2 and q.is_contiguous() and q.shape[1] == nh * kd and q.dtype == torch.bfloat16, "q shape")
+    _require(out.shape == (q.shape[0], nh * vd) and out.dtype == q.dtype and out.is_contiguous(), "out must be [T, heads * value_dim]")
+    _require(score_mix is None or (score_mix.dtype == torch.float32 and score_mix.is_contiguous()
+                                   and score_mix.shape == (nh, nh)), "score_mix: float32 [heads, heads]")
+    pages, page_size = _cache_geometry(kv_cache, nkv, kd, vd, q.dtype)
+    n_tiles = tile_row.numel()
+    scratch = None
+    if not single or n_tiles == 0:
+        splits = 1
+    elif splits is None:
+        keys = max(1, max_context if window <= 0 else min(max_context, window + keep_first))
+        most = -(-keys // max(1, int(library().zb_heads_attention_tile_keys(nh, nkv, kd, vd)))) + 1
+        splits = max(1, min(most, _sm_count() // n_tiles))
+    if splits > 1:
+        scratch, _ = _decode_workspace(q.device, n_tiles * splits * nh * (vd + 2), 1)
+    _check(library().zb_heads_attention(
+        _ptr(out), _ptr(q), _ptr(kv_cache), _ptr(block_table), block_table.shape[1], page_size, pages,
+        block_table.shape[0], _ptr(tile_row), _ptr(tile_q0), n_tiles, _ptr(row_q_start), _ptr(row_q_len), _ptr(row_ctx),
+        nh, nkv, kd, vd, int(window), int(keep_first), float(scale), _ptr(score_mix), _ptr(r1), _ptr(r2), int(single),
+        int(splits), _ptr(scratch), _ptr(status), _stream()), "heads_attention", kernels=2 if splits > 1 else 1)
     return out
 
 
@@ -920,15 +1004,16 @@ QK_NORMS = {"none": 0, "per_head": 1, "whole": 2}
 def qkv_halves(qkv: torch.Tensor, nh: int, nkv: int, kd: int, vd: int, norm: str, q_norm_w: torch.Tensor | None,
                k_norm_w: torch.Tensor | None, eps: float, freqs: torch.Tensor | None, rot_dims: int, rot_mult: float,
                value_unit_norm: bool, positions: torch.Tensor, token_row: torch.Tensor, kv_cache: torch.Tensor | None,
-               block_table: torch.Tensor, status: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
-    """From a fused q/k/v projection to queries and cache entries, for a rotation of halves: an RMS norm of q
-    and of k (``norm`` "per_head": per head, scales [kd] shared by the heads; "whole": one statistic over all
+               block_table: torch.Tensor, status: torch.Tensor, dtype: torch.dtype,
+               bias: torch.Tensor | None = None) -> torch.Tensor:
+    """From a fused q/k/v projection to queries and cache entries, for a rotation of halves: a float32 bias on
+    every column (``bias``, or None), an RMS norm of q and of k (``norm`` "per_head": per head, scales [kd] shared by the heads; "whole": one statistic over all
     heads of q and one over all heads of k, scales [nh * kd] and [nkv * kd]; "none"; scales may be None),
     the rotation of value i with value i + rot_dims / 2 by position * freqs[i] on the first ``rot_dims``
     values of every q and k head (cosine and sine times ``rot_mult``), every value head divided by its root
     mean square (``value_unit_norm``), and the cache write of k and v.  Returns the queries [T, nh * kd] in
     ``dtype``; ``qkv`` may be float32 whatever ``dtype`` is.  Without ``kv_cache`` only the queries are made."""
-    _cuda(qkv, q_norm_w, k_norm_w, freqs, positions, token_row, kv_cache, block_table, status)
+    _cuda(qkv, q_norm_w, k_norm_w, freqs, positions, token_row, kv_cache, block_table, status, bias)
     _i32(positions, token_row, block_table)
     T = qkv.shape[0]
     width = nh * kd + (nkv * (kd + vd) if kv_cache is not None else 0)
@@ -936,7 +1021,7 @@ def qkv_halves(qkv: torch.Tensor, nh: int, nkv: int, kd: int, vd: int, norm: str
              "qkv must be [T, heads*key_dim + kv_heads*(key_dim + value_dim)] with unit inner stride")
     _require(norm in QK_NORMS, f"the norm of q and k is one of {sorted(QK_NORMS)}")
     sizes = (nh * kd, nkv * kd) if norm == "whole" else (kd, kd)
-    for vector, size in ((q_norm_w, sizes[0]), (k_norm_w, sizes[1]), (freqs, rot_dims // 2)):
+    for vector, size in ((q_norm_w, sizes[0]), (k_norm_w, sizes[1]), (freqs, rot_dims // 2), (bias, width)):
         _require(vector is None or (vector.dtype == torch.float32 and vector.is_contiguous() and vector.numel() == size),
                  f"a float32 vector of {size} values")
     _require(positions.numel() == T and token_row.numel() == T and block_table.dim() == 2, "one position and row per token")
@@ -945,7 +1030,7 @@ def qkv_halves(qkv: torch.Tensor, nh: int, nkv: int, kd: int, vd: int, norm: str
         pages, page_size = _cache_geometry(kv_cache, nkv, kd, vd, dtype)
     q_out = torch.empty((T, nh * kd), dtype=dtype, device=qkv.device)
     _check(library().zb_qkv_halves(
-        _ptr(q_out), _ptr(qkv), qkv.stride(0), QK_NORMS[norm], _ptr(q_norm_w), _ptr(k_norm_w), float(eps), _ptr(freqs),
+        _ptr(q_out), _ptr(qkv), qkv.stride(0), _ptr(bias), QK_NORMS[norm], _ptr(q_norm_w), _ptr(k_norm_w), float(eps), _ptr(freqs),
         int(rot_dims), float(rot_mult), int(value_unit_norm), _ptr(positions), _ptr(token_row), _ptr(kv_cache),
         _ptr(block_table), block_table.shape[1], page_size, pages, block_table.shape[0], T, nh, nkv, kd, vd,
         DTYPE_CODE[qkv.dtype], DTYPE_CODE[dtype], _ptr(status), _stream()), "qkv_halves")
@@ -983,11 +1068,13 @@ def head_mix(a: torch.Tensor, mix: torch.Tensor, nh: int, nkv: int, vd: int, out
 
 
 def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
-    """x *= sigmoid(gate) in place and value by value; ``gate`` float32 [T, width], rows may be strided."""
+    """x *= sigmoid(gate) in place; ``gate`` float32 [T, n], rows may be strided: value by value where n is x's
+    width, else one gate for every run of width / n values (the output of one of n heads)."""
     _cuda(x, gate)
     _require(x.dim() == 2 and x.is_contiguous() and x.dtype in DTYPE_CODE, "x: contiguous [T, width]")
-    _require(gate.dtype == torch.float32 and gate.shape == x.shape and gate.stride(1) == 1, "gate: float32 [T, width]")
-    _check(library().zb_sigmoid_gate(_ptr(x), _ptr(gate), gate.stride(0), x.shape[0], x.shape[1], DTYPE_CODE[x.dtype],
+    _require(gate.dtype == torch.float32 and gate.dim() == 2 and gate.shape[0] == x.shape[0] and gate.shape[1] > 0
+             and x.shape[1] % gate.shape[1] == 0 and (gate.stride(1) == 1 or gate.shape[1] == 1), "gate: float32 [T, width or heads]")
+    _check(library().zb_sigmoid_gate(_ptr(x), _ptr(gate), gate.stride(0), x.shape[0], x.shape[1], x.shape[1] // gate.shape[1], DTYPE_CODE[x.dtype],
                                      _stream()), "sigmoid_gate")
     return x
 
@@ -1156,9 +1243,10 @@ def paged_decode(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.Ten
                  window: int, scale: float, status: torch.Tensor, out: torch.Tensor,
                  scratch: torch.Tensor | None = None, split_size: int | None = None,
                  counters: torch.Tensor | None = None, chunk: int = 0,
-                 sinks: torch.Tensor | None = None, softcap: float = 0.0, keys_only: bool = False) -> torch.Tensor:
+                 sinks: torch.Tensor | None = None, softcap: float = 0.0, keys_only: bool = False,
+                 distance_bias: tuple[torch.Tensor, torch.Tensor] | None = None) -> torch.Tensor:
     """Split-context attention for rows with one new token each; writes those tokens' rows of ``out``.
-    ``chunk``, ``sinks`` and ``softcap`` as in ``paged_attention``; ``keys_only`` as its ``shared_kv``.
+    ``chunk``, ``sinks``, ``softcap`` and ``distance_bias`` as in ``paged_attention``; ``keys_only`` as its ``shared_kv``.
 
     ``max_context`` is at least the longest context of the rows, the new token included.  ``scratch``
     (float32, any contents) and ``counters`` (int32, zero) come from a process-wide workspace unless
@@ -1186,14 +1274,15 @@ def paged_decode(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.Ten
              f"scratch must hold {need} floats")
     _require(counters.dtype == torch.int32 and counters.is_contiguous() and counters.numel() >= n_rows * nkv,
              f"counters must hold {n_rows * nkv} zeroed int32 values")
-    if chunk or sinks is not None or softcap or keys_only:
+    if chunk or sinks is not None or softcap or keys_only or distance_bias is not None:
+        r1, r2 = _distance_bias(distance_bias, nh)
         _cuda(sinks)
         _require(sinks is None or (sinks.dtype == torch.float32 and sinks.is_contiguous() and sinks.numel() == nh),
                  "one float32 sink per query head")
         _check(library().zb_paged_decode_masked(
             _ptr(out), _ptr(q), _ptr(kv_cache), _ptr(block_table), block_table.shape[1], page_size, pages,
             block_table.shape[0], _ptr(rows), n_rows, _ptr(row_q_start), _ptr(row_ctx), nh, nkv, hd, int(window),
-            int(chunk), float(scale), float(softcap), int(keys_only), _ptr(sinks), int(split_size), max_splits,
+            int(chunk), float(scale), float(softcap), int(keys_only), _ptr(sinks), _ptr(r1), _ptr(r2), int(split_size), max_splits,
             _ptr(scratch), _ptr(counters), _ptr(status), _stream()), "paged_decode")
         return out
     _check(library().zb_paged_decode(
@@ -1291,10 +1380,11 @@ def paged_prefill(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.Te
                   out: torch.Tensor, chunk: int = 0, sinks: torch.Tensor | None = None, softcap: float = 0.0,
                   keys_only: bool = False, keep_first: int = 0, pool: int = 0, pool_cache: torch.Tensor | None = None,
                   pool_table: torch.Tensor | None = None, cross_values: bool = False,
-                  by_group: bool = False) -> torch.Tensor:
+                  by_group: bool = False,
+                  distance_bias: tuple[torch.Tensor, torch.Tensor] | None = None) -> torch.Tensor:
     """Tensor-core attention for rows with several new tokens, cut into tiles of
-    ``paged_prefill_tile_tokens()``; writes those tokens' rows of ``out``.  ``chunk``, ``sinks`` and
-    ``softcap`` as in ``paged_attention``, ``keys_only`` as its ``shared_kv``.  Head size 128 runs on tcgen05
+    ``paged_prefill_tile_tokens()``; writes those tokens' rows of ``out``.  ``chunk``, ``sinks``, ``softcap`` and
+    ``distance_bias`` as in ``paged_attention``, ``keys_only`` as its ``shared_kv``.  Head size 128 runs on tcgen05
     with the accumulators in tensor memory (every form but the chunked mask), other sizes and chunked masks
     on mma.sync.  ``keep_first``, ``pool`` with its store, and ``cross_values`` (``out`` is then
     [T, nh * nkv * hd], bfloat16 or float32) as in ``paged_attention``: these run on mma.sync.  ``by_group``: every
@@ -1320,20 +1410,21 @@ def paged_prefill(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.Te
                  and pool_cache.shape[1:] == kv_cache.shape[1:] and pool_cache.dtype == kv_cache.dtype
                  and pool_cache.is_contiguous(), "a pooled store has the pages' shape and a table row per request")
         pool_pages, pool_blocks = pool_cache.shape[0], pool_table.shape[1]
-    tensor_memory = (USE_TCGEN05_PREFILL and not chunk and not windowed
+    r1, r2 = _distance_bias(distance_bias, nh)
+    tensor_memory = (USE_TCGEN05_PREFILL and not chunk and not windowed and not (softcap and r1 is not None)
                      and bool(library().zb_paged_prefill_tc_supported(nh, nkv, hd, DTYPE_CODE[q.dtype], page_size)))
     common = (_ptr(out), _ptr(q), _ptr(kv_cache), _ptr(block_table), block_table.shape[1], page_size, pages,
               block_table.shape[0], _ptr(tile_row), _ptr(tile_q0), tile_row.numel(), _ptr(row_q_start), _ptr(row_q_len),
               _ptr(row_ctx), nh, nkv, hd, int(window))
     if tensor_memory:
         _check(library().zb_paged_prefill_tc_masked(*common, float(scale), float(softcap), int(keys_only), _ptr(sinks),
-                                                    _ptr(status), _stream()), "paged_prefill")
-    elif windowed:
+                                                    _ptr(r1), _ptr(r2), _ptr(status), _stream()), "paged_prefill")
+    elif windowed or r1 is not None:
         _check(library().zb_paged_prefill_windowed(*common, int(chunk), float(scale), float(softcap), int(keys_only),
                                                    _ptr(sinks), int(keep_first), int(pool), _ptr(pool_cache),
                                                    _ptr(pool_table), pool_blocks, pool_pages, int(cross_values),
-                                                   int(out.dtype == torch.float32), int(by_group), _ptr(status),
-                                                   _stream()), "paged_prefill")
+                                                   int(out.dtype == torch.float32), int(by_group), _ptr(r1), _ptr(r2),
+                                                   _ptr(status), _stream()), "paged_prefill")
     else:
         _check(library().zb_paged_prefill_masked(*common, int(chunk), float(scale), float(softcap), int(keys_only),
                                                  _ptr(sinks), _ptr(status), _stream()), "paged_prefill")
@@ -1388,10 +1479,12 @@ def _bounded_args(bounded: BoundedGate, rows: int) -> tuple:
 
 
 def gemm_small(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = None,
-               swiglu: bool = False, act: str = "silu", bounded: BoundedGate | None = None) -> torch.Tensor:
+               swiglu: bool = False, act: str = "silu", bounded: BoundedGate | None = None,
+               gelu: bool = False) -> torch.Tensor:
     """x [M <= 64, K] times w [N, K] transposed, bfloat16, float32 accumulation, weights read once.
     With ``swiglu`` the rows of w are blocks of 8 gate rows each followed by its 8 up rows, and the
-    result is silu(gate) * up, [M, N / 2]; with ``bounded`` as well, the bounded gate of those sums."""
+    result is silu(gate) * up, [M, N / 2]; with ``bounded`` as well, the bounded gate of those sums.  ``gelu``
+    (without ``swiglu``): the tanh form of GELU of the sums."""
     _cuda(x, w)
     _require(x.dim() == 2 and w.dim() == 2 and x.shape[1] == w.shape[1], "x [M, K] and w [N, K]")
     _require(gemm_small_supported(x, w), "gemm_small takes bfloat16, M <= 64, K a multiple of 8, 16-byte aligned rows")
@@ -1399,12 +1492,17 @@ def gemm_small(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None =
     M, K = x.shape
     N = w.shape[0]
     _require(not swiglu or N % 16 == 0, "swiglu needs a multiple of 16 rows")
+    _require(not (swiglu and gelu), "GELU is an epilogue of the ungated product")
     out = torch.empty((M, N // 2 if swiglu else N), dtype=out_dtype, device=x.device)
     if bounded is not None:
         _require(swiglu, "the bounded gate is a gated epilogue")
         _cuda(bounded.bias)
         _check(library().zb_gemm_small_bounded(_ptr(out), _ptr(x), _ptr(w), *_bounded_args(bounded, N), M, N, K, x.stride(0),
                                                w.stride(0), out.stride(0), DTYPE_CODE[out_dtype], _stream()), "gemm_small")
+        return out
+    if gelu:
+        _check(library().zb_gemm_small_gelu(_ptr(out), _ptr(x), _ptr(w), M, N, K, x.stride(0), w.stride(0), out.stride(0),
+                                            DTYPE_CODE[out_dtype], _stream()), "gemm_small")
         return out
     _check(library().zb_gemm_small(_ptr(out), _ptr(x), _ptr(w), M, N, K, x.stride(0), w.stride(0), out.stride(0),
                                    DTYPE_CODE[out_dtype], (2 if act == "relu" else 1) if swiglu else 0, _stream()),
@@ -1430,19 +1528,21 @@ def gemm_tc_supported(x: torch.Tensor, w: torch.Tensor, swiglu: bool = False) ->
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, swiglu: bool = False, block_n: int = 0,
             status: torch.Tensor | None = None, out_dtype: torch.dtype | None = None, act: str = "silu",
-            bounded: BoundedGate | None = None) -> torch.Tensor:
+            bounded: BoundedGate | None = None, gelu: bool = False) -> torch.Tensor:
     """x [M, K] times w [N, K] transposed on tcgen05 tensor cores, bfloat16 with float32 sums in
     tensor memory; the result in bfloat16, or with ``out_dtype=torch.float32`` the sums as they are.
     With ``swiglu`` the rows of w are blocks of 8 gate rows each followed by its 8 up
     rows, and the result is silu(gate) * up, [M, N / 2], taken from the float32 sums and rounded once
-    (with ``bounded`` as well: the bounded gate of those sums and their biases).
+    (with ``bounded`` as well: the bounded gate of those sums and their biases).  ``gelu``: the tanh form of GELU
+    of the float32 sums, rounded once.
     ``block_n`` is the width of an output tile (256, 128; 2: tiles of 256 x 256 on pairs of SMs; 0: chosen).  ``status`` (default: the
     device's status word) receives a report if a wait inside the kernel ran out."""
     _cuda(x, w)
     _require(gemm_tc_supported(x, w, swiglu), "gemm_tc takes bfloat16 x [M, K] and contiguous w [N, K], K a multiple of 8, "
              "16-byte aligned; with swiglu N a multiple of 16")
     wide = out_dtype == torch.float32
-    _require(out_dtype in (None, torch.bfloat16, torch.float32) and not (wide and swiglu), "bfloat16 out, or float32 without the activation")
+    _require(out_dtype in (None, torch.bfloat16, torch.float32) and not (wide and (swiglu or gelu)) and not (swiglu and gelu),
+             "bfloat16 out, or float32 without an activation")
     M, K = x.shape
     N = w.shape[0]
     width = N // 2 if swiglu else N
@@ -1458,7 +1558,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, swiglu: bool = False, block_n: int
         return out if ldy == width else out[:, :width].contiguous()
     _require(act in ACTIVATIONS, f"the gate's activation is one of {sorted(ACTIVATIONS)}")
     gated = 3 if act == "relu" else 1         # the kernel's codes for the two gated epilogues
-    _check(library().zb_gemm_tc(_ptr(out), _ptr(x), _ptr(w), M, N, K, x.stride(0), ldy, 2 if wide else (gated if swiglu else 0),
+    _check(library().zb_gemm_tc(_ptr(out), _ptr(x), _ptr(w), M, N, K, x.stride(0), ldy, 2 if wide else (gated if swiglu else (4 if gelu else 0)),
                                 int(block_n), _ptr(status), _stream()), "gemm_tc")
     return out if ldy == width else out[:, :width].contiguous()
 
@@ -1694,13 +1794,15 @@ def interleave_gate_up(w_gate: torch.Tensor, w_up: torch.Tensor) -> torch.Tensor
 
 
 def routed_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate: torch.Tensor,
-                   w_up: torch.Tensor | None, w_down: torch.Tensor, act: str = "silu") -> torch.Tensor:
+                   w_up: torch.Tensor | None, w_down: torch.Tensor, act: str = "silu",
+                   weigh_inputs: bool = False) -> torch.Tensor:
     """sum_j weights[t, j] * expert_{ids[t, j]}(x[t]) for x [T, width]: expert e < E is
     w_down[e] (act(w_gate[e] x) * (w_up[e] x)) with w_gate, w_up [E, ff, width] and w_down [E, width, ff]; an
     id >= E names an identity expert, whose output is x itself.  Without ``w_up``, ``w_gate`` holds both
     matrices as ``interleave_gate_up`` lays them out.  The tokens are sorted by expert on the device and
     nothing comes back to the host: alignment, the two products (gate/up with the activation, down) and the
-    weighted sum.  bfloat16 with many tokens per expert and the interleaved layout: each product is ONE
+    weighted sum.  ``weigh_inputs``: sum_j expert_{ids[t, j]}(weights[t, j] x[t]) instead (the gate and up sums
+    are multiplied by the weight ahead of the activation; no identity experts).  bfloat16 with many tokens per expert and the interleaved layout: each product is ONE
     grouped launch of the tcgen05 kernel over runs padded to whole tiles; otherwise tiles on mma.sync
     (bfloat16) or CUDA cores (float32)."""
     _cuda(x, ids, weights, w_gate, w_up, w_down)
@@ -1732,17 +1834,18 @@ def routed_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_
         _check(lib.zb_route_align_padded(_ptr(tile_group), _ptr(slots), _ptr(place), _ptr(ids), num_slots, E, tiles,
                                          GROUPED_TILE_ROWS, _stream()), "route_align")
         rows = torch.empty((places, width), dtype=x.dtype, device=device)
-        _check(lib.zb_gather_places(_ptr(rows), _ptr(x), x.stride(0), _ptr(slots), places, width, top, _stream()),
-               "gather_places")
+        place_scale = torch.empty(places, dtype=torch.float32, device=device) if weigh_inputs else None
+        _check(lib.zb_gather_places(_ptr(rows), _ptr(x), x.stride(0), _ptr(slots), places, width, top, _ptr(place_scale),
+                                    _ptr(weights), _stream()), "gather_places")
         status = device_status(device)
         hidden = torch.empty((places, ff), dtype=x.dtype, device=device)
         _check(lib.zb_gemm_tc_grouped(_ptr(hidden), _ptr(rows), _ptr(w_gate), _ptr(tile_group), tiles, E, 2 * ff, width, width,
-                                      ff, 3 if act == "relu" else 1, _ptr(status), _stream()), "gemm_tc_grouped")
+                                      ff, 3 if act == "relu" else 1, _ptr(place_scale), _ptr(status), _stream()), "gemm_tc_grouped")
         # An expert's output takes the model's type before it is weighted on every path: here the product writes it so.
         ldy = width
         y = torch.empty((places, ldy), dtype=x.dtype, device=device)
         _check(lib.zb_gemm_tc_grouped(_ptr(y), _ptr(hidden), _ptr(w_down), _ptr(tile_group), tiles, E, width, ff, ff, ldy, 0,
-                                      _ptr(status), _stream()), "gemm_tc_grouped")
+                                      None, _ptr(status), _stream()), "gemm_tc_grouped")
     else:
         tile_rows = lib.zb_expert_tile_rows(code)          # CUDA-core tiles in float32, tensor-core tiles in bfloat16
         max_tiles = -(-num_slots // tile_rows) + E
@@ -1754,11 +1857,11 @@ def routed_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_
         ldy = width
         y = torch.empty((max(num_slots, 1), width), dtype=torch.float32, device=device)
         _check(lib.zb_expert_product(_ptr(hidden), _ptr(x), x.stride(0), _ptr(w_gate), _ptr(w_up), _ptr(plan), _ptr(slots),
-                                     max_tiles, ff, width, top, ACTIVATIONS[act], 0, code, _stream()), "expert_product")
-        _check(lib.zb_expert_product(_ptr(y), _ptr(hidden), ff, _ptr(w_down), None, _ptr(plan), _ptr(slots), max_tiles,
+                                     _ptr(weights) if weigh_inputs else None, max_tiles, ff, width, top, ACTIVATIONS[act], 0, code, _stream()), "expert_product")
+        _check(lib.zb_expert_product(_ptr(y), _ptr(hidden), ff, _ptr(w_down), None, _ptr(plan), _ptr(slots), None, max_tiles,
                                      width, ff, top, ACTIVATIONS[act], 1, code, _stream()), "expert_product")
-    _check(lib.zb_route_combine(_ptr(out), _ptr(y), ldy, DTYPE_CODE[y.dtype], _ptr(x), x.stride(0), _ptr(ids), _ptr(weights),
-                                _ptr(place), T, width, top, code, _stream()), "route_combine")
+    _check(lib.zb_route_combine(_ptr(out), _ptr(y), ldy, DTYPE_CODE[y.dtype], _ptr(x), x.stride(0), _ptr(ids),
+                                None if weigh_inputs else _ptr(weights), _ptr(place), T, width, top, code, _stream()), "route_combine")
     return out
 
 

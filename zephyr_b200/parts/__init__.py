@@ -9,7 +9,7 @@ from . import norms, position, attention, latent, feed_forward, routed, recurren
 from .attention import Attention
 from .blocks import OutputNormResidual, PreNormResidual, SandwichResidual
 from .ends import Embedding, NormHead
-from .feed_forward import SwiGLU
+from .feed_forward import SwiGLU, UngatedFeedForward
 from .latent import LatentAttention
 from .routed import RoutedFeedForward
 from .model import Model, cache_specs, expected_weights, run_order_for, tile_requests
@@ -19,7 +19,7 @@ from .recurrent import GatedLinearAttention, Mamba2, ParallelMixers
 
 __all__ = [
     "Attention", "BLOCKS", "LatentAttention", "OutputNormResidual", "RoutedFeedForward", "DeferredSum", "GatedLinearAttention", "LayerNorm", "Mamba2", "ParallelMixers", "RopePairs",
-    "SandwichResidual", "run_order_for", "Block", "Embedding", "FEED_FORWARDS", "FeedForward", "INPUTS", "InputPart", "MIXERS",
+    "SandwichResidual", "UngatedFeedForward", "run_order_for", "Block", "Embedding", "FEED_FORWARDS", "FeedForward", "INPUTS", "InputPart", "MIXERS",
     "Mixer", "Model", "NORMS", "NoPosition", "Norm", "NormHead", "OUTPUTS", "OutputPart", "POSITION_ENCODINGS", "Part",
     "PositionEncoding", "PreNormResidual", "RMSNorm", "ResidualStream", "RopeNeox", "StepContext", "SwiGLU",
     "cache_specs", "expected_weights", "lookup", "register_block", "register_feed_forward", "register_input",

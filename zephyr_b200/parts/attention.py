@@ -33,6 +33,14 @@ second store, one entry a block, and a query at position i sees, beside its wind
 or before i - window, in the same softmax), a mixing of the heads' softmax weights (``head_mix``: a matrix M
 [heads, heads]; head h applies sum_g M[h, g] weights_g to the values of its own key/value head), and a
 sigmoid gate on the joined heads before the output projection (``out_gate``: sigmoid(Wg x), value by value).
+These combine with biases on the projections.
+
+Two parameters act between the scores and the softmax: ``score_mix`` (a matrix M [heads, heads]; head h's scaled
+score becomes sum_g M[h, g] times head g's, so every head's score of a key needs every other head's: such a layer
+runs on the kernels that keep all heads of a tile in one CTA, ``ops.heads_attention``, or on the general one), and
+``distance_bias`` (the names of two vectors r1, r2 [heads]: r1_h ln(1 + r2_h d) is taken off head h's score of the
+key d positions back; every attention kernel has it).  ``head_gate``: one sigmoid gate per head on its output,
+sigmoid(Wg x)_h with Wg [heads, hidden], whose product rides along with the projections.
 """
 
 from __future__ import annotations
@@ -113,22 +121,35 @@ class Attention(Mixer):
         self.pool = int(p.get("pool") or 0)
         self.head_mix = weights[p["head_mix"]].float().contiguous() if p.get("head_mix") else None
         self.w_gate = weights[p["out_gate"]] if p.get("out_gate") else None
+        self.score_mix = weights[p["score_mix"]].float().contiguous() if p.get("score_mix") else None
+        self.distance_bias = (tuple(weights[name].float().contiguous() for name in p["distance_bias"])
+                              if p.get("distance_bias") else None)
+        self.head_gate = bool(p.get("head_gate"))
+        if self.head_gate:
+            if self.w_gate is not None:
+                raise ConfigError("an attention layer has a gate per value or a gate per head")
+            self.w_gate = weights[p["head_gate"]]
+        if self.score_mix is not None and (self.head_mix is not None or self.pool or self.chunk or self.sinks is not None
+                                           or self.softcap > 0.0):
+            raise ConfigError("mixed scores do not combine with mixed weights, pooled blocks, chunks, sinks or a bound")
+        if self.distance_bias is not None and self.pool:
+            raise ConfigError("a bias on the distance and pooled blocks do not combine")
         if self.qk_norm not in ("per_head", "whole") or self.keep_first < 0 or self.pool < 0:
             raise ConfigError("qk_norm is 'per_head' or 'whole'; keep_first and pool are not negative")
         if (self.keep_first or self.pool) and self.window <= 0:
             raise ConfigError("kept first tokens and pooled blocks come with a window")
         # What runs through the kernel that rotates halves.
         self.halves = (halves is not None or self.qk_norm == "whole" or self.value_unit_norm or self.keep_first > 0
-                       or self.pool > 0 or self.head_mix is not None or self.w_gate is not None)
-        if self.halves and (pairs is not None or self.qkv_bias is not None or self.values_from_keys or self.unit_norm
-                            or self.q_temp is not None):
-            raise ConfigError("the rotation of halves and its companions do not combine with biases, a rotation of "
+                       or self.pool > 0 or self.head_mix is not None
+                       or (self.w_gate is not None and not self.head_gate))
+        if self.halves and (pairs is not None or self.values_from_keys or self.unit_norm or self.q_temp is not None):
+            raise ConfigError("the rotation of halves and its companions do not combine with a rotation of "
                               "adjacent pairs, keys as values, unit norms or a query multiplier")
         # What only the general path takes.
         self.general = (pairs is not None or self.vd != self.hd or self.chunk > 0 or self.sinks is not None
                         or self.qkv_bias is not None or self.o_bias is not None or p.get("scale") is not None
                         or self.values_from_keys or self.unit_norm or self.softcap > 0.0 or self.q_temp is not None
-                        or self.halves)
+                        or self.halves or self.score_mix is not None or self.distance_bias is not None or self.head_gate)
         if self.general:
             self._init_general(p)
             return
@@ -161,7 +182,7 @@ class Attention(Mixer):
         if (self.position is not None and self.pair_freqs is None and self.half_freqs is None
                 and self.position.as_rotation_tables() != (None, None)):
             raise ConfigError("the general attention path rotates adjacent pairs, halves of part of a head, or nothing")
-        if self.halves and self.w_gate is not None:
+        if self.w_gate is not None:
             self.w_qkv = torch.cat([self.w_qkv, self.w_gate], dim=0).contiguous()
             self.w_q = self.w_qkv[: self.nh * self.hd]
         self.q_norm = self.q_norm.float().contiguous() if self.q_norm is not None else None
@@ -177,6 +198,14 @@ class Attention(Mixer):
         # Kept first tokens, pooled blocks and mixed heads are masks and outputs of the mma.sync prompt kernel
         # (and of the general one); it then serves single tokens too, as tiles of one token.
         self.windowed = bool(self.keep_first or self.pool or self.head_mix is not None)
+        # Tokens a tile of the kernel with all heads in one CTA (0: it does not take the layer).  Mixed scores run
+        # there, and so does what no other tensor-core kernel takes: keys and values of two widths behind a mask of
+        # a window and kept first tokens, with or without a distance bias.
+        plain_mask = not (self.chunk or self.pool or self.sinks is not None or self.softcap > 0.0
+                          or self.head_mix is not None or self.values_from_keys)
+        self.heads_tile_tokens = 0
+        if plain_mask and (self.score_mix is not None or not (equal and ops.paged_prefill_supported(self.nh, self.nkv, self.hd, self.dtype))):
+            self.heads_tile_tokens = ops.heads_attention_tile_tokens(self.nh, self.nkv, self.hd, self.vd, self.dtype)
         self.fast_decode = equal and not self.windowed and ops.paged_decode_supported(self.nh, self.nkv, self.hd, self.dtype)
         self.fast_prefill = equal and ops.paged_prefill_supported(self.nh, self.nkv, self.hd, self.dtype)
         self.prefill_tile_tokens = ops.paged_prefill_tile_tokens()
@@ -204,6 +233,12 @@ class Attention(Mixer):
             decls[p["head_mix"]] = WeightDecl((nh, nh), ROLE_LINEAR)
         if p.get("out_gate"):
             decls[p["out_gate"]] = WeightDecl((nh * vd, hidden), ROLE_LINEAR)
+        if p.get("score_mix"):
+            decls[p["score_mix"]] = WeightDecl((nh, nh), ROLE_LINEAR)
+        for name in p.get("distance_bias") or ():
+            decls[name] = WeightDecl((nh,), ROLE_NORM)
+        if p.get("head_gate"):
+            decls[p["head_gate"]] = WeightDecl((nh, hidden), ROLE_LINEAR)
         for name, size in (("q_bias", nh * hd), ("k_bias", nkv * hd), ("v_bias", nkv * vd), ("o_bias", hidden),
                            ("sinks", nh)):
             if p.get(name) and not (name == "v_bias" and p.get("values_from_keys")):
@@ -211,7 +246,7 @@ class Attention(Mixer):
         return decls
 
     def weights_read(self) -> list[torch.Tensor]:
-        return [t for t in (self.w_qkv, self.w_o, self.q_norm, self.k_norm, self.head_mix) if t is not None]
+        return [t for t in (self.w_qkv, self.w_o, self.q_norm, self.k_norm, self.head_mix, self.score_mix) if t is not None]
 
     @staticmethod
     def cache_spec(spec: MixerSpec) -> "PagedCacheSpec | tuple":
@@ -232,7 +267,12 @@ class Attention(Mixer):
         p = spec.params
         tokens = ops.attention_tile_tokens(int(p["num_heads"]) // int(p["num_kv_heads"]))
         wide = ops.paged_prefill_tile_tokens()
-        return [(tokens, "all"), (tokens, "multi"), (tokens, "single"), (wide, "multi"), (wide, "all")]
+        wanted = [(tokens, "all"), (tokens, "multi"), (tokens, "single"), (wide, "multi"), (wide, "all")]
+        kd, vd = int(p["head_dim"]), int(p.get("value_dim") or p["head_dim"])
+        if not p.get("score_mix") and kd == vd and kd % 32 == 0:
+            return wanted           # (what the other tensor-core kernels take)
+        own = ops.heads_attention_tile_tokens(int(p["num_heads"]), int(p["num_kv_heads"]), kd, vd, torch.bfloat16)
+        return wanted + [(own, which) for which in ("multi", "single") if own > 0 and (own, which) not in wanted]
 
     # ------------------------------------------------------------------ forward
     def _store_projected(self, projected: torch.Tensor, ctx: StepContext, call: LayerCall) -> torch.Tensor:
@@ -278,13 +318,17 @@ class Attention(Mixer):
         goes to the general kernel."""
         cache = ctx.caches[call.cache]
         table = ctx.block_table(call.cache)
-        if self.general and self.windowed:
+        if self.general and self.heads_tile_tokens > 0:
+            return self._attend_all_heads(q, ctx, call, cache, table)
+        if self.general and (self.windowed or self.score_mix is not None):
             return self._attend_windowed(q, ctx, call, cache, table)
         out = torch.empty((q.shape[0], self.nh * self.vd), dtype=q.dtype, device=q.device)
         common = (self.nh, self.nkv, self.hd, self.window, self.scale, ctx.status)
         masks = {"chunk": self.chunk, "sinks": self.sinks} if (self.chunk or self.sinks is not None) else {}
         if self.softcap > 0.0:
             masks["softcap"] = self.softcap
+        if self.general and self.distance_bias is not None:
+            masks["distance_bias"] = self.distance_bias
         decode_done = self.fast_decode and ctx.num_decode_rows > 0
         if decode_done:
             ops.paged_decode(q, cache, table, ctx.decode_rows, ctx.row_q_start, ctx.row_ctx, ctx.max_decode_context,
@@ -305,6 +349,19 @@ class Attention(Mixer):
                                 ctx.row_ctx, *common, out=out, head_slopes=self.score_slopes, value_dim=self.vd, **masks)
         return out
 
+    def _attend_all_heads(self, q: torch.Tensor, ctx: StepContext, call: LayerCall, cache, table) -> torch.Tensor:
+        """Rows with several tokens as tiles of tokens with all heads in one CTA, single tokens with their keys
+        shared by several CTAs."""
+        out = torch.empty((q.shape[0], self.nh * self.vd), dtype=q.dtype, device=q.device)
+        for which, single in (("multi", False), ("single", True)):
+            tile_row, tile_q0 = ctx.tiles[(self.heads_tile_tokens, which)]
+            if tile_row.numel() > 0:
+                ops.heads_attention(q, cache, table, tile_row, tile_q0, ctx.row_q_start, ctx.row_q_len, ctx.row_ctx, self.nh,
+                                    self.nkv, self.hd, self.vd, self.window, self.scale, ctx.status, out,
+                                    keep_first=self.keep_first, score_mix=self.score_mix, distance_bias=self.distance_bias,
+                                    single=single, max_context=ctx.max_decode_context)
+        return out
+
     def _attend_windowed(self, q: torch.Tensor, ctx: StepContext, call: LayerCall, cache, table) -> torch.Tensor:
         """Attention with kept first tokens, pooled blocks or mixed heads: every row, prompts and single
         tokens alike, on the mma.sync prompt kernel where it takes the shape (bfloat16, one width for keys
@@ -315,6 +372,8 @@ class Attention(Mixer):
         masks = {"chunk": self.chunk, "sinks": self.sinks, "keep_first": self.keep_first}
         if self.softcap > 0.0:
             masks["softcap"] = self.softcap
+        if self.distance_bias is not None:
+            masks["distance_bias"] = self.distance_bias
         if self.pool:
             masks.update(pool=self.pool, pool_cache=ctx.caches[call.extra_caches[0]],
                          pool_table=ctx.block_table(call.extra_caches[0]))
@@ -322,7 +381,7 @@ class Attention(Mixer):
         width = self.nh * self.vd * (self.nkv if mixed else 1)
         out = torch.empty((q.shape[0], width), dtype=torch.float32 if mixed else q.dtype, device=q.device)
         common = (self.nh, self.nkv, self.hd, self.window, self.scale, ctx.status)
-        if self.fast_prefill:
+        if self.fast_prefill and self.score_mix is None:
             # Rows with several tokens as tiles of tokens; single tokens as tiles of the heads of a group.
             # (The kernel takes groups of up to 16 heads that way; larger ones run as tiles of one token.)
             for which, by_group in (((self.prefill_tile_tokens, "multi"), False),
@@ -335,7 +394,7 @@ class Attention(Mixer):
             tile_row, tile_q0 = ctx.tiles[(self.tile_tokens, "all")]
             ops.paged_attention(q, cache, table, tile_row, tile_q0, self.tile_tokens, ctx.row_q_start, ctx.row_q_len,
                                 ctx.row_ctx, *common, out=out, value_dim=self.vd, cross_values=mixed,
-                                out_dtype=out.dtype, **masks)
+                                out_dtype=out.dtype, score_mix=self.score_mix, **masks)
         return ops.head_mix(out, self.head_mix, self.nh, self.nkv, self.vd, q.dtype) if mixed else out
 
     takes_out_dtype = True
@@ -347,36 +406,39 @@ class Attention(Mixer):
         table = ctx.block_table(call.cache)
         # A layer that reads another layer's cache needs no k and v.
         weight, bias, cache = self.w_qkv, self.qkv_bias, ctx.caches[call.cache]
+        if not call.writes_cache and self.w_gate is not None:
+            raise ConfigError("a gated layer that reads another layer's cache is not built")
         if not call.writes_cache:
             weight, cache = self.w_q, None
             bias = bias[: self.nh * self.hd] if bias is not None else None
         projected = ops.linear(x, weight, out_dtype=torch.float32)
         if self.halves:
-            return self._forward_halves(projected, ctx, call, cache, table, out_dtype)
+            return self._forward_halves(projected, bias, ctx, call, cache, table, out_dtype)
         q = ops.qkv_pairs(projected, self.nh, self.nkv, self.hd, self.vd, bias, self.q_norm, self.k_norm, self.eps,
                           self.pair_freqs, self.pair_dims, ctx.positions, ctx.token_row, cache, table, ctx.status,
                           self.dtype, unit_norm=self.unit_norm, values_from_keys=self.values_from_keys,
                           q_temp=self.q_temp)
-        attended = self.attend(q, ctx, call)
+        return self._project_out(self.attend(q, ctx, call), projected, out_dtype)
+
+    def _project_out(self, attended: torch.Tensor, projected: torch.Tensor, out_dtype: torch.dtype | None) -> torch.Tensor:
+        """The gate, whose product came along with the projections, and the output projection."""
+        if self.w_gate is not None:
+            at = self.nh * self.hd + self.nkv * (self.hd + (0 if self.values_from_keys else self.vd))
+            ops.sigmoid_gate(attended, projected[:, at:at + self.w_gate.shape[0]])
         return ops.linear(attended, self.w_o, out_dtype=out_dtype, bias=self.o_bias)
 
-    def _forward_halves(self, projected: torch.Tensor, ctx: StepContext, call: LayerCall, cache, table,
+    def _forward_halves(self, projected: torch.Tensor, bias: torch.Tensor | None, ctx: StepContext, call: LayerCall, cache, table,
                         out_dtype: torch.dtype | None) -> torch.Tensor:
-        """Norms, rotation of halves and cache write in one kernel; the blocks that this step's tokens
+        """Biases, norms, rotation of halves and cache write in one kernel; the blocks that this step's tokens
         complete are pooled; attention; the gate; the output projection."""
-        if not call.writes_cache and self.w_gate is not None:
-            raise ConfigError("a gated layer that reads another layer's cache is not built")
         q = ops.qkv_halves(projected, self.nh, self.nkv, self.hd, self.vd, self.qk_norm if self.q_norm is not None else "none",
                            self.q_norm, self.k_norm, self.eps, self.half_freqs, self.half_dims, self.half_mult,
-                           self.value_unit_norm, ctx.positions, ctx.token_row, cache, table, ctx.status, self.dtype)
+                           self.value_unit_norm, ctx.positions, ctx.token_row, cache, table, ctx.status, self.dtype,
+                           bias=bias)
         if self.pool and call.writes_cache:
             ops.pool_blocks(cache, table, ctx.caches[call.extra_caches[0]], ctx.block_table(call.extra_caches[0]),
                             ctx.positions, ctx.token_row, self.nkv, self.hd, self.vd, self.pool, ctx.status)
-        attended = self.attend(q, ctx, call)
-        if self.w_gate is not None:
-            at = (self.nh + 2 * self.nkv) * self.hd if self.vd == self.hd else self.nh * self.hd + self.nkv * (self.hd + self.vd)
-            ops.sigmoid_gate(attended, projected[:, at:at + self.nh * self.vd])
-        return ops.linear(attended, self.w_o, out_dtype=out_dtype, bias=self.o_bias)
+        return self._project_out(self.attend(q, ctx, call), projected, out_dtype)
 
     def forward(self, x: torch.Tensor, ctx: StepContext, call: LayerCall,
                 out_dtype: torch.dtype | None = None) -> torch.Tensor:

@@ -2,7 +2,9 @@
 
 ``prenorm_residual``: r = x + mixer(norm1(x)); x' = r + ffn(norm2(r)), the sums in float32
 (reference: src/model/causal_lm/qwen3.cpp:79-88).  Each sum is folded into the norm that follows
-it, so the block hands its last summand on as ``pending``.
+it, so the block hands its last summand on as ``pending``.  On a float32 stream (an input part that makes one) the
+summands travel as a tuple and join the stream in the kernel of the next norm (``Norm.sum_forward``).  The
+feed-forward may be missing; the layer is then its first half.
 
 ``sandwich_residual``: a norm before and one behind each part, and a multiplier m on what joins the
 stream: r = x + m * mixer_out(mixer(mixer_norm(x))); x' = r + m * ffn_out(ffn(ffn_norm(r))).  The
@@ -32,17 +34,36 @@ from .fused import BlockPlan
 
 class PreNormResidual(Block):
     graph_safe = True
+    feed_forward_optional = True
 
     norm_names = ("mixer", "feed_forward")
 
-    def __init__(self, mixer: Mixer, feed_forward: FeedForward, norms: Mapping[str, Norm]):
+    def __init__(self, mixer: Mixer, feed_forward: FeedForward | None, norms: Mapping[str, Norm]):
         self.mixer = mixer
         self.feed_forward = feed_forward
         self.norms = dict(norms)
         self.mixer_norm = norms["mixer"]
-        self.feed_forward_norm = norms["feed_forward"]
+        self.feed_forward_norm = norms.get("feed_forward")
+
+    def _forward_float32(self, stream: ResidualStream, ctx: StepContext, call: LayerCall) -> ResidualStream:
+        if stream.deferred is not None:
+            stream.flush()
+        pending = stream.pending if stream.pending is not None else ()
+        normed = self.mixer_norm.sum_forward(stream.hidden, pending if isinstance(pending, tuple) else (pending,))
+        stream.rounded = None
+        stream.pending = (self.mixer.forward(normed, ctx, call),)
+        if self.feed_forward is not None:
+            normed = self.feed_forward_norm.sum_forward(stream.hidden, stream.pending)
+            stream.pending = self.feed_forward.forward_summands(normed)
+        return stream
 
     def forward(self, stream: ResidualStream, ctx: StepContext, call: LayerCall) -> ResidualStream:
+        # A stream in the model's own type takes the norms' form for that type (float32 models included, unless
+        # their norms have groups or a layer lacks its second half).
+        own_type = (getattr(self.mixer_norm, "dtype", stream.hidden.dtype) == stream.hidden.dtype
+                    and getattr(self.mixer_norm, "groups", 1) == 1 and self.feed_forward is not None)
+        if stream.hidden.dtype == torch.float32 and (not own_type or isinstance(stream.pending, tuple)):
+            return self._forward_float32(stream, ctx, call)
         if stream.pending is None:
             normed = self.mixer_norm.forward(stream.hidden)
         else:
@@ -52,8 +73,9 @@ class PreNormResidual(Block):
         stream.pending = self.feed_forward.forward(normed)
         return stream
 
-
     def chain_plan(self) -> BlockPlan | None:
+        if self.feed_forward is None:
+            return None
         mixer_norm, ffn_norm = self.mixer_norm.as_rms_scale(), self.feed_forward_norm.as_rms_scale()
         gated = self.feed_forward.as_gated_products()
         if mixer_norm is None or ffn_norm is None or gated is None:

@@ -39,7 +39,8 @@ class Embedding(InputPart):
         self.float32_stream = bool(spec.params.get("float32_stream", False))
         self.scale = float(spec.params.get("scale", 1.0))
         # For models whose first part reads the stream itself: hand on its rounding with it.
-        self.rounded_copy = bool(spec.params.get("rounded_copy", False))
+        # (a multiplier brings the rounding along unless the spec says it is not wanted)
+        self.rounded_copy = bool(spec.params.get("rounded_copy", self.scale != 1.0))
         if self.scale != 1.0 and not self.float32_stream:
             raise ConfigError("an embedding multiplier comes with a float32 stream")
 
@@ -52,14 +53,14 @@ class Embedding(InputPart):
         return []          # a step gathers a few rows of the table; it does not stream it
 
     def forward(self, ctx: StepContext) -> torch.Tensor:
-        if self.float32_stream and (self.scale != 1.0 or self.rounded_copy):
+        if self.float32_stream and self.rounded_copy:
             # The stream, and its rounding for the first part that reads the stream itself.
             if self.table.dtype == torch.float32:
                 return ops.embedding_f32(self.table, ctx.token_ids, ctx.status, self.scale)
             hidden, rounded = ops.embedding_f32(self.table, ctx.token_ids, ctx.status, self.scale, rounded=True)
             return ResidualStream(hidden, rounded=rounded)
         if self.float32_stream:
-            return ops.embedding_f32(self.table, ctx.token_ids, ctx.status)
+            return ops.embedding_f32(self.table, ctx.token_ids, ctx.status, self.scale)
         return ops.embedding(self.table, ctx.token_ids, ctx.status)
 
 

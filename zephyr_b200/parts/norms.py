@@ -2,6 +2,9 @@
 the normalisation and not as (1 + w) (reference: src/layer/normalization.cpp:10-18,
 deps/ttl/src/kernels/normalization/normalization.cu:76-139).
 
+With ``groups`` > 1 each of that many equal consecutive parts of the row is divided by its own root mean square; the
+scale stays one vector over the whole row.  Such a norm reads a float32 stream (``forward``, ``sum_forward``).
+
 LayerNorm: mean and variance of the row, a scale and (where the spec names one) a shift."""
 
 from __future__ import annotations
@@ -10,6 +13,7 @@ from typing import Mapping
 
 import torch
 
+from ..config.errors import ConfigError
 from ..config.spec import NormSpec
 from ..kernels import ops
 from ..weights.loader import ROLE_NORM, ROLE_ZERO, WeightDecl
@@ -22,6 +26,9 @@ class RMSNorm(Norm):
     def __init__(self, spec: NormSpec, weights: Mapping[str, torch.Tensor], dtype: torch.dtype):
         self.size = spec.size
         self.eps = float(spec.eps)
+        self.groups = int(spec.groups)
+        if self.groups <= 0 or spec.size % self.groups != 0:
+            raise ConfigError(f"a norm's groups divide its {spec.size} values evenly, {self.groups} do not")
         self.dtype = dtype
         self.weight = weights[spec.weight]
         self._scale32 = self.weight.float().contiguous()     # what the fused residual form reads
@@ -34,8 +41,9 @@ class RMSNorm(Norm):
         return [self.weight]          # (the float32 copy of the scales stands in for them, not beside them)
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
-        if x.dtype == torch.float32 and self.dtype != torch.float32:
-            return ops.sum_rms_norm(x, None, None, self.weight, self.eps, out_dtype=self.dtype)    # a float32 stream
+        if x.dtype == torch.float32 and (self.dtype != torch.float32 or self.groups > 1):
+            return ops.sum_rms_norm(x, None, None, self.weight, self.eps, out_dtype=self.dtype, groups=self.groups)    # a float32 stream
+        self._needs_one_group("a norm of rows in the model's type")
         return ops.rmsnorm(x, self.weight, self.eps)
 
     def sum_forward(self, stream: torch.Tensor, summands: tuple) -> torch.Tensor:
@@ -53,9 +61,14 @@ class RMSNorm(Norm):
             stream.add_(torch.stack(shifts).sum(0))
         a = rows[0] if len(rows) > 0 else None
         b = rows[1] if len(rows) > 1 else None
-        return ops.sum_rms_norm(stream, a, b, self.weight, self.eps, out_dtype=self.dtype, bias=shift)
+        return ops.sum_rms_norm(stream, a, b, self.weight, self.eps, out_dtype=self.dtype, bias=shift, groups=self.groups)
+
+    def _needs_one_group(self, what: str) -> None:
+        if self.groups > 1:
+            raise ConfigError(f"a norm in groups reads a float32 stream: {what} is not built")
 
     def add_forward(self, residual: torch.Tensor, delta: torch.Tensor) -> torch.Tensor:
+        self._needs_one_group("the sum in the model's type")
         return ops.add_rmsnorm(residual, delta, self.weight, self.eps)
 
     def add_scaled(self, residual: torch.Tensor, delta: torch.Tensor, mult: float,
@@ -63,12 +76,13 @@ class RMSNorm(Norm):
         """residual (float32) += mult * norm(delta), in place and in one kernel; with ``then`` also returns
         then(residual), with ``rounded_sum`` the sum itself in delta's type: the form a block with norms
         behind its parts uses."""
+        self._needs_one_group("the norm of a part's output")
         if then is None:
             return ops.residual_rms_norm(residual, delta, self._scale32, self.eps, mult, rounded_sum=rounded_sum)
         return ops.residual_rms_norm(residual, delta, self._scale32, self.eps, mult, then._scale32, then.eps)
 
-    def as_rms_scale(self) -> tuple[torch.Tensor, float]:
-        return self.weight, self.eps
+    def as_rms_scale(self) -> tuple[torch.Tensor, float] | None:
+        return (self.weight, self.eps) if self.groups == 1 else None
 
 
 class LayerNorm(Norm):

@@ -11,7 +11,8 @@ Further forms, each named by the spec: ``scores`` "sigmoid" (s = sigmoid(z), eve
 its ``top`` largest choice values, and only outputs of the ``keep`` runs with the largest marks can be taken;
 ``weight_scale``: a multiplier on every weight; ``router_bias``: a bias b on the logits, z = Wr x + b;
 ``scores`` "top_softmax": the ``top`` largest logits are taken, and their outputs count with the softmax over
-the taken logits only.
+the taken logits only; ``weigh`` "inputs": the weight goes on the expert's input instead of its output,
+out = sum of expert_e(s_e x) (no identity experts then).
 
 The first ``experts`` router outputs are gated feed-forwards, expert_e(x) = down_e(act(gate_e x) * (up_e x)),
 without biases; the last ``identity`` outputs are identity experts, expert(x) = x, which have no tensors.
@@ -52,6 +53,9 @@ class RoutedFeedForward(FeedForward):
         if self.scores not in ops.ROUTE_SCORES:
             raise ConfigError(f"router scores are one of {sorted(ops.ROUTE_SCORES)}")
         self.weight_scale = float(p.get("weight_scale", 1.0))
+        self.weigh = str(p.get("weigh", "outputs"))
+        if self.weigh not in ("outputs", "inputs") or (self.weigh == "inputs" and self.identity > 0):
+            raise ConfigError("weights go on the experts' outputs, or on their inputs where there are no identity experts")
         self.groups = None
         if p.get("groups"):
             g = p["groups"]
@@ -103,7 +107,8 @@ class RoutedFeedForward(FeedForward):
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         ids, weights = self.route(x)
-        return ops.routed_experts(x, ids, weights, self.w_gate, self.w_up, self.w_down, act=self.activation)
+        return ops.routed_experts(x, ids, weights, self.w_gate, self.w_up, self.w_down, act=self.activation,
+                                  weigh_inputs=self.weigh == "inputs")
 
 
 register_feed_forward("routed", RoutedFeedForward)

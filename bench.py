@@ -90,6 +90,18 @@ RIZOVIK_SIZES = {
                   delta=dict(heads=32, kv_heads=8, dim=128, vdim=128), experts=16, top=4),
 }
 
+# Legilix beside Rizovik: mixed scores beside mixed weights (both over a window that keeps the first tokens), a distance
+# bias over a window beside a window with pooled blocks; ``dense_ff`` is what gives an ungated feed-forward the weights of
+# a gated one of ``ff``.
+LEGILIX_SIZES = {
+    "w1024": dict(width=1024, ff=3072, dense_ff=4608, layers=8, heads=8, kv_heads=4, head_dim=128, window=1024, keep_first=64,
+                  experts=16, top=4),
+    "w2048": dict(width=2048, ff=6144, dense_ff=9216, layers=8, heads=16, kv_heads=8, head_dim=128, window=1024, keep_first=64,
+                  experts=16, top=4),
+    "w4096": dict(width=4096, ff=12288, dense_ff=18432, layers=8, heads=32, kv_heads=8, head_dim=128, window=1024, keep_first=64,
+                  experts=16, top=4),
+}
+
 
 def metric_name(args) -> str:
     """One string for both arms: the driver divides their values only if the strings are equal."""
@@ -322,6 +334,32 @@ def build_rizovik_pair(size: str, batch: int, context: int):
     return rizovik, gefovik, make
 
 
+def build_legilix_pair(size: str, batch: int, context: int):
+    """(Legilix configuration, Rizovik configuration of equal sizes, engine builder) of one entry of ``LEGILIX_SIZES``."""
+    from zephyr_b200.config import LegilixConfig, RizovikConfig
+
+    z = LEGILIX_SIZES[size]
+    hd = z["head_dim"]
+    routed = {"kind": "moe", "expert": {"ff": z["ff"] // z["top"]}, "router": {"experts": z["experts"], "top": z["top"]}}
+    dense = {"kind": "dense", "ff": z["dense_ff"]}
+    sizes = dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=hd, vdim=hd, scale=hd ** -0.5)
+    kept = {"size": z["window"], "keep_first": z["keep_first"]}
+    talking = dict(sizes, mask=kept, rot={"base": 150000.0, "dims": hd // 2,
+                                          "scaling": {"factor": 8.0, "original": 4096, "fast": 16.0, "slow": 1.0}})
+    distant = dict(sizes, mask={"size": z["window"]})
+    layers = [{"type": "attention", "mixer": talking, "mlp": dense}, {"type": "attention_2", "mixer": distant, "mlp": routed},
+              {"type": "attention", "mixer": talking, "mlp": routed}, {"type": "attention_2", "mixer": distant, "mlp": dense}]
+    legilix = LegilixConfig(vocab=32768, width=z["width"], norm_eps=1e-6, norm_groups=4, embedding_scale=8.0, logit_scale=0.25,
+                            layers=tuple((layers * 2)[:z["layers"]]))
+    mixed = {"type": "attention_2", "mlp": routed, "mixer": dict(sizes, mask=kept, rot={"base": 150000.0, "dims": hd // 2})}
+    pooled = {"type": "attention", "mlp": routed,
+              "mixer": dict(sizes, rot={"base": 150000.0, "dims": hd // 2}, mask={"size": z["window"], "pool": 16})}
+    rizovik = RizovikConfig(vocab=32768, width=z["width"], norm_eps=1e-6, residual_mult=1.0,
+                            layers=tuple(([mixed, pooled] * 4)[:z["layers"]]))
+    _, _, make = build_pair("w2048", batch, context)
+    return legilix, rizovik, make
+
+
 def run_legelix(args) -> dict:
     """Prefill of 2048 tokens and a decode step of ``--batch`` requests at ``--context``, device-timed, for
     every entry of ``LEGELIX_SIZES`` (or ``GEFOVIK_SIZES``) and for the Qwen3 decoder of equal size beside it."""
@@ -333,7 +371,8 @@ def run_legelix(args) -> dict:
            "data": "synthetic: seeded random weights and token ids", "sizes": {}}
     table, pair, beside = {"legelix": (LEGELIX_SIZES, build_pair, "qwen3"), "gefovik": (GEFOVIK_SIZES, build_gefovik_pair, "qwen3"),
                            "fekotar": (FEKOTAR_SIZES, build_fekotar_pair, "gefovik"),
-                           "rizovik": (RIZOVIK_SIZES, build_rizovik_pair, "gefovik")}[args.arch]
+                           "rizovik": (RIZOVIK_SIZES, build_rizovik_pair, "gefovik"),
+                           "legilix": (LEGILIX_SIZES, build_legilix_pair, "rizovik")}[args.arch]
     for size in (args.sizes.split(",") if args.sizes else table):
         legelix, qwen, make = pair(size, args.batch, args.context)
         row = {}
@@ -635,10 +674,10 @@ def main() -> int:
     parser.add_argument("--no-points", dest="points", action="store_false", help="skip decode at batch 1 and 64")
     parser.add_argument("--own-products", action="store_true",
                         help="with --only: no product on the vendor library (all on this package's tcgen05 kernel)")
-    parser.add_argument("--arch", choices=("qwen3", "legelix", "gefovik", "fekotar", "rizovik"), default="qwen3",
+    parser.add_argument("--arch", choices=("qwen3", "legelix", "gefovik", "fekotar", "rizovik", "legilix"), default="qwen3",
                         help="legelix, gefovik: prefill and decode of that design at a few layer sizes, beside Qwen3 of equal "
-                             "size; fekotar, rizovik: the same beside Gefovik of equal size")
-    parser.add_argument("--sizes", default="", help="--arch legelix|gefovik|fekotar|rizovik: entries of that design's table of sizes, with commas (default: all)")
+                             "size; fekotar, rizovik: the same beside Gefovik of equal size; legilix: beside Rizovik")
+    parser.add_argument("--sizes", default="", help="--arch legelix|gefovik|fekotar|rizovik|legilix: entries of that design's table of sizes, with commas (default: all)")
     parser.add_argument("--only", choices=("prefill", "decode"), default=None,
                         help="time only the 2048-token prefill, or only the decode step, and print a short line "
                              "(the program a profiler is pointed at)")
@@ -648,7 +687,7 @@ def main() -> int:
         return 2
     if args.warmup < 3:
         args.warmup = 3
-    if args.arch in ("legelix", "gefovik", "fekotar", "rizovik"):
+    if args.arch in ("legelix", "gefovik", "fekotar", "rizovik", "legilix"):
         print(json.dumps(run_legelix(args)))
         return 0
     if args.only is not None and args.impl == "ours":

@@ -9,13 +9,13 @@
 //
 // The scores are float32 from the product to the softmax, the mixing included.
 //
-// One CTA = 8 or 16 consecutive new tokens of one request (or ONE decoded token), eight warps of 1, 2 or 4
-// heads each.  The products put keys on the 16-row side of m16n8k16 and tokens on its 8-column side
+// One CTA = 8 or 16 consecutive new tokens of one request (or ONE decoded token), eight or sixteen warps of one or
+// two heads each.  The products put keys on the 16-row side of m16n8k16 and tokens on its 8-column side
 // (S^T = K Q^T, O^T = V^T P^T), so a warp keeps its heads' queries and outputs in registers whatever the count
-// of tokens, and heads that share a key/value head share its fragments.  A tile of 32 (or 16) keys, with the
+// of tokens.  A tile of 32 (or 16) keys, with the
 // keys and values of every key/value head, goes through three phases:
 //   scores    each warp forms its heads' raw scores and leaves them in shared memory, [head][token][key];
-//   mixing    a thread owns one or two (token, key) pairs: it reads the raw scores of all heads, forms the
+//   mixing    a thread owns one (token, key) pair (or two): it reads the raw scores of all heads, forms the
 //             mixed ones, takes off the bias, applies the mask and writes them back in place;
 //   values    each warp reads its heads' scores as the second product's operand: online softmax in float32 in
 //             base 2, probabilities rounded to bfloat16.
@@ -29,8 +29,6 @@
 
 namespace zb {
 
-constexpr int AH_WARPS = 8;
-constexpr int AH_THREADS = AH_WARPS * 32;
 constexpr size_t AH_SMEM_LIMIT = 227 * 1024;
 
 struct HeadsAttentionArgs {
@@ -57,11 +55,25 @@ struct HeadsAttentionArgs {
 
 __host__ __device__ constexpr int ah_padded(int dim) { return (dim + 15) / 16 * 16 + 8; }      // a row in shared memory
 
-// HPW heads a warp, NT columns of 8 tokens, DM: keys and values of up to 16 DM values, BK keys a tile.
-template <int HPW, int NT, int DM, int BK>
-__global__ void __launch_bounds__(AH_THREADS, 1) heads_attention_kernel(const HeadsAttentionArgs a) {
-  constexpr int HM = AH_WARPS * HPW, NTOK = 8 * NT, SST = BK + 8, MT = BK / 16;
-  constexpr int KPT = NTOK * BK >= 2 * AH_THREADS ? 2 : 1;             // keys a thread mixes at a time
+// ldmatrix at a shared-memory address: the kernel's offsets are then plain 32-bit additions.
+__device__ __forceinline__ void ah_ldmatrix(unsigned (&r)[4], unsigned address) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(address) : "memory");
+}
+__device__ __forceinline__ void ah_ldmatrix_trans(unsigned (&r)[4], unsigned address) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(address) : "memory");
+}
+__device__ __forceinline__ void ah_copy16(unsigned smem, const void* gmem, int bytes) {       // 0 bytes: zeros
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(smem), "l"(gmem), "r"(bytes) : "memory");
+}
+
+// W warps of HPW heads each, NT columns of 8 tokens, DM: keys and values of up to 16 DM values, BK keys a tile.
+template <int W, int HPW, int NT, int DM, int BK>
+__global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel(const HeadsAttentionArgs a) {
+  constexpr int THREADS = W * 32, HM = W * HPW, NTOK = 8 * NT, SST = BK + 8, MT = BK / 16;
+  constexpr int KPT = NTOK * BK >= 2 * THREADS ? 2 : 1;                // keys a thread mixes at a time
+  static_assert(NTOK * BK <= KPT * THREADS, "one turn of the threads mixes a tile");
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int kst = ah_padded(a.kd), vst = ah_padded(a.vd);
   __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smem_raw);                     // [nkv][BK][kst]
@@ -77,7 +89,6 @@ __global__ void __launch_bounds__(AH_THREADS, 1) heads_attention_kernel(const He
     if (threadIdx.x == 0) report(a.status, STATUS_ROW_OUT_OF_RANGE, row, tile);
     return;
   }
-  const int g = a.nh / a.nkv;
   const int q_len = a.row_q_len[row], ctx = a.row_ctx[row], tok0 = a.row_q_start[row] + q0;
   const int n_tok = min(a.splits > 1 ? 1 : NTOK, q_len - q0);
   if (n_tok <= 0) return;
@@ -115,20 +126,28 @@ __global__ void __launch_bounds__(AH_THREADS, 1) heads_attention_kernel(const He
   // The planned tile's rows of every key/value head; zeros for keys that nobody sees.
   auto load_rows = [&](__nv_bfloat16* dst, int stride, int dim, long long part, int buffer) {
     if (dim % 8 == 0) {
+      // A row's 16-byte pieces lie side by side on 4, 8, 16 or 32 lanes; a thread walks its keys, and for each of
+      // them the key/value heads, whose rows lie a page's rows apart.
       const int chunks = dim / 8;
-      const int lanes = chunks <= 4 ? 4 : (chunks <= 8 ? 8 : (chunks <= 16 ? 16 : 32)), rows = 32 / lanes;      // a row
-      for (int r = warp * rows + lane / lanes; r < a.nkv * BK; r += AH_WARPS * rows) {
-        const int kvh = r / BK, key = r % BK;
-        const int2 w = where_s[buffer][key];
-        const int in_page = a.page_shift >= 0 ? w.y & (a.page_size - 1) : w.y % a.page_size;
-        const int swizzle = kv_swizzle(w.y, chunks);
-        const __nv_bfloat16* src = a.kv_cache;
-        if (w.x > 0) src += w.x * page_elems + part + (static_cast<long long>(kvh) * a.page_size + in_page) * dim;
-        for (int c = lane & (lanes - 1); c < chunks; c += lanes)
-          cp_async_16(dst + r * stride + c * 8, w.x > 0 ? src + ((c ^ swizzle) << 3) : src, w.x > 0);
+      const int shift = chunks <= 4 ? 2 : (chunks <= 8 ? 3 : (chunks <= 16 ? 4 : 5)), c = lane & ((1 << shift) - 1);
+      if (c < chunks) {
+        const unsigned step = static_cast<unsigned>(BK * stride) * 2u;
+        const long long head_step = static_cast<long long>(a.page_size) * dim * 2;
+        for (int key = (warp << (5 - shift)) + (lane >> shift); key < BK; key += W << (5 - shift)) {
+          const int2 w = where_s[buffer][key];
+          const int in_page = a.page_shift >= 0 ? w.y & (a.page_size - 1) : w.y % a.page_size;
+          const char* src = reinterpret_cast<const char*>(
+              a.kv_cache + (w.x > 0 ? w.x * page_elems + part + static_cast<long long>(in_page) * dim +
+                                          ((c ^ kv_swizzle(w.y, chunks)) << 3) : 0));
+          const int bytes = w.x > 0 ? 16 : 0;
+          const long long advance = w.x > 0 ? head_step : 0;
+          unsigned to = smem_u32(dst + key * stride + c * 8);
+#pragma unroll 4
+          for (int kvh = 0; kvh < a.nkv; ++kvh, src += advance, to += step) ah_copy16(to, src, bytes);
+        }
       }
     } else {                                           // rows stored as they are, on any boundary
-      for (int r = warp; r < a.nkv * BK; r += AH_WARPS) {
+      for (int r = warp; r < a.nkv * BK; r += W) {
         const int kvh = r / BK, key = r % BK;
         const int2 w = where_s[buffer][key];
         const long long from = w.x * page_elems + part + (static_cast<long long>(kvh) * a.page_size + w.y % a.page_size) * dim;
@@ -143,10 +162,10 @@ __global__ void __launch_bounds__(AH_THREADS, 1) heads_attention_kernel(const He
 
   if (t_begin < t_end) plan(t_begin, 0);
   // The columns that pad a row to whole steps of 16 stay zero for good.
-  for (int e = threadIdx.x; e < a.nkv * BK * (kst + vst) / 8; e += AH_THREADS)
+  for (int e = threadIdx.x; e < a.nkv * BK * (kst + vst) / 8; e += THREADS)
     reinterpret_cast<uint4*>(k_s)[e] = make_uint4(0, 0, 0, 0);
   if (a.score_mix != nullptr)
-    for (int e = threadIdx.x; e < HM * HM; e += AH_THREADS) {
+    for (int e = threadIdx.x; e < HM * HM; e += THREADS) {
       const int h = e / HM, o = e - h * HM;
       mix_s[e] = h < a.nh && o < a.nh ? a.score_mix[h * a.nh + o] * a.scale_log2 : 0.0f;
     }
@@ -156,11 +175,17 @@ __global__ void __launch_bounds__(AH_THREADS, 1) heads_attention_kernel(const He
   if (t_begin < t_end) load_values(0);
   cp_async_commit();
 
-  // This warp's heads; their queries as the B operand (k = dims, n = tokens).
-  const int head0 = warp * HPW;
+  // This warp's heads; their queries as the B operand (k = dims, n = tokens).  A head past the last one runs on the
+  // last head's keys with queries of zero and is never stored.
+  const int head0 = warp * HPW, g = a.nh / a.nkv;
+  const bool works = head0 < a.nh;
+  unsigned k_at[HPW], v_at[HPW];                     // where this lane's rows of the heads' keys and values begin
   unsigned qf[HPW][NT][DM][2];
 #pragma unroll
   for (int i = 0; i < HPW; ++i) {
+    const int kvh = min(head0 + i, a.nh - 1) / g;
+    k_at[i] = smem_u32(k_s + (kvh * BK + ((lane >> 3) & 1) * 8 + (lane & 7)) * kst + (lane >> 4) * 8);
+    v_at[i] = smem_u32(v_s + (kvh * BK + (lane >> 4) * 8 + (lane & 7)) * vst + ((lane >> 3) & 1) * 8);
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt) {
       const int tok = nt * 8 + quad_row, head = head0 + i;
@@ -197,6 +222,9 @@ __global__ void __launch_bounds__(AH_THREADS, 1) heads_attention_kernel(const He
 #pragma unroll
       for (int m = 0; m < DM; ++m) o[i][nt][m][0] = o[i][nt][m][1] = o[i][nt][m][2] = o[i][nt][m][3] = 0.0f;
     }
+  const unsigned k_step = static_cast<unsigned>(16 * kst) * 2u, v_step = static_cast<unsigned>(16 * vst) * 2u;   // 16 keys
+  float* const raw_at = s_s + (head0 * NTOK + 2 * quad) * SST + quad_row;              // where this lane's raw scores go
+  const float* const own_at = s_s + (head0 * NTOK + quad_row) * SST + 2 * quad;        // and where it reads its final ones
 
   cp_async_wait<1>();
   __syncthreads();                                   // the first tile's keys have landed
@@ -205,40 +233,42 @@ __global__ void __launch_bounds__(AH_THREADS, 1) heads_attention_kernel(const He
     const bool more = t + 1 < t_end;
     if (more) plan(t + 1, buffer ^ 1);
     // ------------------------------------------------------------------------------------ raw scores
-    if (head0 < a.nh) {
+    if (works) {
+      float acc[MT][HPW][NT][4];
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt) {
-        float acc[HPW][NT][4];
+      for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
         for (int i = 0; i < HPW; ++i)
 #pragma unroll
-          for (int nt = 0; nt < NT; ++nt) acc[i][nt][0] = acc[i][nt][1] = acc[i][nt][2] = acc[i][nt][3] = 0.0f;
+          for (int nt = 0; nt < NT; ++nt) acc[mt][i][nt][0] = acc[mt][i][nt][1] = acc[mt][i][nt][2] = acc[mt][i][nt][3] = 0.0f;
 #pragma unroll
-        for (int ks = 0; ks < DM; ++ks) {
-          if (ks >= ks_n) break;
-          unsigned ka[4];
-          int held = -1;
+      for (int ks = 0; ks < DM; ++ks) {
+        if (ks < ks_n) {
 #pragma unroll
           for (int i = 0; i < HPW; ++i) {
-            if (head0 + i >= a.nh) break;
-            const int kvh = (head0 + i) / g;
-            if (kvh != held)
-              ldmatrix_x4(ka, k_s + (kvh * BK + mt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * kst + ks * 16 + (lane >> 4) * 8);
-            held = kvh;
 #pragma unroll
-            for (int nt = 0; nt < NT; ++nt) mma_bf16_16816(acc[i][nt], ka, qf[i][nt][ks][0], qf[i][nt][ks][1]);
+            for (int mt = 0; mt < MT; ++mt) {
+              unsigned ka[4];
+              ah_ldmatrix(ka, k_at[i] + mt * k_step + ks * 32);
+#pragma unroll
+              for (int nt = 0; nt < NT; ++nt) mma_bf16_16816(acc[mt][i][nt], ka, qf[i][nt][ks][0], qf[i][nt][ks][1]);
+            }
           }
         }
+      }
 #pragma unroll
-        for (int i = 0; i < HPW; ++i) {
-          if (head0 + i >= a.nh) break;
+      for (int i = 0; i < HPW; ++i) {
+        if (head0 + i < a.nh) {
 #pragma unroll
-          for (int nt = 0; nt < NT; ++nt) {
-            float* dst = s_s + ((head0 + i) * NTOK + nt * 8 + 2 * quad) * SST + mt * 16 + quad_row;
-            dst[0] = acc[i][nt][0];
-            dst[SST] = acc[i][nt][1];
-            dst[8] = acc[i][nt][2];
-            dst[SST + 8] = acc[i][nt][3];
+          for (int mt = 0; mt < MT; ++mt) {
+#pragma unroll
+            for (int nt = 0; nt < NT; ++nt) {
+              float* dst = raw_at + (i * NTOK + nt * 8) * SST + mt * 16;
+              dst[0] = acc[mt][i][nt][0];
+              dst[SST] = acc[mt][i][nt][1];
+              dst[8] = acc[mt][i][nt][2];
+              dst[SST + 8] = acc[mt][i][nt][3];
+            }
           }
         }
       }
@@ -274,21 +304,24 @@ __global__ void __launch_bounds__(AH_THREADS, 1) heads_attention_kernel(const He
           for (int h = 0; h < HM; ++h)
 #pragma unroll
             for (int u = 0; u < KPT; ++u) s[h][u] = h < a.nh ? at[h * NTOK * SST + u] : 0.0f;
+#pragma unroll 2
           for (int h = 0; h < a.nh; ++h) {
-            float v[KPT];
+            float v[KPT], w[KPT];                    // two chains of additions side by side
 #pragma unroll
-            for (int u = 0; u < KPT; ++u) v[u] = 0.0f;
+            for (int u = 0; u < KPT; ++u) v[u] = w[u] = 0.0f;
 #pragma unroll
             for (int o4 = 0; o4 < HM / 4; ++o4) {
               const float4 m = *reinterpret_cast<const float4*>(mix_s + h * HM + 4 * o4);
 #pragma unroll
               for (int u = 0; u < KPT; ++u) {
                 v[u] = fmaf(m.x, s[4 * o4][u], v[u]);
-                v[u] = fmaf(m.y, s[4 * o4 + 1][u], v[u]);
+                w[u] = fmaf(m.y, s[4 * o4 + 1][u], w[u]);
                 v[u] = fmaf(m.z, s[4 * o4 + 2][u], v[u]);
-                v[u] = fmaf(m.w, s[4 * o4 + 3][u], v[u]);
+                w[u] = fmaf(m.w, s[4 * o4 + 3][u], w[u]);
               }
             }
+#pragma unroll
+            for (int u = 0; u < KPT; ++u) v[u] += w[u];
             finish(h, v);
           }
         } else {
@@ -304,19 +337,18 @@ __global__ void __launch_bounds__(AH_THREADS, 1) heads_attention_kernel(const He
     cp_async_wait<1>();
     __syncthreads();                                 // the scores are final, this tile's values have landed
     // ------------------------------------------------------------------------------ softmax and values
-    if (head0 < a.nh) {
+    if (works) {
       unsigned pb[HPW][NT][MT][2];
 #pragma unroll
       for (int i = 0; i < HPW; ++i) {
-        if (head0 + i >= a.nh) break;
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt) {
-          const float* src = s_s + ((head0 + i) * NTOK + nt * 8 + quad_row) * SST + 2 * quad;
           float2 v[BK / 8];
           float top = -INFINITY;
+          const bool real = head0 + i < a.nh;        // (uniform over the warp)
 #pragma unroll
           for (int j = 0; j < BK / 8; ++j) {
-            v[j] = *reinterpret_cast<const float2*>(src + 8 * j);
+            v[j] = real ? *reinterpret_cast<const float2*>(own_at + (i * NTOK + nt * 8) * SST + 8 * j) : make_float2(0.0f, 0.0f);
             top = fmaxf(top, fmaxf(v[j].x, v[j].y));
           }
           top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 1));
@@ -351,20 +383,16 @@ __global__ void __launch_bounds__(AH_THREADS, 1) heads_attention_kernel(const He
       }
 #pragma unroll
       for (int m = 0; m < DM; ++m) {
-        if (m >= vm_n) break;
-#pragma unroll
-        for (int ks = 0; ks < MT; ++ks) {
-          unsigned va[4];
-          int held = -1;
+        if (m < vm_n) {
 #pragma unroll
           for (int i = 0; i < HPW; ++i) {
-            if (head0 + i >= a.nh) break;
-            const int kvh = (head0 + i) / g;
-            if (kvh != held)
-              ldmatrix_x4_trans(va, v_s + (kvh * BK + ks * 16 + (lane >> 4) * 8 + (lane & 7)) * vst + m * 16 + ((lane >> 3) & 1) * 8);
-            held = kvh;
 #pragma unroll
-            for (int nt = 0; nt < NT; ++nt) mma_bf16_16816(o[i][nt][m], va, pb[i][nt][ks][0], pb[i][nt][ks][1]);
+            for (int ks = 0; ks < MT; ++ks) {
+              unsigned va[4];
+              ah_ldmatrix_trans(va, v_at[i] + ks * v_step + m * 32);
+#pragma unroll
+              for (int nt = 0; nt < NT; ++nt) mma_bf16_16816(o[i][nt][m], va, pb[i][nt][ks][0], pb[i][nt][ks][1]);
+            }
           }
         }
       }
@@ -444,35 +472,35 @@ __global__ void __launch_bounds__(128) heads_merge_kernel(const HeadsAttentionAr
 }
 
 struct HeadsShape {
-  int hpw, nt, dm, bk;
+  int warps, hpw, nt, dm, bk;
   size_t smem;
 };
 
-// How the kernel runs this layer (hpw 0: it does not take it); `single`: for tiles of one token.
+// How the kernel runs this layer (warps 0: it does not take it); `single`: for tiles of one token.
 HeadsShape heads_shape(int nh, int nkv, int kd, int vd, bool single) {
-  HeadsShape shape{0, 0, 0, 0, 0};
+  HeadsShape shape{0, 0, 0, 0, 0, 0};
   if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || kd <= 0 || vd <= 0) return shape;
   const int widest = (kd > vd ? kd : vd);
   const int dm = widest <= 64 ? 4 : (widest <= 128 ? 8 : (widest <= 256 ? 16 : 0));
-  const int hpw = nh <= 8 ? 1 : (nh <= 16 ? 2 : (nh <= 32 ? 4 : 0));
-  if (dm == 0 || hpw == 0 || (dm == 16 && hpw == 4)) return shape;
-  const int nt = single || hpw == 4 || (dm == 16 && hpw == 2) ? 1 : 2;
+  const int warps = nh <= 8 ? 8 : 16, hpw = nh <= 16 ? 1 : (nh <= 32 ? 2 : 0);
+  if (dm == 0 || hpw == 0 || (dm == 16 && hpw == 2)) return shape;
+  const int nt = single || hpw == 2 || dm == 16 ? 1 : 2;
   for (int bk = 32; bk >= 16; bk -= 16) {
     const size_t smem = static_cast<size_t>(nkv) * bk * (ah_padded(kd) + ah_padded(vd)) * sizeof(__nv_bfloat16) +
-                        (static_cast<size_t>(64) * hpw * hpw + static_cast<size_t>(nh) * 8 * nt * (bk + 8)) * sizeof(float);
+                        (static_cast<size_t>(warps) * hpw * warps * hpw + static_cast<size_t>(nh) * 8 * nt * (bk + 8)) * sizeof(float);
     if (smem + 1024 <= AH_SMEM_LIMIT) {
-      shape = HeadsShape{hpw, nt, dm, bk, smem};
+      shape = HeadsShape{warps, hpw, nt, dm, bk, smem};
       return shape;
     }
   }
   return shape;
 }
 
-template <int HPW, int NT, int DM, int BK>
+template <int W, int HPW, int NT, int DM, int BK>
 int heads_launch(const HeadsAttentionArgs& a, int n_tiles, size_t smem, cudaStream_t stream) {
-  auto kernel = heads_attention_kernel<HPW, NT, DM, BK>;
+  auto kernel = heads_attention_kernel<W, HPW, NT, DM, BK>;
   if (cuda_failed(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)))) return ERR_CUDA;
-  kernel<<<dim3(a.splits, n_tiles), AH_THREADS, smem, stream>>>(a);
+  kernel<<<dim3(a.splits, n_tiles), W * 32, smem, stream>>>(a);
   return launch_result();
 }
 
@@ -483,7 +511,7 @@ using namespace zb;
 // New tokens of one request that a tile covers for rows with several of them (0: the shape is not taken).
 ZB_API int zb_heads_attention_tile_tokens(int nh, int nkv, int kd, int vd, int dtype) {
   if (dtype != DTYPE_BF16) return 0;
-  if (heads_shape(nh, nkv, kd, vd, true).hpw == 0) return 0;
+  if (heads_shape(nh, nkv, kd, vd, true).warps == 0) return 0;
   return 8 * heads_shape(nh, nkv, kd, vd, false).nt;
 }
 
@@ -504,7 +532,7 @@ ZB_API int zb_heads_attention(void* out, const void* q, const void* kv_cache, co
       reinterpret_cast<uintptr_t>(kv_cache) % 16 != 0)
     return ERR_BAD_ARGUMENT;
   const HeadsShape shape = heads_shape(nh, nkv, kd, vd, single != 0);
-  if (shape.hpw == 0) return ERR_UNSUPPORTED;
+  if (shape.warps == 0) return ERR_UNSUPPORTED;
   if (n_tiles == 0) return OK;
   if (n_tiles > 65535) return ERR_UNSUPPORTED;
   HeadsAttentionArgs a;
@@ -526,12 +554,13 @@ ZB_API int zb_heads_attention(void* out, const void* q, const void* kv_cache, co
   a.status = status;
   auto s = static_cast<cudaStream_t>(stream);
   int rc = ERR_UNSUPPORTED;
-#define ZB_AH(HPW, NT, DM, BK) \
-  if (shape.hpw == HPW && shape.nt == NT && shape.dm == DM && shape.bk == BK) rc = heads_launch<HPW, NT, DM, BK>(a, n_tiles, shape.smem, s);
-#define ZB_AH_BK(HPW, NT, DM) ZB_AH(HPW, NT, DM, 32) ZB_AH(HPW, NT, DM, 16)
-  ZB_AH_BK(1, 1, 4) ZB_AH_BK(1, 2, 4) ZB_AH_BK(2, 1, 4) ZB_AH_BK(2, 2, 4) ZB_AH_BK(4, 1, 4)
-  ZB_AH_BK(1, 1, 8) ZB_AH_BK(1, 2, 8) ZB_AH_BK(2, 1, 8) ZB_AH_BK(2, 2, 8) ZB_AH_BK(4, 1, 8)
-  ZB_AH_BK(1, 1, 16) ZB_AH_BK(1, 2, 16) ZB_AH_BK(2, 1, 16)
+#define ZB_AH(W, HPW, NT, DM, BK)                                                                                  \
+  if (shape.warps == W && shape.hpw == HPW && shape.nt == NT && shape.dm == DM && shape.bk == BK)                  \
+    rc = heads_launch<W, HPW, NT, DM, BK>(a, n_tiles, shape.smem, s);
+#define ZB_AH_BK(W, HPW, NT, DM) ZB_AH(W, HPW, NT, DM, 32) ZB_AH(W, HPW, NT, DM, 16)
+  ZB_AH_BK(8, 1, 1, 4) ZB_AH_BK(8, 1, 2, 4) ZB_AH_BK(16, 1, 1, 4) ZB_AH_BK(16, 1, 2, 4) ZB_AH_BK(16, 2, 1, 4)
+  ZB_AH_BK(8, 1, 1, 8) ZB_AH_BK(8, 1, 2, 8) ZB_AH_BK(16, 1, 1, 8) ZB_AH_BK(16, 1, 2, 8) ZB_AH_BK(16, 2, 1, 8)
+  ZB_AH_BK(8, 1, 1, 16) ZB_AH_BK(16, 1, 1, 16)
 #undef ZB_AH_BK
 #undef ZB_AH
   if (rc != OK || splits == 1) return rc;

@@ -107,7 +107,8 @@ __global__ void store_last_token_kernel(int* last_token, const int* ids, const i
 // ------------------------------------------------------------------------------------ sum + RMS norm
 // One CTA a row, or a group of a row (the grid's y counts the groups of H values; a norm without groups has
 // one).  The values are summed into the stream first (and kept in registers where they fit), then normed.
-// PER: elements a thread keeps; rows longer than PER * threads re-read the stream.
+// PER: elements a thread keeps; rows longer than PER * threads re-read the stream.  Short groups take fewer
+// threads (the block's size), so that many of them share an SM.
 constexpr int SN_THREADS = 256;
 constexpr int SN_PER = 16;
 
@@ -116,6 +117,7 @@ __global__ void __launch_bounds__(SN_THREADS)
 sum_rms_norm_kernel(OUT* out, long long out_stride, float* x, long long x_stride, const A* a, const B* b,
                     const float* bias, const void* w, int w_dtype, float eps, int H) {
   __shared__ float scratch[33];
+  const int threads = blockDim.x;
   const long long r = blockIdx.x, summand_stride = static_cast<long long>(H) * gridDim.y;
   const int g0 = blockIdx.y * H;             // where this group begins in its row
   float* xr = x + r * x_stride + g0;
@@ -136,11 +138,11 @@ sum_rms_norm_kernel(OUT* out, long long out_stride, float* x, long long x_stride
   float ss = 0.0f;
 #pragma unroll
   for (int k = 0; k < SN_PER; ++k) {
-    const int i = threadIdx.x + k * SN_THREADS;
+    const int i = threadIdx.x + k * threads;
     keep[k] = i < H ? summed(i) : 0.0f;
     ss += keep[k] * keep[k];
   }
-  for (int i = threadIdx.x + SN_PER * SN_THREADS; i < H; i += SN_THREADS) {
+  for (int i = threadIdx.x + SN_PER * threads; i < H; i += threads) {
     const float v = summed(i);
     ss += v * v;
   }
@@ -149,10 +151,10 @@ sum_rms_norm_kernel(OUT* out, long long out_stride, float* x, long long x_stride
   OUT* o = out + r * out_stride + g0;
 #pragma unroll
   for (int k = 0; k < SN_PER; ++k) {
-    const int i = threadIdx.x + k * SN_THREADS;
+    const int i = threadIdx.x + k * threads;
     if (i < H) o[i] = from_float<OUT>(keep[k] * inv * load_scale(w, w_dtype, g0 + i));
   }
-  for (int i = threadIdx.x + SN_PER * SN_THREADS; i < H; i += SN_THREADS)
+  for (int i = threadIdx.x + SN_PER * threads; i < H; i += threads)
     o[i] = from_float<OUT>(xr[i] * inv * load_scale(w, w_dtype, g0 + i));
 }
 
@@ -162,6 +164,7 @@ __global__ void __launch_bounds__(SN_THREADS)
 sum_rms_norm_vec_kernel(OUT* out, long long out_stride, float* x, long long x_stride, const A* a, const B* b,
                         const float* bias, const void* w, int w_dtype, float eps, int H) {
   __shared__ float scratch[33];
+  const int threads = blockDim.x;
   const long long r = blockIdx.x, summand_stride = static_cast<long long>(H) * gridDim.y;
   const int g0 = blockIdx.y * H;             // where this group begins in its row
   float* xr = x + r * x_stride + g0;
@@ -193,11 +196,11 @@ sum_rms_norm_vec_kernel(OUT* out, long long out_stride, float* x, long long x_st
   float ss = 0.0f;
 #pragma unroll
   for (int k = 0; k < PER; ++k) {
-    const int i = 4 * (threadIdx.x + k * SN_THREADS);
+    const int i = 4 * (threadIdx.x + k * threads);
     keep[k] = i < H ? summed(i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
     ss += keep[k].x * keep[k].x + keep[k].y * keep[k].y + keep[k].z * keep[k].z + keep[k].w * keep[k].w;
   }
-  for (int i = 4 * (threadIdx.x + PER * SN_THREADS); i < H; i += 4 * SN_THREADS) {
+  for (int i = 4 * (threadIdx.x + PER * threads); i < H; i += 4 * threads) {
     const float4 v = summed(i);
     ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
   }
@@ -206,10 +209,10 @@ sum_rms_norm_vec_kernel(OUT* out, long long out_stride, float* x, long long x_st
   OUT* o = out + r * out_stride + g0;
 #pragma unroll
   for (int k = 0; k < PER; ++k) {
-    const int i = 4 * (threadIdx.x + k * SN_THREADS);
+    const int i = 4 * (threadIdx.x + k * threads);
     if (i < H) store4(o + i, scaled(keep[k], inv, i));
   }
-  for (int i = 4 * (threadIdx.x + PER * SN_THREADS); i < H; i += 4 * SN_THREADS) store4(o + i, scaled(load4(xr + i), inv, i));
+  for (int i = 4 * (threadIdx.x + PER * threads); i < H; i += 4 * threads) store4(o + i, scaled(load4(xr + i), inv, i));
 }
 
 // -------------------------------------------------------------------------------------- clamped gate
@@ -363,15 +366,16 @@ ZB_API int zb_sum_rms_norm(void* out, long long out_stride, int out_dtype, float
   auto fits = [](const void* p, int bytes) { return reinterpret_cast<uintptr_t>(p) % bytes == 0; };
   const int part = H / groups;
   const dim3 grid(rows, groups);
+  const int threads = groups == 1 ? SN_THREADS : std::min(SN_THREADS, (part + 255) / 256 * 32);      // about eight values each
   const bool vectors = part % 4 == 0 && x_stride % 4 == 0 && out_stride % 4 == 0 && fits(x, 16) && fits(a, a_bytes) &&
                        fits(b, b_bytes) && fits(out, o_bytes) && fits(w, w_bytes) && fits(bias, 16);
 #define ZB_SN(A_, B_, OUT_)                                                                                          \
   {                                                                                                                  \
     if (vectors)                                                                                                     \
-      sum_rms_norm_vec_kernel<A_, B_, OUT_><<<grid, SN_THREADS, 0, s>>>((OUT_*)out, out_stride, x, x_stride,         \
+      sum_rms_norm_vec_kernel<A_, B_, OUT_><<<grid, threads, 0, s>>>((OUT_*)out, out_stride, x, x_stride,         \
                                                                          (const A_*)a, (const B_*)b, bias, w, w_dtype, eps, part); \
     else                                                                                                             \
-      sum_rms_norm_kernel<A_, B_, OUT_><<<grid, SN_THREADS, 0, s>>>((OUT_*)out, out_stride, x, x_stride, (const A_*)a, \
+      sum_rms_norm_kernel<A_, B_, OUT_><<<grid, threads, 0, s>>>((OUT_*)out, out_stride, x, x_stride, (const A_*)a, \
                                                                      (const B_*)b, bias, w, w_dtype, eps, part);     \
   }
 #define ZB_SN_OUT(A_, B_)                              \

@@ -269,6 +269,23 @@ sigmoid_gate_kernel(T* x, const float* gate, long long gate_stride, int width, i
   }
 }
 
+// The same for bfloat16 rows and runs of whole 16-byte pieces: a thread owns a piece and its run's gate.
+__global__ void __launch_bounds__(256)
+sigmoid_gate_pieces_kernel(uint4* x, const float* gate, long long gate_stride, int pieces, int per_pieces) {
+  const long long t = blockIdx.x;
+  for (int c = threadIdx.x; c < pieces; c += blockDim.x) {
+    const float g = 1.0f / (1.0f + expf(-gate[t * gate_stride + c / per_pieces]));
+    uint4 v = x[t * pieces + c];
+    __nv_bfloat162* pair = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const float2 f = __bfloat1622float2(pair[u]);
+      pair[u] = __floats2bfloat162_rn(f.x * g, f.y * g);
+    }
+    x[t * pieces + c] = v;
+  }
+}
+
 }  // namespace zb
 
 using namespace zb;
@@ -347,6 +364,10 @@ ZB_API int zb_sigmoid_gate(void* x, const float* gate, long long gate_stride, in
   if (tokens < 0 || width <= 0 || per <= 0 || width % per != 0 || gate_stride < width / per) return ERR_BAD_ARGUMENT;
   if (tokens == 0) return OK;
   auto s = static_cast<cudaStream_t>(stream);
+  if (dtype == DTYPE_BF16 && per % 8 == 0 && reinterpret_cast<uintptr_t>(x) % 16 == 0) {
+    sigmoid_gate_pieces_kernel<<<tokens, 256, 0, s>>>(static_cast<uint4*>(x), gate, gate_stride, width / 8, per / 8);
+    return launch_result();
+  }
   if (dtype == DTYPE_F32) sigmoid_gate_kernel<float><<<tokens, 256, 0, s>>>(static_cast<float*>(x), gate, gate_stride, width, per);
   else sigmoid_gate_kernel<__nv_bfloat16><<<tokens, 256, 0, s>>>(static_cast<__nv_bfloat16*>(x), gate, gate_stride, width, per);
   return launch_result();

@@ -718,6 +718,151 @@ def window_parts(args) -> dict:
     return out
 
 
+def mixed_scores(args) -> dict:
+    """Attention over a window of ``--window`` (default 1024) with 64 kept first tokens whose heads' scores are mixed
+    ahead of the softmax (all heads of a tile in one CTA), a prompt of ``--tokens`` tokens and ``--batch`` single tokens
+    at ``--context``; the same without the matrix; beside them the kept window on the mma.sync prompt kernel, with one
+    value head a query head and with every pair of heads (what a mixing of the weights behind the softmax takes)."""
+    device = torch.device("cuda")
+    H, G, d, page = args.heads, args.kv_heads, args.head_dim, args.page_size
+    window, keep = args.window or 1024, 64
+    status = ops.new_status(device)
+    mix = torch.eye(H, device=device) + torch.randn((H, H), device=device) * 0.1
+    # What a query's scores and values take, and a mixing of the scores, over the keys of its window.
+    seen = sum(min(p + 1, window + min(keep, max(0, p + 1 - window))) for p in range(args.tokens))
+    flops = seen * (4 * H * d + 2 * H * H)
+    out = {"heads": H, "kv_heads": G, "head_dim": d, "window": window, "prompt_gflop": round(flops / 1e9, 1)}
+
+    def run(kernel: str, new_tokens: int, before: int, requests: int, with_mix: bool) -> float:
+        T = new_tokens * requests
+        q = torch.randn((T, H * d), device=device, dtype=torch.bfloat16)
+        caches, table = _paged_inputs(requests, before + new_tokens, G, d, page, device)
+        start = torch.arange(0, T, new_tokens, dtype=torch.int32, device=device)
+        lens = torch.full((requests,), new_tokens, dtype=torch.int32, device=device)
+        ctx = torch.full((requests,), before, dtype=torch.int32, device=device)
+        single = new_tokens == 1
+        cross = kernel == "pairs"
+        tile = 1 if single else (ops.heads_attention_tile_tokens(H, G, d, d, torch.bfloat16) if kernel == "heads"
+                                 else ops.paged_prefill_tile_tokens())
+        per = -(-new_tokens // tile)
+        tile_row = torch.arange(requests, dtype=torch.int32, device=device).repeat_interleave(per)
+        tile_q0 = (torch.arange(per, dtype=torch.int32, device=device) * tile).repeat(requests)
+        result = torch.empty((T, H * d * (G if cross else 1)), device=device, dtype=torch.float32 if cross else torch.bfloat16)
+        if kernel == "heads":
+            return _time(lambda i: ops.heads_attention(q, caches[i % len(caches)], table, tile_row, tile_q0, start, lens, ctx, H, G, d, d,
+                                                       window, d ** -0.5, status, result, keep_first=keep,
+                                                       score_mix=mix if with_mix else None, single=single, max_context=before + new_tokens),
+                         args.warmup, args.iters)
+        return _time(lambda i: ops.paged_prefill(q, caches[i % len(caches)], table, tile_row, tile_q0, start, lens, ctx, H, G, d,
+                                                 window, d ** -0.5, status, result, keep_first=keep, cross_values=cross,
+                                                 by_group=single and H // G <= 16), args.warmup, args.iters)
+
+    for name, kernel, with_mix in (("mixed scores", "heads", True), ("all heads in one CTA, no matrix", "heads", False),
+                                   ("like: kept window on mma.sync", "plain", False), ("like: pairs of heads", "pairs", False)):
+        prompt = run(kernel, args.tokens, 0, 1, with_mix)
+        out[name] = {"prompt_us": round(prompt, 1), "prompt_tflops": round(flops / prompt / 1e6, 1),
+                     "single_tokens_us": round(run(kernel, 1, args.context - 1, args.batch, with_mix), 1)}
+    out["single_tokens_mb"] = round(args.batch * (window + keep) * 2 * G * d * 2 / 1e6, 1)
+    ops.check_status(status, "mixed_scores")
+    return out
+
+
+def distance_bias(args) -> dict:
+    """The logarithmic bias on the distance over a window of ``--window`` (default 1024): the prompt kernel (tcgen05 at
+    head size 128) and the split-context kernel, with and without the bias, and beside them a bound on the scores."""
+    device = torch.device("cuda")
+    H, G, d, page = args.heads, args.kv_heads, args.head_dim, args.page_size
+    window = args.window or 1024
+    status = ops.new_status(device)
+    bias = (torch.rand(H, device=device) + 0.1, torch.rand(H, device=device) * 0.4 + 0.05)
+    seen = sum(min(p + 1, window) for p in range(args.tokens))
+    flops = seen * 4 * H * d
+    T, B = args.tokens, args.batch
+    out = {"heads": H, "kv_heads": G, "head_dim": d, "window": window, "prompt_gflop": round(flops / 1e9, 1),
+           "single_tokens_mb": round(B * window * 2 * G * d * 2 / 1e6, 1)}
+    q = torch.randn((T, H * d), device=device, dtype=torch.bfloat16)
+    caches, table = _paged_inputs(1, T, G, d, page, device)
+    zero, length = torch.zeros(1, dtype=torch.int32, device=device), torch.full((1,), T, dtype=torch.int32, device=device)
+    tile_q0 = torch.arange(0, T, ops.paged_prefill_tile_tokens(), dtype=torch.int32, device=device)
+    result = torch.empty_like(q)
+    dq = torch.randn((B, H * d), device=device, dtype=torch.bfloat16)
+    dcaches, dtable = _paged_inputs(B, args.context, G, d, page, device)
+    rows = torch.arange(B, dtype=torch.int32, device=device)
+    ctx = torch.full((B,), args.context - 1, dtype=torch.int32, device=device)
+    dresult = torch.empty_like(dq)
+    for name, masks in (("window alone", {}), ("distance bias", {"distance_bias": bias}), ("like: bound on the scores", {"softcap": 50.0})):
+        us = _time(lambda i: ops.paged_prefill(q, caches[i % len(caches)], table, torch.zeros_like(tile_q0), tile_q0, zero, length, zero,
+                                               H, G, d, window, d ** -0.5, status, result, **masks), args.warmup, args.iters)
+        ds = _time(lambda i: ops.paged_decode(dq, dcaches[i % len(dcaches)], dtable, rows, rows, ctx, args.context, H, G, d, window,
+                                              d ** -0.5, status, dresult, **masks), args.warmup, args.iters)
+        out[name] = {"prompt_us": round(us, 1), "prompt_tflops": round(flops / us / 1e6, 1), "single_tokens_us": round(ds, 1)}
+    ops.check_status(status, "distance_bias")
+    return out
+
+
+def prenorm_parts(args) -> dict:
+    """The small kernels of a pre-norm design on a float32 stream, each beside its like: sum + norm in groups beside one
+    group; biases + per-head norms + rotation of halves + cache write beside the whole-projection form; biases + cache
+    write; the gate per head beside the gate per value; the ungated product with GELU beside the gated one of as many
+    weights, for a prompt and for a few rows; a routed layer with its weights on the inputs beside on the outputs."""
+    device = torch.device("cuda")
+    T, W, H, G, d, page = args.tokens, args.hidden, args.heads, args.kv_heads, args.head_dim, args.page_size
+    bf = torch.bfloat16
+    status = ops.new_status(device)
+    out = {"tokens": T, "hidden": W}
+    n = _copies(T * W * 8)
+    stream = [torch.randn((T, W), device=device) for _ in range(n)]
+    delta = [torch.randn((T, W), device=device, dtype=bf) for _ in range(n)]
+    w = torch.ones(W, device=device, dtype=bf)
+    for name, groups in (("sum_rms_norm, 4 groups", 4), ("like: one group", 1)):
+        us = _time(lambda i: ops.sum_rms_norm(stream[i % n], delta[i % n], None, w, 1e-6, bf, groups=groups), args.warmup, args.iters)
+        out[name] = {"us": round(us, 2), "gbs": round(T * W * 12 / us / 1e3, 1)}
+    blocks = -(-T // page)
+    table = torch.arange(1, blocks + 1, dtype=torch.int32, device=device).view(1, -1)
+    cache = torch.zeros((blocks + 1, 2, G, page, d), dtype=bf, device=device)
+    positions, rows = torch.arange(T, dtype=torch.int32, device=device), torch.zeros(T, dtype=torch.int32, device=device)
+    width = (H + 2 * G) * d
+    m = _copies(T * width * 4)
+    projected = [torch.randn((T, width), device=device) for _ in range(m)]
+    bias, head_w, freqs = torch.randn(width, device=device), torch.ones(d, device=device), torch.rand(d // 4, device=device)
+    q_w, k_w = torch.ones(H * d, device=device), torch.ones(G * d, device=device)
+    gbs = lambda us: {"us": round(us, 2), "gbs": round(T * width * 6 / us / 1e3, 1)}
+    out["qkv_halves, biases and norms per head"] = gbs(_time(lambda i: ops.qkv_halves(
+        projected[i % m], H, G, d, d, "per_head", head_w, head_w, 1e-6, freqs, d // 2, 1.1, False, positions, rows, cache, table, status,
+        bf, bias=bias), args.warmup, args.iters))
+    out["like: qkv_halves, whole norms"] = gbs(_time(lambda i: ops.qkv_halves(
+        projected[i % m], H, G, d, d, "whole", q_w, k_w, 1e-6, freqs, d // 2, 1.0, True, positions, rows, cache, table, status, bf),
+        args.warmup, args.iters))
+    out["qkv_pairs, biases alone"] = gbs(_time(lambda i: ops.qkv_pairs(
+        projected[i % m], H, G, d, d, bias, None, None, 1e-6, None, 0, positions, rows, cache, table, status, bf), args.warmup, args.iters))
+    attended = torch.randn((T, H * d), device=device, dtype=bf)
+    head_gate, gate = torch.randn((T, H), device=device), torch.randn((T, H * d), device=device)
+    us = _time(lambda i: ops.sigmoid_gate(attended, head_gate), args.warmup, args.iters)
+    out["sigmoid_gate per head"] = {"us": round(us, 2), "gbs": round(T * H * d * 4 / us / 1e3, 1)}
+    us = _time(lambda i: ops.sigmoid_gate(attended, gate), args.warmup, args.iters)
+    out["like: sigmoid_gate per value"] = {"us": round(us, 2), "gbs": round(T * H * d * 8 / us / 1e3, 1)}
+    F = args.ffn // 16 * 16
+    k = _copies(F * W * 2)
+    mats = [torch.randn((F, W), device=device, dtype=bf) * W ** -0.5 for _ in range(k)]
+    x, few = torch.randn((T, W), device=device, dtype=bf), torch.randn((args.rows, W), device=device, dtype=bf)
+    for name, kwargs in (("gelu", {"gelu": True}), ("like: swiglu", {"swiglu": True})):
+        us = _time(lambda i: ops.gemm_tc(x, mats[i % k], **kwargs), args.warmup, args.iters)
+        small = _time(lambda i: ops.gemm_small(few, mats[i % k], **kwargs), args.warmup, args.iters)
+        out[f"product with {name}"] = {"us": round(us, 1), "tflops": round(2 * T * F * W / us / 1e6, 1), "few_rows_us": round(small, 2),
+                                       "few_rows_gbs": round(F * W * 2 / small / 1e3, 1)}
+    E, top, ff = args.experts, args.top, F // args.top // 16 * 8
+    gate_up = ops.interleave_gate_up(*(torch.randn((E, ff, W), device=device, dtype=bf) * W ** -0.5 for _ in range(2)))
+    down = torch.randn((E, W, ff), device=device, dtype=bf) * ff ** -0.5
+    for rows_of, tokens in (("prompt", x), ("few rows", few)):
+        ids, weights = ops.route(torch.randn((tokens.shape[0], E), device=device), None, top, "sigmoid")
+        for name, inputs in (("routed, weights on inputs", True), ("like: weights on outputs", False)):
+            us = _time(lambda i: ops.routed_experts(tokens, ids, weights, gate_up, None, down, weigh_inputs=inputs), args.warmup, args.iters)
+            out[f"{name}, {rows_of}"] = {"us": round(us, 1), "tflops": round(6 * tokens.shape[0] * top * ff * W / us / 1e6, 1)}
+    ops.check_status(status, "prenorm_parts")
+    return out
+
+
+CASES.update({"mixed_scores": mixed_scores, "distance_bias": distance_bias, "prenorm_parts": prenorm_parts})
 CASES.update({"delta_rule": delta_rule, "windowed_attention": windowed_attention, "window_parts": window_parts})
 
 

@@ -15,8 +15,10 @@
 // of tokens.  A tile of 32 (or 16) keys, with the
 // keys and values of every key/value head, goes through three phases:
 //   scores    each warp forms its heads' raw scores and leaves them in shared memory, [head][token][key];
-//   mixing    a thread owns one (token, key) pair (or two): it reads the raw scores of all heads, forms the
-//             mixed ones, takes off the bias, applies the mask and writes them back in place;
+//   mixing    S' = M S over the heads, for 8 keys of a token at a time, on the tensor cores and exact to float32: a
+//             raw score is the sum of three bfloat16 values (24 bits), a matrix entry of one (an entry that is a
+//             bfloat16 value, as in a bfloat16 checkpoint) or of three, and the products that count are added up in
+//             float32; the bias is taken off, the mask applied, and the scores go back in place;
 //   values    each warp reads its heads' scores as the second product's operand: online softmax in float32 in
 //             base 2, probabilities rounded to bfloat16.
 // The next tile's keys are fetched (16-byte asynchronous copies, straight from the pages) while this tile is
@@ -53,6 +55,7 @@ struct HeadsAttentionArgs {
   int* status;
 };
 
+__host__ __device__ constexpr int ah_head_stride(int tokens, int keys) { return tokens * (keys + 8) + 4; }
 __host__ __device__ constexpr int ah_padded(int dim) { return (dim + 15) / 16 * 16 + 8; }      // a row in shared memory
 
 // ldmatrix at a shared-memory address: the kernel's offsets are then plain 32-bit additions.
@@ -64,23 +67,41 @@ __device__ __forceinline__ void ah_ldmatrix_trans(unsigned (&r)[4], unsigned add
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(address) : "memory");
 }
+__device__ __forceinline__ float ah_exp2(float x) {      // the special-function unit's: relative error about 2^-22
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ void ah_copy16(unsigned smem, const void* gmem, int bytes) {       // 0 bytes: zeros
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(smem), "l"(gmem), "r"(bytes) : "memory");
 }
 
-// W warps of HPW heads each, NT columns of 8 tokens, DM: keys and values of up to 16 DM values, BK keys a tile.
-template <int W, int HPW, int NT, int DM, int BK>
+// A float as the sum of three bfloat16 values, two floats at a time (the first in the low halves).
+__device__ __forceinline__ void ah_split(float x, float y, unsigned& hi, unsigned& mid, unsigned& lo) {
+  hi = pack_bf16(x, y);
+  x -= __uint_as_float(hi << 16);
+  y -= __uint_as_float(hi & 0xffff0000u);
+  mid = pack_bf16(x, y);
+  lo = pack_bf16(x - __uint_as_float(mid << 16), y - __uint_as_float(mid & 0xffff0000u));
+}
+
+// W warps in CG column groups; a warp has HPW heads and NT columns of 8 tokens.  DM: keys and values of up to 16 DM
+// values, BK keys a tile.
+template <int W, int HPW, int NT, int CG, int DM, int BK>
 __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel(const HeadsAttentionArgs a) {
-  constexpr int THREADS = W * 32, HM = W * HPW, NTOK = 8 * NT, SST = BK + 8, MT = BK / 16;
-  constexpr int KPT = NTOK * BK >= 2 * THREADS ? 2 : 1;                // keys a thread mixes at a time
-  static_assert(NTOK * BK <= KPT * THREADS, "one turn of the threads mixes a tile");
+  constexpr int THREADS = W * 32, WH = W / CG, HM = WH * HPW < 16 ? 16 : WH * HPW, NTOK = 8 * NT * CG, SST = BK + 8, MT = BK / 16;
+  constexpr int HST = ah_head_stride(NTOK, BK);                        // floats between two heads' scores
+  constexpr int MST = HM + 8;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int kst = ah_padded(a.kd), vst = ah_padded(a.vd);
   __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smem_raw);                     // [nkv][BK][kst]
   __nv_bfloat16* v_s = k_s + a.nkv * BK * kst;                                         // [nkv][BK][vst]
-  float* mix_s = reinterpret_cast<float*>(v_s + a.nkv * BK * vst);                     // [HM][HM], times scale and log2(e)
-  float* s_s = mix_s + HM * HM;                                                        // [nh][NTOK][SST]
-  __shared__ int2 where_s[2][BK];                    // a tile's keys: (page, position), page 0: not in sight of anyone
+  __nv_bfloat16* mix_s = v_s + a.nkv * BK * vst;                                       // [3][HM][MST], the matrix's three parts
+  float* s_s = reinterpret_cast<float*>(mix_s + 3 * HM * MST);                         // [nh][HST]: [NTOK][SST] of each head
+  // A tile's keys: where their first key/value head's key row and value row begin in the cache (bytes, multiples of
+  // 16, the row's chunk permutation in the low bits; or bytes of any value for rows stored as they are), or -1 for a
+  // key that nobody sees.
+  __shared__ longlong2 where_s[2][BK];
 
   // The host lists the tiles by the number of keys they see, fewest first: the longest work starts first.
   const int tile = gridDim.y - 1 - blockIdx.y, split = blockIdx.x;
@@ -108,6 +129,8 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
   const int t_end = static_cast<int>(static_cast<long long>(all_tiles) * (split + 1) / a.splits);
   auto tile_start = [&](int t) { return t < kept_tiles ? t * BK : first_tile + (t - kept_tiles) * BK; };
 
+  const long long page_elems = static_cast<long long>(a.nkv) * a.page_size * (a.kd + a.vd);
+  const long long value_part = static_cast<long long>(a.nkv) * a.page_size * a.kd;
   auto plan = [&](int t, int buffer) {               // by the first BK threads
     if (threadIdx.x >= BK) return;
     const int pos = tile_start(t) + static_cast<int>(threadIdx.x);
@@ -120,11 +143,19 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
         page = 0;
       }
     }
-    where_s[buffer][threadIdx.x] = make_int2(page, pos);
+    longlong2 at = make_longlong2(-1, -1);
+    if (page > 0) {
+      const int in_page = a.page_shift >= 0 ? pos & (a.page_size - 1) : pos % a.page_size;
+      at.x = (page * page_elems + static_cast<long long>(in_page) * a.kd) * 2;
+      at.y = (page * page_elems + value_part + static_cast<long long>(in_page) * a.vd) * 2;
+      if (a.kd % 8 == 0) at.x += kv_swizzle(pos, a.kd / 8);
+      if (a.vd % 8 == 0) at.y += kv_swizzle(pos, a.vd / 8);
+    }
+    where_s[buffer][threadIdx.x] = at;
   };
-  const long long page_elems = static_cast<long long>(a.nkv) * a.page_size * (a.kd + a.vd);
   // The planned tile's rows of every key/value head; zeros for keys that nobody sees.
-  auto load_rows = [&](__nv_bfloat16* dst, int stride, int dim, long long part, int buffer) {
+  auto load_rows = [&](__nv_bfloat16* dst, int stride, int dim, bool values, int buffer) {
+    const char* cache = reinterpret_cast<const char*>(a.kv_cache);
     if (dim % 8 == 0) {
       // A row's 16-byte pieces lie side by side on 4, 8, 16 or 32 lanes; a thread walks its keys, and for each of
       // them the key/value heads, whose rows lie a page's rows apart.
@@ -134,13 +165,11 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
         const unsigned step = static_cast<unsigned>(BK * stride) * 2u;
         const long long head_step = static_cast<long long>(a.page_size) * dim * 2;
         for (int key = (warp << (5 - shift)) + (lane >> shift); key < BK; key += W << (5 - shift)) {
-          const int2 w = where_s[buffer][key];
-          const int in_page = a.page_shift >= 0 ? w.y & (a.page_size - 1) : w.y % a.page_size;
-          const char* src = reinterpret_cast<const char*>(
-              a.kv_cache + (w.x > 0 ? w.x * page_elems + part + static_cast<long long>(in_page) * dim +
-                                          ((c ^ kv_swizzle(w.y, chunks)) << 3) : 0));
-          const int bytes = w.x > 0 ? 16 : 0;
-          const long long advance = w.x > 0 ? head_step : 0;
+          const long long from = values ? where_s[buffer][key].y : where_s[buffer][key].x;
+          const bool seen = from >= 0;
+          const char* src = cache + (seen ? (from & ~15LL) + ((c ^ static_cast<int>(from & 15)) << 4) : 0);
+          const int bytes = seen ? 16 : 0;
+          const long long advance = seen ? head_step : 0;
           unsigned to = smem_u32(dst + key * stride + c * 8);
 #pragma unroll 4
           for (int kvh = 0; kvh < a.nkv; ++kvh, src += advance, to += step) ah_copy16(to, src, bytes);
@@ -149,27 +178,34 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
     } else {                                           // rows stored as they are, on any boundary
       for (int r = warp; r < a.nkv * BK; r += W) {
         const int kvh = r / BK, key = r % BK;
-        const int2 w = where_s[buffer][key];
-        const long long from = w.x * page_elems + part + (static_cast<long long>(kvh) * a.page_size + w.y % a.page_size) * dim;
-        for (int i = lane; i < dim; i += 32)
-          dst[r * stride + i] = w.x > 0 ? a.kv_cache[from + i] : __float2bfloat16_rn(0.0f);
+        const long long from = values ? where_s[buffer][key].y : where_s[buffer][key].x;
+        const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(
+            cache + (from >= 0 ? from + static_cast<long long>(kvh) * a.page_size * dim * 2 : 0));
+        for (int i = lane; i < dim; i += 32) dst[r * stride + i] = from >= 0 ? src[i] : __float2bfloat16_rn(0.0f);
       }
     }
   };
-  const long long value_part = static_cast<long long>(a.nkv) * a.page_size * a.kd;
-  auto load_keys = [&](int buffer) { load_rows(k_s, kst, a.kd, 0, buffer); };
-  auto load_values = [&](int buffer) { load_rows(v_s, vst, a.vd, value_part, buffer); };
+  auto load_keys = [&](int buffer) { load_rows(k_s, kst, a.kd, false, buffer); };
+  auto load_values = [&](int buffer) { load_rows(v_s, vst, a.vd, true, buffer); };
 
   if (t_begin < t_end) plan(t_begin, 0);
   // The columns that pad a row to whole steps of 16 stay zero for good.
   for (int e = threadIdx.x; e < a.nkv * BK * (kst + vst) / 8; e += THREADS)
     reinterpret_cast<uint4*>(k_s)[e] = make_uint4(0, 0, 0, 0);
+  int inexact = 0;
   if (a.score_mix != nullptr)
     for (int e = threadIdx.x; e < HM * HM; e += THREADS) {
       const int h = e / HM, o = e - h * HM;
-      mix_s[e] = h < a.nh && o < a.nh ? a.score_mix[h * a.nh + o] * a.scale_log2 : 0.0f;
+      float v = h < a.nh && o < a.nh ? a.score_mix[h * a.nh + o] : 0.0f;
+#pragma unroll
+      for (int part = 0; part < 3; ++part) {
+        const __nv_bfloat16 b = __float2bfloat16_rn(v);
+        mix_s[(part * HM + h) * MST + o] = b;
+        v -= __bfloat162float(b);
+        if (part == 0 && v != 0.0f) inexact = 1;
+      }
     }
-  __syncthreads();
+  const bool one_part = __syncthreads_or(inexact) == 0;      // (a barrier: the plan is there, the pads are zero)
   if (t_begin < t_end) load_keys(0);
   cp_async_commit();
   if (t_begin < t_end) load_values(0);
@@ -177,8 +213,8 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
 
   // This warp's heads; their queries as the B operand (k = dims, n = tokens).  A head past the last one runs on the
   // last head's keys with queries of zero and is never stored.
-  const int head0 = warp * HPW, g = a.nh / a.nkv;
-  const bool works = head0 < a.nh;
+  const int head0 = warp % WH * HPW, col0 = warp / WH * (8 * NT), g = a.nh / a.nkv;
+  const bool works = head0 < a.nh && col0 < n_tok;
   unsigned k_at[HPW], v_at[HPW];                     // where this lane's rows of the heads' keys and values begin
   unsigned qf[HPW][NT][DM][2];
 #pragma unroll
@@ -188,7 +224,7 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
     v_at[i] = smem_u32(v_s + (kvh * BK + (lane >> 4) * 8 + (lane & 7)) * vst + ((lane >> 3) & 1) * 8);
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt) {
-      const int tok = nt * 8 + quad_row, head = head0 + i;
+      const int tok = col0 + nt * 8 + quad_row, head = head0 + i;
       const bool ok = tok < n_tok && head < a.nh;
       const __nv_bfloat16* src = a.q + (static_cast<size_t>(tok0 + (ok ? tok : 0)) * a.nh + (ok ? head : 0)) * a.kd;
       const bool pairs = a.kd % 2 == 0;
@@ -223,8 +259,9 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
       for (int m = 0; m < DM; ++m) o[i][nt][m][0] = o[i][nt][m][1] = o[i][nt][m][2] = o[i][nt][m][3] = 0.0f;
     }
   const unsigned k_step = static_cast<unsigned>(16 * kst) * 2u, v_step = static_cast<unsigned>(16 * vst) * 2u;   // 16 keys
-  float* const raw_at = s_s + (head0 * NTOK + 2 * quad) * SST + quad_row;              // where this lane's raw scores go
-  const float* const own_at = s_s + (head0 * NTOK + quad_row) * SST + 2 * quad;        // and where it reads its final ones
+  const int lane_raw = 2 * quad * HST + quad_row;    // a lane's raw scores of two heads and one key of a piece
+  float* const raw_at = s_s + head0 * HST + (col0 + 2 * quad) * SST + quad_row;           // where this lane's raw scores go
+  const float* const own_at = s_s + head0 * HST + (col0 + quad_row) * SST + 2 * quad;      // and where it reads its final ones
 
   cp_async_wait<1>();
   __syncthreads();                                   // the first tile's keys have landed
@@ -263,7 +300,7 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
           for (int mt = 0; mt < MT; ++mt) {
 #pragma unroll
             for (int nt = 0; nt < NT; ++nt) {
-              float* dst = raw_at + (i * NTOK + nt * 8) * SST + mt * 16;
+              float* dst = raw_at + i * HST + nt * 8 * SST + mt * 16;
               dst[0] = acc[mt][i][nt][0];
               dst[SST] = acc[mt][i][nt][1];
               dst[8] = acc[mt][i][nt][2];
@@ -277,61 +314,64 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
     if (more) load_keys(buffer ^ 1);
     cp_async_commit();
     // --------------------------------------------------------------------- mixing, bias, mask, in place
-    {
-      const int e = threadIdx.x * KPT, tok = e / BK, key = e % BK;
-      if (tok < n_tok) {
-        const int k0 = tile_start(t), qp = ctx + q0 + tok;
-        bool valid[KPT];
-        float distance[KPT];
+    // A warp takes 8 keys of a token at a time: the lane's columns are keys 2 quad and 2 quad + 1, its rows heads.
+    for (int piece = warp; piece < n_tok * (BK / 8); piece += W) {
+      const int tok = piece / (BK / 8), key8 = piece % (BK / 8) * 8;
+      const int pos = tile_start(t) + key8 + 2 * quad, qp = ctx + q0 + tok;
+      bool valid[2];
 #pragma unroll
-        for (int u = 0; u < KPT; ++u) {
-          const int pos = k0 + key + u;
-          valid[u] = t < kept_tiles ? pos < kept
-                                    : pos <= qp && pos >= lo && (a.window == 0 || pos > qp - a.window || pos < a.keep_first);
-          distance[u] = static_cast<float>(qp - pos);
+      for (int u = 0; u < 2; ++u)
+        valid[u] = t < kept_tiles ? pos + u < kept
+                                  : pos + u <= qp && pos + u >= lo &&
+                                        (a.window == 0 || pos + u > qp - a.window || pos + u < a.keep_first);
+      float* at = s_s + tok * SST + key8;
+      auto finish = [&](int h, float x, float y) {
+        x *= a.scale_log2;
+        y *= a.scale_log2;
+        if (a.bias_r1 != nullptr) {
+          const float r1 = a.bias_r1[h], r2 = a.bias_r2[h];
+          x = fmaf(-r1, __log2f(fmaf(r2, static_cast<float>(qp - pos), 1.0f)), x);
+          y = fmaf(-r1, __log2f(fmaf(r2, static_cast<float>(qp - pos - 1), 1.0f)), y);
         }
-        float* at = s_s + tok * SST + key;
-        auto finish = [&](int h, float (&v)[KPT]) {
+        *reinterpret_cast<float2*>(at + h * HST + 2 * quad) = make_float2(valid[0] ? x : -INFINITY, valid[1] ? y : -INFINITY);
+      };
+      if (a.score_mix != nullptr) {
+        unsigned hi[HM / 16][2], mid[HM / 16][2], low[HM / 16][2];
 #pragma unroll
-          for (int u = 0; u < KPT; ++u) {
-            if (a.bias_r1 != nullptr) v[u] = fmaf(-a.bias_r1[h], __log2f(fmaf(a.bias_r2[h], distance[u], 1.0f)), v[u]);
-            at[h * NTOK * SST + u] = valid[u] ? v[u] : -INFINITY;
+        for (int kk = 0; kk < HM / 16; ++kk)
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const int h = kk * 16 + half * 8 + 2 * quad;
+            const float* raw = at + (kk * 16 + half * 8) * HST + lane_raw;
+            const float x = h < a.nh ? raw[0] : 0.0f, y = h + 1 < a.nh ? raw[HST] : 0.0f;
+            ah_split(x, y, hi[kk][half], mid[kk][half], low[kk][half]);
           }
-        };
-        if (a.score_mix != nullptr) {
-          float s[HM][KPT];
+        __syncwarp();                                // the raw scores of these keys are read
 #pragma unroll
-          for (int h = 0; h < HM; ++h)
+        for (int mt = 0; mt < HM / 16; ++mt) {
+          float c[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
-            for (int u = 0; u < KPT; ++u) s[h][u] = h < a.nh ? at[h * NTOK * SST + u] : 0.0f;
-#pragma unroll 2
-          for (int h = 0; h < a.nh; ++h) {
-            float v[KPT], w[KPT];                    // two chains of additions side by side
-#pragma unroll
-            for (int u = 0; u < KPT; ++u) v[u] = w[u] = 0.0f;
-#pragma unroll
-            for (int o4 = 0; o4 < HM / 4; ++o4) {
-              const float4 m = *reinterpret_cast<const float4*>(mix_s + h * HM + 4 * o4);
-#pragma unroll
-              for (int u = 0; u < KPT; ++u) {
-                v[u] = fmaf(m.x, s[4 * o4][u], v[u]);
-                w[u] = fmaf(m.y, s[4 * o4 + 1][u], w[u]);
-                v[u] = fmaf(m.z, s[4 * o4 + 2][u], v[u]);
-                w[u] = fmaf(m.w, s[4 * o4 + 3][u], w[u]);
-              }
+          for (int kk = 0; kk < HM / 16; ++kk) {
+            const __nv_bfloat16* m_at = mix_s + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * MST + kk * 16 + (lane >> 4) * 8;
+            unsigned m[4];
+            if (!one_part) {                         // the smaller products first
+              ldmatrix_x4(m, m_at + 2 * HM * MST);
+              mma_bf16_16816(c, m, hi[kk][0], hi[kk][1]);
+              ldmatrix_x4(m, m_at + HM * MST);
+              mma_bf16_16816(c, m, mid[kk][0], mid[kk][1]);
+              mma_bf16_16816(c, m, hi[kk][0], hi[kk][1]);
             }
-#pragma unroll
-            for (int u = 0; u < KPT; ++u) v[u] += w[u];
-            finish(h, v);
+            ldmatrix_x4(m, m_at);
+            mma_bf16_16816(c, m, low[kk][0], low[kk][1]);
+            mma_bf16_16816(c, m, mid[kk][0], mid[kk][1]);
+            mma_bf16_16816(c, m, hi[kk][0], hi[kk][1]);
           }
-        } else {
-          for (int h = 0; h < a.nh; ++h) {
-            float v[KPT];
-#pragma unroll
-            for (int u = 0; u < KPT; ++u) v[u] = at[h * NTOK * SST + u] * a.scale_log2;
-            finish(h, v);
-          }
+          const int h = mt * 16 + quad_row;
+          if (h < a.nh) finish(h, c[0], c[1]);
+          if (h + 8 < a.nh) finish(h + 8, c[2], c[3]);
         }
+      } else {
+        for (int h = quad_row; h < a.nh; h += 8) finish(h, at[h * HST + 2 * quad], at[h * HST + 2 * quad + 1]);
       }
     }
     cp_async_wait<1>();
@@ -348,20 +388,20 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
           const bool real = head0 + i < a.nh;        // (uniform over the warp)
 #pragma unroll
           for (int j = 0; j < BK / 8; ++j) {
-            v[j] = real ? *reinterpret_cast<const float2*>(own_at + (i * NTOK + nt * 8) * SST + 8 * j) : make_float2(0.0f, 0.0f);
+            v[j] = real ? *reinterpret_cast<const float2*>(own_at + i * HST + nt * 8 * SST + 8 * j) : make_float2(0.0f, 0.0f);
             top = fmaxf(top, fmaxf(v[j].x, v[j].y));
           }
           top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 1));
           top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 2));
           const float new_m = fmaxf(m_run[i][nt], top);
           const float m_use = new_m == -INFINITY ? 0.0f : new_m;      // a token that has seen no key yet
-          const float corr = exp2f(m_run[i][nt] - m_use);
+          const float corr = ah_exp2(m_run[i][nt] - m_use);
           m_run[i][nt] = new_m;
           float sum = 0.0f;
 #pragma unroll
           for (int j = 0; j < BK / 8; ++j) {
-            v[j].x = exp2f(v[j].x - m_use);
-            v[j].y = exp2f(v[j].y - m_use);
+            v[j].x = ah_exp2(v[j].x - m_use);
+            v[j].y = ah_exp2(v[j].y - m_use);
             sum += v[j].x + v[j].y;
           }
           sum += __shfl_xor_sync(0xffffffffu, sum, 1);
@@ -407,7 +447,7 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
 #pragma unroll
   for (int i = 0; i < HPW; ++i) {
     const int head = head0 + i;
-    if (head >= a.nh) break;
+    if (head >= a.nh || col0 >= n_tok) break;
     if (a.splits > 1) {                              // one token: column 0 of the first tokens' column
       const size_t slot = (static_cast<size_t>(tile) * a.splits + split) * a.nh + head;
       if (lane == 0) {
@@ -430,7 +470,7 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
       const float inv[2] = {l0 > 0.0f ? 1.0f / l0 : 0.0f, l1 > 0.0f ? 1.0f / l1 : 0.0f};
 #pragma unroll
       for (int u = 0; u < 2; ++u) {
-        const int tok = nt * 8 + 2 * quad + u;
+        const int tok = col0 + nt * 8 + 2 * quad + u;
         if (tok >= n_tok) continue;
         __nv_bfloat16* dst = a.out + (static_cast<size_t>(tok0 + tok) * a.nh + head) * a.vd;
 #pragma unroll
@@ -472,33 +512,37 @@ __global__ void __launch_bounds__(128) heads_merge_kernel(const HeadsAttentionAr
 }
 
 struct HeadsShape {
-  int warps, hpw, nt, dm, bk;
+  int warps, hpw, nt, cg, dm, bk;
   size_t smem;
 };
 
 // How the kernel runs this layer (warps 0: it does not take it); `single`: for tiles of one token.
 HeadsShape heads_shape(int nh, int nkv, int kd, int vd, bool single) {
-  HeadsShape shape{0, 0, 0, 0, 0, 0};
+  HeadsShape shape{0, 0, 0, 0, 0, 0, 0};
   if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || kd <= 0 || vd <= 0) return shape;
   const int widest = (kd > vd ? kd : vd);
   const int dm = widest <= 64 ? 4 : (widest <= 128 ? 8 : (widest <= 256 ? 16 : 0));
-  const int warps = nh <= 8 ? 8 : 16, hpw = nh <= 16 ? 1 : (nh <= 32 ? 2 : 0);
+  const int hpw = nh <= 16 ? 1 : (nh <= 32 ? 2 : 0);
   if (dm == 0 || hpw == 0 || (dm == 16 && hpw == 2)) return shape;
-  const int nt = single || hpw == 2 || dm == 16 ? 1 : 2;
+  // Up to 8 heads: eight warps for a token, sixteen in two column groups for a prompt.
+  const int cg = nh <= 8 && !single ? 2 : 1, warps = nh <= 8 && single ? 8 : 16;
+  const int nt = single || nh <= 8 || hpw == 2 || dm == 16 ? 1 : 2;
+  const int hm = nh <= 16 ? 16 : 32;
   for (int bk = 32; bk >= 16; bk -= 16) {
     const size_t smem = static_cast<size_t>(nkv) * bk * (ah_padded(kd) + ah_padded(vd)) * sizeof(__nv_bfloat16) +
-                        (static_cast<size_t>(warps) * hpw * warps * hpw + static_cast<size_t>(nh) * 8 * nt * (bk + 8)) * sizeof(float);
+                        static_cast<size_t>(3) * hm * (hm + 8) * sizeof(__nv_bfloat16) +
+                        static_cast<size_t>(nh) * ah_head_stride(8 * nt * cg, bk) * sizeof(float);
     if (smem + 1024 <= AH_SMEM_LIMIT) {
-      shape = HeadsShape{warps, hpw, nt, dm, bk, smem};
+      shape = HeadsShape{warps, hpw, nt, cg, dm, bk, smem};
       return shape;
     }
   }
   return shape;
 }
 
-template <int W, int HPW, int NT, int DM, int BK>
+template <int W, int HPW, int NT, int CG, int DM, int BK>
 int heads_launch(const HeadsAttentionArgs& a, int n_tiles, size_t smem, cudaStream_t stream) {
-  auto kernel = heads_attention_kernel<W, HPW, NT, DM, BK>;
+  auto kernel = heads_attention_kernel<W, HPW, NT, CG, DM, BK>;
   if (cuda_failed(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)))) return ERR_CUDA;
   kernel<<<dim3(a.splits, n_tiles), W * 32, smem, stream>>>(a);
   return launch_result();
@@ -512,7 +556,8 @@ using namespace zb;
 ZB_API int zb_heads_attention_tile_tokens(int nh, int nkv, int kd, int vd, int dtype) {
   if (dtype != DTYPE_BF16) return 0;
   if (heads_shape(nh, nkv, kd, vd, true).warps == 0) return 0;
-  return 8 * heads_shape(nh, nkv, kd, vd, false).nt;
+  const HeadsShape shape = heads_shape(nh, nkv, kd, vd, false);
+  return shape.warps == 0 ? 0 : 8 * shape.nt * shape.cg;
 }
 
 // Keys of a tile of a decoded token: its keys can be cut into at most ceil(keys / this) splits that all have work.
@@ -554,13 +599,13 @@ ZB_API int zb_heads_attention(void* out, const void* q, const void* kv_cache, co
   a.status = status;
   auto s = static_cast<cudaStream_t>(stream);
   int rc = ERR_UNSUPPORTED;
-#define ZB_AH(W, HPW, NT, DM, BK)                                                                                  \
-  if (shape.warps == W && shape.hpw == HPW && shape.nt == NT && shape.dm == DM && shape.bk == BK)                  \
-    rc = heads_launch<W, HPW, NT, DM, BK>(a, n_tiles, shape.smem, s);
-#define ZB_AH_BK(W, HPW, NT, DM) ZB_AH(W, HPW, NT, DM, 32) ZB_AH(W, HPW, NT, DM, 16)
-  ZB_AH_BK(8, 1, 1, 4) ZB_AH_BK(8, 1, 2, 4) ZB_AH_BK(16, 1, 1, 4) ZB_AH_BK(16, 1, 2, 4) ZB_AH_BK(16, 2, 1, 4)
-  ZB_AH_BK(8, 1, 1, 8) ZB_AH_BK(8, 1, 2, 8) ZB_AH_BK(16, 1, 1, 8) ZB_AH_BK(16, 1, 2, 8) ZB_AH_BK(16, 2, 1, 8)
-  ZB_AH_BK(8, 1, 1, 16) ZB_AH_BK(16, 1, 1, 16)
+#define ZB_AH(W, HPW, NT, CG, DM, BK)                                                                              \
+  if (shape.warps == W && shape.hpw == HPW && shape.nt == NT && shape.cg == CG && shape.dm == DM && shape.bk == BK) \
+    rc = heads_launch<W, HPW, NT, CG, DM, BK>(a, n_tiles, shape.smem, s);
+#define ZB_AH_BK(W, HPW, NT, CG, DM) ZB_AH(W, HPW, NT, CG, DM, 32) ZB_AH(W, HPW, NT, CG, DM, 16)
+  ZB_AH_BK(8, 1, 1, 1, 4) ZB_AH_BK(16, 1, 1, 2, 4) ZB_AH_BK(16, 1, 1, 1, 4) ZB_AH_BK(16, 1, 2, 1, 4) ZB_AH_BK(16, 2, 1, 1, 4)
+  ZB_AH_BK(8, 1, 1, 1, 8) ZB_AH_BK(16, 1, 1, 2, 8) ZB_AH_BK(16, 1, 1, 1, 8) ZB_AH_BK(16, 1, 2, 1, 8) ZB_AH_BK(16, 2, 1, 1, 8)
+  ZB_AH_BK(8, 1, 1, 1, 16) ZB_AH_BK(16, 1, 1, 2, 16) ZB_AH_BK(16, 1, 1, 1, 16)
 #undef ZB_AH_BK
 #undef ZB_AH
   if (rc != OK || splits == 1) return rc;

@@ -97,7 +97,7 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
   __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smem_raw);                     // [nkv][BK][kst]
   __nv_bfloat16* v_s = k_s + a.nkv * BK * kst;                                         // [nkv][BK][vst]
   __nv_bfloat16* mix_s = v_s + a.nkv * BK * vst;                                       // [3][HM][MST], the matrix's three parts
-  float* s_s = reinterpret_cast<float*>(mix_s + 3 * HM * MST);                         // [nh][HST]: [NTOK][SST] of each head
+  float* s_s = reinterpret_cast<float*>(mix_s + 3 * HM * MST);                         // [HM][HST]: [NTOK][SST] of each head, zeros past the last
   // A tile's keys: where their first key/value head's key row and value row begin in the cache (bytes, multiples of
   // 16, the row's chunk permutation in the low bits; or bytes of any value for rows stored as they are), or -1 for a
   // key that nobody sees.
@@ -192,6 +192,7 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
   // The columns that pad a row to whole steps of 16 stay zero for good.
   for (int e = threadIdx.x; e < a.nkv * BK * (kst + vst) / 8; e += THREADS)
     reinterpret_cast<uint4*>(k_s)[e] = make_uint4(0, 0, 0, 0);
+  for (int e = a.nh * HST + threadIdx.x; e < HM * HST; e += THREADS) s_s[e] = 0.0f;
   int inexact = 0;
   if (a.score_mix != nullptr)
     for (int e = threadIdx.x; e < HM * HM; e += THREADS) {
@@ -259,7 +260,10 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
       for (int m = 0; m < DM; ++m) o[i][nt][m][0] = o[i][nt][m][1] = o[i][nt][m][2] = o[i][nt][m][3] = 0.0f;
     }
   const unsigned k_step = static_cast<unsigned>(16 * kst) * 2u, v_step = static_cast<unsigned>(16 * vst) * 2u;   // 16 keys
-  const int lane_raw = 2 * quad * HST + quad_row;    // a lane's raw scores of two heads and one key of a piece
+  // In a piece of 8 keys: a lane's raw scores of two heads and one key, its final ones of one head and two keys, and its
+  // rows of the mixing matrix.
+  const int lane_raw = 2 * quad * HST + quad_row, lane_final = quad_row * HST + 2 * quad;
+  const unsigned mix_at = smem_u32(mix_s + ((lane & 7) + ((lane >> 3) & 1) * 8) * MST + (lane >> 4) * 8);
   float* const raw_at = s_s + head0 * HST + (col0 + 2 * quad) * SST + quad_row;           // where this lane's raw scores go
   const float* const own_at = s_s + head0 * HST + (col0 + quad_row) * SST + 2 * quad;      // and where it reads its final ones
 
@@ -314,18 +318,17 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
     if (more) load_keys(buffer ^ 1);
     cp_async_commit();
     // --------------------------------------------------------------------- mixing, bias, mask, in place
-    // A warp takes 8 keys of a token at a time: the lane's columns are keys 2 quad and 2 quad + 1, its rows heads.
-    for (int piece = warp; piece < n_tok * (BK / 8); piece += W) {
-      const int tok = piece / (BK / 8), key8 = piece % (BK / 8) * 8;
-      const int pos = tile_start(t) + key8 + 2 * quad, qp = ctx + q0 + tok;
-      bool valid[2];
-#pragma unroll
-      for (int u = 0; u < 2; ++u)
-        valid[u] = t < kept_tiles ? pos + u < kept
-                                  : pos + u <= qp && pos + u >= lo &&
-                                        (a.window == 0 || pos + u > qp - a.window || pos + u < a.keep_first);
-      float* at = s_s + tok * SST + key8;
-      auto finish = [&](int h, float x, float y) {
+    // A warp takes 8 keys of a token at a time, the same keys of every token it takes: the lane's columns are keys
+    // 2 quad and 2 quad + 1, its rows heads.
+    {
+      constexpr int PER_TOKEN = BK / 8, TOKENS = W / PER_TOKEN, PIECES = (NTOK + TOKENS - 1) / TOKENS, AT_ONCE = HM == 16 ? 2 : 1;
+      const int key8 = warp % PER_TOKEN * 8, tok_first = warp / PER_TOKEN;
+      const int k0 = tile_start(t), pos = k0 + key8 + 2 * quad;
+      // A tile that every token sees whole needs no mask: most tiles of a long window are such.
+      const bool whole = t < kept_tiles ? k0 + BK <= kept
+                                        : k0 + BK - 1 <= ctx + q0 && k0 >= lo && (a.window == 0 || k0 > hi - 1 - a.window);
+      auto finish = [&](float* at, int tok, int h, float x, float y) {
+        const int qp = ctx + q0 + tok;
         x *= a.scale_log2;
         y *= a.scale_log2;
         if (a.bias_r1 != nullptr) {
@@ -333,45 +336,83 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
           x = fmaf(-r1, __log2f(fmaf(r2, static_cast<float>(qp - pos), 1.0f)), x);
           y = fmaf(-r1, __log2f(fmaf(r2, static_cast<float>(qp - pos - 1), 1.0f)), y);
         }
-        *reinterpret_cast<float2*>(at + h * HST + 2 * quad) = make_float2(valid[0] ? x : -INFINITY, valid[1] ? y : -INFINITY);
+        if (!whole) {
+          auto valid = [&](int p) {
+            return t < kept_tiles ? p < kept : p <= qp && p >= lo && (a.window == 0 || p > qp - a.window || p < a.keep_first);
+          };
+          if (!valid(pos)) x = -INFINITY;
+          if (!valid(pos + 1)) y = -INFINITY;
+        }
+        *reinterpret_cast<float2*>(at + lane_final) = make_float2(x, y);
       };
       if (a.score_mix != nullptr) {
-        unsigned hi[HM / 16][2], mid[HM / 16][2], low[HM / 16][2];
 #pragma unroll
-        for (int kk = 0; kk < HM / 16; ++kk)
+        for (int j0 = 0; j0 < PIECES; j0 += AT_ONCE) {
+          if (tok_first + j0 * TOKENS >= n_tok) break;           // (the same for the whole warp, as are the tokens below)
+          float* at[AT_ONCE];
+          unsigned hi3[AT_ONCE][HM / 16][2], mid3[AT_ONCE][HM / 16][2], low3[AT_ONCE][HM / 16][2];
 #pragma unroll
-          for (int half = 0; half < 2; ++half) {
-            const int h = kk * 16 + half * 8 + 2 * quad;
-            const float* raw = at + (kk * 16 + half * 8) * HST + lane_raw;
-            const float x = h < a.nh ? raw[0] : 0.0f, y = h + 1 < a.nh ? raw[HST] : 0.0f;
-            ah_split(x, y, hi[kk][half], mid[kk][half], low[kk][half]);
+          for (int u = 0; u < AT_ONCE; ++u) {
+            // (a token past the last one has scores of whatever lies there, which nobody reads)
+            at[u] = s_s + min(tok_first + (j0 + u) * TOKENS, NTOK - 1) * SST + key8;
+#pragma unroll
+            for (int kk = 0; kk < HM / 16; ++kk)
+#pragma unroll
+              for (int half = 0; half < 2; ++half) {
+                const float* raw = at[u] + (kk * 16 + half * 8) * HST + lane_raw;
+                ah_split(raw[0], raw[HST], hi3[u][kk][half], mid3[u][kk][half], low3[u][kk][half]);
+              }
           }
-        __syncwarp();                                // the raw scores of these keys are read
+          __syncwarp();                              // the raw scores of these keys are read
 #pragma unroll
-        for (int mt = 0; mt < HM / 16; ++mt) {
-          float c[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+          for (int mt = 0; mt < HM / 16; ++mt) {
+            float c[AT_ONCE][4];
 #pragma unroll
-          for (int kk = 0; kk < HM / 16; ++kk) {
-            const __nv_bfloat16* m_at = mix_s + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * MST + kk * 16 + (lane >> 4) * 8;
-            unsigned m[4];
-            if (!one_part) {                         // the smaller products first
-              ldmatrix_x4(m, m_at + 2 * HM * MST);
-              mma_bf16_16816(c, m, hi[kk][0], hi[kk][1]);
-              ldmatrix_x4(m, m_at + HM * MST);
-              mma_bf16_16816(c, m, mid[kk][0], mid[kk][1]);
-              mma_bf16_16816(c, m, hi[kk][0], hi[kk][1]);
+            for (int u = 0; u < AT_ONCE; ++u) c[u][0] = c[u][1] = c[u][2] = c[u][3] = 0.0f;
+#pragma unroll
+            for (int kk = 0; kk < HM / 16; ++kk) {
+              const unsigned m_at = mix_at + static_cast<unsigned>(mt * 16 * MST + kk * 16) * 2u;
+              unsigned m[4];
+              if (!one_part) {                       // the smaller products first
+                ah_ldmatrix(m, m_at + 2u * (2 * HM * MST));
+#pragma unroll
+                for (int u = 0; u < AT_ONCE; ++u) mma_bf16_16816(c[u], m, hi3[u][kk][0], hi3[u][kk][1]);
+                ah_ldmatrix(m, m_at + 2u * (HM * MST));
+#pragma unroll
+                for (int u = 0; u < AT_ONCE; ++u) {
+                  mma_bf16_16816(c[u], m, mid3[u][kk][0], mid3[u][kk][1]);
+                  mma_bf16_16816(c[u], m, hi3[u][kk][0], hi3[u][kk][1]);
+                }
+              }
+              ah_ldmatrix(m, m_at);
+#pragma unroll
+              for (int u = 0; u < AT_ONCE; ++u) mma_bf16_16816(c[u], m, low3[u][kk][0], low3[u][kk][1]);
+#pragma unroll
+              for (int u = 0; u < AT_ONCE; ++u) mma_bf16_16816(c[u], m, mid3[u][kk][0], mid3[u][kk][1]);
+#pragma unroll
+              for (int u = 0; u < AT_ONCE; ++u) mma_bf16_16816(c[u], m, hi3[u][kk][0], hi3[u][kk][1]);
             }
-            ldmatrix_x4(m, m_at);
-            mma_bf16_16816(c, m, low[kk][0], low[kk][1]);
-            mma_bf16_16816(c, m, mid[kk][0], mid[kk][1]);
-            mma_bf16_16816(c, m, hi[kk][0], hi[kk][1]);
+#pragma unroll
+            for (int u = 0; u < AT_ONCE; ++u) {
+              const int tok = tok_first + (j0 + u) * TOKENS, h = mt * 16 + quad_row;
+              if (tok < n_tok) {
+                if (h < a.nh) finish(at[u] + mt * 16 * HST, tok, h, c[u][0], c[u][1]);
+                if (h + 8 < a.nh) finish(at[u] + (mt * 16 + 8) * HST, tok, h + 8, c[u][2], c[u][3]);
+              }
+            }
           }
-          const int h = mt * 16 + quad_row;
-          if (h < a.nh) finish(h, c[0], c[1]);
-          if (h + 8 < a.nh) finish(h + 8, c[2], c[3]);
         }
       } else {
-        for (int h = quad_row; h < a.nh; h += 8) finish(h, at[h * HST + 2 * quad], at[h * HST + 2 * quad + 1]);
+        for (int tok = tok_first; tok < n_tok; tok += TOKENS) {
+          float* at = s_s + tok * SST + key8;
+#pragma unroll
+          for (int h8 = 0; h8 < HM; h8 += 8) {
+            if (h8 + quad_row < a.nh) {
+              const float2 raw = *reinterpret_cast<const float2*>(at + h8 * HST + lane_final);
+              finish(at + h8 * HST, tok, h8 + quad_row, raw.x, raw.y);
+            }
+          }
+        }
       }
     }
     cp_async_wait<1>();
@@ -531,7 +572,7 @@ HeadsShape heads_shape(int nh, int nkv, int kd, int vd, bool single) {
   for (int bk = 32; bk >= 16; bk -= 16) {
     const size_t smem = static_cast<size_t>(nkv) * bk * (ah_padded(kd) + ah_padded(vd)) * sizeof(__nv_bfloat16) +
                         static_cast<size_t>(3) * hm * (hm + 8) * sizeof(__nv_bfloat16) +
-                        static_cast<size_t>(nh) * ah_head_stride(8 * nt * cg, bk) * sizeof(float);
+                        static_cast<size_t>(hm) * ah_head_stride(8 * nt * cg, bk) * sizeof(float);
     if (smem + 1024 <= AH_SMEM_LIMIT) {
       shape = HeadsShape{warps, hpw, nt, cg, dm, bk, smem};
       return shape;

@@ -573,7 +573,7 @@ HeadsShape heads_shape(int nh, int nkv, int kd, int vd, bool single) {
     const size_t smem = static_cast<size_t>(nkv) * bk * (ah_padded(kd) + ah_padded(vd)) * sizeof(__nv_bfloat16) +
                         static_cast<size_t>(3) * hm * (hm + 8) * sizeof(__nv_bfloat16) +
                         static_cast<size_t>(hm) * ah_head_stride(8 * nt * cg, bk) * sizeof(float);
-    if (smem + 1024 <= AH_SMEM_LIMIT) {
+    if (smem + 2048 <= AH_SMEM_LIMIT) {
       shape = HeadsShape{warps, hpw, nt, cg, dm, bk, smem};
       return shape;
     }

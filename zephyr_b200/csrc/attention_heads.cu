@@ -526,28 +526,38 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
 }
 
 // The splits' partial results of one token and head, in the order of the context.
-__global__ void __launch_bounds__(128) heads_merge_kernel(const HeadsAttentionArgs a) {
-  const int tile = blockIdx.x, head = blockIdx.y;
+constexpr int AH_MERGE_THREADS = 128;
+constexpr int AH_MAX_SPLITS = AH_MERGE_THREADS;      // a thread each
+
+__global__ void __launch_bounds__(AH_MERGE_THREADS) heads_merge_kernel(const HeadsAttentionArgs a) {
+  __shared__ float weight_s[AH_MAX_SPLITS];
+  __shared__ float warp_note[AH_MERGE_THREADS / 32];
+  __shared__ float scratch[33];
+  const int tile = blockIdx.x, head = blockIdx.y, split = threadIdx.x;
   const int row = a.tile_row[tile];
   if (row < 0 || row >= a.num_rows || a.row_q_len[row] - a.tile_q0[tile] <= 0) return;       // (reported by the other kernel)
   const size_t slot0 = static_cast<size_t>(tile) * a.splits * a.nh + head;
-  float top = -INFINITY;
-  for (int s = 0; s < a.splits; ++s) top = fmaxf(top, a.part_ml[2 * (slot0 + static_cast<size_t>(s) * a.nh)]);
-  float l = 0.0f;
-  for (int s = 0; s < a.splits; ++s) {
-    const size_t slot = slot0 + static_cast<size_t>(s) * a.nh;
-    const float m = a.part_ml[2 * slot];
-    if (m > -INFINITY) l = fmaf(a.part_ml[2 * slot + 1], exp2f(m - top), l);
+  float m = -INFINITY, l = 0.0f;
+  if (split < a.splits) {
+    const float2 ml = *reinterpret_cast<const float2*>(a.part_ml + 2 * (slot0 + static_cast<size_t>(split) * a.nh));
+    m = ml.x;
+    l = ml.y;
   }
-  const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+  const float warp_top = warp_max(m);
+  if ((threadIdx.x & 31) == 0) warp_note[threadIdx.x >> 5] = warp_top;
+  __syncthreads();
+  float top = warp_note[0];
+#pragma unroll
+  for (int i = 1; i < AH_MERGE_THREADS / 32; ++i) top = fmaxf(top, warp_note[i]);
+  const float weight = m > -INFINITY ? exp2f(m - top) : 0.0f;
+  weight_s[split] = weight;
+  const float sum = block_sum(l * weight, scratch);  // (a barrier: the weights are there)
+  const float inv = sum > 0.0f ? 1.0f / sum : 0.0f;
   const size_t token = a.row_q_start[row] + a.tile_q0[tile];
-  for (int d = threadIdx.x; d < a.vd; d += blockDim.x) {
+  for (int d = threadIdx.x; d < a.vd; d += AH_MERGE_THREADS) {
     float v = 0.0f;
-    for (int s = 0; s < a.splits; ++s) {
-      const size_t slot = slot0 + static_cast<size_t>(s) * a.nh;
-      const float m = a.part_ml[2 * slot];
-      if (m > -INFINITY) v = fmaf(a.part_o[slot * a.vd + d], exp2f(m - top), v);
-    }
+#pragma unroll 8
+    for (int s = 0; s < a.splits; ++s) v = fmaf(a.part_o[(slot0 + static_cast<size_t>(s) * a.nh) * a.vd + d], weight_s[s], v);
     a.out[(token * a.nh + head) * a.vd + d] = __float2bfloat16_rn(v * inv);
   }
 }
@@ -606,14 +616,14 @@ ZB_API int zb_heads_attention_tile_keys(int nh, int nkv, int kd, int vd) { retur
 
 // Attention of the tiles' tokens over their requests' pages; writes those tokens' rows of `out` [T, nh * vd].
 // `single`: every tile is one token, whose keys `splits` CTAs share; with splits > 1 `scratch` holds
-// n_tiles * splits * nh * (vd + 2) floats (contents irrelevant).
+// n_tiles * splits * nh * (vd + 2) floats (contents irrelevant); at most 128 splits.
 ZB_API int zb_heads_attention(void* out, const void* q, const void* kv_cache, const int* block_table, int max_blocks,
                               int page_size, int num_pages, int num_rows, const int* tile_row, const int* tile_q0,
                               int n_tiles, const int* row_q_start, const int* row_q_len, const int* row_ctx, int nh,
                               int nkv, int kd, int vd, int window, int keep_first, float scale, const float* score_mix,
                               const float* bias_r1, const float* bias_r2, int single, int splits, float* scratch,
                               int* status, void* stream) {
-  if (n_tiles < 0 || page_size <= 0 || window < 0 || keep_first < 0 || splits <= 0 || (splits > 1 && (!single || scratch == nullptr)) ||
+  if (n_tiles < 0 || page_size <= 0 || window < 0 || keep_first < 0 || splits <= 0 || splits > AH_MAX_SPLITS || (splits > 1 && (!single || scratch == nullptr)) ||
       (bias_r1 == nullptr) != (bias_r2 == nullptr) || reinterpret_cast<uintptr_t>(q) % 4 != 0 ||
       reinterpret_cast<uintptr_t>(kv_cache) % 16 != 0)
     return ERR_BAD_ARGUMENT;
@@ -635,8 +645,8 @@ ZB_API int zb_heads_attention(void* out, const void* q, const void* kv_cache, co
   a.scale_log2 = scale * 1.4426950408889634f;
   a.score_mix = score_mix; a.bias_r1 = bias_r1; a.bias_r2 = bias_r2;
   a.splits = splits;
-  a.part_o = scratch;
-  a.part_ml = scratch != nullptr ? scratch + static_cast<size_t>(n_tiles) * splits * nh * vd : nullptr;
+  a.part_ml = scratch;                               // pairs of floats first: they stay on 8-byte boundaries
+  a.part_o = scratch != nullptr ? scratch + static_cast<size_t>(n_tiles) * splits * nh * 2 : nullptr;
   a.status = status;
   auto s = static_cast<cudaStream_t>(stream);
   int rc = ERR_UNSUPPORTED;
@@ -650,6 +660,6 @@ ZB_API int zb_heads_attention(void* out, const void* q, const void* kv_cache, co
 #undef ZB_AH_BK
 #undef ZB_AH
   if (rc != OK || splits == 1) return rc;
-  heads_merge_kernel<<<dim3(n_tiles, nh), 128, 0, s>>>(a);
+  heads_merge_kernel<<<dim3(n_tiles, nh), AH_MERGE_THREADS, 0, s>>>(a);
   return launch_result();
 }

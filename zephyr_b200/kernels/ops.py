@@ -987,7 +987,7 @@ def heads_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.
     elif splits is None:
         keys = max(1, max_context if window <= 0 else min(max_context, window + keep_first))
         most = -(-keys // max(1, int(library().zb_heads_attention_tile_keys(nh, nkv, kd, vd)))) + 1
-        splits = max(1, min(most, _sm_count() // n_tiles))
+        splits = max(1, min(most, _sm_count() // n_tiles, 128))
     if splits > 1:
         scratch, _ = _decode_workspace(q.device, n_tiles * splits * nh * (vd + 2), 1)
     _check(library().zb_heads_attention(

@@ -74,7 +74,8 @@ struct PrefillArgs {
 
 // NS: stages of the ring of key/value tiles.  Two leave room for two CTAs an SM; three and four were measured
 // for tiles of one token (a decode step of 8 requests: 2.63 against 2.59 ms) and are not used.
-template <int HD, bool DEC, int NS>
+// DISTANT: with the distance bias (a form of its own, so that the others keep their registers).
+template <int HD, bool DEC, int NS, bool DISTANT>
 __global__ void __launch_bounds__(PRE_WARPS * 32, 1)
 paged_prefill_kernel(const PrefillArgs a) {
   static_assert(HD % 32 == 0 && HD <= 256, "head sizes that are multiples of 32, up to 256");
@@ -184,9 +185,8 @@ paged_prefill_kernel(const PrefillArgs a) {
   const int warp_seen_first = a.pool > 0 ? (warp_pos0 - a.window + 1) / a.pool : 0;      // what the warp's first row sees
 
   // The distance bias of this lane's two rows (in powers of two: r1 ln(x) log2(e) = r1 log2(x)).
-  const bool distant = a.bias_r1 != nullptr;
   float r1[2] = {0.0f, 0.0f}, r2[2] = {0.0f, 0.0f};
-  if (distant) {
+  if (DISTANT) {
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       const int row_head = DEC ? head + min(quad_row + 8 * h, g - 1) : head;
@@ -197,7 +197,7 @@ paged_prefill_kernel(const PrefillArgs a) {
   // A raw score of this lane's row h whose key lies at `pos`, scaled, bounded and biased.
   auto finished = [&](float raw, int h, int pos) {
     float v = a.softcap_log2 > 0.0f ? a.softcap_log2 * tanhf(raw * a.scale_over_cap) : raw * a.scale_log2;
-    if (distant) v = fmaf(-r1[h], __log2f(fmaf(r2[h], static_cast<float>(qpos[h] - pos), 1.0f)), v);
+    if (DISTANT) v = fmaf(-r1[h], __log2f(fmaf(r2[h], static_cast<float>(qpos[h] - pos), 1.0f)), v);
     return v;
   };
 
@@ -410,7 +410,9 @@ int prefill_launch(const PrefillArgs& a, int n_tiles, cudaStream_t stream, bool 
   constexpr int GROUP_STAGES = 2;
   const int stages = by_group ? GROUP_STAGES : 2;
   const size_t smem = (static_cast<size_t>(PRE_BM) + 2 * stages * PRE_BN) * (HD + 8) * sizeof(__nv_bfloat16);
-  auto kernel = by_group ? paged_prefill_kernel<HD, true, GROUP_STAGES> : paged_prefill_kernel<HD, false, 2>;
+  const bool distant = a.bias_r1 != nullptr;
+  auto kernel = by_group ? (distant ? paged_prefill_kernel<HD, true, GROUP_STAGES, true> : paged_prefill_kernel<HD, true, GROUP_STAGES, false>)
+                         : (distant ? paged_prefill_kernel<HD, false, 2, true> : paged_prefill_kernel<HD, false, 2, false>);
   if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess)
     return ERR_CUDA;
   const int across = by_group ? a.nkv : a.nh;

@@ -161,6 +161,8 @@ __device__ __forceinline__ void softmax_pass(unsigned tmem_row, unsigned (&words
   row_sum = (sum4[0] + sum4[1]) + (sum4[2] + sum4[3]);
 }
 
+// BIASED_SCORES: with the distance bias (a form of its own, so that the other keeps its registers).
+template <bool BIASED_SCORES>
 __global__ void __launch_bounds__(TC_THREADS, 1)
 paged_prefill_tc_kernel(const __grid_constant__ PrefillTcArgs a) {
   // Shared memory holds keys and values only (three stages of each, tiles of 32 KB on 1024-byte
@@ -444,7 +446,8 @@ paged_prefill_tc_kernel(const __grid_constant__ PrefillTcArgs a) {
     const unsigned tmem_o = tmem_base + lane_base + 2 * TC_BN;
     const int qp = ctx + q0 + r;
     float m_used = -INFINITY, l_run = 0.0f;
-    const bool capped = a.softcap_log2 > 0.0f, biased = a.bias_r1 != nullptr;
+    const bool capped = !BIASED_SCORES && a.softcap_log2 > 0.0f;
+    constexpr bool biased = BIASED_SCORES;
     const float r1 = biased ? a.bias_r1[head] : 0.0f, r2 = biased ? a.bias_r2[head] : 0.0f;
     bool failed = false;
     for (int j = 0; j < n_tiles; ++j) {
@@ -684,9 +687,10 @@ ZB_API int zb_paged_prefill_tc_masked(void* out, const void* q, const void* kv_c
   a.status = status;
   a.trace = prefill_tc_trace();
   const size_t smem = 2 * TC_STAGES * TC_TILE_BYTES;
-  if (cudaFuncSetAttribute(paged_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess)
+  auto kernel = bias_r1 != nullptr ? paged_prefill_tc_kernel<true> : paged_prefill_tc_kernel<false>;
+  if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess)
     return ERR_CUDA;
-  paged_prefill_tc_kernel<<<dim3(nh, n_tiles), TC_THREADS, smem, static_cast<cudaStream_t>(stream)>>>(a);
+  kernel<<<dim3(nh, n_tiles), TC_THREADS, smem, static_cast<cudaStream_t>(stream)>>>(a);
   return launch_result();
 }
 

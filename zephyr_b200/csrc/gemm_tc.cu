@@ -41,6 +41,7 @@ constexpr int GT_EPI_PLAIN = 0;
 constexpr int GT_EPI_GELU = 4;             // the sums through the tanh form of GELU
 constexpr int GT_EPI_RELU_GATE = 3;        // the interface's code for the gated epilogue with max(gate, 0) in SiLU's place
 constexpr int GT_EPI_SWIGLU = 1;           // columns 16 j .. 16 j + 7 are gates, 16 j + 8 .. 16 j + 15 their ups
+constexpr int GT_EPI_SWIGLU_SCALED = 5;    // the same, both sums of a row times its scale first (GateForm::row_scale)
 constexpr int GT_EPI_FLOAT = 2;            // the sums as they are, float32 (logits)
 constexpr int GT_A_BYTES = GT_BM * GT_BK * 2;
 constexpr int GT_STAGING_BYTES = 32 * 128;  // an epilogue warp's 32 rows x 64 output columns on their way out; two a warp
@@ -104,6 +105,8 @@ template <int N> __device__ __forceinline__ void bulk_wait_read() {
 }
 __device__ __forceinline__ void bulk_wait_all() { asm volatile("cp.async.bulk.wait_group 0;\n" ::: "memory"); }
 
+__host__ __device__ constexpr bool gt_gated(int epilogue) { return epilogue == GT_EPI_SWIGLU || epilogue == GT_EPI_SWIGLU_SCALED; }
+
 // An epilogue warp's 32 rows of a tile (its TMEM lanes, accumulator columns tmem_row .. + BN) -> y:
 // the sums are read 32 columns at a time, the epilogue applied in float32, and groups of 64 output
 // columns go through one of the warp's two staging buffers to a tiled store, which leaves out
@@ -113,14 +116,15 @@ __device__ __forceinline__ void write_out_rows(const CUtensorMap& y_map, unsigne
                                                unsigned char* staging, int& stores, int lane, const GateForm& form, int n_end) {
   // A group = 128 bytes of a row's output: 64 bfloat16 columns from two reads of 32 sums (four reads with
   // the activation, which halves them), or 32 float32 columns from one read.
-  constexpr int READS = EPI == GT_EPI_SWIGLU ? 4 : EPI == GT_EPI_FLOAT ? 1 : 2;
+  constexpr bool GATED = gt_gated(EPI);
+  constexpr int READS = GATED ? 4 : EPI == GT_EPI_FLOAT ? 1 : 2;
   constexpr int PIECES = 8 / READS;                                  // 16-byte pieces a read leaves
   constexpr int GROUP_COLUMNS = EPI == GT_EPI_FLOAT ? 32 : 64;       // output columns of a group
   // (rows of a grouped product are whole tiles, so every row has its scale)
-  const float scale = EPI == GT_EPI_SWIGLU && form.row_scale != nullptr ? __ldg(form.row_scale + row0 + lane) : 1.0f;
+  const float scale = EPI == GT_EPI_SWIGLU_SCALED ? __ldg(form.row_scale + row0 + lane) : 1.0f;
 #pragma unroll 1
   for (int group = 0; group < BN / (32 * READS); ++group) {
-    const int out_col = (EPI == GT_EPI_SWIGLU ? n0 / 2 : n0) + group * GROUP_COLUMNS;
+    const int out_col = (GATED ? n0 / 2 : n0) + group * GROUP_COLUMNS;
     if (out_col >= width) break;                // the same for the whole warp
     unsigned char* buffer = staging + (stores & 1) * GT_STAGING_BYTES;
     if (stores >= 2) {                          // the store before last has read this buffer
@@ -158,8 +162,12 @@ __device__ __forceinline__ void write_out_rows(const CUtensorMap& y_map, unsigne
           } else {
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
-              if (EPI == GT_EPI_SWIGLU) {
-                const float gate = __uint_as_float(v[16 * j + i]) * scale, up = __uint_as_float(v[16 * j + 8 + i]) * scale;
+              if (GATED) {
+                float gate = __uint_as_float(v[16 * j + i]), up = __uint_as_float(v[16 * j + 8 + i]);
+                if (EPI == GT_EPI_SWIGLU_SCALED) {
+                  gate *= scale;
+                  up *= scale;
+                }
                 o[i] = (form.kind == GATE_RELU ? fmaxf(gate, 0.0f) : silu_fast(gate)) * up;
               } else if (EPI == GT_EPI_GELU) {
                 o[i] = gelu_tanh_fast(__uint_as_float(v[8 * j + i]));
@@ -281,7 +289,7 @@ __global__ void __launch_bounds__(GT_THREADS, 1) gemm_tc_kernel(const __grid_con
   } else {
     const int quarter = warp & 3;                   // the TMEM lanes this warp may read: 32 quarter .. + 31
     unsigned char* staging = ring + Shape::STAGES * Shape::STAGE_BYTES + (warp - 2) * 2 * GT_STAGING_BYTES;
-    const int width = EPI == GT_EPI_SWIGLU ? a.N / 2 : a.N;
+    const int width = gt_gated(EPI) ? a.N / 2 : a.N;
     int acc = 0, stores = 0;
     unsigned acc_phase = 0;
     for (int tile = blockIdx.x; tile < a.tiles && !sh.failed; tile += gridDim.x) {
@@ -678,6 +686,8 @@ ZB_API int zb_gemm_tc_grouped(void* y, const void* x, const void* w, const int* 
   const bool wide = N >= 256;
   if (epilogue == GT_EPI_FLOAT)
     return wide ? gemm_tc_launch<256, GT_EPI_FLOAT>(a, w, sms, s) : gemm_tc_launch<128, GT_EPI_FLOAT>(a, w, sms, s);
+  if (epilogue == GT_EPI_SWIGLU && row_scale != nullptr)
+    return wide ? gemm_tc_launch<256, GT_EPI_SWIGLU_SCALED>(a, w, sms, s) : gemm_tc_launch<128, GT_EPI_SWIGLU_SCALED>(a, w, sms, s);
   if (epilogue == GT_EPI_SWIGLU)
     return wide ? gemm_tc_launch<256, GT_EPI_SWIGLU>(a, w, sms, s) : gemm_tc_launch<128, GT_EPI_SWIGLU>(a, w, sms, s);
   return wide ? gemm_tc_launch<256, GT_EPI_PLAIN>(a, w, sms, s) : gemm_tc_launch<128, GT_EPI_PLAIN>(a, w, sms, s);

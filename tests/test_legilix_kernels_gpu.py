@@ -360,18 +360,18 @@ def test_gelu_far_from_zero_and_in_every_form(cuda_device):
     from zephyr_b200.kernels import ops
 
     z = torch.cat([torch.linspace(-12.0, 12.0, 1001), torch.tensor([-1e4, 1e4, 0.0])])
-    got = ops.gelu_rows(z.to(cuda_device)).cpu().double()
+    got = ops.act_rows(z.to(cuda_device), "gelu_tanh").cpu().double()
     assert (got - gelu_tanh(z.double())).abs().max() < 2e-6 and float(got[-3]) == 0.0 and float(got[-2]) == 1e4
-    rounded = ops.gelu_rows(z.to(cuda_device), torch.bfloat16).cpu().double()
+    rounded = ops.act_rows(z.to(cuda_device), "gelu_tanh", torch.bfloat16).cpu().double()
     assert ((rounded - gelu_tanh(z.double())).abs() <= 2.0 ** -8 * gelu_tanh(z.double()).abs() + 1e-6).all()
     g = torch.Generator().manual_seed(1)
     w = (torch.randn(304, 64, generator=g) * 0.4).to(torch.bfloat16)
     x = torch.randn(600, 64, generator=g).to(torch.bfloat16)
     expected = gelu_tanh(x.double() @ w.double().T)
     for block_n in (0, 2, 128, 256):
-        y = ops.gemm_tc(x.to(cuda_device), w.to(cuda_device), gelu=True, block_n=block_n).cpu().double()
+        y = ops.gemm_tc(x.to(cuda_device), w.to(cuda_device), product_act="gelu_tanh", block_n=block_n).cpu().double()
         assert ((y - expected).abs() <= 2.0 ** -8 * expected.abs() + 2e-5).all()
-    y = ops.gemm_small(x[:9].to(cuda_device), w.to(cuda_device), gelu=True).cpu().double()
+    y = ops.gemm_small(x[:9].to(cuda_device), w.to(cuda_device), product_act="gelu_tanh").cpu().double()
     assert ((y - expected[:9]).abs() <= 2.0 ** -8 * expected[:9].abs() + 2e-5).all()
 
 

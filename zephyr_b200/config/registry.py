@@ -23,6 +23,7 @@ from .legilix import LegilixConfig
 from .qwen3 import Qwen3Config
 from .rizovik import RizovikConfig
 from .spec import ModelSpec
+from .tedulorn import TedulornConfig
 
 
 @dataclass(frozen=True)
@@ -115,3 +116,4 @@ register_architecture(GefovikConfig.model_type, GefovikConfig.architecture, Gefo
 register_architecture(FekotarConfig.model_type, FekotarConfig.architecture, FekotarConfig)
 register_architecture(RizovikConfig.model_type, RizovikConfig.architecture, RizovikConfig)
 register_architecture(LegilixConfig.model_type, LegilixConfig.architecture, LegilixConfig)
+register_architecture(TedulornConfig.model_type, TedulornConfig.architecture, TedulornConfig)

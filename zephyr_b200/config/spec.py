@@ -58,6 +58,14 @@ class FeedForwardSpec:
 
 
 @dataclass(frozen=True)
+class SideSpec:
+    """What joins the stream behind a layer's mixer and feed-forward, made from the stream itself."""
+
+    kind: str          # key in parts.SIDES, e.g. "token_gate"
+    params: Mapping[str, Any]
+
+
+@dataclass(frozen=True)
 class LayerSpec:
     """One layer: which block arrangement, and the parts placed in it.
 
@@ -70,6 +78,7 @@ class LayerSpec:
     feed_forward: FeedForwardSpec | None      # None: a layer without a feed-forward (where the block allows it)
     norms: Mapping[str, NormSpec]
     block_params: Mapping[str, Any] = field(default_factory=dict)   # the arrangement's own constants
+    side: SideSpec | None = None      # for arrangements that take one (``Block.takes_side``)
 
 
 @dataclass(frozen=True)

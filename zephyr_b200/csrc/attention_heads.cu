@@ -5,7 +5,8 @@
 //   s_h(i, j) = scale q_h(i) . k_c(h)(j)              c(h) = h / (heads / kv_heads)
 //   s_h <- sum_g M[h, g] s_g                          `score_mix` [nh, nh], or nothing
 //   s_h <- s_h - r1_h ln(1 + r2_h (i - j))            `bias_r1`, `bias_r2` [nh], or nothing
-//   softmax over the keys in sight (a window that may keep the first `keep_first` tokens), then the values
+//   softmax over the keys in sight (a window that may keep the first `keep_first` tokens), exp(sink_h) joining its
+//   denominator where there are `sinks` [nh] (a key of that score with a value of zero), then the values
 //
 // The scores are float32 from the product to the softmax, the mixing included.
 //
@@ -49,6 +50,7 @@ struct HeadsAttentionArgs {
   const float* score_mix;        // null, or [nh, nh]
   const float* bias_r1;          // null, or [nh] each
   const float* bias_r2;
+  const float* sinks;            // null, or [nh]
   int splits;                    // > 1: every tile is one token, and its keys' tiles are shared by this many CTAs
   float* part_o;                 // [n_tiles, splits, nh, vd]
   float* part_ml;                // [n_tiles, splits, nh, 2]
@@ -254,8 +256,10 @@ __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1) heads_attention_kernel
   for (int i = 0; i < HPW; ++i)
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt) {
-      m_run[i][nt] = -INFINITY;
-      l_run[i][nt] = 0.0f;
+      // A sink is a key that every token sees first, in the first split.
+      const bool sink = a.sinks != nullptr && split == 0 && head0 + i < a.nh;
+      m_run[i][nt] = sink ? a.sinks[head0 + i] * 1.4426950408889634f : -INFINITY;
+      l_run[i][nt] = sink ? 1.0f : 0.0f;
 #pragma unroll
       for (int m = 0; m < DM; ++m) o[i][nt][m][0] = o[i][nt][m][1] = o[i][nt][m][2] = o[i][nt][m][3] = 0.0f;
     }
@@ -621,7 +625,7 @@ ZB_API int zb_heads_attention(void* out, const void* q, const void* kv_cache, co
                               int page_size, int num_pages, int num_rows, const int* tile_row, const int* tile_q0,
                               int n_tiles, const int* row_q_start, const int* row_q_len, const int* row_ctx, int nh,
                               int nkv, int kd, int vd, int window, int keep_first, float scale, const float* score_mix,
-                              const float* bias_r1, const float* bias_r2, int single, int splits, float* scratch,
+                              const float* bias_r1, const float* bias_r2, const float* sinks, int single, int splits, float* scratch,
                               int* status, void* stream) {
   if (n_tiles < 0 || page_size <= 0 || window < 0 || keep_first < 0 || splits <= 0 || splits > AH_MAX_SPLITS || (splits > 1 && (!single || scratch == nullptr)) ||
       (bias_r1 == nullptr) != (bias_r2 == nullptr) || reinterpret_cast<uintptr_t>(q) % 4 != 0 ||
@@ -643,7 +647,7 @@ ZB_API int zb_heads_attention(void* out, const void* q, const void* kv_cache, co
     if (page_size == (1 << shift)) a.page_shift = shift;
   a.nh = nh; a.nkv = nkv; a.kd = kd; a.vd = vd; a.window = window; a.keep_first = window > 0 ? keep_first : 0;
   a.scale_log2 = scale * 1.4426950408889634f;
-  a.score_mix = score_mix; a.bias_r1 = bias_r1; a.bias_r2 = bias_r2;
+  a.score_mix = score_mix; a.bias_r1 = bias_r1; a.bias_r2 = bias_r2; a.sinks = sinks;
   a.splits = splits;
   a.part_ml = scratch;                               // pairs of floats first: they stay on 8-byte boundaries
   a.part_o = scratch != nullptr ? scratch + static_cast<size_t>(n_tiles) * splits * nh * 2 : nullptr;

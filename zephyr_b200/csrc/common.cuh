@@ -87,7 +87,17 @@ __device__ __forceinline__ float bounded_gate(float g, float u, const GateForm& 
   return g * s * (u + f.shift);
 }
 
-// What an ungated feed-forward's product may do to its sums: the tanh form of GELU,
+// What an ungated feed-forward's product may do to its sums.
+constexpr int ACT_NONE = 0;
+constexpr int ACT_GELU = 1;
+constexpr int ACT_RELU2 = 2;        // max(z, 0)^2
+
+__device__ __forceinline__ float relu_squared(float z) {
+  z = fmaxf(z, 0.0f);
+  return z * z;
+}
+
+// The tanh form of GELU,
 // 0.5 z (1 + tanh(u)) with u = sqrt(2 / pi) (z + 0.044715 z^3), as z / (1 + e^(-2u)).
 __device__ __forceinline__ float gelu_tanh(float z) {
   const float u = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);

@@ -10,7 +10,7 @@
 //
 // One CTA owns 16 rows of W; its four warps split K, and for matrices with few rows a cluster of
 // up to 8 CTAs splits K further.  Partial sums meet in (distributed) shared memory and are added in
-// a fixed order, so the result does not depend on timing.  GELU takes each sum through the tanh form.  With SWIGLU the 16 rows are 8 gate
+// a fixed order, so the result does not depend on timing.  ACT takes each sum through GELU's tanh form or a squared ReLU.  With SWIGLU the 16 rows are 8 gate
 // rows followed by their 8 up rows, and the epilogue writes silu(gate) * up: the activation costs
 // no extra pass over memory (reference: src/layer/mlp.cpp:29-36, src/layer/activation.cu:31-33).
 #include <cooperative_groups.h>
@@ -46,7 +46,7 @@ template <> __device__ __forceinline__ void store_out<__nv_bfloat16>(__nv_bfloat
   *p = __float2bfloat16_rn(v);
 }
 
-template <int MT, typename TOut, bool SWIGLU, bool GELU>
+template <int MT, typename TOut, bool SWIGLU, int ACT>
 __global__ void __launch_bounds__(GS_WARPS * 32)
 gemm_small_kernel(const SmallGemmArgs a) {
   // Partial sums of this CTA's warps: [warp][mt][row][token].
@@ -146,14 +146,14 @@ gemm_small_kernel(const SmallGemmArgs a) {
           for (int w = 0; w < GS_WARPS; ++w) sum += parts[c][w * PER_WARP + e];
         const int token = mt * 8 + tok;
         if (token < a.M && n0 + r < a.N)
-          store_out<TOut>(y + static_cast<size_t>(token) * a.ldy + n0 + r, GELU ? gelu_tanh(sum) : sum);
+          store_out<TOut>(y + static_cast<size_t>(token) * a.ldy + n0 + r, ACT == ACT_GELU ? gelu_tanh(sum) : ACT == ACT_RELU2 ? relu_squared(sum) : sum);
       }
     }
   }
   if (ksplit > 1) cluster.sync();           // nobody leaves while its shared memory may still be read
 }
 
-template <int MT, typename TOut, bool SWIGLU, bool GELU>
+template <int MT, typename TOut, bool SWIGLU, int ACT>
 int small_gemm_launch(const SmallGemmArgs& a, int ksplit, cudaStream_t stream) {
   cudaLaunchConfig_t config = {};
   config.gridDim = dim3((a.N + GS_ROWS - 1) / GS_ROWS, ksplit, 1);
@@ -167,17 +167,17 @@ int small_gemm_launch(const SmallGemmArgs& a, int ksplit, cudaStream_t stream) {
   attribute[0].val.clusterDim.z = 1;
   config.attrs = attribute;
   config.numAttrs = 1;
-  if (cudaLaunchKernelEx(&config, gemm_small_kernel<MT, TOut, SWIGLU, GELU>, a) != cudaSuccess) return ERR_CUDA;
+  if (cudaLaunchKernelEx(&config, gemm_small_kernel<MT, TOut, SWIGLU, ACT>, a) != cudaSuccess) return ERR_CUDA;
   return launch_result();
 }
 
-template <typename TOut, bool SWIGLU, bool GELU>
+template <typename TOut, bool SWIGLU, int ACT>
 int small_gemm_dispatch(const SmallGemmArgs& a, int ksplit, cudaStream_t stream) {
   switch ((a.M + 7) / 8) {
-    case 1: return small_gemm_launch<1, TOut, SWIGLU, GELU>(a, ksplit, stream);
-    case 2: return small_gemm_launch<2, TOut, SWIGLU, GELU>(a, ksplit, stream);
-    case 3: case 4: return small_gemm_launch<4, TOut, SWIGLU, GELU>(a, ksplit, stream);
-    default: return small_gemm_launch<8, TOut, SWIGLU, GELU>(a, ksplit, stream);
+    case 1: return small_gemm_launch<1, TOut, SWIGLU, ACT>(a, ksplit, stream);
+    case 2: return small_gemm_launch<2, TOut, SWIGLU, ACT>(a, ksplit, stream);
+    case 3: case 4: return small_gemm_launch<4, TOut, SWIGLU, ACT>(a, ksplit, stream);
+    default: return small_gemm_launch<8, TOut, SWIGLU, ACT>(a, ksplit, stream);
   }
 }
 
@@ -206,7 +206,7 @@ ZB_API int zb_gemm_small_ksplit(int N, int K) {
 // out_dtype: bfloat16 or float32.
 static int small_gemm(void* y, const void* x, const void* w, int M, int N, int K, long long ldx, long long ldw,
                       long long ldy, int out_dtype, bool gated, const GateForm& gate, void* stream,
-                      bool gelu = false) {
+                      int act = ACT_NONE) {
   if (!zb_gemm_small_supported(M, N, K)) return ERR_UNSUPPORTED;
   if (ldx < K || ldw < K || ldx % 8 != 0 || ldw % 8 != 0 || reinterpret_cast<uintptr_t>(x) % 16 != 0 ||
       reinterpret_cast<uintptr_t>(w) % 16 != 0 || (gated && N % 16 != 0))
@@ -219,14 +219,17 @@ static int small_gemm(void* y, const void* x, const void* w, int M, int N, int K
   a.gate = gate;
   const int ksplit = zb_gemm_small_ksplit(N, K);
   auto s = static_cast<cudaStream_t>(stream);
-  if (gelu)
-    return out_dtype == DTYPE_F32 ? small_gemm_dispatch<float, false, true>(a, ksplit, s)
-                                  : small_gemm_dispatch<__nv_bfloat16, false, true>(a, ksplit, s);
+  if (act == ACT_GELU)
+    return out_dtype == DTYPE_F32 ? small_gemm_dispatch<float, false, ACT_GELU>(a, ksplit, s)
+                                  : small_gemm_dispatch<__nv_bfloat16, false, ACT_GELU>(a, ksplit, s);
+  if (act == ACT_RELU2)
+    return out_dtype == DTYPE_F32 ? small_gemm_dispatch<float, false, ACT_RELU2>(a, ksplit, s)
+                                  : small_gemm_dispatch<__nv_bfloat16, false, ACT_RELU2>(a, ksplit, s);
   if (gated)
-    return out_dtype == DTYPE_F32 ? small_gemm_dispatch<float, true, false>(a, ksplit, s)
-                                  : small_gemm_dispatch<__nv_bfloat16, true, false>(a, ksplit, s);
-  return out_dtype == DTYPE_F32 ? small_gemm_dispatch<float, false, false>(a, ksplit, s)
-                                : small_gemm_dispatch<__nv_bfloat16, false, false>(a, ksplit, s);
+    return out_dtype == DTYPE_F32 ? small_gemm_dispatch<float, true, ACT_NONE>(a, ksplit, s)
+                                  : small_gemm_dispatch<__nv_bfloat16, true, ACT_NONE>(a, ksplit, s);
+  return out_dtype == DTYPE_F32 ? small_gemm_dispatch<float, false, ACT_NONE>(a, ksplit, s)
+                                : small_gemm_dispatch<__nv_bfloat16, false, ACT_NONE>(a, ksplit, s);
 }
 
 ZB_API int zb_gemm_small(void* y, const void* x, const void* w, int M, int N, int K, long long ldx, long long ldw,
@@ -235,10 +238,11 @@ ZB_API int zb_gemm_small(void* y, const void* x, const void* w, int M, int N, in
                     plain_gate(swiglu == 2 ? GATE_RELU : GATE_SILU), stream);
 }
 
-// y = gelu_tanh(x w^T).
-ZB_API int zb_gemm_small_gelu(void* y, const void* x, const void* w, int M, int N, int K, long long ldx, long long ldw,
-                              long long ldy, int out_dtype, void* stream) {
-  return small_gemm(y, x, w, M, N, K, ldx, ldw, ldy, out_dtype, false, plain_gate(GATE_SILU), stream, true);
+// y = act(x w^T); act: 1 gelu_tanh, 2 the square of max(., 0).
+ZB_API int zb_gemm_small_act(void* y, const void* x, const void* w, int M, int N, int K, long long ldx, long long ldw,
+                             long long ldy, int out_dtype, int act, void* stream) {
+  if (act != ACT_GELU && act != ACT_RELU2) return ERR_BAD_ARGUMENT;
+  return small_gemm(y, x, w, M, N, K, ldx, ldw, ldy, out_dtype, false, plain_gate(GATE_SILU), stream, act);
 }
 
 // The gated form with the bounded gate: y[:, 8j + r] from the sums of w's rows 16j + r (gate) and 16j + 8 + r

@@ -42,6 +42,8 @@ constexpr int GT_EPI_GELU = 4;             // the sums through the tanh form of 
 constexpr int GT_EPI_RELU_GATE = 3;        // the interface's code for the gated epilogue with max(gate, 0) in SiLU's place
 constexpr int GT_EPI_SWIGLU = 1;           // columns 16 j .. 16 j + 7 are gates, 16 j + 8 .. 16 j + 15 their ups
 constexpr int GT_EPI_SWIGLU_SCALED = 5;    // the same, both sums of a row times its scale first (GateForm::row_scale)
+constexpr int GT_EPI_RELU2 = 6;            // the square of max(sum, 0)
+constexpr int GT_EPI_BOUNDED_GATE = 7;     // the interface's code for the gated epilogue with the bounded gate (grouped products)
 constexpr int GT_EPI_FLOAT = 2;            // the sums as they are, float32 (logits)
 constexpr int GT_A_BYTES = GT_BM * GT_BK * 2;
 constexpr int GT_STAGING_BYTES = 32 * 128;  // an epilogue warp's 32 rows x 64 output columns on their way out; two a warp
@@ -171,6 +173,8 @@ __device__ __forceinline__ void write_out_rows(const CUtensorMap& y_map, unsigne
                 o[i] = (form.kind == GATE_RELU ? fmaxf(gate, 0.0f) : silu_fast(gate)) * up;
               } else if (EPI == GT_EPI_GELU) {
                 o[i] = gelu_tanh_fast(__uint_as_float(v[8 * j + i]));
+              } else if (EPI == GT_EPI_RELU2) {
+                o[i] = relu_squared(__uint_as_float(v[8 * j + i]));
               } else {
                 o[i] = __uint_as_float(v[8 * j + i]);
               }
@@ -584,16 +588,17 @@ using namespace zb;
 
 // 1 if zb_gemm_tc takes these sizes (x [M, K] with ldx elements between rows, w [N, K], y with ldy).
 ZB_API int zb_gemm_tc_supported(int M, int N, int K, long long ldx, int ldy, int epilogue) {
-  if (epilogue == GT_EPI_RELU_GATE) epilogue = GT_EPI_SWIGLU;
+  if (epilogue == GT_EPI_RELU_GATE || epilogue == GT_EPI_BOUNDED_GATE) epilogue = GT_EPI_SWIGLU;
   if (M <= 0 || N <= 0 || K <= 0 || K % 8 != 0 || ldx % 8 != 0 || ldx < K || (epilogue != GT_EPI_FLOAT && ldy % 8 != 0)) return 0;
   if (epilogue == GT_EPI_SWIGLU) return N % 16 == 0 && ldy >= N / 2;
   if (epilogue == GT_EPI_FLOAT) return ldy % 4 == 0 && ldy >= N;          // ldy counts float32 elements then
-  return (epilogue == GT_EPI_PLAIN || epilogue == GT_EPI_GELU) && ldy >= N;
+  return (epilogue == GT_EPI_PLAIN || epilogue == GT_EPI_GELU || epilogue == GT_EPI_RELU2) && ldy >= N;
 }
 
 // y = epilogue(x w^T), x and w bfloat16.  epilogue 0: y [M, N] bfloat16; 2: the same in float32;
 // 1: y [M, N / 2] = silu(gate) * up for w's rows in
-// blocks of 8 gate rows and their 8 up rows; 3: the same with max(gate, 0) * up; 4: y [M, N] bfloat16 = gelu_tanh of the sums.  block_n is 256 or 128, or 2 for tiles of 256 x 256 on pairs of
+// blocks of 8 gate rows and their 8 up rows; 3: the same with max(gate, 0) * up; 4: y [M, N] bfloat16 = gelu_tanh of the sums; 6: the square of
+// max(sum, 0).  block_n is 256 or 128, or 2 for tiles of 256 x 256 on pairs of
 // SMs (0: chosen from the sizes).
 static int gemm_tc_run(void* y, const void* x, const void* w, int M, int N, int K, long long ldx, int ldy, int epilogue,
                        const GateForm& gate, int block_n, int* status, void* stream) {
@@ -625,9 +630,12 @@ static int gemm_tc_run(void* y, const void* x, const void* w, int M, int N, int 
   if (block_n == GT_PAIR)
     return epilogue == GT_EPI_SWIGLU ? gemm_tc_pair_launch<GT_EPI_SWIGLU>(a, w, sms, s)
            : epilogue == GT_EPI_FLOAT ? gemm_tc_pair_launch<GT_EPI_FLOAT>(a, w, sms, s)
-           : epilogue == GT_EPI_GELU ? gemm_tc_pair_launch<GT_EPI_GELU>(a, w, sms, s) : gemm_tc_pair_launch<GT_EPI_PLAIN>(a, w, sms, s);
+           : epilogue == GT_EPI_GELU ? gemm_tc_pair_launch<GT_EPI_GELU>(a, w, sms, s)
+           : epilogue == GT_EPI_RELU2 ? gemm_tc_pair_launch<GT_EPI_RELU2>(a, w, sms, s) : gemm_tc_pair_launch<GT_EPI_PLAIN>(a, w, sms, s);
   if (epilogue == GT_EPI_GELU)
     return block_n == 256 ? gemm_tc_launch<256, GT_EPI_GELU>(a, w, sms, s) : gemm_tc_launch<128, GT_EPI_GELU>(a, w, sms, s);
+  if (epilogue == GT_EPI_RELU2)
+    return block_n == 256 ? gemm_tc_launch<256, GT_EPI_RELU2>(a, w, sms, s) : gemm_tc_launch<128, GT_EPI_RELU2>(a, w, sms, s);
   if (epilogue == GT_EPI_FLOAT)
     return block_n == 256 ? gemm_tc_launch<256, GT_EPI_FLOAT>(a, w, sms, s) : gemm_tc_launch<128, GT_EPI_FLOAT>(a, w, sms, s);
   if (epilogue == GT_EPI_SWIGLU)
@@ -656,16 +664,20 @@ ZB_API int zb_gemm_tc_bounded(void* y, const void* x, const void* w, const float
 // The same over several matrices stacked in w ([groups * N, K]): x [tiles_m * 128, K] is cut into tiles of
 // 128 rows, and tile i multiplies with matrix tile_group[i] (a device array; a negative entry leaves the
 // tile out, its rows of y unwritten).  Rows sorted by expert and padded to whole tiles make a routed
-// feed-forward's products one launch.  Tiles of one SM; epilogues as zb_gemm_tc (not 4).  `row_scale`: null, or one
-// float32 per row of x that goes on both sums of the gated epilogue.
+// feed-forward's products one launch.  Tiles of one SM; epilogues as zb_gemm_tc (not 4 and
+// 6), and 7: the gated one with the bounded gate (`limit`, `alpha`, `shift`; no biases).  `row_scale`: null, or one float32
+// per row of x that goes on both sums of the gated epilogue (1 and 3).
 ZB_API int zb_gemm_tc_grouped(void* y, const void* x, const void* w, const int* tile_group, int tiles_m, int groups,
-                              int N, int K, long long ldx, int ldy, int epilogue, const float* row_scale, int* status,
-                              void* stream) {
-  if (tiles_m <= 0 || groups <= 0 || tile_group == nullptr || epilogue == GT_EPI_GELU) return ERR_BAD_ARGUMENT;
+                              int N, int K, long long ldx, int ldy, int epilogue, const float* row_scale, float limit,
+                              float alpha, float shift, int* status, void* stream) {
+  if (tiles_m <= 0 || groups <= 0 || tile_group == nullptr || epilogue == GT_EPI_GELU || epilogue == GT_EPI_RELU2)
+    return ERR_BAD_ARGUMENT;
+  const bool bounded = epilogue == GT_EPI_BOUNDED_GATE;
+  if (bounded && (row_scale != nullptr || !(limit > 0.0f))) return ERR_BAD_ARGUMENT;
   const int M = tiles_m * GT_BM;
   if (!zb_gemm_tc_supported(M, N, K, ldx, ldy, epilogue)) return ERR_UNSUPPORTED;
   const int relu_gate = epilogue == GT_EPI_RELU_GATE;
-  if (relu_gate) epilogue = GT_EPI_SWIGLU;
+  if (relu_gate || bounded) epilogue = GT_EPI_SWIGLU;
   if (reinterpret_cast<uintptr_t>(y) % 16 != 0 || reinterpret_cast<uintptr_t>(x) % 16 != 0 ||
       reinterpret_cast<uintptr_t>(w) % 16 != 0)
     return ERR_BAD_ARGUMENT;
@@ -675,7 +687,7 @@ ZB_API int zb_gemm_tc_grouped(void* y, const void* x, const void* w, const int* 
     return ERR_CUDA;
   GemmTcArgs a;
   a.M = M; a.N = N; a.K = K;
-  a.gate = plain_gate(relu_gate ? GATE_RELU : GATE_SILU);
+  a.gate = bounded ? GateForm{GATE_BOUNDED, nullptr, limit, alpha, shift, nullptr} : plain_gate(relu_gate ? GATE_RELU : GATE_SILU);
   a.gate.row_scale = row_scale;
   a.tile_group = tile_group;
   a.groups = groups;

@@ -6,9 +6,11 @@
 //   * the causal convolution over a few taps per channel with its SiLU, whose last taps - 1 inputs
 //     live in the request's state slot;
 //   * the decayed outer-product recurrence  S_t = diag(a_t) S_{t-1} + k_t v_t^T,  o_t = S_t^T q_t
-//     per head, S [D, V] float32 in the request's state slot, in two settings: a decay per key channel
+//     per head, S [D, V] float32 in the request's state slot, in three settings: a decay per key channel
 //     a = sigmoid(z)^(1/tau) (gated linear attention), and one decay per head a = exp(-exp(A) dt)
-//     with k = dt B, q = C and a skip term D x (the state-space form of Mamba-2);
+//     with k = dt B, q = C and a skip term D x (the state-space form of Mamba-2), and a constant decay per
+//     head (retention; long portions of it run on tensor cores, retention.cu);
+//   * the rotation of halves on the q and k heads of a fused projection, k with a multiplier;
 //   * the RMS norm over equal groups of a row with a SiLU gate before or behind it.
 //
 // Everything that enters the recurrence is float32: decays, their logarithms, softplus, step sizes,
@@ -397,6 +399,7 @@ constexpr int SCAN_V_REGS = SCAN_CHUNK * SCAN_COLS / 64;   // values a thread fe
 
 constexpr int SCAN_GATED = 0;        // a[d] given per key channel (made from the logits by gated_decay_kernel), q scaled
 constexpr int SCAN_STATE_SPACE = 1;  // a = exp(-exp(A_log[h]) dt), k = dt B, q = C, o += skip[h] v, dt = softplus(. + dt_bias[h])
+constexpr int SCAN_FIXED = 2;        // a = decay[h], the same for every token
 
 struct ScanArgs {
   const void* q; long long q_stride;   // [tokens, .]: head h (or its group) at column h * D
@@ -405,6 +408,7 @@ struct ScanArgs {
   const float* z; long long z_stride;  // gated: decays [tokens, H * D], float32
   const void* dt; long long dt_stride; // state space: [tokens, H]
   const void* dt_bias; const void* a_log; const void* skip;   // state space: [H] each
+  const float* decay;                  // fixed: [H]
   int w_dtype;
   float* state; long long slot_stride; // slot s at state + s * slot_stride: [H][D][V]
   float* out;                          // [tokens, H * V] float32
@@ -502,6 +506,7 @@ __global__ void __launch_bounds__(512) decayed_state_scan_kernel(const ScanArgs 
   const T* vp = static_cast<const T*>(a.v);
   const int qk_col = (MODE == SCAN_STATE_SPACE ? h / a.heads_per_group : h) * D;
   float head_decay = 0.0f, head_dt_bias = 0.0f, head_skip = 0.0f;
+  if (MODE == SCAN_FIXED) head_decay = a.decay[h];
   if (MODE == SCAN_STATE_SPACE) {
     head_decay = -expf(load_scale(a.a_log, a.w_dtype, h));
     head_dt_bias = load_scale(a.dt_bias, a.w_dtype, h);
@@ -563,6 +568,9 @@ __global__ void __launch_bounds__(512) decayed_state_scan_kernel(const ScanArgs 
         a_s[e] = pa[j];
         k_s[e] = to_float(pk[j]);
         q_s[e] = to_float(pq[j]) * a.q_scale;
+      } else if (MODE == SCAN_FIXED) {
+        k_s[e] = to_float(pk[j]);
+        q_s[e] = to_float(pq[j]) * a.q_scale;
       } else {
         a_s[e] = t < nc ? step_s[SCAN_CHUNK + t] : 0.0f;
         k_s[e] = t < nc ? to_float(pk[j]) * step_s[t] : 0.0f;
@@ -584,7 +592,8 @@ __global__ void __launch_bounds__(512) decayed_state_scan_kernel(const ScanArgs 
       float o0 = 0.0f, o1 = 0.0f, o2 = 0.0f, o3 = 0.0f, p0 = 0.0f, p1 = 0.0f, p2 = 0.0f, p3 = 0.0f;
 #pragma unroll
       for (int d4 = 0; d4 < SCAN_ROWS / 4; ++d4) {
-        const float4 av = at[d4], kv = kt[d4], qv = qt[d4];
+        const float4 av = MODE == SCAN_FIXED ? make_float4(head_decay, head_decay, head_decay, head_decay) : at[d4];
+        const float4 kv = kt[d4], qv = qt[d4];
         const int d = 4 * d4;
         S[d] = fmaf(av.x, S[d], kv.x * vt);
         S[d + 1] = fmaf(av.y, S[d + 1], kv.y * vt);
@@ -640,6 +649,35 @@ __global__ void __launch_bounds__(512) decayed_state_scan_kernel(const ScanArgs 
       if (d0 + d < D && col < V) state[static_cast<long long>(d0 + d) * V + col] = S[d];
       if (d0 + d < D && col2 < V) state[static_cast<long long>(d0 + d) * V + col2] = S2[d];
     }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// From a fused projection (float32 rows: q heads, then k heads) to rotated queries and keys: value i of the first
+// `rot_dims` values of a head turns with value i + rot_dims / 2 by position * freqs[i] (float32 products); k times
+// `k_scale` behind the rotation.  One CTA a token, which works its angles out once for all heads.
+__global__ void __launch_bounds__(256) rotate_qk_kernel(float* out, const float* x, long long stride, const float* freqs, int rot_dims,
+                                                        float k_scale, const int* positions, int heads, int dim) {
+  extern __shared__ float2 turn_s[];                        // [rot_dims / 2]: cosine, sine
+  const long long t = blockIdx.x;
+  const int half = rot_dims / 2, cols = heads * dim;
+  const float pos = static_cast<float>(positions[t]);
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float s, c;
+    sincosf(pos * freqs[i], &s, &c);
+    turn_s[i] = make_float2(c, s);
+  }
+  __syncthreads();
+  const float* src = x + t * stride;
+  float* dst = out + t * 2 * cols;
+  for (int e = threadIdx.x; e < 2 * cols; e += blockDim.x) {
+    const int i = e % dim;
+    float y = src[e];
+    if (i < rot_dims) {
+      const float2 cs = turn_s[i < half ? i : i - half];
+      y = i < half ? y * cs.x - src[e + half] * cs.y : y * cs.x + src[e - half] * cs.y;
+    }
+    dst[e] = e < cols ? y : y * k_scale;
   }
 }
 
@@ -885,7 +923,8 @@ ZB_API int zb_state_scan_max_channels() { return 16 * SCAN_ROWS; }
 ZB_API int zb_decayed_state_scan(float* out, const void* q, long long q_stride, const void* k, long long k_stride,
                                  const void* v, long long v_stride, float* z, long long z_stride,
                                  const void* z_bias, const void* dt, long long dt_stride, const void* dt_bias,
-                                 const void* a_log, const void* skip, int w_dtype, float* state, long long slot_stride,
+                                 const void* a_log, const void* skip, const float* decay, int w_dtype, float* state,
+                                 long long slot_stride,
                                  const int* slots, const int* row_q_start, const int* row_q_len, int rows, int tokens,
                                  int H, int D, int V, int heads_per_group, int num_slots, int write_state,
                                  float q_scale, float inv_tau, int mode, int dtype, int seg_len, float* ws_state,
@@ -894,7 +933,7 @@ ZB_API int zb_decayed_state_scan(float* out, const void* q, long long q_stride, 
       (seg_len > 0 && (ws_state == nullptr || ws_decay == nullptr)))
     return ERR_BAD_ARGUMENT;
   if (D > 16 * SCAN_ROWS) return ERR_UNSUPPORTED;
-  if (mode != SCAN_GATED && mode != SCAN_STATE_SPACE) return ERR_BAD_ARGUMENT;
+  if (mode < SCAN_GATED || mode > SCAN_FIXED || (mode == SCAN_FIXED && decay == nullptr)) return ERR_BAD_ARGUMENT;
   if (rows == 0 || tokens == 0) return OK;
   auto s = static_cast<cudaStream_t>(stream);
   if (mode == SCAN_GATED) {
@@ -905,6 +944,7 @@ ZB_API int zb_decayed_state_scan(float* out, const void* q, long long q_stride, 
   ScanArgs a;
   a.q = q; a.q_stride = q_stride; a.k = k; a.k_stride = k_stride; a.v = v; a.v_stride = v_stride;
   a.z = z; a.z_stride = z_stride; a.dt = dt; a.dt_stride = dt_stride; a.dt_bias = dt_bias;
+  a.decay = decay;
   a.a_log = a_log; a.skip = skip; a.w_dtype = w_dtype; a.state = state; a.slot_stride = slot_stride; a.out = out;
   a.slots = slots; a.row_q_start = row_q_start; a.row_q_len = row_q_len; a.H = H; a.D = D; a.V = V;
   a.heads_per_group = heads_per_group; a.num_slots = num_slots; a.write_state = write_state; a.q_scale = q_scale;
@@ -931,11 +971,27 @@ ZB_API int zb_decayed_state_scan(float* out, const void* q, long long q_stride, 
     kernel<<<grid, warps * 32, smem, s>>>(a);                                                                  \
   }
   if (dtype == DTYPE_F32) {
-    if (mode == SCAN_GATED) ZB_SCAN(float, SCAN_GATED) else ZB_SCAN(float, SCAN_STATE_SPACE)
+    if (mode == SCAN_GATED) ZB_SCAN(float, SCAN_GATED)
+    else if (mode == SCAN_FIXED) ZB_SCAN(float, SCAN_FIXED)
+    else ZB_SCAN(float, SCAN_STATE_SPACE)
   } else {
-    if (mode == SCAN_GATED) ZB_SCAN(__nv_bfloat16, SCAN_GATED) else ZB_SCAN(__nv_bfloat16, SCAN_STATE_SPACE)
+    if (mode == SCAN_GATED) ZB_SCAN(__nv_bfloat16, SCAN_GATED)
+    else if (mode == SCAN_FIXED) ZB_SCAN(__nv_bfloat16, SCAN_FIXED)
+    else ZB_SCAN(__nv_bfloat16, SCAN_STATE_SPACE)
   }
 #undef ZB_SCAN
+  return launch_result();
+}
+
+// out [T, 2 heads * dim] float32 = the rotated q and k heads of x's rows (float32, `stride` apart), k times k_scale.
+ZB_API int zb_rotate_qk(float* out, const float* x, long long stride, const float* freqs, int rot_dims, float k_scale,
+                        const int* positions, int tokens, int heads, int dim, void* stream) {
+  if (tokens < 0 || heads <= 0 || dim <= 0 || rot_dims < 0 || rot_dims > dim || rot_dims % 2 != 0 || stride < 2LL * heads * dim ||
+      (rot_dims > 0 && freqs == nullptr) || rot_dims > 4096)
+    return ERR_BAD_ARGUMENT;
+  if (tokens == 0) return OK;
+  rotate_qk_kernel<<<tokens, 256, sizeof(float2) * (rot_dims / 2 + 1), static_cast<cudaStream_t>(stream)>>>(
+      out, x, stride, freqs, rot_dims, k_scale, positions, heads, dim);
   return launch_result();
 }
 

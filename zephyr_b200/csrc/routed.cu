@@ -37,14 +37,15 @@ constexpr int ROUTE_WARPS = 4;
 // outputs of the `keep` groups with the largest marks can be taken; ties: the lower group); and a
 // multiplier on the weights (`weight_scale`); a bias on the logits (`logit_bias`, part of the logit for the
 // choice and for the weight alike); and scores that are the logits themselves (`score_kind` 2): the `top`
-// largest logits are taken and weigh their outputs by the softmax over the taken logits only.
+// largest logits are taken and weigh their outputs by the softmax over the taken logits only.  `normalize`: the
+// weights of a token's taken outputs are divided by their sum (+ 1e-20) ahead of the multiplier.
 constexpr int ROUTE_GROUP_TOP_MAX = 4;
 constexpr int SCORES_SOFTMAX = 0, SCORES_SIGMOID = 1, SCORES_TOP_SOFTMAX = 2;
 
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 route_kernel(int* ids, float* weights, const float* logits, long long logits_stride, const float* correction,
              int tokens, int outputs, int top, int score_kind, int groups, int keep, int group_top,
-             float weight_scale, const float* logit_bias) {
+             float weight_scale, const float* logit_bias, int normalize) {
   __shared__ float choice_of[ROUTE_WARPS][32 * ROUTE_PER_LANE];
   __shared__ float mark_of[ROUTE_WARPS][32 * ROUTE_PER_LANE];
   const int warp = threadIdx.x >> 5;
@@ -163,7 +164,7 @@ route_kernel(int* ids, float* weights, const float* logits, long long logits_str
     w = __shfl_sync(0xffffffffu, w, best_e & 31);
     if (lane == 0) {
       ids[static_cast<size_t>(t) * top + j] = best_e;
-      weights[static_cast<size_t>(t) * top + j] = score_kind == SCORES_TOP_SOFTMAX ? w : w * weight_scale;
+      weights[static_cast<size_t>(t) * top + j] = (score_kind == SCORES_TOP_SOFTMAX || normalize) ? w : w * weight_scale;
     }
   }
   if (score_kind == SCORES_TOP_SOFTMAX && lane == 0) {
@@ -176,6 +177,11 @@ route_kernel(int* ids, float* weights, const float* logits, long long logits_str
       sum += w[j];
     }
     for (int j = 0; j < top; ++j) w[j] = w[j] / sum * weight_scale;
+  } else if (normalize && lane == 0) {
+    float* w = weights + static_cast<size_t>(t) * top;
+    float sum = 0.0f;
+    for (int j = 0; j < top; ++j) sum += w[j];
+    for (int j = 0; j < top; ++j) w[j] = w[j] / (sum + 1e-20f) * weight_scale;
   }
 }
 
@@ -287,6 +293,7 @@ struct ExpertProductArgs {
   long long x_stride;
   int N, K, top, act;
   const float* weights;    // null, or per slot what both sums of the gate/up product are multiplied by
+  float limit, alpha, shift;   // the bounded gate's constants (act 2)
   int interleaved;         // gate/up: w0 is [experts, 2 N, K], blocks of 8 gate rows each followed by its 8 up rows
 };
 
@@ -309,8 +316,10 @@ __device__ __forceinline__ float expert_act(float g, int act) {
 
 // What a gate sum and its up sum become.  Without weights on the inputs both are rounded to the model's type
 // before the activation, as separate products would leave them.
+// The bounded gate (act 2) takes the unrounded sums, as the products' epilogues do.
 template <typename T>
 __device__ __forceinline__ float gated_value(float gate, float up, float scale, const ExpertProductArgs& a) {
+  if (a.act == 2) return bounded_gate<false>(gate, up, GateForm{GATE_BOUNDED, nullptr, a.limit, a.alpha, a.shift, nullptr});
   if (a.weights != nullptr) return expert_act(scale * gate, a.act) * (scale * up);
   return expert_act(to_float(from_float<T>(gate)), a.act) * to_float(from_float<T>(up));
 }
@@ -503,7 +512,8 @@ ZB_API int zb_expert_tile_rows(int dtype) { return dtype == DTYPE_F32 ? TP_BM : 
 // `group_top` largest choice values) can be taken from: keep * (outputs / groups) must reach `top`.
 ZB_API int zb_route_biased(int* ids, float* weights, const float* logits, long long logits_stride,
                            const float* correction, int tokens, int outputs, int top, int sigmoid_scores, int groups,
-                           int keep, int group_top, float weight_scale, const float* logit_bias, void* stream) {
+                           int keep, int group_top, float weight_scale, const float* logit_bias, int normalize,
+                           void* stream) {
   if (tokens < 0 || outputs <= 0 || top <= 0 || top > outputs || sigmoid_scores < 0 || sigmoid_scores > 2)
     return ERR_BAD_ARGUMENT;
   if (groups > 1 && (outputs % groups != 0 || keep <= 0 || keep > groups || group_top <= 0 ||
@@ -513,7 +523,7 @@ ZB_API int zb_route_biased(int* ids, float* weights, const float* logits, long l
   if (tokens == 0) return OK;
   route_kernel<<<(tokens + ROUTE_WARPS - 1) / ROUTE_WARPS, ROUTE_WARPS * 32, 0, static_cast<cudaStream_t>(stream)>>>(
       ids, weights, logits, logits_stride, correction, tokens, outputs, top, sigmoid_scores, groups, keep, group_top,
-      weight_scale, logit_bias);
+      weight_scale, logit_bias, normalize);
   return launch_result();
 }
 
@@ -521,7 +531,7 @@ ZB_API int zb_route_grouped(int* ids, float* weights, const float* logits, long 
                             const float* correction, int tokens, int outputs, int top, int sigmoid_scores, int groups,
                             int keep, int group_top, float weight_scale, void* stream) {
   return zb_route_biased(ids, weights, logits, logits_stride, correction, tokens, outputs, top, sigmoid_scores, groups,
-                         keep, group_top, weight_scale, nullptr, stream);
+                         keep, group_top, weight_scale, nullptr, 0, stream);
 }
 
 ZB_API int zb_route(int* ids, float* weights, const float* logits, long long logits_stride, const float* correction,
@@ -542,17 +552,22 @@ ZB_API int zb_route_align(int* plan, int* slots, int* place_of_slot, const int* 
 
 // `down` = 0: hidden = act(gate x) * (up x), N = ff, K = width; 1: y = down hidden, N = width, K = ff.
 // `input_weights` (gate/up only; null: none): one float32 per slot that goes on both sums ahead of the activation.
+// act: 0 SiLU, 1 ReLU, 2 the bounded gate with `limit`, `alpha` and `shift` (no input weights).
 // Without w1 the gate/up product reads w0 as [experts, 2 N, K] in blocks of 8 gate rows and their 8 up rows.
 ZB_API int zb_expert_product(void* out, const void* x, long long x_stride, const void* w0, const void* w1,
                              const int* plan, const int* slots, const float* input_weights, int max_tiles, int N,
-                             int K, int top, int act, int down, int dtype, void* stream) {
-  if ((down && input_weights != nullptr) || max_tiles < 0 || N <= 0 || K <= 0 || top <= 0 || (act != 0 && act != 1)) return ERR_BAD_ARGUMENT;
+                             int K, int top, int act, float limit, float alpha, float shift, int down, int dtype,
+                             void* stream) {
+  if ((down && input_weights != nullptr) || max_tiles < 0 || N <= 0 || K <= 0 || top <= 0 || act < 0 || act > 2 ||
+      (act == 2 && (input_weights != nullptr || !(limit > 0.0f))))
+    return ERR_BAD_ARGUMENT;
   if (!down && w1 == nullptr && N % 8 != 0) return ERR_BAD_ARGUMENT;
   if (max_tiles == 0) return OK;
   ExpertProductArgs a;
   a.out = out; a.x = x; a.w0 = w0; a.w1 = w1; a.plan = plan; a.slots = slots; a.x_stride = x_stride;
   a.N = N; a.K = K; a.top = top; a.act = act;
   a.weights = input_weights;
+  a.limit = limit; a.alpha = alpha; a.shift = shift;
   a.interleaved = !down && w1 == nullptr;
   const dim3 grid(max_tiles, (N + TP_BN - 1) / TP_BN);       // both tile forms are 64 outputs wide
   static_assert(TP_BN == TM_BN, "one grid for both forms");

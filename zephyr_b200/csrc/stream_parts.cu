@@ -8,12 +8,14 @@
 //   sum + RMS norm          x += (a + b) in float32 (either summand may be absent), then
 //                           y = x / sqrt(mean(x^2) + eps) * w in the model's type; also the plain norm of
 //                           float32 rows that are a slice of wider rows; and the norm in groups, where each
-//                           of several equal consecutive parts of a row has a mean square of its own.
+//                           of several equal consecutive parts of a row has a mean square of its own; and the sum
+//                           alone with its rounding (no scale: what a part that reads the stream itself takes).
 //   clamped gate            g = min(G + b_g, limit), u = clamp(U + b_u, -limit, limit),
 //                           y = g * sigmoid(alpha * g) * (u + shift), from a float32 or bfloat16 product.
 //   scale                   y *= s on float32 rows (a multiplier on logits).
-//   activation              y = gelu(x), element by element (an ungated feed-forward whose product has no
-//                           epilogue for it).
+//   activation              y = gelu(x) or max(x, 0)^2, element by element (an ungated feed-forward whose product
+//                           has no epilogue for it).
+//   token gate              y[t, i] = gelu(z[t, i]) * E[id_t, offset + i]: a gate on part of the token's row of a table.
 #include "common.cuh"
 
 #include <algorithm>
@@ -147,15 +149,16 @@ sum_rms_norm_kernel(OUT* out, long long out_stride, float* x, long long x_stride
     ss += v * v;
   }
   if (out == nullptr) return;
-  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(H) + eps);
+  const float inv = w != nullptr ? 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(H) + eps) : 1.0f;
   OUT* o = out + r * out_stride + g0;
+  auto scale = [&](int i) { return w != nullptr ? load_scale(w, w_dtype, g0 + i) : 1.0f; };
 #pragma unroll
   for (int k = 0; k < SN_PER; ++k) {
     const int i = threadIdx.x + k * threads;
-    if (i < H) o[i] = from_float<OUT>(keep[k] * inv * load_scale(w, w_dtype, g0 + i));
+    if (i < H) o[i] = from_float<OUT>(keep[k] * inv * scale(i));
   }
   for (int i = threadIdx.x + SN_PER * threads; i < H; i += threads)
-    o[i] = from_float<OUT>(xr[i] * inv * load_scale(w, w_dtype, g0 + i));
+    o[i] = from_float<OUT>(xr[i] * inv * scale(i));
 }
 
 // The same with four values a thread and step: H a multiple of 4, every row and base aligned for that.
@@ -187,6 +190,7 @@ sum_rms_norm_vec_kernel(OUT* out, long long out_stride, float* x, long long x_st
     return v;
   };
   auto scaled = [&](float4 v, float inv, int i) {
+    if (w == nullptr) return v;
     const float4 s = w_dtype == DTYPE_F32 ? load4(static_cast<const float*>(w) + g0 + i)
                                           : load4(static_cast<const __nv_bfloat16*>(w) + g0 + i);
     return make_float4(v.x * inv * s.x, v.y * inv * s.y, v.z * inv * s.z, v.w * inv * s.w);
@@ -205,7 +209,7 @@ sum_rms_norm_vec_kernel(OUT* out, long long out_stride, float* x, long long x_st
     ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
   }
   if (out == nullptr) return;
-  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(H) + eps);
+  const float inv = w != nullptr ? 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(H) + eps) : 1.0f;
   OUT* o = out + r * out_stride + g0;
 #pragma unroll
   for (int k = 0; k < PER; ++k) {
@@ -285,21 +289,36 @@ __global__ void scale_rows_kernel(float* y, long long total, float scale) {
     y[at] *= scale;
 }
 
-template <typename IN, typename OUT>
-__global__ void __launch_bounds__(256) gelu_rows_kernel(OUT* out, const IN* x, long long total) {
+template <int ACT> __device__ __forceinline__ float act_value(float z) { return ACT == ACT_GELU ? gelu_tanh(z) : relu_squared(z); }
+
+template <int ACT, typename IN, typename OUT>
+__global__ void __launch_bounds__(256) act_rows_kernel(OUT* out, const IN* x, long long total) {
   for (long long at = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; at < total;
        at += static_cast<long long>(gridDim.x) * blockDim.x)
-    out[at] = from_float<OUT>(gelu_tanh(to_float(x[at])));
+    out[at] = from_float<OUT>(act_value<ACT>(to_float(x[at])));
 }
 
 // The same four values at a time.
-template <typename IN, typename OUT>
-__global__ void __launch_bounds__(256) gelu_rows_vec_kernel(OUT* out, const IN* x, long long total4) {
+template <int ACT, typename IN, typename OUT>
+__global__ void __launch_bounds__(256) act_rows_vec_kernel(OUT* out, const IN* x, long long total4) {
   for (long long at = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; at < total4;
        at += static_cast<long long>(gridDim.x) * blockDim.x) {
     const float4 v = load4(x + 4 * at);
-    store4(out + 4 * at, make_float4(gelu_tanh(v.x), gelu_tanh(v.y), gelu_tanh(v.z), gelu_tanh(v.w)));
+    store4(out + 4 * at, make_float4(act_value<ACT>(v.x), act_value<ACT>(v.y), act_value<ACT>(v.z), act_value<ACT>(v.w)));
   }
+}
+
+// out[t, i] = gelu_tanh(z[t, i]) * table[ids[t], offset + i], i < dim.
+template <typename IN, typename T>
+__global__ void __launch_bounds__(128) token_gate_kernel(T* out, const IN* z, long long z_stride, const T* table, long long table_stride,
+                                                         const int* ids, int dim, int vocab, int* status) {
+  const long long t = blockIdx.x;
+  const int id = ids[t];
+  const bool ok = id >= 0 && id < vocab;
+  if (!ok && threadIdx.x == 0) report(status, STATUS_TOKEN_OUT_OF_RANGE, id, static_cast<int>(t));
+  const T* e = table + static_cast<long long>(ok ? id : 0) * table_stride;
+  for (int i = threadIdx.x; i < dim; i += blockDim.x)
+    out[t * dim + i] = from_float<T>(ok ? gelu_tanh(to_float(z[t * z_stride + i])) * to_float(e[i]) : 0.0f);
 }
 
 inline int grid_for(long long total, int threads) {
@@ -351,11 +370,11 @@ ZB_API int zb_store_last_token(int* last_token, const int* ids, const int* row_q
 // x [rows, H] float32 (rows x_stride apart) += (a + b + bias), a and b contiguous [rows, H] of their own types
 // or null, bias float32 [H] (a shift of one of the summands, added to every row; only beside a summand) or
 // null; then, unless out is null, out [rows, H] (rows out_stride apart) = rmsnorm(x) * w, each of `groups` equal
-// consecutive parts of a row divided by its own root mean square.
+// consecutive parts of a row divided by its own root mean square; or, without w, x itself.
 ZB_API int zb_sum_rms_norm(void* out, long long out_stride, int out_dtype, float* x, long long x_stride, const void* a,
                            int a_dtype, const void* b, int b_dtype, const float* bias, const void* w, int w_dtype,
                            float eps, int rows, int H, int groups, void* stream) {
-  if (groups <= 0 || groups > 65535 || rows < 0 || H <= 0 || H % groups != 0 || x_stride < H || (out != nullptr && (out_stride < H || w == nullptr)) ||
+  if (groups <= 0 || groups > 65535 || rows < 0 || H <= 0 || H % groups != 0 || x_stride < H || (out != nullptr && out_stride < H) ||
       (bias != nullptr && a == nullptr && b == nullptr))
     return ERR_BAD_ARGUMENT;
   if (rows == 0) return OK;
@@ -434,22 +453,51 @@ ZB_API int zb_scale_rows(float* y, long long total, float scale, void* stream) {
   return launch_result();
 }
 
-// out [total] = gelu_tanh(x [total]) in float32, rounded once; both contiguous.
-ZB_API int zb_gelu_rows(void* out, int out_dtype, const void* x, int in_dtype, long long total, void* stream) {
-  if (total < 0 || (out_dtype == DTYPE_F32 && in_dtype != DTYPE_F32)) return ERR_BAD_ARGUMENT;
+// out [T, dim] (contiguous) = gelu_tanh(z) * the values offset .. offset + dim of the tokens' rows of `table`
+// [vocab, table_stride], in float32, rounded once to the table's type; z may be float32 whatever that is.
+ZB_API int zb_token_gate(void* out, const void* z, long long z_stride, int z_dtype, const void* table, long long table_stride,
+                         int offset, const int* ids, int T, int dim, int vocab, int dtype, int* status, void* stream) {
+  if (T < 0 || dim <= 0 || vocab <= 0 || offset < 0 || offset + dim > table_stride || z_stride < dim ||
+      (dtype == DTYPE_F32 && z_dtype != DTYPE_F32))
+    return ERR_BAD_ARGUMENT;
+  if (T == 0) return OK;
+  auto s = static_cast<cudaStream_t>(stream);
+  using bf16 = __nv_bfloat16;
+  const int threads = dim >= 128 ? 128 : (dim + 31) / 32 * 32;
+  if (dtype == DTYPE_F32)
+    token_gate_kernel<float, float><<<T, threads, 0, s>>>((float*)out, (const float*)z, z_stride, (const float*)table + offset,
+                                                          table_stride, ids, dim, vocab, status);
+  else if (z_dtype == DTYPE_F32)
+    token_gate_kernel<float, bf16><<<T, threads, 0, s>>>((bf16*)out, (const float*)z, z_stride, (const bf16*)table + offset,
+                                                         table_stride, ids, dim, vocab, status);
+  else
+    token_gate_kernel<bf16, bf16><<<T, threads, 0, s>>>((bf16*)out, (const bf16*)z, z_stride, (const bf16*)table + offset,
+                                                        table_stride, ids, dim, vocab, status);
+  return launch_result();
+}
+
+// out [total] = act(x [total]) in float32, rounded once; both contiguous.  act: 1 gelu_tanh, 2 the square of max(., 0).
+ZB_API int zb_act_rows(void* out, int out_dtype, const void* x, int in_dtype, long long total, int act, void* stream) {
+  if ((act != ACT_GELU && act != ACT_RELU2) || total < 0 || (out_dtype == DTYPE_F32 && in_dtype != DTYPE_F32)) return ERR_BAD_ARGUMENT;
   if (total == 0) return OK;
   auto s = static_cast<cudaStream_t>(stream);
   using bf16 = __nv_bfloat16;
-#define ZB_GELU(IN, OUT)                                                                                       \
+#define ZB_ACT2(ACT, IN, OUT)                                                                                       \
   {                                                                                                            \
     if (total % 4 == 0 && aligned_for4<IN>(x) && aligned_for4<OUT>(out))                                       \
-      gelu_rows_vec_kernel<IN, OUT><<<grid_for(total / 4, 256), 256, 0, s>>>((OUT*)out, (const IN*)x, total / 4); \
+      act_rows_vec_kernel<ACT, IN, OUT><<<grid_for(total / 4, 256), 256, 0, s>>>((OUT*)out, (const IN*)x, total / 4); \
     else                                                                                                       \
-      gelu_rows_kernel<IN, OUT><<<grid_for(total, 256), 256, 0, s>>>((OUT*)out, (const IN*)x, total);          \
+      act_rows_kernel<ACT, IN, OUT><<<grid_for(total, 256), 256, 0, s>>>((OUT*)out, (const IN*)x, total);          \
   }
-  if (out_dtype == DTYPE_F32) ZB_GELU(float, float)
-  else if (in_dtype == DTYPE_F32) ZB_GELU(float, bf16)
-  else ZB_GELU(bf16, bf16)
-#undef ZB_GELU
+#define ZB_ACT(IN, OUT)                                \
+  {                                                    \
+    if (act == ACT_GELU) ZB_ACT2(ACT_GELU, IN, OUT)    \
+    else ZB_ACT2(ACT_RELU2, IN, OUT)                   \
+  }
+  if (out_dtype == DTYPE_F32) ZB_ACT(float, float)
+  else if (in_dtype == DTYPE_F32) ZB_ACT(float, bf16)
+  else ZB_ACT(bf16, bf16)
+#undef ZB_ACT
+#undef ZB_ACT2
   return launch_result();
 }

@@ -7,7 +7,8 @@
 //                  the rotation of halves on the first `rot_dims` values of every q and k head: value i
 //                  pairs with value i + rot_dims / 2, (u, v) -> (u c - v s, v c + u s), c, s = cos, sin of
 //                  position * f_i (float32 products, f a table the host made);
-//                  optionally every value head divided by its root mean square (no scales);
+//                  optionally every value head divided by its root mean square (no scales), or the values mixed
+//                  with another layer's values of the same token, v <- (1 - m) v + m v_first with m from the device;
 //                  and the write of k and v into the pages.  One CTA per token; everything in float32
 //                  with one rounding at the store.
 //   pool_blocks  entry b of a pooled store = the mean over positions b P .. b P + P - 1 of the keys and
@@ -41,6 +42,9 @@ struct QkvHalvesArgs {
   int rot_dims;
   float rot_mult;            // a multiplier on cosine and sine
   int value_unit_norm;
+  const float* v_first;      // null, or [T, v_first_stride]: what the values are mixed with
+  long long v_first_stride;
+  const float* v_share;      // its share, one float32
   const int* positions;
   const int* token_row;
   void* cache;               // null: only the queries are made
@@ -90,6 +94,7 @@ __global__ void __launch_bounds__(QH_THREADS) qkv_halves_kernel(const QkvHalvesA
   }
   const long long page_elems = static_cast<long long>(a.nkv) * a.page_size * (a.kd + a.vd);
   const int half = a.rot_dims / 2;
+  const float share = a.v_first != nullptr ? *a.v_share : 0.0f;
   for (int h = warp; h < heads; h += QH_WARPS) {
     const bool is_q = h < a.nh, is_v = h >= a.nh + kv_heads;
     const int dim = is_v ? a.vd : a.kd;
@@ -125,6 +130,8 @@ __global__ void __launch_bounds__(QH_THREADS) qkv_halves_kernel(const QkvHalvesA
     }
     for (int i = lane; i < dim; i += 32) {
       float y = row[i];
+      if (is_v && a.v_first != nullptr)
+        y = (1.0f - share) * y + share * a.v_first[static_cast<long long>(t) * a.v_first_stride + own * a.vd + i];
       if (!is_v && a.freqs != nullptr && i < a.rot_dims) {
         const int f = i < half ? i : i - half;
         float s, c;
@@ -292,7 +299,8 @@ using namespace zb;
 
 ZB_API int zb_qkv_halves(void* q_out, const void* qkv, long long stride, const float* bias, int norm_mode, const float* q_norm_w,
                          const float* k_norm_w, float eps, const float* freqs, int rot_dims, float rot_mult,
-                         int value_unit_norm, const int* positions, const int* token_row, void* cache,
+                         int value_unit_norm, const float* v_first, long long v_first_stride, const float* v_share,
+                         const int* positions, const int* token_row, void* cache,
                          const int* block_table, int max_blocks, int page_size, int num_pages, int num_rows,
                          int tokens, int nh, int nkv, int kd, int vd, int in_dtype, int dtype, int* status,
                          void* stream) {
@@ -301,8 +309,10 @@ ZB_API int zb_qkv_halves(void* q_out, const void* qkv, long long stride, const f
       ((q_norm_w == nullptr) != (k_norm_w == nullptr)))
     return ERR_BAD_ARGUMENT;
   if (dtype == DTYPE_F32 && in_dtype != DTYPE_F32) return ERR_BAD_ARGUMENT;
+  if (v_first != nullptr && (v_share == nullptr || v_first_stride < static_cast<long long>(nkv) * vd)) return ERR_BAD_ARGUMENT;
   if (tokens == 0) return OK;
   QkvHalvesArgs a;
+  a.v_first = v_first; a.v_first_stride = v_first_stride; a.v_share = v_share;
   a.q_out = q_out; a.qkv = qkv; a.stride = stride; a.bias = bias; a.norm_mode = norm_mode; a.q_norm_w = q_norm_w;
   a.k_norm_w = k_norm_w; a.eps = eps; a.freqs = freqs; a.rot_dims = freqs != nullptr ? rot_dims : 0;
   a.rot_mult = rot_mult; a.value_unit_norm = value_unit_norm; a.positions = positions; a.token_row = token_row;

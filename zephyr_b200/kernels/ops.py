@@ -67,7 +67,9 @@ _SIGNATURES = {
     "zb_store_last_token": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
     "zb_sum_rms_norm": [c_void_p, c_longlong, c_int, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_int, c_void_p,
                         c_void_p, c_int, c_float, c_int, c_int, c_int, c_void_p],
-    "zb_gelu_rows": [c_void_p, c_int, c_void_p, c_int, c_longlong, c_void_p],
+    "zb_act_rows": [c_void_p, c_int, c_void_p, c_int, c_longlong, c_int, c_void_p],
+    "zb_token_gate": [c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_int,
+                      c_void_p, c_void_p],
     "zb_clamped_gate": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float,
                         c_void_p],
     "zb_scale_rows": [c_void_p, c_longlong, c_float, c_void_p],
@@ -79,11 +81,11 @@ _SIGNATURES = {
     "zb_route": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_void_p],
     "zb_route_align": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "zb_expert_product": [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                          c_int, c_int, c_int, c_int, c_int, c_void_p],
+                          c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_int, c_void_p],
     "zb_route_align_padded": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "zb_gather_places": [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
     "zb_gemm_tc_grouped": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_longlong, c_int, c_int,
-                           c_void_p, c_void_p, c_void_p],
+                           c_void_p, c_float, c_float, c_float, c_void_p, c_void_p],
     "zb_route_combine": [c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int,
                          c_int, c_int, c_int, c_void_p],
     "zb_add_bias": [c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
@@ -103,9 +105,9 @@ _SIGNATURES = {
     "zb_heads_attention_tile_keys": [c_int, c_int, c_int, c_int],
     "zb_heads_attention": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
                            c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p,
-                           c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p],
+                           c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p],
     "zb_qkv_halves": [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_float,
-                      c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                      c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                       c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "zb_pool_blocks": [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int,
                        c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
@@ -121,7 +123,7 @@ _SIGNATURES = {
     "zb_residual_rms_norm": [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_float, c_float, c_int,
                              c_int, c_int, c_void_p],
     "zb_route_biased": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                        c_int, c_float, c_void_p, c_void_p],
+                        c_int, c_float, c_void_p, c_int, c_void_p],
     "zb_qkv_pairs": [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_void_p,
                      c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                      c_int, c_int, c_float, c_int, c_int, c_int, c_void_p, c_void_p],
@@ -134,9 +136,10 @@ _SIGNATURES = {
                             c_void_p],
     "zb_state_scan_max_channels": [],
     "zb_decayed_state_scan": [c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p,
-                              c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                              c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                               c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                               c_float, c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
+    "zb_rotate_qk": [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
     "zb_gated_group_rms_norm": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                 c_float, c_int, c_int, c_void_p],
     "zb_scaled_sum": [c_void_p, c_void_p, c_void_p, c_float, c_float, c_longlong, c_int, c_int, c_void_p],
@@ -179,8 +182,8 @@ _SIGNATURES = {
                            c_int, c_int, c_void_p, c_void_p],
     "zb_gemm_small_bounded": [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_float, c_int, c_int, c_int,
                               c_longlong, c_longlong, c_longlong, c_int, c_void_p],
-    "zb_gemm_small_gelu": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong, c_int,
-                           c_void_p],
+    "zb_gemm_small_act": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong, c_int, c_int,
+                          c_void_p],
     "zb_gemm_nt_simt": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong,
                         c_int, c_int, c_void_p],
     "zb_fused_chain_stage_supported": [c_int, c_int, c_int, c_int, c_int],
@@ -429,14 +432,33 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor | None = None, blocked: bo
     return out
 
 
-def gelu_rows(x: torch.Tensor, out_dtype: torch.dtype | None = None) -> torch.Tensor:
-    """The tanh form of GELU, 0.5 x (1 + tanh(sqrt(2 / pi) (x + 0.044715 x^3))), of a contiguous tensor, in float32
-    with one rounding."""
+PRODUCT_ACTS = {"gelu_tanh": 1, "relu_squared": 2}      # what an ungated product may do to its sums
+
+
+def act_rows(x: torch.Tensor, act: str, out_dtype: torch.dtype | None = None) -> torch.Tensor:
+    """The tanh form of GELU, 0.5 x (1 + tanh(sqrt(2 / pi) (x + 0.044715 x^3))), or max(x, 0)^2 ("relu_squared"), of a
+    contiguous tensor, in float32 with one rounding."""
+    _require(act in PRODUCT_ACTS, f"the activation is one of {sorted(PRODUCT_ACTS)}")
     _cuda(x)
     _require(x.is_contiguous() and x.dtype in DTYPE_CODE, "a contiguous float32 or bfloat16 tensor")
     out = torch.empty(x.shape, dtype=out_dtype or x.dtype, device=x.device)
-    _check(library().zb_gelu_rows(_ptr(out), DTYPE_CODE[out.dtype], _ptr(x), DTYPE_CODE[x.dtype], x.numel(), _stream()),
-           "gelu_rows")
+    _check(library().zb_act_rows(_ptr(out), DTYPE_CODE[out.dtype], _ptr(x), DTYPE_CODE[x.dtype], x.numel(), PRODUCT_ACTS[act],
+                                 _stream()), "act_rows")
+    return out
+
+
+def token_gate(z: torch.Tensor, table: torch.Tensor, offset: int, ids: torch.Tensor, status: torch.Tensor) -> torch.Tensor:
+    """gelu_tanh(z[t, i]) * table[ids[t], offset + i] for z [T, dim] (unit inner stride; float32 or the table's type) and a
+    table [vocab, >= offset + dim], in float32, rounded once to the table's type."""
+    _cuda(z, table, ids, status)
+    _i32(ids)
+    _require(z.dim() == 2 and z.stride(1) == 1 and z.dtype in (torch.float32, table.dtype) and ids.numel() == z.shape[0], "z: [T, dim]")
+    _require(table.dim() == 2 and table.stride(1) == 1 and table.dtype in DTYPE_CODE and 0 <= offset
+             and offset + z.shape[1] <= table.shape[1], "a table row holds the gate's values")
+    out = torch.empty(z.shape, dtype=table.dtype, device=z.device)
+    _check(library().zb_token_gate(_ptr(out), _ptr(z), z.stride(0), DTYPE_CODE[z.dtype], _ptr(table), table.stride(0), int(offset),
+                                   _ptr(ids), z.shape[0], z.shape[1], table.shape[0], DTYPE_CODE[table.dtype], _ptr(status),
+                                   _stream()), "token_gate")
     return out
 
 
@@ -548,12 +570,13 @@ def pair_embedding(table: torch.Tensor, pair_table: torch.Tensor, ctx_ids: torch
 
 def sum_rms_norm(x: torch.Tensor, a: torch.Tensor | None, b: torch.Tensor | None, w: torch.Tensor | None,
                  eps: float, out_dtype: torch.dtype | None = None, bias: torch.Tensor | None = None,
-                 groups: int = 1) -> torch.Tensor | None:
+                 groups: int = 1, rounded_sum: bool = False) -> torch.Tensor | None:
     """x (float32 [rows, H], unit inner stride, rows may be slices of wider rows) += (a + b + bias) in place,
     where a and b are contiguous [rows, H] summands of either type or None and ``bias`` is a float32 [H] shift
     of one of them (added to every row), or None; then, with a scale ``w``, returns
     x / sqrt(mean(x^2) + eps) * w in ``out_dtype``; with ``groups`` > 1 each of that many equal consecutive parts
-    of a row has a mean square of its own.  Statistics and sums are float32."""
+    of a row has a mean square of its own.  Without a scale and with ``rounded_sum`` it returns the sum itself in
+    ``out_dtype``.  Statistics and sums are float32."""
     _cuda(x, a, b, w, bias)
     _f32_vector(bias, x.shape[-1], "the shift")
     _require(bias is None or a is not None or b is not None, "a shift comes with a summand")
@@ -564,7 +587,7 @@ def sum_rms_norm(x: torch.Tensor, a: torch.Tensor | None, b: torch.Tensor | None
         _require(summand is None or (summand.shape == x.shape and summand.is_contiguous() and summand.dtype in DTYPE_CODE),
                  "summands are contiguous [rows, H]")
     out = None
-    if w is not None:
+    if w is not None or rounded_sum:
         out = torch.empty((rows, H), dtype=out_dtype or torch.float32, device=x.device)
     _check(library().zb_sum_rms_norm(_ptr(out), H, DTYPE_CODE[out.dtype] if out is not None else 0, _ptr(x), x.stride(0),
                                      _ptr(a), DTYPE_CODE[a.dtype] if a is not None else 0, _ptr(b),
@@ -676,7 +699,8 @@ def decayed_state_scan(mode: str, q: torch.Tensor, k: torch.Tensor, v: torch.Ten
                        row_q_len: torch.Tensor, status: torch.Tensor, *, decay_logits: torch.Tensor | None = None,
                        decay_bias: torch.Tensor | None = None, inv_tau: float = 1.0, q_scale: float = 1.0,
                        dt: torch.Tensor | None = None, dt_bias: torch.Tensor | None = None,
-                       a_log: torch.Tensor | None = None, skip: torch.Tensor | None = None, heads_per_group: int = 1,
+                       a_log: torch.Tensor | None = None, skip: torch.Tensor | None = None,
+                       decay: torch.Tensor | None = None, heads_per_group: int = 1,
                        write_state: bool = True, segment: int | None = None) -> torch.Tensor:
     """S_t = diag(a_t) S_{t-1} + k_t v_t^T, o_t = S_t^T q_t per head over each row's new tokens, from and
     to ``state`` [slots, heads * key_dim * value_dim] float32 (rows may be strided); returns o as float32
@@ -684,7 +708,8 @@ def decayed_state_scan(mode: str, q: torch.Tensor, k: torch.Tensor, v: torch.Ten
     ``mode`` "gated": a = sigmoid(decay_logits + decay_bias)^inv_tau per key channel (logits float32
     [T, heads * key_dim], overwritten with the decays), q times ``q_scale``.  ``mode`` "state_space": step = softplus(dt + dt_bias),
     a = exp(-exp(a_log) step) per head, k times step, o += skip * v; q and k belong to the head's group
-    (head // heads_per_group at column group * key_dim).
+    (head // heads_per_group at column group * key_dim).  ``mode`` "fixed": a = ``decay`` (float32 [heads]), q times
+    ``q_scale``.
     ``segment``: long requests are cut into segments of this many tokens that run side by side (a pass
     from zero states, a carry of the state from segment to segment, a pass with the outputs: twice the
     arithmetic on many times the threads); 0: never; None: chosen, for steps whose requests bring 256
@@ -699,12 +724,17 @@ def decayed_state_scan(mode: str, q: torch.Tensor, k: torch.Tensor, v: torch.Ten
     _require(state.dim() == 2 and state.dtype == torch.float32 and state.stride(1) == 1
              and state.shape[1] == heads * key_dim * value_dim, "state must be float32 [slots, heads * key_dim * value_dim]")
     gated = mode == "gated"
-    _require(gated or mode == "state_space", "mode is 'gated' or 'state_space'")
+    fixed = mode == "fixed"
+    _require(gated or fixed or mode == "state_space", "mode is 'gated', 'state_space' or 'fixed'")
     if gated:
         _require(decay_logits is not None and decay_logits.dtype == torch.float32 and decay_logits.dim() == 2
                  and decay_logits.stride(1) == 1 and decay_logits.shape == (T, heads * key_dim), "decay logits: float32 [T, heads * key_dim]")
         _f32_vector(decay_bias, heads * key_dim, "the decay bias")
         _require(decay_bias is not None, "the gated mode needs a decay bias")
+    elif fixed:
+        _cuda(decay)
+        _require(decay is not None, "the fixed mode needs decays")
+        _f32_vector(decay, heads, "the decays")
     else:
         _require(dt is not None and dt.dim() == 2 and dt.stride(1) == 1 and dt.shape[0] == T and dt.shape[1] >= heads
                  and dt.dtype == v.dtype, "dt must be [T, heads] of the model's type")
@@ -724,12 +754,29 @@ def decayed_state_scan(mode: str, q: torch.Tensor, k: torch.Tensor, v: torch.Ten
         ws_decay = torch.empty((pieces, heads * key_dim), dtype=torch.float32, device=v.device)
     _check(library().zb_decayed_state_scan(
         _ptr(out), _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(decay_logits),
-        decay_logits.stride(0) if gated else 0, _ptr(decay_bias), _ptr(dt), dt.stride(0) if not gated else 0,
-        _ptr(dt_bias), _ptr(a_log), _ptr(skip), 0, _ptr(state), state.stride(0), _ptr(slots), _ptr(row_q_start),
+        decay_logits.stride(0) if gated else 0, _ptr(decay_bias), _ptr(dt), dt.stride(0) if dt is not None else 0,
+        _ptr(dt_bias), _ptr(a_log), _ptr(skip), _ptr(decay), 0, _ptr(state), state.stride(0), _ptr(slots), _ptr(row_q_start),
         _ptr(row_q_len), slots.numel(), T, heads, key_dim, value_dim, int(heads_per_group), state.shape[0],
-        int(write_state), float(q_scale), float(inv_tau), 0 if gated else 1, DTYPE_CODE[v.dtype], int(segment),
+        int(write_state), float(q_scale), float(inv_tau), {"gated": 0, "state_space": 1, "fixed": 2}[mode], DTYPE_CODE[v.dtype], int(segment),
         _ptr(ws_state), _ptr(ws_decay), _ptr(status), _stream()), "decayed_state_scan",
         kernels=(2 if gated else 1) + (2 if segment else 0))
+    return out
+
+
+def rotate_qk(qk: torch.Tensor, heads: int, dim: int, freqs: torch.Tensor | None, rot_dims: int, k_scale: float,
+              positions: torch.Tensor) -> torch.Tensor:
+    """The q and k heads of a fused float32 projection ([T, >= 2 * heads * dim], unit inner stride, q first), value i of a
+    head's first ``rot_dims`` values turned with value i + rot_dims / 2 by position * freqs[i]; k times ``k_scale``
+    behind that.  Returns float32 [T, 2 * heads * dim]."""
+    _cuda(qk, freqs, positions)
+    _i32(positions)
+    _require(qk.dim() == 2 and qk.stride(1) == 1 and qk.dtype == torch.float32 and qk.shape[1] >= 2 * heads * dim
+             and positions.numel() == qk.shape[0], "float32 rows of q and k heads")
+    _require(rot_dims == 0 or freqs is not None, "a rotation needs frequencies")
+    _f32_vector(freqs, rot_dims // 2, "the frequencies")
+    out = torch.empty((qk.shape[0], 2 * heads * dim), dtype=torch.float32, device=qk.device)
+    _check(library().zb_rotate_qk(_ptr(out), _ptr(qk), qk.stride(0), _ptr(freqs), int(rot_dims), float(k_scale), _ptr(positions),
+                                  qk.shape[0], heads, dim, _stream()), "rotate_qk")
     return out
 
 
@@ -965,9 +1012,9 @@ def heads_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.
                     nh: int, nkv: int, kd: int, vd: int, window: int, scale: float, status: torch.Tensor,
                     out: torch.Tensor, keep_first: int = 0, score_mix: torch.Tensor | None = None,
                     distance_bias: tuple[torch.Tensor, torch.Tensor] | None = None, single: bool = False,
-                    max_context: int = 0, splits: int | None = None) -> torch.Tensor:
+                    max_context: int = 0, splits: int | None = None, sinks: torch.Tensor | None = None) -> torch.Tensor:
     """Tensor-core attention with all heads of a tile in one CTA, for layers that mix the heads' scores ahead
-    of the softmax (``score_mix``) and for keys and values of any two widths; ``keep_first``, ``score_mix`` and
+    of the softmax (``score_mix``) and for keys and values of any two widths; ``keep_first``, ``score_mix``, ``sinks`` and
     ``distance_bias`` as in ``paged_attention``.  Tiles hold ``heads_attention_tile_tokens`` tokens, or with
     ``single`` one token each, whose keys are then shared by ``splits`` CTAs (default: as many as fill the SMs,
     with ``max_context`` at least the longest context of the rows, the new token included).  Writes the tiles'
@@ -979,6 +1026,8 @@ def heads_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.
     _require(out.shape == (q.shape[0], nh * vd) and out.dtype == q.dtype and out.is_contiguous(), "out must be [T, heads * value_dim]")
     _require(score_mix is None or (score_mix.dtype == torch.float32 and score_mix.is_contiguous()
                                    and score_mix.shape == (nh, nh)), "score_mix: float32 [heads, heads]")
+    _cuda(sinks)
+    _f32_vector(sinks, nh, "sinks")
     pages, page_size = _cache_geometry(kv_cache, nkv, kd, vd, q.dtype)
     n_tiles = tile_row.numel()
     scratch = None
@@ -993,7 +1042,7 @@ def heads_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.
     _check(library().zb_heads_attention(
         _ptr(out), _ptr(q), _ptr(kv_cache), _ptr(block_table), block_table.shape[1], page_size, pages,
         block_table.shape[0], _ptr(tile_row), _ptr(tile_q0), n_tiles, _ptr(row_q_start), _ptr(row_q_len), _ptr(row_ctx),
-        nh, nkv, kd, vd, int(window), int(keep_first), float(scale), _ptr(score_mix), _ptr(r1), _ptr(r2), int(single),
+        nh, nkv, kd, vd, int(window), int(keep_first), float(scale), _ptr(score_mix), _ptr(r1), _ptr(r2), _ptr(sinks), int(single),
         int(splits), _ptr(scratch), _ptr(status), _stream()), "heads_attention", kernels=2 if splits > 1 else 1)
     return out
 
@@ -1005,13 +1054,16 @@ def qkv_halves(qkv: torch.Tensor, nh: int, nkv: int, kd: int, vd: int, norm: str
                k_norm_w: torch.Tensor | None, eps: float, freqs: torch.Tensor | None, rot_dims: int, rot_mult: float,
                value_unit_norm: bool, positions: torch.Tensor, token_row: torch.Tensor, kv_cache: torch.Tensor | None,
                block_table: torch.Tensor, status: torch.Tensor, dtype: torch.dtype,
-               bias: torch.Tensor | None = None) -> torch.Tensor:
+               bias: torch.Tensor | None = None, v_first: torch.Tensor | None = None,
+               v_share: torch.Tensor | None = None) -> torch.Tensor:
     """From a fused q/k/v projection to queries and cache entries, for a rotation of halves: a float32 bias on
     every column (``bias``, or None), an RMS norm of q and of k (``norm`` "per_head": per head, scales [kd] shared by the heads; "whole": one statistic over all
     heads of q and one over all heads of k, scales [nh * kd] and [nkv * kd]; "none"; scales may be None),
     the rotation of value i with value i + rot_dims / 2 by position * freqs[i] on the first ``rot_dims``
     values of every q and k head (cosine and sine times ``rot_mult``), every value head divided by its root
-    mean square (``value_unit_norm``), and the cache write of k and v.  Returns the queries [T, nh * kd] in
+    mean square (``value_unit_norm``), the values mixed with another layer's values of the same tokens,
+    v <- (1 - m) v + m v_first (``v_first`` float32 [T, nkv * vd], rows may be strided; ``v_share`` float32, m), and the
+    cache write of k and v.  Returns the queries [T, nh * kd] in
     ``dtype``; ``qkv`` may be float32 whatever ``dtype`` is.  Without ``kv_cache`` only the queries are made."""
     _cuda(qkv, q_norm_w, k_norm_w, freqs, positions, token_row, kv_cache, block_table, status, bias)
     _i32(positions, token_row, block_table)
@@ -1028,10 +1080,16 @@ def qkv_halves(qkv: torch.Tensor, nh: int, nkv: int, kd: int, vd: int, norm: str
     pages, page_size = (0, 1)
     if kv_cache is not None:
         pages, page_size = _cache_geometry(kv_cache, nkv, kd, vd, dtype)
+    if v_first is not None:
+        _cuda(v_first, v_share)
+        _f32_vector(v_share, 1, "the share")
+        _require(v_share is not None and v_first.dim() == 2 and v_first.dtype == torch.float32 and v_first.shape == (T, nkv * vd)
+                 and v_first.stride(1) == 1, "v_first: float32 [T, kv_heads * value_dim]")
     q_out = torch.empty((T, nh * kd), dtype=dtype, device=qkv.device)
     _check(library().zb_qkv_halves(
         _ptr(q_out), _ptr(qkv), qkv.stride(0), _ptr(bias), QK_NORMS[norm], _ptr(q_norm_w), _ptr(k_norm_w), float(eps), _ptr(freqs),
-        int(rot_dims), float(rot_mult), int(value_unit_norm), _ptr(positions), _ptr(token_row), _ptr(kv_cache),
+        int(rot_dims), float(rot_mult), int(value_unit_norm), _ptr(v_first), v_first.stride(0) if v_first is not None else 0,
+        _ptr(v_share), _ptr(positions), _ptr(token_row), _ptr(kv_cache),
         _ptr(block_table), block_table.shape[1], page_size, pages, block_table.shape[0], T, nh, nkv, kd, vd,
         DTYPE_CODE[qkv.dtype], DTYPE_CODE[dtype], _ptr(status), _stream()), "qkv_halves")
     return q_out
@@ -1480,11 +1538,11 @@ def _bounded_args(bounded: BoundedGate, rows: int) -> tuple:
 
 def gemm_small(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = None,
                swiglu: bool = False, act: str = "silu", bounded: BoundedGate | None = None,
-               gelu: bool = False) -> torch.Tensor:
+               product_act: str | None = None) -> torch.Tensor:
     """x [M <= 64, K] times w [N, K] transposed, bfloat16, float32 accumulation, weights read once.
     With ``swiglu`` the rows of w are blocks of 8 gate rows each followed by its 8 up rows, and the
-    result is silu(gate) * up, [M, N / 2]; with ``bounded`` as well, the bounded gate of those sums.  ``gelu``
-    (without ``swiglu``): the tanh form of GELU of the sums."""
+    result is silu(gate) * up, [M, N / 2]; with ``bounded`` as well, the bounded gate of those sums.
+    ``product_act`` (without ``swiglu``): one of ``PRODUCT_ACTS`` of the sums."""
     _cuda(x, w)
     _require(x.dim() == 2 and w.dim() == 2 and x.shape[1] == w.shape[1], "x [M, K] and w [N, K]")
     _require(gemm_small_supported(x, w), "gemm_small takes bfloat16, M <= 64, K a multiple of 8, 16-byte aligned rows")
@@ -1492,7 +1550,7 @@ def gemm_small(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None =
     M, K = x.shape
     N = w.shape[0]
     _require(not swiglu or N % 16 == 0, "swiglu needs a multiple of 16 rows")
-    _require(not (swiglu and gelu), "GELU is an epilogue of the ungated product")
+    _require(product_act is None or (not swiglu and product_act in PRODUCT_ACTS), f"an ungated product's epilogue is one of {sorted(PRODUCT_ACTS)}")
     out = torch.empty((M, N // 2 if swiglu else N), dtype=out_dtype, device=x.device)
     if bounded is not None:
         _require(swiglu, "the bounded gate is a gated epilogue")
@@ -1500,9 +1558,9 @@ def gemm_small(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None =
         _check(library().zb_gemm_small_bounded(_ptr(out), _ptr(x), _ptr(w), *_bounded_args(bounded, N), M, N, K, x.stride(0),
                                                w.stride(0), out.stride(0), DTYPE_CODE[out_dtype], _stream()), "gemm_small")
         return out
-    if gelu:
-        _check(library().zb_gemm_small_gelu(_ptr(out), _ptr(x), _ptr(w), M, N, K, x.stride(0), w.stride(0), out.stride(0),
-                                            DTYPE_CODE[out_dtype], _stream()), "gemm_small")
+    if product_act is not None:
+        _check(library().zb_gemm_small_act(_ptr(out), _ptr(x), _ptr(w), M, N, K, x.stride(0), w.stride(0), out.stride(0),
+                                           DTYPE_CODE[out_dtype], PRODUCT_ACTS[product_act], _stream()), "gemm_small")
         return out
     _check(library().zb_gemm_small(_ptr(out), _ptr(x), _ptr(w), M, N, K, x.stride(0), w.stride(0), out.stride(0),
                                    DTYPE_CODE[out_dtype], (2 if act == "relu" else 1) if swiglu else 0, _stream()),
@@ -1528,20 +1586,21 @@ def gemm_tc_supported(x: torch.Tensor, w: torch.Tensor, swiglu: bool = False) ->
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, swiglu: bool = False, block_n: int = 0,
             status: torch.Tensor | None = None, out_dtype: torch.dtype | None = None, act: str = "silu",
-            bounded: BoundedGate | None = None, gelu: bool = False) -> torch.Tensor:
+            bounded: BoundedGate | None = None, product_act: str | None = None) -> torch.Tensor:
     """x [M, K] times w [N, K] transposed on tcgen05 tensor cores, bfloat16 with float32 sums in
     tensor memory; the result in bfloat16, or with ``out_dtype=torch.float32`` the sums as they are.
     With ``swiglu`` the rows of w are blocks of 8 gate rows each followed by its 8 up
     rows, and the result is silu(gate) * up, [M, N / 2], taken from the float32 sums and rounded once
-    (with ``bounded`` as well: the bounded gate of those sums and their biases).  ``gelu``: the tanh form of GELU
-    of the float32 sums, rounded once.
+    (with ``bounded`` as well: the bounded gate of those sums and their biases).  ``product_act``: one of
+    ``PRODUCT_ACTS`` of the float32 sums, rounded once.
     ``block_n`` is the width of an output tile (256, 128; 2: tiles of 256 x 256 on pairs of SMs; 0: chosen).  ``status`` (default: the
     device's status word) receives a report if a wait inside the kernel ran out."""
     _cuda(x, w)
     _require(gemm_tc_supported(x, w, swiglu), "gemm_tc takes bfloat16 x [M, K] and contiguous w [N, K], K a multiple of 8, "
              "16-byte aligned; with swiglu N a multiple of 16")
     wide = out_dtype == torch.float32
-    _require(out_dtype in (None, torch.bfloat16, torch.float32) and not (wide and (swiglu or gelu)) and not (swiglu and gelu),
+    _require(product_act is None or product_act in PRODUCT_ACTS, f"a product's activation is one of {sorted(PRODUCT_ACTS)}")
+    _require(out_dtype in (None, torch.bfloat16, torch.float32) and not (wide and (swiglu or product_act)) and not (swiglu and product_act),
              "bfloat16 out, or float32 without an activation")
     M, K = x.shape
     N = w.shape[0]
@@ -1558,7 +1617,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, swiglu: bool = False, block_n: int
         return out if ldy == width else out[:, :width].contiguous()
     _require(act in ACTIVATIONS, f"the gate's activation is one of {sorted(ACTIVATIONS)}")
     gated = 3 if act == "relu" else 1         # the kernel's codes for the two gated epilogues
-    _check(library().zb_gemm_tc(_ptr(out), _ptr(x), _ptr(w), M, N, K, x.stride(0), ldy, 2 if wide else (gated if swiglu else (4 if gelu else 0)),
+    _check(library().zb_gemm_tc(_ptr(out), _ptr(x), _ptr(w), M, N, K, x.stride(0), ldy, 2 if wide else (gated if swiglu else {"gelu_tanh": 4, "relu_squared": 6}.get(product_act, 0)),
                                 int(block_n), _ptr(status), _stream()), "gemm_tc")
     return out if ldy == width else out[:, :width].contiguous()
 
@@ -1757,14 +1816,15 @@ ROUTE_SCORES = {"softmax": 0, "sigmoid": 1, "top_softmax": 2}
 
 def route(logits: torch.Tensor, correction: torch.Tensor | None, top: int, scores: str = "softmax",
           groups: tuple[int, int, int] | None = None, weight_scale: float = 1.0,
-          logit_bias: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
+          logit_bias: torch.Tensor | None = None, normalize: bool = False) -> tuple[torch.Tensor, torch.Tensor]:
     """Token-choice routing: s = softmax(logits) over all outputs (``scores`` "sigmoid": the logistic function
     of each logit on its own); the ``top`` outputs with the largest s + correction are taken (ties: the lower
     index), each with the weight s * ``weight_scale``.  ``groups`` = (count, keep, group_top): the outputs
     form ``count`` equal runs of neighbours, a run's mark is the sum of its ``group_top`` largest choice
     values, and only outputs of the ``keep`` runs with the largest marks can be taken.  ``logit_bias``
     (float32 [outputs]) is added to the logits before anything else.  ``scores`` "top_softmax": the ``top``
-    largest logits are taken and weigh their outputs by the softmax over the taken logits only.  Returns
+    largest logits are taken and weigh their outputs by the softmax over the taken logits only.  ``normalize``: a
+    token's weights are divided by their sum (+ 1e-20) ahead of ``weight_scale``.  Returns
     (ids int32 [T, top], weights float32 [T, top]), in the order of choice."""
     _cuda(logits, correction, logit_bias)
     _f32_vector(logit_bias, logits.shape[1], "the logits' bias")
@@ -1777,7 +1837,7 @@ def route(logits: torch.Tensor, correction: torch.Tensor | None, top: int, score
     weights = torch.empty((T, top), dtype=torch.float32, device=logits.device)
     _check(library().zb_route_biased(_ptr(ids), _ptr(weights), _ptr(logits), logits.stride(0), _ptr(correction), T,
                                      outputs, int(top), ROUTE_SCORES[scores], count, keep, group_top,
-                                     float(weight_scale), _ptr(logit_bias), _stream()), "route")
+                                     float(weight_scale), _ptr(logit_bias), int(normalize), _stream()), "route")
     return ids, weights
 
 
@@ -1795,14 +1855,15 @@ def interleave_gate_up(w_gate: torch.Tensor, w_up: torch.Tensor) -> torch.Tensor
 
 def routed_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate: torch.Tensor,
                    w_up: torch.Tensor | None, w_down: torch.Tensor, act: str = "silu",
-                   weigh_inputs: bool = False) -> torch.Tensor:
+                   weigh_inputs: bool = False, bounded: BoundedGate | None = None) -> torch.Tensor:
     """sum_j weights[t, j] * expert_{ids[t, j]}(x[t]) for x [T, width]: expert e < E is
     w_down[e] (act(w_gate[e] x) * (w_up[e] x)) with w_gate, w_up [E, ff, width] and w_down [E, width, ff]; an
     id >= E names an identity expert, whose output is x itself.  Without ``w_up``, ``w_gate`` holds both
     matrices as ``interleave_gate_up`` lays them out.  The tokens are sorted by expert on the device and
     nothing comes back to the host: alignment, the two products (gate/up with the activation, down) and the
     weighted sum.  ``weigh_inputs``: sum_j expert_{ids[t, j]}(weights[t, j] x[t]) instead (the gate and up sums
-    are multiplied by the weight ahead of the activation; no identity experts).  bfloat16 with many tokens per expert and the interleaved layout: each product is ONE
+    are multiplied by the weight ahead of the activation; no identity experts).  ``bounded`` (without biases): the
+    bounded gate of the unrounded gate and up sums in the activation's place.  bfloat16 with many tokens per expert and the interleaved layout: each product is ONE
     grouped launch of the tcgen05 kernel over runs padded to whole tiles; otherwise tiles on mma.sync
     (bfloat16) or CUDA cores (float32)."""
     _cuda(x, ids, weights, w_gate, w_up, w_down)
@@ -1817,6 +1878,10 @@ def routed_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_
              and w_down.shape == (E, width, ff) and (not interleaved or ff % 8 == 0),
              "expert matrices [E, ff, width] (or [E, 2 ff, width] interleaved), [E, width, ff]")
     _require(act in ACTIVATIONS, f"the gate's activation is one of {sorted(ACTIVATIONS)}")
+    _require(bounded is None or (bounded.bias is None and bounded.limit > 0.0 and not weigh_inputs),
+             "experts' bounded gates have a positive limit, no biases and weights on the outputs")
+    act_code = ACTIVATIONS[act] if bounded is None else 2
+    bounds = (float(bounded.limit), float(bounded.alpha), float(bounded.shift)) if bounded is not None else (0.0, 1.0, 0.0)
     _i32(ids)
     _require(weights.dtype == torch.float32 and weights.is_contiguous() and weights.shape == ids.shape, "one weight per choice")
     lib, device = library(), x.device
@@ -1840,12 +1905,12 @@ def routed_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_
         status = device_status(device)
         hidden = torch.empty((places, ff), dtype=x.dtype, device=device)
         _check(lib.zb_gemm_tc_grouped(_ptr(hidden), _ptr(rows), _ptr(w_gate), _ptr(tile_group), tiles, E, 2 * ff, width, width,
-                                      ff, 3 if act == "relu" else 1, _ptr(place_scale), _ptr(status), _stream()), "gemm_tc_grouped")
+                                      ff, (1, 3, 7)[act_code], _ptr(place_scale), *bounds, _ptr(status), _stream()), "gemm_tc_grouped")
         # An expert's output takes the model's type before it is weighted on every path: here the product writes it so.
         ldy = width
         y = torch.empty((places, ldy), dtype=x.dtype, device=device)
         _check(lib.zb_gemm_tc_grouped(_ptr(y), _ptr(hidden), _ptr(w_down), _ptr(tile_group), tiles, E, width, ff, ff, ldy, 0,
-                                      None, _ptr(status), _stream()), "gemm_tc_grouped")
+                                      None, *bounds, _ptr(status), _stream()), "gemm_tc_grouped")
     else:
         tile_rows = lib.zb_expert_tile_rows(code)          # CUDA-core tiles in float32, tensor-core tiles in bfloat16
         max_tiles = -(-num_slots // tile_rows) + E
@@ -1857,9 +1922,9 @@ def routed_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_
         ldy = width
         y = torch.empty((max(num_slots, 1), width), dtype=torch.float32, device=device)
         _check(lib.zb_expert_product(_ptr(hidden), _ptr(x), x.stride(0), _ptr(w_gate), _ptr(w_up), _ptr(plan), _ptr(slots),
-                                     _ptr(weights) if weigh_inputs else None, max_tiles, ff, width, top, ACTIVATIONS[act], 0, code, _stream()), "expert_product")
+                                     _ptr(weights) if weigh_inputs else None, max_tiles, ff, width, top, act_code, *bounds, 0, code, _stream()), "expert_product")
         _check(lib.zb_expert_product(_ptr(y), _ptr(hidden), ff, _ptr(w_down), None, _ptr(plan), _ptr(slots), None, max_tiles,
-                                     width, ff, top, ACTIVATIONS[act], 1, code, _stream()), "expert_product")
+                                     width, ff, top, act_code, *bounds, 1, code, _stream()), "expert_product")
     _check(lib.zb_route_combine(_ptr(out), _ptr(y), ldy, DTYPE_CODE[y.dtype], _ptr(x), x.stride(0), _ptr(ids),
                                 None if weigh_inputs else _ptr(weights), _ptr(place), T, width, top, code, _stream()), "route_combine")
     return out

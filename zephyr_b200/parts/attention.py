@@ -41,6 +41,11 @@ runs on the kernels that keep all heads of a tile in one CTA, ``ops.heads_attent
 ``distance_bias`` (the names of two vectors r1, r2 [heads]: r1_h ln(1 + r2_h d) is taken off head h's score of the
 key d positions back; every attention kernel has it).  ``head_gate``: one sigmoid gate per head on its output,
 sigmoid(Wg x)_h with Wg [heads, hidden], whose product rides along with the projections.
+
+``zero_sinks``: every head's softmax has one added to its denominator (a sink whose score is 0, without a tensor).
+``value_mix`` = {"group", "share"}: layers that name one group hand values on within a step.  Its first layer (``share``
+None) leaves its values as projected; every later one caches (1 - m) v + m v_first, m being the tensor ``share`` and
+v_first the first layer's values of the same tokens, both unrounded.
 """
 
 from __future__ import annotations
@@ -111,6 +116,13 @@ class Attention(Mixer):
         self.qkv_bias = torch.cat([b.float() for b in biases]).contiguous() if biases[0] is not None else None
         self.o_bias = weights[p["o_bias"]].float().contiguous() if p.get("o_bias") else None
         self.sinks = weights[p["sinks"]].float().contiguous() if p.get("sinks") else None
+        if p.get("zero_sinks"):
+            if self.sinks is not None:
+                raise ConfigError("sinks are learned or zero")
+            self.sinks = torch.zeros(self.nh, dtype=torch.float32, device=device)
+        self.value_group = p["value_mix"]["group"] if p.get("value_mix") else None
+        share = p["value_mix"].get("share") if p.get("value_mix") else None
+        self.value_share = weights[share].float().reshape(1).contiguous() if share else None
         pairs = getattr(self.position, "as_pair_frequencies", None)
         self.pair_freqs, self.pair_dims = pairs() if pairs is not None else (None, 0)
         halves = getattr(self.position, "as_half_frequencies", None)
@@ -138,8 +150,10 @@ class Attention(Mixer):
             raise ConfigError("qk_norm is 'per_head' or 'whole'; keep_first and pool are not negative")
         if (self.keep_first or self.pool) and self.window <= 0:
             raise ConfigError("kept first tokens and pooled blocks come with a window")
+        if self.value_group is not None and (self.value_unit_norm or biases[0] is not None):
+            raise ConfigError("mixed values combine with neither biases nor unit norms of the values")
         # What runs through the kernel that rotates halves.
-        self.halves = (halves is not None or self.qk_norm == "whole" or self.value_unit_norm or self.keep_first > 0
+        self.halves = (self.value_group is not None or halves is not None or self.qk_norm == "whole" or self.value_unit_norm or self.keep_first > 0
                        or self.pool > 0 or self.head_mix is not None
                        or (self.w_gate is not None and not self.head_gate))
         if self.halves and (pairs is not None or self.values_from_keys or self.unit_norm or self.q_temp is not None):
@@ -200,8 +214,8 @@ class Attention(Mixer):
         self.windowed = bool(self.keep_first or self.pool or self.head_mix is not None)
         # Tokens a tile of the kernel with all heads in one CTA (0: it does not take the layer).  Mixed scores run
         # there, and so does what no other tensor-core kernel takes: keys and values of two widths behind a mask of
-        # a window and kept first tokens, with or without a distance bias.
-        plain_mask = not (self.chunk or self.pool or self.sinks is not None or self.softcap > 0.0
+        # a window and kept first tokens, with or without a distance bias or sinks.
+        plain_mask = not (self.chunk or self.pool or self.softcap > 0.0
                           or self.head_mix is not None or self.values_from_keys)
         self.heads_tile_tokens = 0
         if plain_mask and (self.score_mix is not None or not (equal and ops.paged_prefill_supported(self.nh, self.nkv, self.hd, self.dtype))):
@@ -235,6 +249,8 @@ class Attention(Mixer):
             decls[p["out_gate"]] = WeightDecl((nh * vd, hidden), ROLE_LINEAR)
         if p.get("score_mix"):
             decls[p["score_mix"]] = WeightDecl((nh, nh), ROLE_LINEAR)
+        if p.get("value_mix") and p["value_mix"].get("share"):
+            decls[p["value_mix"]["share"]] = WeightDecl((), ROLE_NORM)
         for name in p.get("distance_bias") or ():
             decls[name] = WeightDecl((nh,), ROLE_NORM)
         if p.get("head_gate"):
@@ -359,7 +375,7 @@ class Attention(Mixer):
                 ops.heads_attention(q, cache, table, tile_row, tile_q0, ctx.row_q_start, ctx.row_q_len, ctx.row_ctx, self.nh,
                                     self.nkv, self.hd, self.vd, self.window, self.scale, ctx.status, out,
                                     keep_first=self.keep_first, score_mix=self.score_mix, distance_bias=self.distance_bias,
-                                    single=single, max_context=ctx.max_decode_context)
+                                    sinks=self.sinks, single=single, max_context=ctx.max_decode_context)
         return out
 
     def _attend_windowed(self, q: torch.Tensor, ctx: StepContext, call: LayerCall, cache, table) -> torch.Tensor:
@@ -406,8 +422,8 @@ class Attention(Mixer):
         table = ctx.block_table(call.cache)
         # A layer that reads another layer's cache needs no k and v.
         weight, bias, cache = self.w_qkv, self.qkv_bias, ctx.caches[call.cache]
-        if not call.writes_cache and self.w_gate is not None:
-            raise ConfigError("a gated layer that reads another layer's cache is not built")
+        if not call.writes_cache and (self.w_gate is not None or self.value_group is not None):
+            raise ConfigError("a layer with a gate or mixed values that reads another layer's cache is not built")
         if not call.writes_cache:
             weight, cache = self.w_q, None
             bias = bias[: self.nh * self.hd] if bias is not None else None
@@ -431,10 +447,16 @@ class Attention(Mixer):
                         out_dtype: torch.dtype | None) -> torch.Tensor:
         """Biases, norms, rotation of halves and cache write in one kernel; the blocks that this step's tokens
         complete are pooled; attention; the gate; the output projection."""
+        first = None
+        if self.value_group is not None and self.value_share is None:      # (the projection's tensor stays alive with its view)
+            at = (self.nh + self.nkv) * self.hd
+            ctx.shared[self.value_group] = projected[:, at:at + self.nkv * self.vd]
+        elif self.value_group is not None:
+            first = ctx.shared[self.value_group]
         q = ops.qkv_halves(projected, self.nh, self.nkv, self.hd, self.vd, self.qk_norm if self.q_norm is not None else "none",
                            self.q_norm, self.k_norm, self.eps, self.half_freqs, self.half_dims, self.half_mult,
                            self.value_unit_norm, ctx.positions, ctx.token_row, cache, table, ctx.status, self.dtype,
-                           bias=bias)
+                           bias=bias, v_first=first, v_share=self.value_share if first is not None else None)
         if self.pool and call.writes_cache:
             ops.pool_blocks(cache, table, ctx.caches[call.extra_caches[0]], ctx.block_table(call.extra_caches[0]),
                             ctx.positions, ctx.token_row, self.nkv, self.hd, self.vd, self.pool, ctx.status)

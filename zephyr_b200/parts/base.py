@@ -19,7 +19,7 @@ import torch
 
 from ..cache import CacheStorage, PagedCacheSpec, StateCacheSpec
 from ..config.errors import ConfigError
-from ..config.spec import FeedForwardSpec, InputSpec, LayerCall, MixerSpec, NormSpec, OutputSpec, PositionSpec
+from ..config.spec import FeedForwardSpec, InputSpec, LayerCall, MixerSpec, NormSpec, OutputSpec, PositionSpec, SideSpec
 from ..weights.loader import WeightDecl
 
 
@@ -55,6 +55,8 @@ class StepContext:
     host_q_len: list[int] = field(default_factory=list)
     host_ctx: list[int] = field(default_factory=list)
     host_slots: list[int] = field(default_factory=list)
+    # What a layer hands on to later layers of the same step (values that they mix in), by a name their specs give.
+    shared: dict[str, torch.Tensor] = field(default_factory=dict)
 
     def block_table(self, cache_id: int) -> torch.Tensor:
         return self.block_tables[self.group_of_cache[cache_id]]
@@ -173,6 +175,17 @@ class FeedForward(Part):
         return None
 
 
+class SidePart(Part):
+    """What joins the stream behind a layer's two halves and is not made from a norm's output: a block that takes one
+    (``Block`` with ``side``) sums the stream up first."""
+
+    def __init__(self, spec: SideSpec, weights: Mapping[str, torch.Tensor], dtype: torch.dtype): ...
+
+    def forward(self, x: torch.Tensor, ctx: StepContext) -> "DeferredSum":
+        """The summand for the stream's value ``x`` ([T, hidden] in the model's type), not yet added."""
+        raise NotImplementedError
+
+
 @dataclass
 class DeferredSum:
     """hidden += mult * norm(delta), not yet done: the consumer of the stream either does it in the
@@ -284,6 +297,7 @@ POSITION_ENCODINGS: dict[str, type] = {}
 MIXERS: dict[str, type] = {}
 FEED_FORWARDS: dict[str, type] = {}
 BLOCKS: dict[str, type] = {}
+SIDES: dict[str, type] = {}
 
 
 def _register(table: dict[str, type], what: str, kind: str, cls: type, replace: bool) -> None:
@@ -310,6 +324,10 @@ def register_feed_forward(kind: str, cls: type, replace: bool = False) -> None:
 
 def register_block(kind: str, cls: type, replace: bool = False) -> None:
     _register(BLOCKS, "block", kind, cls, replace)
+
+
+def register_side(kind: str, cls: type, replace: bool = False) -> None:
+    _register(SIDES, "side part", kind, cls, replace)
 
 
 def register_input(kind: str, cls: type, replace: bool = False) -> None:

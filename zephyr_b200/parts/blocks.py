@@ -4,7 +4,9 @@
 (reference: src/model/causal_lm/qwen3.cpp:79-88).  Each sum is folded into the norm that follows
 it, so the block hands its last summand on as ``pending``.  On a float32 stream (an input part that makes one) the
 summands travel as a tuple and join the stream in the kernel of the next norm (``Norm.sum_forward``).  The
-feed-forward may be missing; the layer is then its first half.
+feed-forward may be missing; the layer is then its first half.  A side part (``LayerSpec.side``), x'' = x' + side(x'),
+reads the summed stream's rounding, which the kernel of the sum writes in the same pass; its own summand, a norm's
+output, is taken up by the next layer's norm (``DeferredSum``).
 
 ``sandwich_residual``: a norm before and one behind each part, and a multiplier m on what joins the
 stream: r = x + m * mixer_out(mixer(mixer_norm(x))); x' = r + m * ffn_out(ffn(ffn_norm(r))).  The
@@ -28,7 +30,7 @@ from typing import Mapping
 import torch
 
 from ..config.spec import LayerCall
-from .base import Block, DeferredSum, FeedForward, Mixer, Norm, ResidualStream, StepContext, register_block
+from .base import Block, DeferredSum, FeedForward, Mixer, Norm, ResidualStream, SidePart, StepContext, register_block
 from .fused import BlockPlan
 
 
@@ -37,8 +39,10 @@ class PreNormResidual(Block):
     feed_forward_optional = True
 
     norm_names = ("mixer", "feed_forward")
+    takes_side = True
 
-    def __init__(self, mixer: Mixer, feed_forward: FeedForward | None, norms: Mapping[str, Norm]):
+    def __init__(self, mixer: Mixer, feed_forward: FeedForward | None, norms: Mapping[str, Norm], side: SidePart | None = None):
+        self.side = side
         self.mixer = mixer
         self.feed_forward = feed_forward
         self.norms = dict(norms)
@@ -46,21 +50,28 @@ class PreNormResidual(Block):
         self.feed_forward_norm = norms.get("feed_forward")
 
     def _forward_float32(self, stream: ResidualStream, ctx: StepContext, call: LayerCall) -> ResidualStream:
-        if stream.deferred is not None:
-            stream.flush()
-        pending = stream.pending if stream.pending is not None else ()
-        normed = self.mixer_norm.sum_forward(stream.hidden, pending if isinstance(pending, tuple) else (pending,))
+        if stream.deferred is not None and stream.pending is None:
+            normed = stream.deferred.apply(stream.hidden, then=self.mixer_norm)
+            stream.deferred = None
+        else:
+            if stream.deferred is not None:
+                stream.flush()
+            pending = stream.pending if stream.pending is not None else ()
+            normed = self.mixer_norm.sum_forward(stream.hidden, pending if isinstance(pending, tuple) else (pending,))
         stream.rounded = None
         stream.pending = (self.mixer.forward(normed, ctx, call),)
         if self.feed_forward is not None:
             normed = self.feed_forward_norm.sum_forward(stream.hidden, stream.pending)
             stream.pending = self.feed_forward.forward_summands(normed)
+        if self.side is not None:
+            x = self.mixer_norm.sum_rounded(stream.hidden, stream.pending)
+            stream.pending, stream.deferred = None, self.side.forward(x, ctx)
         return stream
 
     def forward(self, stream: ResidualStream, ctx: StepContext, call: LayerCall) -> ResidualStream:
         # A stream in the model's own type takes the norms' form for that type (float32 models included, unless
         # their norms have groups or a layer lacks its second half).
-        own_type = (getattr(self.mixer_norm, "dtype", stream.hidden.dtype) == stream.hidden.dtype
+        own_type = (self.side is None and stream.deferred is None and getattr(self.mixer_norm, "dtype", stream.hidden.dtype) == stream.hidden.dtype
                     and getattr(self.mixer_norm, "groups", 1) == 1 and self.feed_forward is not None)
         if stream.hidden.dtype == torch.float32 and (not own_type or isinstance(stream.pending, tuple)):
             return self._forward_float32(stream, ctx, call)
@@ -74,7 +85,7 @@ class PreNormResidual(Block):
         return stream
 
     def chain_plan(self) -> BlockPlan | None:
-        if self.feed_forward is None:
+        if self.feed_forward is None or self.side is not None:
             return None
         mixer_norm, ffn_norm = self.mixer_norm.as_rms_scale(), self.feed_forward_norm.as_rms_scale()
         gated = self.feed_forward.as_gated_products()

@@ -27,7 +27,7 @@ from ..cache import StateCacheSpec
 from ..config.spec import InputSpec, OutputSpec
 from ..kernels import ops
 from ..weights.loader import ROLE_EMBEDDING, ROLE_LINEAR, WeightDecl
-from .base import NORMS, InputPart, OutputPart, ResidualStream, StepContext, lookup, register_input, register_output
+from .base import NORMS, DeferredSum, InputPart, OutputPart, ResidualStream, StepContext, lookup, register_input, register_output
 
 
 class Embedding(InputPart):
@@ -123,10 +123,11 @@ class NormHead(OutputPart):
         wanted = ctx.logit_tokens
         if wanted.numel() == 0:
             return torch.empty((0, self.vocab_size), dtype=torch.float32, device=stream.hidden.device)
-        if stream.deferred is not None:
-            stream.flush()
         rows = ops.gather_rows(stream.hidden, wanted, ctx.status)
-        if isinstance(stream.pending, tuple):       # summands that are added to each other first, then to the stream
+        if stream.deferred is not None and stream.pending is None:
+            own = DeferredSum(ops.gather_rows(stream.deferred.delta, wanted, ctx.status), stream.deferred.norm, stream.deferred.mult)
+            normed = own.apply(rows, then=self.norm)
+        elif isinstance(stream.pending, tuple):       # summands that are added to each other first, then to the stream
             normed = self.norm.sum_forward(rows, tuple(ops.gather_rows(part, wanted, ctx.status) if part.dim() == 2 else part
                                                        for part in stream.pending))
         elif stream.pending is not None:

@@ -7,8 +7,8 @@ out = down(y).  Biases, bounds and the activation act on the product's unrounded
 product's kernel for few rows and for many (one pass over the float32 product otherwise); the down product's
 bias joins the float32 sum into the stream.
 
-``ungated`` is the form without a gate: down(gelu(up(x))), gelu in its tanh form, no biases; the activation acts
-on the product's unrounded float32 sums, inside the product's kernel for few rows and for many.
+``ungated`` is the form without a gate: down(act(up(x))), act being GELU in its tanh form or the square of max(., 0),
+no biases; the activation acts on the product's unrounded float32 sums, inside the product's kernel for few rows and for many.
 
 Gate and up run as one product over one packed weight [2I, H], as the reference packs them at
 load (src/layer/mlp.cpp:16-36); the reference puts all gate rows first, this part alternates blocks
@@ -126,14 +126,16 @@ class SwiGLU(FeedForward):
 
 
 class UngatedFeedForward(FeedForward):
-    """out = down(gelu(up(x))), gelu(z) = 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))."""
+    """out = down(act(up(x))); ``activation`` "gelu_tanh" (the default), 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))),
+    or "relu_squared", max(z, 0)^2."""
 
     graph_safe = True
 
     def __init__(self, spec: FeedForwardSpec, weights: Mapping[str, torch.Tensor], dtype: torch.dtype):
         p = spec.params
-        if str(p.get("activation", "gelu_tanh")) != "gelu_tanh":
-            raise ConfigError("an ungated feed-forward's activation is gelu_tanh")
+        self.activation = str(p.get("activation", "gelu_tanh"))
+        if self.activation not in ops.PRODUCT_ACTS:
+            raise ConfigError(f"an ungated feed-forward's activation is one of {sorted(ops.PRODUCT_ACTS)}")
         self.dtype = dtype
         self.w_up, self.w_down = weights[p["up_proj"]], weights[p["down_proj"]]
 
@@ -145,12 +147,12 @@ class UngatedFeedForward(FeedForward):
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         if x.shape[0] <= ops.SMALL_GEMM_ROWS and ops.gemm_small_supported(x, self.w_up):
-            hidden = ops.gemm_small(x, self.w_up, gelu=True)
+            hidden = ops.gemm_small(x, self.w_up, product_act=self.activation)
         elif ((x.shape[0] >= ops.GEMM_TC_MIN_ROWS or not ops.USE_LIBRARY_PRODUCTS)
               and self.w_up.shape[0] % 8 == 0 and ops.gemm_tc_supported(x, self.w_up)):
-            hidden = ops.gemm_tc(x, self.w_up, gelu=True)
+            hidden = ops.gemm_tc(x, self.w_up, product_act=self.activation)
         else:
-            hidden = ops.gelu_rows(ops.linear(x, self.w_up, out_dtype=torch.float32), self.dtype)
+            hidden = ops.act_rows(ops.linear(x, self.w_up, out_dtype=torch.float32), self.activation, self.dtype)
         return ops.linear(hidden, self.w_down)
 
 

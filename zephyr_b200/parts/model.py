@@ -16,7 +16,7 @@ from ..config.errors import ConfigError
 from ..config.spec import LayerSpec, ModelSpec
 from ..kernels import ops
 from ..weights.loader import WeightDecl, WeightStore, load_weights
-from .base import (BLOCKS, FEED_FORWARDS, INPUTS, MIXERS, NORMS, OUTPUTS, ResidualStream, StepContext, lookup)
+from .base import (BLOCKS, FEED_FORWARDS, INPUTS, MIXERS, NORMS, OUTPUTS, SIDES, ResidualStream, StepContext, lookup)
 from .fused import DecodeChains
 
 
@@ -29,6 +29,8 @@ def _layer_classes(layer: LayerSpec):
         raise ConfigError(f"block '{layer.block}' places the norms {sorted(wanted)}, the layer brings {sorted(given)}")
     if layer.feed_forward is None and not getattr(block, "feed_forward_optional", False):
         raise ConfigError(f"block '{layer.block}' needs a feed-forward")
+    if layer.side is not None and not getattr(block, "takes_side", False):
+        raise ConfigError(f"block '{layer.block}' takes no side part")
     return (block, lookup(MIXERS, "mixer", layer.mixer.kind),
             lookup(FEED_FORWARDS, "feed-forward", layer.feed_forward.kind) if layer.feed_forward is not None else None,
             {name: lookup(NORMS, "norm", norm.kind) for name, norm in layer.norms.items()})
@@ -55,6 +57,8 @@ def expected_weights(spec: ModelSpec) -> dict[str, WeightDecl]:
             merge(ffn.weight_decls(layer.feed_forward))
         for name, norm in norms.items():
             merge(norm.weight_decls(layer.norms[name]))
+        if layer.side is not None:
+            merge(lookup(SIDES, "side part", layer.side.kind).weight_decls(layer.side))
     merge(lookup(OUTPUTS, "output part", spec.output.kind).weight_decls(spec.output))
     return decls
 
@@ -116,6 +120,8 @@ class Model:
         for layer in spec.layers:
             block, mixer, ffn, norms = _layer_classes(layer)
             extra = {"params": layer.block_params} if layer.block_params else {}
+            if layer.side is not None:
+                extra["side"] = lookup(SIDES, "side part", layer.side.kind)(layer.side, weights, dtype)
             self.layers.append(block(mixer(layer.mixer, weights, dtype, device),
                                      ffn(layer.feed_forward, weights, dtype) if ffn is not None else None,
                                      {name: cls(layer.norms[name], weights, dtype) for name, cls in norms.items()},
@@ -125,7 +131,7 @@ class Model:
             self.input.cache_id = spec.num_caches
         parts = [self.input, self.output]
         for block in self.layers:
-            parts += [block, block.mixer, block.feed_forward, *getattr(block, "norms", {}).values(),
+            parts += [block, block.mixer, block.feed_forward, getattr(block, "side", None), *getattr(block, "norms", {}).values(),
                       getattr(block.mixer, "position", None), *getattr(block.mixer, "branches", ())]
         self.graph_safe = all(getattr(part, "graph_safe", False) for part in parts if part is not None)
         self.tile_requests = tile_requests(spec)
@@ -166,7 +172,7 @@ class Model:
                 add(tensor)
         for call in self.spec.run_order:
             block = self.layers[call.layer]
-            for part in (block.mixer, block.feed_forward, *getattr(block, "norms", {}).values()):
+            for part in (block.mixer, block.feed_forward, getattr(block, "side", None), *getattr(block, "norms", {}).values()):
                 for tensor in (part.weights_read() if part is not None else ()):
                     add(tensor)
         # Tensors that share a storage overlap (a matrix and a view of its first rows): such a storage

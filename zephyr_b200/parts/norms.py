@@ -46,10 +46,9 @@ class RMSNorm(Norm):
         self._needs_one_group("a norm of rows in the model's type")
         return ops.rmsnorm(x, self.weight, self.eps)
 
-    def sum_forward(self, stream: torch.Tensor, summands: tuple) -> torch.Tensor:
-        """stream (float32) += (the summands added to each other), in place and in float32; returns the norm
-        of the sum in the model's type.  A summand is [rows, H], or a float32 [H] shift that goes on every
-        row.  Two summands and a shift take one kernel for the sums and the norm."""
+    @staticmethod
+    def _two_summands(stream: torch.Tensor, summands: tuple):
+        """(a, b, shift) of a tuple of summands; what goes beyond two rows and a shift joins the stream here."""
         rows = [s for s in summands if s.dim() == 2]
         shifts = [s for s in summands if s.dim() == 1]
         for more in rows[2:]:
@@ -61,7 +60,22 @@ class RMSNorm(Norm):
             stream.add_(torch.stack(shifts).sum(0))
         a = rows[0] if len(rows) > 0 else None
         b = rows[1] if len(rows) > 1 else None
+        return a, b, shift
+
+    def sum_forward(self, stream: torch.Tensor, summands: tuple) -> torch.Tensor:
+        """stream (float32) += (the summands added to each other), in place and in float32; returns the norm
+        of the sum in the model's type.  A summand is [rows, H], or a float32 [H] shift that goes on every
+        row.  Two summands and a shift take one kernel for the sums and the norm."""
+        a, b, shift = self._two_summands(stream, summands)
         return ops.sum_rms_norm(stream, a, b, self.weight, self.eps, out_dtype=self.dtype, bias=shift, groups=self.groups)
+
+    def sum_rounded(self, stream: torch.Tensor, summands: tuple) -> torch.Tensor:
+        """The same sums without the norm: stream += the summands; returns the stream's value in the model's type
+        (in float32 the stream itself)."""
+        a, b, shift = self._two_summands(stream, summands)
+        rounded = self.dtype != torch.float32
+        out = ops.sum_rms_norm(stream, a, b, None, 0.0, out_dtype=self.dtype, bias=shift, rounded_sum=rounded)
+        return out if rounded else stream
 
     def _needs_one_group(self, what: str) -> None:
         if self.groups > 1:

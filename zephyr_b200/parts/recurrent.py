@@ -1,7 +1,7 @@
 """Mixers that carry a state of fixed size per request instead of a growing cache, and a mixer that
 runs several mixers side by side.
 
-Both recurrent mixers are the same recurrence per head,
+Three recurrent mixers are the same recurrence per head,
 
     S_t = diag(a_t) S_{t-1} + k_t v_t^T        (S: key channels x value channels, float32)
     o_t = S_t^T q_t
@@ -29,6 +29,10 @@ S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q; each head's o is RMS-
 channels with one scale vector shared by the heads, the heads are joined, multiplied by silu(Wg h) and
 projected by Wo.  The state and the convolution's last taps - 1 inputs live in the request's slot.
 
+``retention``: q = Wq h and k = Wk h, rotated in halves by the position (position kind ``rope_halves``), k times
+dim^(-1/2) behind the rotation, v = Wv h; a_t is a constant per head; each head's o is divided by its root mean square
+over the value channels (no scales), the heads are joined, multiplied by silu(Wg h) and projected by Wo.
+
 ``parallel``: the sum of several mixers over the same input, each with a weight.  Every branch keeps
 its own store; the call's first cache id goes to the first branch and its ``extra_caches`` to the
 others.
@@ -49,7 +53,7 @@ from ..config.errors import ConfigError
 from ..config.spec import LayerCall, MixerSpec
 from ..kernels import ops
 from ..weights.loader import ROLE_LINEAR, ROLE_NORM, ROLE_ZERO, WeightDecl
-from .base import MIXERS, Mixer, StepContext, lookup, register_mixer
+from .base import MIXERS, POSITION_ENCODINGS, Mixer, StepContext, lookup, register_mixer
 
 MAX_KEY_CHANNELS = 256        # what the scan kernel takes per head (csrc/recurrent.cu: 16 warps of 16 channels)
 
@@ -272,6 +276,62 @@ class GatedDeltaRule(Mixer):
         return ops.linear(normed, self.w_o, out_dtype=out_dtype)
 
 
+class Retention(Mixer):
+    graph_safe = True
+    takes_out_dtype = True
+
+    def __init__(self, spec: MixerSpec, weights: Mapping[str, torch.Tensor], dtype: torch.dtype,
+                 device: torch.device | str):
+        p = spec.params
+        self.hidden, self.heads = int(p["hidden_size"]), int(p["heads"])
+        self.dim, self.vdim, self.eps = int(p["key_dim"]), int(p["value_dim"]), float(p["norm_eps"])
+        _check_sizes(self.heads, self.dim, self.vdim)
+        if len(p["decay"]) != self.heads:
+            raise ConfigError("retention needs one decay per head")
+        self.decay = torch.tensor([float(a) for a in p["decay"]], dtype=torch.float32, device=device)
+        self.position = (lookup(POSITION_ENCODINGS, "position encoding", spec.position.kind)(spec.position, dtype, device)
+                         if spec.position is not None else None)
+        halves = getattr(self.position, "as_half_frequencies", None)
+        if self.position is not None and halves is None:
+            raise ConfigError("retention rotates halves, or nothing")
+        self.freqs, self.rot_dims, mult = halves() if halves is not None else (None, 0, 1.0)
+        if mult != 1.0:
+            raise ConfigError("retention's rotation takes no multiplier")
+        # One product with float32 sums out for everything that enters the recurrence, q | k | v (behind the unit
+        # norm of o a rounding of q or k counts in full where q . k is small); the gate comes out of a second
+        # product, in the model's type.
+        self.w_in = torch.cat([weights[p[n]] for n in ("q", "k", "v")], dim=0).contiguous()
+        self.w_g, self.w_o = weights[p["g"]], weights[p["o"]]
+        self.unit = torch.ones(self.vdim, dtype=torch.float32, device=self.w_o.device)
+
+    @staticmethod
+    def weight_decls(spec: MixerSpec) -> dict[str, WeightDecl]:
+        p = spec.params
+        hidden, hd, hv = int(p["hidden_size"]), int(p["heads"]) * int(p["key_dim"]), int(p["heads"]) * int(p["value_dim"])
+        return {p["q"]: WeightDecl((hd, hidden), ROLE_LINEAR), p["k"]: WeightDecl((hd, hidden), ROLE_LINEAR),
+                p["v"]: WeightDecl((hv, hidden), ROLE_LINEAR), p["g"]: WeightDecl((hv, hidden), ROLE_LINEAR),
+                p["o"]: WeightDecl((hidden, hv), ROLE_LINEAR)}
+
+    def weights_read(self) -> list[torch.Tensor]:
+        return [self.w_in, self.w_g, self.w_o]
+
+    @staticmethod
+    def cache_spec(spec: MixerSpec) -> StateCacheSpec:
+        p = spec.params
+        return StateCacheSpec(shape=(int(p["heads"]) * int(p["key_dim"]) * int(p["value_dim"]),), dtype="float32")
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, call: LayerCall,
+                out_dtype: torch.dtype | None = None) -> torch.Tensor:
+        hd = self.heads * self.dim
+        projected = ops.linear(x, self.w_in, out_dtype=torch.float32)      # q | k | v
+        turned = ops.rotate_qk(projected, self.heads, self.dim, self.freqs, self.rot_dims, self.dim ** -0.5, ctx.positions)
+        o = ops.decayed_state_scan("fixed", turned[:, :hd], turned[:, hd:], projected[:, 2 * hd:], self.heads, self.dim, self.vdim,
+                                   ctx.caches[call.cache], ctx.state_slots, ctx.row_q_start, ctx.row_q_len, ctx.status,
+                                   decay=self.decay, write_state=call.writes_cache)
+        normed = ops.gated_group_rms_norm(o, ops.linear(x, self.w_g), self.unit, self.vdim, self.eps, gate_first=False)
+        return ops.linear(normed, self.w_o, out_dtype=out_dtype)
+
+
 def _check_sizes(heads: int, key_channels: int, value_channels: int) -> None:
     if heads <= 0 or key_channels <= 0 or value_channels <= 0:
         raise ConfigError("a recurrent mixer needs positive head counts and widths")
@@ -349,4 +409,5 @@ def _store_count(sub: MixerSpec) -> int:
 register_mixer("gated_delta", GatedDeltaRule)
 register_mixer("gla", GatedLinearAttention)
 register_mixer("mamba2", Mamba2)
+register_mixer("retention", Retention)
 register_mixer("parallel", ParallelMixers)

@@ -12,7 +12,11 @@ its ``top`` largest choice values, and only outputs of the ``keep`` runs with th
 ``weight_scale``: a multiplier on every weight; ``router_bias``: a bias b on the logits, z = Wr x + b;
 ``scores`` "top_softmax": the ``top`` largest logits are taken, and their outputs count with the softmax over
 the taken logits only; ``weigh`` "inputs": the weight goes on the expert's input instead of its output,
-out = sum of expert_e(s_e x) (no identity experts then).
+out = sum of expert_e(s_e x) (no identity experts then); ``normalize``: the taken outputs' weights are divided by their
+sum (+ 1e-20); ``activation`` "clamped_swish" with ``limit``, ``alpha`` and ``up_shift``: the experts' gate is bounded,
+g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(alpha g) * (u + up_shift), on the products' float32
+sums; ``shared``: a gated feed-forward of its own (the parameters of the ``gated`` kind) that runs for every token
+beside the routed experts, whose outputs and its own join the stream as two summands.
 
 The first ``experts`` router outputs are gated feed-forwards, expert_e(x) = down_e(act(gate_e x) * (up_e x)),
 without biases; the last ``identity`` outputs are identity experts, expert(x) = x, which have no tensors.
@@ -32,7 +36,7 @@ from ..config.errors import ConfigError
 from ..config.spec import FeedForwardSpec
 from ..kernels import ops
 from ..weights.loader import ROLE_LINEAR, ROLE_ZERO, WeightDecl
-from .base import FeedForward, register_feed_forward
+from .base import FEED_FORWARDS, FeedForward, lookup, register_feed_forward
 
 
 class RoutedFeedForward(FeedForward):
@@ -47,8 +51,16 @@ class RoutedFeedForward(FeedForward):
         outputs = self.experts + self.identity
         if self.experts <= 0 or self.identity < 0 or not 0 < self.top <= outputs:
             raise ConfigError("a routed feed-forward needs experts, and takes between one and all of its outputs")
-        if self.activation not in ops.ACTIVATIONS:
-            raise ConfigError(f"an expert's activation is one of {sorted(ops.ACTIVATIONS)}")
+        if self.activation not in ops.ACTIVATIONS and self.activation != "clamped_swish":
+            raise ConfigError(f"an expert's activation is one of {sorted(ops.ACTIVATIONS) + ['clamped_swish']}")
+        self.bounded = None
+        if self.activation == "clamped_swish":
+            self.bounded = ops.BoundedGate(None, float(p["limit"]), float(p.get("alpha", 1.0)), float(p.get("up_shift", 0.0)))
+            if not self.bounded.limit > 0.0:
+                raise ConfigError("the bounded activation needs a positive limit")
+        self.normalize = bool(p.get("normalize", False))
+        if self.normalize and str(p.get("scores", "softmax")) == "top_softmax":
+            raise ConfigError("the softmax over the taken logits is normalised as it is")
         self.scores = str(p.get("scores", "softmax"))
         if self.scores not in ops.ROUTE_SCORES:
             raise ConfigError(f"router scores are one of {sorted(ops.ROUTE_SCORES)}")
@@ -56,6 +68,8 @@ class RoutedFeedForward(FeedForward):
         self.weigh = str(p.get("weigh", "outputs"))
         if self.weigh not in ("outputs", "inputs") or (self.weigh == "inputs" and self.identity > 0):
             raise ConfigError("weights go on the experts' outputs, or on their inputs where there are no identity experts")
+        if self.bounded is not None and self.weigh == "inputs":
+            raise ConfigError("bounded experts take weights on their outputs")
         self.groups = None
         if p.get("groups"):
             g = p["groups"]
@@ -78,6 +92,9 @@ class RoutedFeedForward(FeedForward):
             # Blocks of 8 gate rows and their 8 up rows: the layout whose product applies the activation
             # where the sums leave the tensor cores.  The separate matrices are not kept beside it.
             self.w_gate, self.w_up = ops.interleave_gate_up(self.w_gate, self.w_up), None
+        self.shared = None
+        if p.get("shared"):
+            self.shared = lookup(FEED_FORWARDS, "feed-forward", "gated")(FeedForwardSpec("gated", p["shared"]), weights, dtype)
 
     @staticmethod
     def weight_decls(spec: FeedForwardSpec) -> dict[str, WeightDecl]:
@@ -95,20 +112,32 @@ class RoutedFeedForward(FeedForward):
             decls[gate] = WeightDecl((inter, hidden), ROLE_LINEAR)
             decls[up] = WeightDecl((inter, hidden), ROLE_LINEAR)
             decls[down] = WeightDecl((hidden, inter), ROLE_LINEAR)
+        if p.get("shared"):
+            decls.update(lookup(FEED_FORWARDS, "feed-forward", "gated").weight_decls(FeedForwardSpec("gated", p["shared"])))
         return decls
 
     def weights_read(self) -> list[torch.Tensor]:
-        return [w for w in (self.w_router, self.w_gate, self.w_up, self.w_down) if w is not None]
+        own = [w for w in (self.w_router, self.w_gate, self.w_up, self.w_down) if w is not None]
+        return own + (self.shared.weights_read() if self.shared is not None else [])
 
     def route(self, x: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
         logits = ops.linear(x, self.w_router, out_dtype=torch.float32)
         return ops.route(logits, self.correction, self.top, self.scores, self.groups, self.weight_scale,
-                         logit_bias=self.router_bias)
+                         logit_bias=self.router_bias, normalize=self.normalize)
+
+    def _routed(self, x: torch.Tensor) -> torch.Tensor:
+        ids, weights = self.route(x)
+        return ops.routed_experts(x, ids, weights, self.w_gate, self.w_up, self.w_down,
+                                  act="silu" if self.bounded is not None else self.activation,
+                                  weigh_inputs=self.weigh == "inputs", bounded=self.bounded)
+
+    def forward_summands(self, x: torch.Tensor) -> tuple[torch.Tensor, ...]:
+        routed = self._routed(x)
+        return (routed,) if self.shared is None else (routed, self.shared.forward(x))
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
-        ids, weights = self.route(x)
-        return ops.routed_experts(x, ids, weights, self.w_gate, self.w_up, self.w_down, act=self.activation,
-                                  weigh_inputs=self.weigh == "inputs")
+        summands = self.forward_summands(x)
+        return summands[0] if len(summands) == 1 else ops.scaled_sum(*summands, 1.0, 1.0)
 
 
 register_feed_forward("routed", RoutedFeedForward)

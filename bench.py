@@ -102,6 +102,18 @@ LEGILIX_SIZES = {
                   experts=16, top=4),
 }
 
+# Tedulorn beside Legilix: retention beside mixed scores, a window that keeps the first tokens with one added to the
+# denominator beside a window with a distance bias, bounded experts (a quarter of the routed width in a shared one) beside
+# plain ones, a gate on the token's row behind every layer.
+TEDULORN_SIZES = {
+    "w1024": dict(width=1024, ff=3072, dense_ff=4608, layers=8, heads=8, kv_heads=4, head_dim=128, window=1024, keep_first=64,
+                  ret_heads=8, ret_dim=128, ret_vdim=128, experts=16, top=4, side=128),
+    "w2048": dict(width=2048, ff=6144, dense_ff=9216, layers=8, heads=16, kv_heads=8, head_dim=128, window=1024, keep_first=64,
+                  ret_heads=16, ret_dim=128, ret_vdim=128, experts=16, top=4, side=256),
+    "w4096": dict(width=4096, ff=12288, dense_ff=18432, layers=8, heads=32, kv_heads=8, head_dim=128, window=1024, keep_first=64,
+                  ret_heads=32, ret_dim=128, ret_vdim=128, experts=16, top=4, side=256),
+}
+
 
 def metric_name(args) -> str:
     """One string for both arms: the driver divides their values only if the strings are equal."""
@@ -360,6 +372,29 @@ def build_legilix_pair(size: str, batch: int, context: int):
     return legilix, rizovik, make
 
 
+def build_tedulorn_pair(size: str, batch: int, context: int):
+    """(Tedulorn configuration, Legilix configuration of equal sizes, engine builder) of one entry of ``TEDULORN_SIZES``."""
+    from zephyr_b200.config import TedulornConfig
+
+    z = TEDULORN_SIZES[size]
+    hd = z["head_dim"]
+    # Five experts' worth of a token's routed width: four routed ones and the shared one.
+    part = z["ff"] // (z["top"] + 1) // 16 * 16
+    routed = {"kind": "moe", "expert": {"ff": part, "limit": 7.0}, "shared": {"ff": part, "limit": 7.0},
+              "router": {"experts": z["experts"], "top": z["top"], "groups": {"count": 4, "keep": 2}}}
+    dense = {"kind": "dense", "ff": z["dense_ff"]}
+    keeping = dict(heads=z["ret_heads"], dim=z["ret_dim"], vdim=z["ret_vdim"], rot={"base": 10000.0, "dims": z["ret_dim"]},
+                   decay=[1.0 - 2.0 ** -(5 + h % 8) for h in range(z["ret_heads"])])
+    seeing = dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=hd, vdim=hd, scale=hd ** -0.5, v_mix=True,
+                  rot={"base": 150000.0, "dims": hd // 2}, mask={"size": z["window"], "keep_first": z["keep_first"]})
+    layers = [{"type": "retention", "mixer": keeping, "mlp": dense}, {"type": "attention", "mixer": seeing, "mlp": routed},
+              {"type": "retention", "mixer": keeping, "mlp": routed}, {"type": "attention", "mixer": seeing, "mlp": dense}]
+    tedulorn = TedulornConfig(vocab=32768, width=z["width"], norm_eps=1e-6, embedding_scale=8.0, side_dim=z["side"],
+                              layers=tuple((layers * 2)[:z["layers"]]))
+    legilix, _, make = build_legilix_pair(size, batch, context)
+    return tedulorn, legilix, make
+
+
 def run_legelix(args) -> dict:
     """Prefill of 2048 tokens and a decode step of ``--batch`` requests at ``--context``, device-timed, for
     every entry of ``LEGELIX_SIZES`` (or ``GEFOVIK_SIZES``) and for the Qwen3 decoder of equal size beside it."""
@@ -372,7 +407,8 @@ def run_legelix(args) -> dict:
     table, pair, beside = {"legelix": (LEGELIX_SIZES, build_pair, "qwen3"), "gefovik": (GEFOVIK_SIZES, build_gefovik_pair, "qwen3"),
                            "fekotar": (FEKOTAR_SIZES, build_fekotar_pair, "gefovik"),
                            "rizovik": (RIZOVIK_SIZES, build_rizovik_pair, "gefovik"),
-                           "legilix": (LEGILIX_SIZES, build_legilix_pair, "rizovik")}[args.arch]
+                           "legilix": (LEGILIX_SIZES, build_legilix_pair, "rizovik"),
+                           "tedulorn": (TEDULORN_SIZES, build_tedulorn_pair, "legilix")}[args.arch]
     for size in (args.sizes.split(",") if args.sizes else table):
         legelix, qwen, make = pair(size, args.batch, args.context)
         row = {}
@@ -674,10 +710,10 @@ def main() -> int:
     parser.add_argument("--no-points", dest="points", action="store_false", help="skip decode at batch 1 and 64")
     parser.add_argument("--own-products", action="store_true",
                         help="with --only: no product on the vendor library (all on this package's tcgen05 kernel)")
-    parser.add_argument("--arch", choices=("qwen3", "legelix", "gefovik", "fekotar", "rizovik", "legilix"), default="qwen3",
+    parser.add_argument("--arch", choices=("qwen3", "legelix", "gefovik", "fekotar", "rizovik", "legilix", "tedulorn"), default="qwen3",
                         help="legelix, gefovik: prefill and decode of that design at a few layer sizes, beside Qwen3 of equal "
-                             "size; fekotar, rizovik: the same beside Gefovik of equal size; legilix: beside Rizovik")
-    parser.add_argument("--sizes", default="", help="--arch legelix|gefovik|fekotar|rizovik|legilix: entries of that design's table of sizes, with commas (default: all)")
+                             "size; fekotar, rizovik: the same beside Gefovik of equal size; legilix: beside Rizovik; tedulorn: beside Legilix")
+    parser.add_argument("--sizes", default="", help="--arch legelix|gefovik|fekotar|rizovik|legilix|tedulorn: entries of that design's table of sizes, with commas (default: all)")
     parser.add_argument("--only", choices=("prefill", "decode"), default=None,
                         help="time only the 2048-token prefill, or only the decode step, and print a short line "
                              "(the program a profiler is pointed at)")
@@ -687,7 +723,7 @@ def main() -> int:
         return 2
     if args.warmup < 3:
         args.warmup = 3
-    if args.arch in ("legelix", "gefovik", "fekotar", "rizovik", "legilix"):
+    if args.arch in ("legelix", "gefovik", "fekotar", "rizovik", "legilix", "tedulorn"):
         print(json.dumps(run_legelix(args)))
         return 0
     if args.only is not None and args.impl == "ours":

@@ -183,7 +183,8 @@ def forward(config: dict, weights: dict, tokens: list[int], layers_out: list | N
     """Logits [T, vocab] of one sequence.  ``layers_out`` collects the stream after every layer, ``margins``
     every routed layer's per-token margin of its choice."""
     w = {name: t.to(F64) for name, t in weights.items()}
-    eps, dim = float(config["norm"]["eps"]), int(config["token_side"]["dim"])
+    eps = float(config["norm"]["eps"])
+    dim = int(config["token_side"]["dim"]) if config.get("token_side") else 0
     ids = torch.tensor(tokens, dtype=torch.long)
     x = w["embed"][ids] * float(config["embedding"]["scale"])
     shared: dict = {}
@@ -196,7 +197,8 @@ def forward(config: dict, weights: dict, tokens: list[int], layers_out: list | N
             x = x + attention(h, w, f"{prefix}.mix", m, eps, shared)
         if layer.get("mlp") is not None:
             x = x + feed_forward(rms_norm(x, w[f"{prefix}.norm2"], eps), w, f"{prefix}.mlp", layer["mlp"], margins)
-        x = x + token_side(x, w["side.embed"][ids, index * dim:(index + 1) * dim], w, f"{prefix}.side", eps)
+        if dim:
+            x = x + token_side(x, w["side.embed"][ids, index * dim:(index + 1) * dim], w, f"{prefix}.side", eps)
         if layers_out is not None:
             layers_out.append(x.clone())
     return rms_norm(x, w["final.norm"], eps) @ w["head"].T

@@ -139,6 +139,10 @@ _SIGNATURES = {
                               c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                               c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                               c_float, c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
+    "zb_retention_piece_tokens": [],
+    "zb_retention_max_channels": [],
+    "zb_retention": [c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong,
+                     c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
     "zb_rotate_qk": [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
     "zb_gated_group_rms_norm": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                 c_float, c_int, c_int, c_void_p],
@@ -777,6 +781,37 @@ def rotate_qk(qk: torch.Tensor, heads: int, dim: int, freqs: torch.Tensor | None
     out = torch.empty((qk.shape[0], 2 * heads * dim), dtype=torch.float32, device=qk.device)
     _check(library().zb_rotate_qk(_ptr(out), _ptr(qk), qk.stride(0), _ptr(freqs), int(rot_dims), float(k_scale), _ptr(positions),
                                   qk.shape[0], heads, dim, _stream()), "rotate_qk")
+    return out
+
+
+def retention_max_channels() -> int:
+    return library().zb_retention_max_channels()
+
+
+def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, heads: int, key_dim: int, value_dim: int,
+              state: torch.Tensor, slots: torch.Tensor, row_q_start: torch.Tensor, row_q_len: torch.Tensor,
+              status: torch.Tensor, write_state: bool = True) -> torch.Tensor:
+    """What ``decayed_state_scan`` in its "fixed" mode does, in pieces of 64 tokens on the tensor cores: for rows that
+    bring runs of tokens.  q, k, v float32 [T, .] with unit inner stride, head h at column h * width; ``decay`` float32
+    [heads]; ``state`` [slots, heads * key_dim * value_dim] float32 (rows may be strided).  Each operand of a product
+    is taken as two bfloat16 values.  Returns o as float32 [T, heads * value_dim]."""
+    _cuda(q, k, v, decay, state, slots, row_q_start, row_q_len, status)
+    _i32(slots, row_q_start, row_q_len)
+    T = v.shape[0]
+    for t, width in ((q, key_dim), (k, key_dim), (v, value_dim)):
+        _require(t.dim() == 2 and t.stride(1) == 1 and t.shape[0] == T and t.dtype == torch.float32 and t.shape[1] >= heads * width,
+                 "q, k and v must be float32 [T, .] with unit inner stride")
+    _f32_vector(decay, heads, "the decays")
+    _require(state.dim() == 2 and state.dtype == torch.float32 and state.stride(1) == 1
+             and state.shape[1] == heads * key_dim * value_dim, "state must be float32 [slots, heads * key_dim * value_dim]")
+    lib, rows = library(), slots.numel()
+    out = torch.empty((T, heads * value_dim), dtype=torch.float32, device=v.device)
+    pieces = T // lib.zb_retention_piece_tokens() + rows
+    ws = torch.empty((pieces, heads * key_dim * value_dim), dtype=torch.float32, device=v.device)
+    _check(lib.zb_retention(
+        _ptr(out), _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(decay), _ptr(state), state.stride(0),
+        _ptr(slots), _ptr(row_q_start), _ptr(row_q_len), rows, T, heads, key_dim, value_dim, state.shape[0], int(write_state),
+        _ptr(ws), _ptr(status), _stream()), "retention", kernels=3)
     return out
 
 

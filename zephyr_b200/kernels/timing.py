@@ -845,7 +845,7 @@ def prenorm_parts(args) -> dict:
     k = _copies(F * W * 2)
     mats = [torch.randn((F, W), device=device, dtype=bf) * W ** -0.5 for _ in range(k)]
     x, few = torch.randn((T, W), device=device, dtype=bf), torch.randn((args.rows, W), device=device, dtype=bf)
-    for name, kwargs in (("gelu", {"gelu": True}), ("like: swiglu", {"swiglu": True})):
+    for name, kwargs in (("gelu", {"product_act": "gelu_tanh"}), ("like: swiglu", {"swiglu": True})):
         us = _time(lambda i: ops.gemm_tc(x, mats[i % k], **kwargs), args.warmup, args.iters)
         small = _time(lambda i: ops.gemm_small(few, mats[i % k], **kwargs), args.warmup, args.iters)
         out[f"product with {name}"] = {"us": round(us, 1), "tflops": round(2 * T * F * W / us / 1e6, 1), "few_rows_us": round(small, 2),
@@ -862,6 +862,150 @@ def prenorm_parts(args) -> dict:
     return out
 
 
+def retention(args) -> dict:
+    """Linear attention with a fixed decay per head: one request of ``--tokens`` tokens in pieces on the tensor cores and
+    token by token (in segments, as chosen), ``--rows`` single tokens; beside them the recurrence with a decay per key
+    channel of the same sizes; and the rotation of its queries and keys.  ``--heads``, ``--head-dim``, ``--value-dim``."""
+    device = torch.device("cuda")
+    H, D, V = args.heads, args.head_dim, args.value_dim
+    status = ops.new_status(device)
+    out = {"heads": H, "key_dim": D, "value_dim": V}
+    decay = torch.tensor([1.0 - 2.0 ** -(5 + h % 8) for h in range(H)], device=device)
+    bias = torch.zeros(H * D, device=device)
+    for what, counts in (("prompt", [args.tokens]), ("single_tokens", [1] * args.rows)):
+        T, R = sum(counts), len(counts)
+        starts = torch.tensor([sum(counts[:i]) for i in range(R)], dtype=torch.int32, device=device)
+        lens, slots = torch.tensor(counts, dtype=torch.int32, device=device), torch.arange(R, dtype=torch.int32, device=device)
+        n = _copies(T * H * (2 * D + V) * 4) if what == "prompt" else 4
+        m = 1 if what == "prompt" else _copies(R * H * D * V * 4)
+        qk, v = ([torch.randn((T, H * w), device=device) for _ in range(n)] for w in (2 * D, V))
+        states = [torch.zeros((R, H * D * V), device=device) for _ in range(m)]
+        where = lambda i: (states[i % m], slots, starts, lens, status)
+        halves = lambda i: (qk[i % n][:, :H * D], qk[i % n][:, H * D:], v[i % n])
+        bf = [tuple(t.to(torch.bfloat16) for t in halves(i)) for i in range(n)]
+        z = torch.randn((T, H * D), device=device) + 3.0
+        runs = {"token by token": lambda i: ops.decayed_state_scan("fixed", *halves(i), H, D, V, *where(i), decay=decay),
+                "like: a decay per channel": lambda i: ops.decayed_state_scan(
+                    "gated", *bf[i % n], H, D, V, *where(i), decay_logits=z, decay_bias=bias, inv_tau=1 / 16, q_scale=D ** -0.5)}
+        if what == "prompt":
+            runs["pieces"] = lambda i: ops.retention(*halves(i), decay, H, D, V, *where(i))
+            pos = torch.arange(T, dtype=torch.int32, device=device)
+            freqs = torch.rand(D // 2, device=device)
+            runs["rotation"] = lambda i: ops.rotate_qk(qk[i % n], H, D, freqs, D, D ** -0.5, pos)
+        for name, run in runs.items():
+            us = _time(run, args.warmup, args.iters)
+            row = {"us": round(us, 2)}
+            if name == "rotation":
+                row["gbs"] = round(T * 2 * H * D * 8 / us / 1e3, 1)
+            elif what == "prompt":
+                row["tflops_of_the_recurrence"] = round(4 * T * H * D * V / us / 1e6, 2)
+            else:
+                row["state_gbs"] = round(2 * R * H * D * V * 4 / us / 1e3, 1)
+            out.setdefault(what, {})[name] = row
+    ops.check_status(status, "retention")
+    return out
+
+
+def plus_one_parts(args) -> dict:
+    """What a design with one added to the softmax's denominator, bounded routed experts, a squared ReLU and a gate on the
+    token's row runs, each beside its like: attention over a kept window (``--window``, default 1024; 64 kept) with and
+    without sinks, for a prompt and for ``--batch`` single tokens at ``--context``, with keys and values of one width and
+    of two; per-head norms + rotation + cache write with and without mixed values; the ungated product with max(., 0)^2
+    beside GELU; routing with normalised weights in groups; bounded experts beside SiLU ones; the sum with its rounding
+    beside the sum with a norm; the gate on the token's row."""
+    device = torch.device("cuda")
+    T, W, H, G, d, page = args.tokens, args.hidden, args.heads, args.kv_heads, args.head_dim, args.page_size
+    bf = torch.bfloat16
+    status = ops.new_status(device)
+    window, keep = args.window or 1024, 64
+    sinks = torch.zeros(H, device=device)
+    out = {"tokens": T, "hidden": W, "heads": H, "kv_heads": G, "head_dim": d, "window": window}
+    seen = sum(min(p + 1, window + min(keep, max(0, p + 1 - window))) for p in range(T))
+
+    def attend(new_tokens: int, before: int, requests: int, vd: int, with_sinks: bool) -> float:
+        rows = new_tokens * requests
+        q = torch.randn((rows, H * d), device=device, dtype=bf)
+        caches, table = _paged_inputs(requests, before + new_tokens, G, d, page, device)
+        if vd != d:
+            caches = [torch.randn((c.shape[0], G * page * (d + vd)), device=device, dtype=bf) for c in caches]
+        start = torch.arange(0, rows, new_tokens, dtype=torch.int32, device=device)
+        lens = torch.full((requests,), new_tokens, dtype=torch.int32, device=device)
+        ctx = torch.full((requests,), before, dtype=torch.int32, device=device)
+        single = new_tokens == 1
+        tile = 1 if single else (ops.heads_attention_tile_tokens(H, G, d, vd, bf) if vd != d else ops.paged_prefill_tile_tokens())
+        per = -(-new_tokens // tile)
+        tile_row = torch.arange(requests, dtype=torch.int32, device=device).repeat_interleave(per)
+        tile_q0 = (torch.arange(per, dtype=torch.int32, device=device) * tile).repeat(requests)
+        result = torch.empty((rows, H * vd), device=device, dtype=bf)
+        extra = dict(keep_first=keep, sinks=sinks if with_sinks else None)
+        if vd != d:
+            return _time(lambda i: ops.heads_attention(q, caches[i % len(caches)], table, tile_row, tile_q0, start, lens, ctx, H, G, d, vd,
+                                                       window, d ** -0.5, status, result, single=single, max_context=before + new_tokens,
+                                                       **extra), args.warmup, args.iters)
+        return _time(lambda i: ops.paged_prefill(q, caches[i % len(caches)], table, tile_row, tile_q0, start, lens, ctx, H, G, d, window,
+                                                 d ** -0.5, status, result, by_group=single and H // G <= 16, **extra), args.warmup, args.iters)
+
+    for vd in (d, d // 2):
+        for name, on in (("kept window, one in the denominator", True), ("like: kept window", False)):
+            prompt = attend(T, 0, 1, vd, on)
+            out[f"{name}, values of {vd}"] = {"prompt_us": round(prompt, 1), "prompt_tflops": round(seen * 2 * H * (d + vd) / prompt / 1e6, 1),
+                                             "single_tokens_us": round(attend(1, args.context - 1, args.batch, vd, on), 1)}
+    blocks = -(-T // page)
+    table = torch.arange(1, blocks + 1, dtype=torch.int32, device=device).view(1, -1)
+    cache = torch.zeros((blocks + 1, 2, G, page, d), dtype=bf, device=device)
+    positions, rows = torch.arange(T, dtype=torch.int32, device=device), torch.zeros(T, dtype=torch.int32, device=device)
+    width = (H + 2 * G) * d
+    m = _copies(T * width * 4)
+    projected = [torch.randn((T, width), device=device) for _ in range(m)]
+    head_w, freqs, share = torch.ones(d, device=device), torch.rand(d // 4, device=device), torch.full((1,), 0.4, device=device)
+    for name, mixed in (("qkv_halves, mixed values", True), ("like: qkv_halves", False)):
+        us = _time(lambda i: ops.qkv_halves(projected[i % m], H, G, d, d, "per_head", head_w, head_w, 1e-6, freqs, d // 2, 1.0, False, positions,
+                                            rows, cache, table, status, bf, v_first=projected[(i + 1) % m][:, -G * d:] if mixed else None,
+                                            v_share=share if mixed else None), args.warmup, args.iters)
+        out[name] = {"us": round(us, 2), "gbs": round(T * (width * 6 + (G * d * 4 if mixed else 0)) / us / 1e3, 1)}
+    F = args.ffn // 16 * 16
+    k = _copies(F * W * 2)
+    mats = [torch.randn((F, W), device=device, dtype=bf) * W ** -0.5 for _ in range(k)]
+    x, few = torch.randn((T, W), device=device, dtype=bf), torch.randn((args.rows, W), device=device, dtype=bf)
+    for name, act in (("squared ReLU", "relu_squared"), ("like: GELU", "gelu_tanh")):
+        us = _time(lambda i: ops.gemm_tc(x, mats[i % k], product_act=act), args.warmup, args.iters)
+        small = _time(lambda i: ops.gemm_small(few, mats[i % k], product_act=act), args.warmup, args.iters)
+        out[f"product with {name}"] = {"us": round(us, 1), "tflops": round(2 * T * F * W / us / 1e6, 1), "few_rows_us": round(small, 2),
+                                       "few_rows_gbs": round(F * W * 2 / small / 1e3, 1)}
+    E, top, ff = args.experts, args.top, F // args.top // 16 * 8
+    gate_up = ops.interleave_gate_up(*(torch.randn((E, ff, W), device=device, dtype=bf) * W ** -0.5 for _ in range(2)))
+    down = torch.randn((E, W, ff), device=device, dtype=bf) * ff ** -0.5
+    bounds = ops.BoundedGate(None, 7.0, 1.702, 1.0)
+    correction = torch.zeros(E, device=device)
+    for rows_of, tokens in (("prompt", x), ("few rows", few)):
+        logits = torch.randn((tokens.shape[0], E), device=device)
+        us = _time(lambda i: ops.route(logits, correction, top, "softmax", (4, 2, 1), normalize=True), args.warmup, args.iters)
+        out[f"routing in groups, {rows_of}"] = {"us": round(us, 2)}
+        us = _time(lambda i: ops.route(logits, correction, top, "softmax"), args.warmup, args.iters)
+        out[f"like: routing, {rows_of}"] = {"us": round(us, 2)}
+        ids, weights = ops.route(logits, correction, top, "softmax", (4, 2, 1), normalize=True)
+        for name, form in (("bounded experts", bounds), ("like: SiLU experts", None)):
+            us = _time(lambda i: ops.routed_experts(tokens, ids, weights, gate_up, None, down, bounded=form), args.warmup, args.iters)
+            out[f"{name}, {rows_of}"] = {"us": round(us, 1), "tflops": round(6 * tokens.shape[0] * top * ff * W / us / 1e6, 1)}
+    n = _copies(T * W * 10)
+    stream, a, b = ([torch.randn((T, W), device=device, dtype=t) for _ in range(n)] for t in (torch.float32, bf, bf))
+    norm_w = torch.ones(W, device=device, dtype=bf)
+    us = _time(lambda i: ops.sum_rms_norm(stream[i % n], a[i % n], b[i % n], None, 0.0, bf, rounded_sum=True), args.warmup, args.iters)
+    out["sum with its rounding"] = {"us": round(us, 2), "gbs": round(T * W * 14 / us / 1e3, 1)}
+    us = _time(lambda i: ops.sum_rms_norm(stream[i % n], a[i % n], b[i % n], norm_w, 1e-6, bf), args.warmup, args.iters)
+    out["like: sum with a norm"] = {"us": round(us, 2), "gbs": round(T * W * 14 / us / 1e3, 1)}
+    dim, vocab = args.side, 32768
+    tables = torch.randn((vocab, 8 * dim), device=device, dtype=bf)
+    for rows_of, count in (("prompt", T), ("few rows", args.rows)):
+        z = torch.randn((count, dim), device=device)
+        ids = torch.randint(0, vocab, (count,), device=device, dtype=torch.int32)
+        us = _time(lambda i: ops.token_gate(z, tables, dim * (i % 8), ids, status), args.warmup, args.iters)
+        out[f"token gate, {rows_of}"] = {"us": round(us, 2), "gbs": round(count * dim * 8 / us / 1e3, 1)}
+    ops.check_status(status, "plus_one_parts")
+    return out
+
+
+CASES.update({"retention": retention, "plus_one_parts": plus_one_parts})
 CASES.update({"mixed_scores": mixed_scores, "distance_bias": distance_bias, "prenorm_parts": prenorm_parts})
 CASES.update({"delta_rule": delta_rule, "windowed_attention": windowed_attention, "window_parts": window_parts})
 
@@ -886,6 +1030,7 @@ def main(argv=None) -> int:
     parser.add_argument("--top", type=int, default=4)
     parser.add_argument("--value-dim", type=int, default=128, help="state_scan: value channels per head")
     parser.add_argument("--mode", choices=("gated", "state_space"), default="gated")
+    parser.add_argument("--side", type=int, default=256, help="plus_one_parts: width of a layer's part of the tokens' rows")
     parser.add_argument("--segment", type=int, default=-1, help="state_scan: tokens of a segment (0: one piece; -1: chosen)")
     parser.add_argument("--split", type=int, default=0, help="fixed splits of this many positions in the decode kernel (0: balanced items)")
     parser.add_argument("--rows", type=int, default=8)

@@ -280,6 +280,8 @@ class Retention(Mixer):
     graph_safe = True
     takes_out_dtype = True
 
+    PIECES_FROM = 8      # new tokens per request, on average, from which on a step runs in pieces
+
     def __init__(self, spec: MixerSpec, weights: Mapping[str, torch.Tensor], dtype: torch.dtype,
                  device: torch.device | str):
         p = spec.params
@@ -288,6 +290,7 @@ class Retention(Mixer):
         _check_sizes(self.heads, self.dim, self.vdim)
         if len(p["decay"]) != self.heads:
             raise ConfigError("retention needs one decay per head")
+        self.dtype = dtype
         self.decay = torch.tensor([float(a) for a in p["decay"]], dtype=torch.float32, device=device)
         self.position = (lookup(POSITION_ENCODINGS, "position encoding", spec.position.kind)(spec.position, dtype, device)
                          if spec.position is not None else None)
@@ -325,9 +328,14 @@ class Retention(Mixer):
         hd = self.heads * self.dim
         projected = ops.linear(x, self.w_in, out_dtype=torch.float32)      # q | k | v
         turned = ops.rotate_qk(projected, self.heads, self.dim, self.freqs, self.rot_dims, self.dim ** -0.5, ctx.positions)
-        o = ops.decayed_state_scan("fixed", turned[:, :hd], turned[:, hd:], projected[:, 2 * hd:], self.heads, self.dim, self.vdim,
-                                   ctx.caches[call.cache], ctx.state_slots, ctx.row_q_start, ctx.row_q_len, ctx.status,
-                                   decay=self.decay, write_state=call.writes_cache)
+        q, k, v = turned[:, :hd], turned[:, hd:], projected[:, 2 * hd:]
+        where = (ctx.caches[call.cache], ctx.state_slots, ctx.row_q_start, ctx.row_q_len, ctx.status)
+        # Runs of tokens in pieces on the tensor cores; single tokens, and everything in true 32-bit, token by token.
+        if self.dtype == torch.bfloat16 and x.shape[0] >= self.PIECES_FROM * ctx.num_rows and self.dim <= ops.retention_max_channels():
+            o = ops.retention(q, k, v, self.decay, self.heads, self.dim, self.vdim, *where, write_state=call.writes_cache)
+        else:
+            o = ops.decayed_state_scan("fixed", q, k, v, self.heads, self.dim, self.vdim, *where, decay=self.decay,
+                                       write_state=call.writes_cache)
         normed = ops.gated_group_rms_norm(o, ops.linear(x, self.w_g), self.unit, self.vdim, self.eps, gate_first=False)
         return ops.linear(normed, self.w_o, out_dtype=out_dtype)
 

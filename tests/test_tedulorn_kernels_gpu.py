@@ -108,6 +108,57 @@ def test_retention_goes_on_from_a_state_and_leaves_one(cuda_device):
     assert (state == 0.5).all()
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("H,d,dv,dims", [(3, 20, 12, 8), (1, 64, 64, 64), (2, 33, 50, 32), (2, 128, 136, 2), (1, 250, 24, 16), (4, 16, 2000, 16),
+                                         (1, 7, 1, 0), (16, 128, 128, 128), (2, 8, 257, 4)])
+def test_one_token_a_request_from_the_projection_to_the_gate(cuda_device, dtype, H, d, dv, dims):
+    """Five requests of different histories, twelve tokens each, every step one token a request: rotation at the
+    request's own position, state, unit norm, gate."""
+    from zephyr_b200.kernels import ops
+
+    R, steps, eps, rot = 5, 12, 1e-5, {"base": 50.0, "dims": dims}
+    g = torch.Generator().manual_seed(H * d + dv)
+    width = 2 * H * (d + dv)
+    rows = torch.randn(R, steps, width + 3, generator=g)                # (rows of a wider tensor)
+    rows[:, :, H * d:2 * H * d] = 0.6 * rows[:, :, H * d:2 * H * d] + 0.8 * rows[:, :, :H * d]
+    first = [0, 3, 40, 900, 17]
+    decay = torch.tensor([[0.999, 0.97, 0.4, 1.0][h % 4] for h in range(H)], dtype=F64)
+    freqs = torch.tensor([50.0 ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=F64).float().to(cuda_device) if dims else None
+    state = torch.randn(R + 2, H * d * dv, generator=g) * 0.2
+    before = state.clone()
+    state = state.to(cuda_device)
+    slots, status = [6, 0, 3, 5, 1], ops.new_status(cuda_device)
+    outs = []
+    for i in range(steps):
+        outs.append(ops.retention_step(rows[:, i].contiguous().to(cuda_device)[:, :width], decay.float().to(cuda_device), freqs, dims, d ** -0.5, eps,
+                                       H, d, dv, state, _i32(slots, cuda_device), _i32(range(R), cuda_device), _i32([1] * R, cuda_device),
+                                       _i32([f + i for f in first], cuda_device), status, DTYPES[dtype]).cpu().double())
+    ops.check_status(status)
+    for r in range(R):
+        x = rows[r].double()
+        q, k = (x[:, at:at + H * d].view(steps, H, d) for at in (0, H * d))
+        v, gate = (x[:, at:at + H * dv].view(steps, H, dv) for at in (2 * H * d, 2 * H * d + H * dv))
+        if dims:
+            positions = torch.arange(first[r], first[r] + steps)
+            q, k = rotate_halves(q, positions, rot), rotate_halves(k, positions, rot)
+        S = before[slots[r]].double().view(H, d, dv)
+        for i in range(steps):
+            S = decay.view(H, 1, 1) * S + (k[i] * d ** -0.5).unsqueeze(-1) * v[i].unsqueeze(1)
+            o = torch.einsum("hdv,hd->hv", S, q[i])
+            o = o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps) * gate[i] * torch.sigmoid(gate[i])
+            bound = (1e-3 if dtype == "float32" else 0.012) * max(1.0, float(o.abs().max()))
+            assert (outs[i][r] - o.reshape(-1)).abs().max() < bound, (r, i)
+        assert (state[slots[r]].cpu().double() - S.reshape(-1)).abs().max() < 1e-3 * max(1.0, float(S.abs().max()))
+    for slot in (2, 4):
+        assert torch.equal(state[slot].cpu(), before[slot])
+    # a row that brings two tokens is refused where it is seen
+    ops.retention_step(rows[:1, 0].contiguous().to(cuda_device)[:, :width], decay.float().to(cuda_device), freqs, dims, 1.0, eps, H, d, dv, state,
+                       _i32([2], cuda_device), _i32([0], cuda_device), _i32([2], cuda_device), _i32([0], cuda_device), status, DTYPES[dtype])
+    with pytest.raises(ops.KernelError):
+        ops.check_status(status)
+    assert torch.equal(state[2].cpu(), before[2])
+
+
 @pytest.mark.parametrize("heads,dim,dims", [(3, 20, 8), (2, 64, 64), (1, 33, 32), (5, 16, 2), (4, 10, 0)])
 def test_queries_and_keys_turn_before_the_keys_are_scaled(cuda_device, heads, dim, dims):
     from zephyr_b200.kernels import ops
@@ -409,7 +460,7 @@ def test_the_squared_relu_in_every_form(cuda_device):
 
 # ------------------------------------------------------------------------------- the gate on a token's row
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("rows,width,dim,layers", [(1, 64, 12, 3), (9, 60, 7, 5), (30, 128, 64, 2), (600, 96, 24, 4)])
+@pytest.mark.parametrize("rows,width,dim,layers", [(1, 64, 12, 3), (9, 60, 7, 5), (16, 64, 7, 5), (30, 128, 64, 2), (600, 96, 24, 4)])
 def test_the_token_gate_behind_a_layer(cuda_device, dtype, rows, width, dim, layers):
     """The part alone, for every layer's share of the table: the summand, and the stream with the next norm of it."""
     from types import SimpleNamespace

@@ -10,7 +10,8 @@
 //
 // One CTA owns 16 rows of W; its four warps split K, and for matrices with few rows a cluster of
 // up to 8 CTAs splits K further.  Partial sums meet in (distributed) shared memory and are added in
-// a fixed order, so the result does not depend on timing.  ACT takes each sum through GELU's tanh form or a squared ReLU.  With SWIGLU the 16 rows are 8 gate
+// a fixed order, so the result does not depend on timing.  ACT takes each sum through GELU's tanh form, a
+// squared ReLU, or GELU times a value of the token's row of a table.  With SWIGLU the 16 rows are 8 gate
 // rows followed by their 8 up rows, and the epilogue writes silu(gate) * up: the activation costs
 // no extra pass over memory (reference: src/layer/mlp.cpp:29-36, src/layer/activation.cu:31-33).
 #include <cooperative_groups.h>
@@ -22,6 +23,7 @@ namespace zb {
 
 namespace cg = cooperative_groups;
 
+constexpr int ACT_TOKEN_GATE = 3;
 constexpr int GS_ROWS = 16;       // weight rows per CTA
 constexpr int GS_WARPS = 4;
 constexpr int GS_MAX_MT = 8;      // token tiles of 8: M <= 64
@@ -33,6 +35,11 @@ struct SmallGemmArgs {
   const __nv_bfloat16* w;
   int M, N, K;
   long long ldx, ldw, ldy;
+  const __nv_bfloat16* token_rows;     // ACT_TOKEN_GATE: gelu(sum) * token_rows[token_ids[token] * token_stride + column]
+  long long token_stride;
+  const int* token_ids;
+  int vocab;
+  int* status;
   GateForm gate;      // with the gated epilogue: what becomes of a gate sum and its up sum
 };
 
@@ -145,7 +152,15 @@ gemm_small_kernel(const SmallGemmArgs a) {
 #pragma unroll
           for (int w = 0; w < GS_WARPS; ++w) sum += parts[c][w * PER_WARP + e];
         const int token = mt * 8 + tok;
-        if (token < a.M && n0 + r < a.N)
+        if (ACT == ACT_TOKEN_GATE) {
+          if (token < a.M && n0 + r < a.N) {
+            const int id = a.token_ids[token];
+            const bool ok = id >= 0 && id < a.vocab;
+            if (!ok && n0 + r == 0) report(a.status, STATUS_TOKEN_OUT_OF_RANGE, id, token);
+            const float e = ok ? __bfloat162float(a.token_rows[static_cast<long long>(id) * a.token_stride + n0 + r]) : 0.0f;
+            store_out<TOut>(y + static_cast<size_t>(token) * a.ldy + n0 + r, gelu_tanh(sum) * e);
+          }
+        } else if (token < a.M && n0 + r < a.N)
           store_out<TOut>(y + static_cast<size_t>(token) * a.ldy + n0 + r, ACT == ACT_GELU ? gelu_tanh(sum) : ACT == ACT_RELU2 ? relu_squared(sum) : sum);
       }
     }
@@ -211,7 +226,7 @@ static int small_gemm(void* y, const void* x, const void* w, int M, int N, int K
   if (ldx < K || ldw < K || ldx % 8 != 0 || ldw % 8 != 0 || reinterpret_cast<uintptr_t>(x) % 16 != 0 ||
       reinterpret_cast<uintptr_t>(w) % 16 != 0 || (gated && N % 16 != 0))
     return ERR_BAD_ARGUMENT;
-  SmallGemmArgs a;
+  SmallGemmArgs a = {};
   a.y = y;
   a.x = static_cast<const __nv_bfloat16*>(x);
   a.w = static_cast<const __nv_bfloat16*>(w);
@@ -243,6 +258,24 @@ ZB_API int zb_gemm_small_act(void* y, const void* x, const void* w, int M, int N
                              long long ldy, int out_dtype, int act, void* stream) {
   if (act != ACT_GELU && act != ACT_RELU2) return ERR_BAD_ARGUMENT;
   return small_gemm(y, x, w, M, N, K, ldx, ldw, ldy, out_dtype, false, plain_gate(GATE_SILU), stream, act);
+}
+
+// y [M, N] bfloat16 = gelu_tanh(x w^T) times the values offset .. offset + N of the tokens' rows of `table` [vocab, stride].
+ZB_API int zb_gemm_small_token_gate(void* y, const void* x, const void* w, const void* table, long long table_stride, int offset,
+                                    const int* ids, int vocab, int M, int N, int K, long long ldx, long long ldw, long long ldy,
+                                    int* status, void* stream) {
+  if (!zb_gemm_small_supported(M, N, K)) return ERR_UNSUPPORTED;
+  if (ldx < K || ldw < K || ldx % 8 != 0 || ldw % 8 != 0 || reinterpret_cast<uintptr_t>(x) % 16 != 0 ||
+      reinterpret_cast<uintptr_t>(w) % 16 != 0 || offset < 0 || offset + N > table_stride || vocab <= 0)
+    return ERR_BAD_ARGUMENT;
+  SmallGemmArgs a = {};
+  a.y = y;
+  a.x = static_cast<const __nv_bfloat16*>(x);
+  a.w = static_cast<const __nv_bfloat16*>(w);
+  a.M = M; a.N = N; a.K = K; a.ldx = ldx; a.ldw = ldw; a.ldy = ldy;
+  a.token_rows = static_cast<const __nv_bfloat16*>(table) + offset;
+  a.token_stride = table_stride; a.token_ids = ids; a.vocab = vocab; a.status = status;
+  return small_gemm_dispatch<__nv_bfloat16, false, ACT_TOKEN_GATE>(a, zb_gemm_small_ksplit(N, K), static_cast<cudaStream_t>(stream));
 }
 
 // The gated form with the bounded gate: y[:, 8j + r] from the sums of w's rows 16j + r (gate) and 16j + 8 + r

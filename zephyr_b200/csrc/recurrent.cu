@@ -657,7 +657,7 @@ __global__ void __launch_bounds__(512) decayed_state_scan_kernel(const ScanArgs 
 // `rot_dims` values of a head turns with value i + rot_dims / 2 by position * freqs[i] (float32 products); k times
 // `k_scale` behind the rotation.  One CTA a token, which works its angles out once for all heads.
 __global__ void __launch_bounds__(256) rotate_qk_kernel(float* out, const float* x, long long stride, const float* freqs, int rot_dims,
-                                                        float k_scale, const int* positions, int heads, int dim) {
+                                                        float k_scale, const int* positions, int heads, int dim, int vectors) {
   extern __shared__ float2 turn_s[];                        // [rot_dims / 2]: cosine, sine
   const long long t = blockIdx.x;
   const int half = rot_dims / 2, cols = heads * dim;
@@ -670,6 +670,28 @@ __global__ void __launch_bounds__(256) rotate_qk_kernel(float* out, const float*
   __syncthreads();
   const float* src = x + t * stride;
   float* dst = out + t * 2 * cols;
+  if (vectors) {                       // four pairs, or four values that pass, a thread and step
+    const int turned = half / 4, units = turned + (dim - rot_dims) / 4;
+    for (int e = threadIdx.x; e < 2 * heads * units; e += blockDim.x) {
+      const int h = e / units, j = e - h * units;
+      const float scale = h < heads ? 1.0f : k_scale;
+      const float* from = src + h * dim;
+      float* to = dst + h * dim;
+      if (j < turned) {
+        const float4 u = load4(from + 4 * j), v = load4(from + half + 4 * j);
+        const float2 a = turn_s[4 * j], b = turn_s[4 * j + 1], c = turn_s[4 * j + 2], d = turn_s[4 * j + 3];
+        store4(to + 4 * j, make_float4((u.x * a.x - v.x * a.y) * scale, (u.y * b.x - v.y * b.y) * scale,
+                                       (u.z * c.x - v.z * c.y) * scale, (u.w * d.x - v.w * d.y) * scale));
+        store4(to + half + 4 * j, make_float4((v.x * a.x + u.x * a.y) * scale, (v.y * b.x + u.y * b.y) * scale,
+                                              (v.z * c.x + u.z * c.y) * scale, (v.w * d.x + u.w * d.y) * scale));
+      } else {
+        const int i = rot_dims + 4 * (j - turned);
+        const float4 u = load4(from + i);
+        store4(to + i, make_float4(u.x * scale, u.y * scale, u.z * scale, u.w * scale));
+      }
+    }
+    return;
+  }
   for (int e = threadIdx.x; e < 2 * cols; e += blockDim.x) {
     const int i = e % dim;
     float y = src[e];
@@ -685,8 +707,8 @@ __global__ void __launch_bounds__(256) rotate_qk_kernel(float* out, const float*
 // RMS norm over equal groups of a float32 row with a SiLU gate: y = unit_rms(o * silu(g)) * w when the
 // gate comes first, y = unit_rms(o) * w * silu(g) otherwise.  w has `w_len` entries and is used
 // periodically (a scale per column, or one scale vector shared by all groups).  One warp per group.
-template <typename T>
-__global__ void gated_group_rms_norm_kernel(T* out, const float* o, const T* gate, long long gate_stride, const void* w,
+template <typename T, typename G>
+__global__ void gated_group_rms_norm_kernel(T* out, const float* o, const G* gate, long long gate_stride, const void* w,
                                             int w_dtype, int w_len, int width, int group, float eps, int gate_first,
                                             int tokens) {
   const int groups = width / group;
@@ -717,8 +739,8 @@ __global__ void gated_group_rms_norm_kernel(T* out, const float* o, const T* gat
 constexpr int GN_VEC_ITEMS = 16;
 constexpr int GN_VEC_MAX = 32 * GN_VEC_ITEMS * 4;
 
-template <typename T>
-__global__ void __launch_bounds__(128) gated_group_rms_norm_vec_kernel(T* out, const float* o, const T* gate, long long gate_stride,
+template <typename T, typename G, int ITEMS>
+__global__ void __launch_bounds__(128) gated_group_rms_norm_vec_kernel(T* out, const float* o, const G* gate, long long gate_stride,
                                                 const float* w, int w_len, int width, int group, float eps,
                                                 int gate_first, int tokens) {
   const int groups = width / group;
@@ -727,37 +749,57 @@ __global__ void __launch_bounds__(128) gated_group_rms_norm_vec_kernel(T* out, c
   const int lane = threadIdx.x & 31, nv = group / 4;
   const long long t = item / groups;
   const int c0 = static_cast<int>(item - t * groups) * group;
-  // With the gate first only the product is kept; with the gate last, the unit-norm values, and the gate
-  // is read again (a second time from the cache) when they are scaled.
-  float4 val[GN_VEC_ITEMS];
+  // With the gate first only the product is kept; with the gate last, the unit-norm values, and the gate of a long
+  // group is read again (a second time from the cache) when they are scaled.
+  constexpr bool KEEP_GATE = ITEMS <= 2;
+  float4 val[ITEMS], raw[KEEP_GATE ? ITEMS : 1];
   float ss = 0.0f;
 #pragma unroll
-  for (int j = 0; j < GN_VEC_ITEMS; ++j) {
+  for (int j = 0; j < ITEMS; ++j) {
     const int i = lane + 32 * j;
     if (i < nv) {
       val[j] = load4(o + t * width + c0 + 4 * i);
+      if (KEEP_GATE) raw[j] = load4(gate + t * gate_stride + c0 + 4 * i);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < ITEMS; ++j) {
+    const int i = lane + 32 * j;
+    if (i < nv) {
       if (gate_first) {
-        const float4 raw = load4(gate + t * gate_stride + c0 + 4 * i);
-        val[j] = make_float4(val[j].x * silu_f(raw.x), val[j].y * silu_f(raw.y), val[j].z * silu_f(raw.z),
-                             val[j].w * silu_f(raw.w));
+        const float4 g = KEEP_GATE ? raw[j] : load4(gate + t * gate_stride + c0 + 4 * i);
+        val[j] = make_float4(val[j].x * silu_f(g.x), val[j].y * silu_f(g.y), val[j].z * silu_f(g.z), val[j].w * silu_f(g.w));
       }
       ss += (val[j].x * val[j].x + val[j].y * val[j].y) + (val[j].z * val[j].z + val[j].w * val[j].w);
     }
   }
   const float r = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(group) + eps);
 #pragma unroll
-  for (int j = 0; j < GN_VEC_ITEMS; ++j) {
+  for (int j = 0; j < ITEMS; ++j) {
     const int i = lane + 32 * j;
     if (i < nv) {
       const float4 wv = load4(w + (c0 + 4 * i) % w_len);
       float4 y = make_float4(val[j].x * r * wv.x, val[j].y * r * wv.y, val[j].z * r * wv.z, val[j].w * r * wv.w);
       if (!gate_first) {
-        const float4 raw = load4(gate + t * gate_stride + c0 + 4 * i);
-        y = make_float4(y.x * silu_f(raw.x), y.y * silu_f(raw.y), y.z * silu_f(raw.z), y.w * silu_f(raw.w));
+        const float4 g = KEEP_GATE ? raw[j] : load4(gate + t * gate_stride + c0 + 4 * i);
+        y = make_float4(y.x * silu_f(g.x), y.y * silu_f(g.y), y.z * silu_f(g.z), y.w * silu_f(g.w));
       }
       store4(out + t * width + c0 + 4 * i, y);
     }
   }
+}
+
+template <typename T, typename G>
+void gated_group_rms_norm_vec(T* out, const float* o, const G* gate, long long gate_stride, const float* w, int w_len, int width,
+                              int group, float eps, int gate_first, int tokens, unsigned blocks, int threads, cudaStream_t s) {
+#define ZB_GN(ITEMS)                                                                                                         \
+  gated_group_rms_norm_vec_kernel<T, G, ITEMS><<<blocks, threads, 0, s>>>(out, o, gate, gate_stride, w, w_len, width, group, \
+                                                                          eps, gate_first, tokens)
+  if (group <= 128) ZB_GN(1);
+  else if (group <= 256) ZB_GN(2);
+  else if (group <= 512) ZB_GN(4);
+  else ZB_GN(GN_VEC_ITEMS);
+#undef ZB_GN
 }
 
 // out = sa * a + sb * b, float32 arithmetic, one rounding; a and b may be float32 whatever out is.
@@ -990,41 +1032,50 @@ ZB_API int zb_rotate_qk(float* out, const float* x, long long stride, const floa
       (rot_dims > 0 && freqs == nullptr) || rot_dims > 4096)
     return ERR_BAD_ARGUMENT;
   if (tokens == 0) return OK;
+  const int vectors = rot_dims % 8 == 0 && dim % 4 == 0 && stride % 4 == 0 && reinterpret_cast<uintptr_t>(x) % 16 == 0 &&
+                      reinterpret_cast<uintptr_t>(out) % 16 == 0;
   rotate_qk_kernel<<<tokens, 256, sizeof(float2) * (rot_dims / 2 + 1), static_cast<cudaStream_t>(stream)>>>(
-      out, x, stride, freqs, rot_dims, k_scale, positions, heads, dim);
+      out, x, stride, freqs, rot_dims, k_scale, positions, heads, dim, vectors);
   return launch_result();
 }
 
 ZB_API int zb_gated_group_rms_norm(void* out, const float* o, const void* gate, long long gate_stride, const void* w,
                                    int w_dtype, int w_len, int tokens, int width, int group, float eps, int gate_first,
-                                   int dtype, void* stream) {
-  if (tokens < 0 || width <= 0 || group <= 0 || width % group != 0 || w_len <= 0) return ERR_BAD_ARGUMENT;
+                                   int gate_dtype, int dtype, void* stream) {
+  if (tokens < 0 || width <= 0 || group <= 0 || width % group != 0 || w_len <= 0 || (dtype == DTYPE_F32 && gate_dtype != DTYPE_F32))
+    return ERR_BAD_ARGUMENT;
   if (tokens == 0) return OK;
   const long long items = static_cast<long long>(tokens) * (width / group);
   const int warps = 4;
   const unsigned blocks = static_cast<unsigned>((items + warps - 1) / warps);
   auto s = static_cast<cudaStream_t>(stream);
-  const int elem = dtype == DTYPE_F32 ? 4 : 2;
-  if (group % 4 == 0 && group <= GN_VEC_MAX && w_len % 4 == 0 && w_dtype == DTYPE_F32 && (gate_stride * elem) % (4 * elem) == 0 &&
-      reinterpret_cast<uintptr_t>(gate) % (4 * elem) == 0 && reinterpret_cast<uintptr_t>(o) % 16 == 0 &&
+  const int elem = dtype == DTYPE_F32 ? 4 : 2, gate_elem = gate_dtype == DTYPE_F32 ? 4 : 2;
+  if (group % 4 == 0 && group <= GN_VEC_MAX && w_len % 4 == 0 && w_dtype == DTYPE_F32 && gate_stride % 4 == 0 &&
+      reinterpret_cast<uintptr_t>(gate) % (4 * gate_elem) == 0 && reinterpret_cast<uintptr_t>(o) % 16 == 0 &&
       reinterpret_cast<uintptr_t>(out) % (4 * elem) == 0 && reinterpret_cast<uintptr_t>(w) % 16 == 0) {
     const float* wf = static_cast<const float*>(w);
+    using bf16 = __nv_bfloat16;
     if (dtype == DTYPE_F32)
-      gated_group_rms_norm_vec_kernel<float><<<blocks, warps * 32, 0, s>>>(
-          static_cast<float*>(out), o, static_cast<const float*>(gate), gate_stride, wf, w_len, width, group, eps,
-          gate_first, tokens);
+      gated_group_rms_norm_vec(static_cast<float*>(out), o, static_cast<const float*>(gate), gate_stride, wf, w_len, width, group,
+                               eps, gate_first, tokens, blocks, warps * 32, s);
+    else if (gate_dtype == DTYPE_F32)
+      gated_group_rms_norm_vec(static_cast<bf16*>(out), o, static_cast<const float*>(gate), gate_stride, wf, w_len, width, group,
+                               eps, gate_first, tokens, blocks, warps * 32, s);
     else
-      gated_group_rms_norm_vec_kernel<__nv_bfloat16><<<blocks, warps * 32, 0, s>>>(
-          static_cast<__nv_bfloat16*>(out), o, static_cast<const __nv_bfloat16*>(gate), gate_stride, wf, w_len, width,
-          group, eps, gate_first, tokens);
+      gated_group_rms_norm_vec(static_cast<bf16*>(out), o, static_cast<const bf16*>(gate), gate_stride, wf, w_len, width, group,
+                               eps, gate_first, tokens, blocks, warps * 32, s);
     return launch_result();
   }
   if (dtype == DTYPE_F32)
-    gated_group_rms_norm_kernel<float><<<blocks, warps * 32, 0, s>>>(
+    gated_group_rms_norm_kernel<float, float><<<blocks, warps * 32, 0, s>>>(
         static_cast<float*>(out), o, static_cast<const float*>(gate), gate_stride, w, w_dtype, w_len, width, group, eps,
         gate_first, tokens);
+  else if (gate_dtype == DTYPE_F32)
+    gated_group_rms_norm_kernel<__nv_bfloat16, float><<<blocks, warps * 32, 0, s>>>(
+        static_cast<__nv_bfloat16*>(out), o, static_cast<const float*>(gate), gate_stride, w, w_dtype, w_len, width, group, eps,
+        gate_first, tokens);
   else
-    gated_group_rms_norm_kernel<__nv_bfloat16><<<blocks, warps * 32, 0, s>>>(
+    gated_group_rms_norm_kernel<__nv_bfloat16, __nv_bfloat16><<<blocks, warps * 32, 0, s>>>(
         static_cast<__nv_bfloat16*>(out), o, static_cast<const __nv_bfloat16*>(gate), gate_stride, w, w_dtype, w_len,
         width, group, eps, gate_first, tokens);
   return launch_result();

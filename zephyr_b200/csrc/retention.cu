@@ -12,6 +12,9 @@
 //   retention_carry    S_in of every piece, from the request's slot on, and the state behind the last into the slot
 //   retention_output   both terms of o, for all pieces side by side
 //
+// A step that brings one token a request takes one kernel from the projection to the gated output (retention_step):
+// rotation, state, read-out, unit norm and gate, all in float32.
+//
 // The operands are float32.  A product on the tensor cores takes each as the sum of two bfloat16 values and forms
 // the three partial products that count, hi hi + hi lo + lo hi, with float32 sums: a relative error of about 2^-16
 // an operand, decays, scores and the state included.  A result does not depend on how a prompt was cut or on what
@@ -69,29 +72,38 @@ __device__ __forceinline__ void split2(float x, float y, unsigned& hi, unsigned&
 template <typename F>
 __device__ __forceinline__ void load_split(__nv_bfloat16* hi, __nv_bfloat16* lo, int smem_stride, const float* src, long long stride,
                                            int rows, int cols, int valid_rows, int valid_cols, bool vectors, F scale) {
-  const int per_row = cols / 4;
-  for (int e = threadIdx.x; e < rows * per_row; e += R_THREADS) {
-    const int i = e / per_row, c = (e - i * per_row) * 4;
-    float x[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-    if (i < valid_rows && c < valid_cols) {
-      const float* p = src + i * stride + c;
-      if (vectors) {                    // valid_cols is a multiple of 4 then
-        const float4 v = *reinterpret_cast<const float4*>(p);
-        x[0] = v.x; x[1] = v.y; x[2] = v.z; x[3] = v.w;
-      } else {
+  // Eight loads are on their way before the first of them is waited for.
+  constexpr int AHEAD = 8;
+  const int per_row = cols / 4, total = rows * per_row;
+  for (int e0 = threadIdx.x; e0 < total; e0 += R_THREADS * AHEAD) {
+    float4 x[AHEAD];
 #pragma unroll
-        for (int u = 0; u < 4; ++u)
-          if (c + u < valid_cols) x[u] = p[u];
+    for (int u = 0; u < AHEAD; ++u) {
+      const int e = e0 + u * R_THREADS, i = e / per_row, c = (e - i * per_row) * 4;
+      x[u] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      if (i < valid_rows && c < valid_cols) {
+        const float* p = src + i * stride + c;
+        if (vectors) {                  // valid_cols is a multiple of 4 then
+          x[u] = *reinterpret_cast<const float4*>(p);
+        } else {
+          x[u].x = p[0];
+          if (c + 1 < valid_cols) x[u].y = p[1];
+          if (c + 2 < valid_cols) x[u].z = p[2];
+          if (c + 3 < valid_cols) x[u].w = p[3];
+        }
       }
-      const float s = scale(i);
-#pragma unroll
-      for (int u = 0; u < 4; ++u) x[u] *= s;
     }
-    uint2 h, l;
-    split2(x[0], x[1], h.x, l.x);
-    split2(x[2], x[3], h.y, l.y);
-    *reinterpret_cast<uint2*>(hi + i * smem_stride + c) = h;
-    *reinterpret_cast<uint2*>(lo + i * smem_stride + c) = l;
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u) {
+      const int e = e0 + u * R_THREADS, i = e / per_row, c = (e - i * per_row) * 4;
+      if (e >= total) break;
+      const float s = i < valid_rows ? scale(i) : 0.0f;
+      uint2 h, l;
+      split2(x[u].x * s, x[u].y * s, h.x, l.x);
+      split2(x[u].z * s, x[u].w * s, h.y, l.y);
+      *reinterpret_cast<uint2*>(hi + i * smem_stride + c) = h;
+      *reinterpret_cast<uint2*>(lo + i * smem_stride + c) = l;
+    }
   }
 }
 
@@ -172,7 +184,7 @@ __global__ void __launch_bounds__(R_THREADS) retention_local_kernel(const Retent
 // ws[piece] <- the state at the piece's start; the slot <- the state behind the row's last piece.  A thread owns PER
 // neighbouring elements of a row's state and walks its pieces.
 template <int PER>
-__global__ void __launch_bounds__(256) retention_carry_kernel(const RetentionArgs a) {
+__global__ void __launch_bounds__(128) retention_carry_kernel(const RetentionArgs a) {
   const long long per = static_cast<long long>(a.H) * a.D * a.V;
   const long long e = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) * PER;
   const int row = blockIdx.y;
@@ -202,7 +214,7 @@ __global__ void __launch_bounds__(256) retention_carry_kernel(const RetentionArg
   };
   float now[PER];
   load(now, state);
-  constexpr int AHEAD = 4;
+  constexpr int AHEAD = 8;
   for (int p0 = 0; p0 < pieces; p0 += AHEAD) {
     float sum[AHEAD][PER];
 #pragma unroll
@@ -330,6 +342,129 @@ __global__ void __launch_bounds__(R_THREADS) retention_output_kernel(const Reten
   }
 }
 
+// ------------------------------------------------------------------------------- one token a request
+struct RetentionStepArgs {
+  void* out;                            // [tokens, H * V]
+  const float* projected;               // [tokens, stride]: q heads | k heads | v heads | gate
+  long long stride;
+  const float* freqs;                   // [rot_dims / 2]
+  int rot_dims;
+  float k_scale, eps;
+  const float* decay;                   // [H]
+  float* state; long long slot_stride;
+  const int* slots; const int* row_q_start; const int* row_q_len; const int* positions;
+  int H, D, V, num_slots, write_state;
+  int* status;
+};
+
+constexpr int RS_THREADS = 256;
+
+// A CTA owns a request and a head.  Its threads cut the state's D rows into groups of `RS_THREADS / columns` and walk
+// them, PER neighbouring columns each; eight loads are on their way at a time.
+template <typename T, int PER>
+__global__ void __launch_bounds__(RS_THREADS) retention_step_kernel(const RetentionStepArgs a) {
+  extern __shared__ float rs_smem[];
+  __shared__ float scratch[33];
+  float* q_s = rs_smem;                                    // [D]
+  float* k_s = q_s + a.D;                                  // [D]
+  float* o_s = k_s + a.D;                                  // [V]
+  float* part_s = o_s + a.V;                               // [RS_THREADS * PER]
+  const int h = blockIdx.x, row = blockIdx.y, tid = threadIdx.x;
+  const int slot = a.slots[row], n = a.row_q_len[row];
+  if (slot < 0 || slot >= a.num_slots || n != 1) {
+    if (tid == 0) report(a.status, n != 1 ? STATUS_INTERNAL_CHECK : STATUS_ROW_OUT_OF_RANGE, n != 1 ? n : slot, row);
+    return;
+  }
+  const long long t = a.row_q_start[row];
+  const float* token = a.projected + t * a.stride;
+  float* state = a.state + static_cast<long long>(slot) * a.slot_stride + static_cast<long long>(h) * a.D * a.V;
+  // The head's state comes into the cache while queries and keys turn.
+  for (long long line = tid; line * 32 < static_cast<long long>(a.D) * a.V; line += RS_THREADS)
+    asm volatile("prefetch.global.L2 [%0];\n" ::"l"(state + line * 32));
+  const float pos = static_cast<float>(a.positions[t]);
+  const int half = a.rot_dims / 2, qk = a.H * a.D;
+  for (int i = tid; i < a.D; i += RS_THREADS) {
+    if (i >= half && i < a.rot_dims) continue;             // the partner of one below
+    const float qu = token[h * a.D + i], ku = token[qk + h * a.D + i];
+    if (i >= a.rot_dims) {
+      q_s[i] = qu;
+      k_s[i] = ku * a.k_scale;
+      continue;
+    }
+    const float qv = token[h * a.D + i + half], kv = token[qk + h * a.D + i + half];
+    float s, c;
+    sincosf(pos * a.freqs[i], &s, &c);
+    q_s[i] = qu * c - qv * s;
+    q_s[i + half] = qv * c + qu * s;
+    k_s[i] = (ku * c - kv * s) * a.k_scale;
+    k_s[i + half] = (kv * c + ku * s) * a.k_scale;
+  }
+  __syncthreads();
+  const float decay = a.decay[h];
+  const float* values = token + 2 * qk + h * a.V;
+  const int all = a.V / PER;                               // columns in runs of PER (PER divides V)
+  float ss = 0.0f;
+  for (int c0 = 0; c0 < all; c0 += RS_THREADS) {
+    const int cols = min(RS_THREADS, all - c0), groups = RS_THREADS / cols;
+    const int group = tid / cols, col = tid - group * cols, at = (c0 + col) * PER;
+    float o[PER], v[PER];
+#pragma unroll
+    for (int u = 0; u < PER; ++u) {
+      o[u] = 0.0f;
+      v[u] = group < groups ? values[at + u] : 0.0f;
+    }
+    if (group < groups) {
+      constexpr int AHEAD = 8;
+      for (int d0 = group; d0 < a.D; d0 += groups * AHEAD) {
+        float s[AHEAD][PER];
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) {
+          const int d = d0 + i * groups;
+          if (d < a.D) {
+            const float* p = state + static_cast<long long>(d) * a.V + at;
+            if (PER == 4) *reinterpret_cast<float4*>(&s[i][0]) = *reinterpret_cast<const float4*>(p);
+            else s[i][0] = *p;
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) {
+          const int d = d0 + i * groups;
+          if (d < a.D) {
+            const float kd = k_s[d], qd = q_s[d];
+#pragma unroll
+            for (int u = 0; u < PER; ++u) {
+              s[i][u] = fmaf(decay, s[i][u], kd * v[u]);
+              o[u] = fmaf(s[i][u], qd, o[u]);
+            }
+            if (a.write_state) {
+              float* p = state + static_cast<long long>(d) * a.V + at;
+              if (PER == 4) *reinterpret_cast<float4*>(p) = *reinterpret_cast<const float4*>(&s[i][0]);
+              else *p = s[i][0];
+            }
+          }
+        }
+      }
+#pragma unroll
+      for (int u = 0; u < PER; ++u) part_s[(group * cols + col) * PER + u] = o[u];
+    }
+    __syncthreads();
+    for (int c = tid; c < cols * PER; c += RS_THREADS) {
+      float sum = 0.0f;
+      for (int g = 0; g < groups; ++g) sum += part_s[g * cols * PER + c];
+      o_s[c0 * PER + c] = sum;
+      ss = fmaf(sum, sum, ss);
+    }
+    __syncthreads();
+  }
+  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(a.V) + a.eps);
+  const float* gate = token + 2 * qk + a.H * a.V + h * a.V;
+  T* out = static_cast<T*>(a.out) + (t * a.H + h) * a.V;
+  for (int c = tid; c < a.V; c += RS_THREADS) {
+    const float g = gate[c];
+    out[c] = from_float<T>(o_s[c] * inv * (g / (1.0f + expf(-g))));
+  }
+}
+
 inline size_t retention_local_smem(int D) { return sizeof(__nv_bfloat16) * 2 * (static_cast<size_t>(RC) * retention_kst(D) + RC * R_VST); }
 inline size_t retention_output_smem(int D) {
   const size_t keys = static_cast<size_t>(2) * RC * retention_kst(D);
@@ -379,9 +514,39 @@ ZB_API int zb_retention(float* out, const float* q, long long q_stride, const fl
   const long long per = static_cast<long long>(H) * D * V;
   const bool four = D * V % 4 == 0 && aligned(ws) && aligned(state) && slot_stride % 4 == 0;
   const long long threads = four ? per / 4 : per;
-  const dim3 carry(static_cast<unsigned>((threads + 255) / 256), rows);
-  if (four) retention_carry_kernel<4><<<carry, 256, 0, s>>>(a);
-  else retention_carry_kernel<1><<<carry, 256, 0, s>>>(a);
+  const dim3 carry(static_cast<unsigned>((threads + 127) / 128), rows);
+  if (four) retention_carry_kernel<4><<<carry, 128, 0, s>>>(a);
+  else retention_carry_kernel<1><<<carry, 128, 0, s>>>(a);
   retention_output_kernel<<<dim3((tiles + a.tiles_per_cta - 1) / a.tiles_per_cta, H, pieces), R_THREADS, output_smem, s>>>(a);
+  return launch_result();
+}
+
+// One token a request, from the projection's float32 rows (q | k | v | gate) to the gated, unit-normed output [tokens,
+// H * V] in `dtype`, the requests' states brought up to date.
+ZB_API int zb_retention_step(void* out, const float* projected, long long stride, const float* freqs, int rot_dims, float k_scale,
+                             float eps, const float* decay, float* state, long long slot_stride, const int* slots,
+                             const int* row_q_start, const int* row_q_len, const int* positions, int rows, int H, int D, int V,
+                             int num_slots, int write_state, int dtype, int* status, void* stream) {
+  if (rows < 0 || H <= 0 || D <= 0 || V <= 0 || num_slots <= 0 || rot_dims < 0 || rot_dims > D || rot_dims % 2 != 0 ||
+      (rot_dims > 0 && freqs == nullptr) || stride < 2LL * H * (static_cast<long long>(D) + V))
+    return ERR_BAD_ARGUMENT;
+  if (rows > 65535 || 2LL * D + V > 10000) return ERR_UNSUPPORTED;
+  if (rows == 0) return OK;
+  RetentionStepArgs a;
+  a.out = out; a.projected = projected; a.stride = stride; a.freqs = freqs; a.rot_dims = rot_dims; a.k_scale = k_scale; a.eps = eps;
+  a.decay = decay; a.state = state; a.slot_stride = slot_stride; a.slots = slots; a.row_q_start = row_q_start;
+  a.row_q_len = row_q_len; a.positions = positions; a.H = H; a.D = D; a.V = V; a.num_slots = num_slots;
+  a.write_state = write_state; a.status = status;
+  auto s = static_cast<cudaStream_t>(stream);
+  const dim3 grid(H, rows);
+  const bool four = V % 4 == 0 && slot_stride % 4 == 0 && reinterpret_cast<uintptr_t>(state) % 16 == 0;
+  const size_t smem = sizeof(float) * (2 * D + V + RS_THREADS * (four ? 4 : 1));
+  if (dtype == DTYPE_F32) {
+    if (four) retention_step_kernel<float, 4><<<grid, RS_THREADS, smem, s>>>(a);
+    else retention_step_kernel<float, 1><<<grid, RS_THREADS, smem, s>>>(a);
+  } else {
+    if (four) retention_step_kernel<__nv_bfloat16, 4><<<grid, RS_THREADS, smem, s>>>(a);
+    else retention_step_kernel<__nv_bfloat16, 1><<<grid, RS_THREADS, smem, s>>>(a);
+  }
   return launch_result();
 }

@@ -63,6 +63,7 @@ __global__ void __launch_bounds__(QH_THREADS) qkv_halves_kernel(const QkvHalvesA
   const int cols = q_cols + k_cols + v_cols, heads = a.nh + 2 * kv_heads;
   float* x = qh_smem;                    // [cols]
   float* head_ss = qh_smem + cols;       // [heads]
+  float* turn = head_ss + heads;         // [rot_dims]: cosines, then sines, of the token's angles, once for all heads
   const IN* src = static_cast<const IN*>(a.qkv) + static_cast<long long>(t) * a.stride;
   for (int i = threadIdx.x; i < cols; i += QH_THREADS) x[i] = to_float(src[i]) + (a.bias != nullptr ? a.bias[i] : 0.0f);
   __syncthreads();
@@ -77,8 +78,15 @@ __global__ void __launch_bounds__(QH_THREADS) qkv_halves_kernel(const QkvHalvesA
     ss = warp_sum(ss);
     if (lane == 0) head_ss[h] = ss;
   }
-  __syncthreads();
   const int pos = a.positions[t];
+  const int half = a.rot_dims / 2;
+  for (int i = threadIdx.x; i < half; i += QH_THREADS) {
+    float s, c;
+    sincosf(static_cast<float>(pos) * a.freqs[i], &s, &c);
+    turn[i] = c * a.rot_mult;
+    turn[half + i] = s * a.rot_mult;
+  }
+  __syncthreads();
   int page = 0;
   if (a.cache != nullptr) {
     const int row = a.token_row[t], block = pos / a.page_size;
@@ -93,7 +101,6 @@ __global__ void __launch_bounds__(QH_THREADS) qkv_halves_kernel(const QkvHalvesA
     }
   }
   const long long page_elems = static_cast<long long>(a.nkv) * a.page_size * (a.kd + a.vd);
-  const int half = a.rot_dims / 2;
   const float share = a.v_first != nullptr ? *a.v_share : 0.0f;
   for (int h = warp; h < heads; h += QH_WARPS) {
     const bool is_q = h < a.nh, is_v = h >= a.nh + kv_heads;
@@ -134,13 +141,139 @@ __global__ void __launch_bounds__(QH_THREADS) qkv_halves_kernel(const QkvHalvesA
         y = (1.0f - share) * y + share * a.v_first[static_cast<long long>(t) * a.v_first_stride + own * a.vd + i];
       if (!is_v && a.freqs != nullptr && i < a.rot_dims) {
         const int f = i < half ? i : i - half;
-        float s, c;
-        sincosf(static_cast<float>(pos) * a.freqs[f], &s, &c);
-        s *= a.rot_mult;
-        c *= a.rot_mult;
+        const float c = turn[f], s = turn[half + f];
         y = i < half ? row[i] * c - row[i + half] * s : row[i] * c + row[i - half] * s;
       }
       dst[swizzle_pos >= 0 ? kv_element_index(i, swizzle_pos, dim, sizeof(T)) : i] = from_float<T>(y);
+    }
+  }
+}
+
+// The same four values at a time: widths, rotated halves and row starts that are multiples of four values, heads of
+// whole 16-byte pieces.  A head's values stay where the load put them; norm, rotation and the store are one pass.
+template <typename T> __device__ __forceinline__ void store_four(T* p, float4 v);
+template <> __device__ __forceinline__ void store_four<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+template <> __device__ __forceinline__ void store_four<__nv_bfloat16>(__nv_bfloat16* p, float4 v) {
+  uint2 raw;
+  *reinterpret_cast<__nv_bfloat162*>(&raw.x) = __floats2bfloat162_rn(v.x, v.y);
+  *reinterpret_cast<__nv_bfloat162*>(&raw.y) = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = raw;
+}
+__device__ __forceinline__ float4 scaled4(float4 v, float s, const float* w, int i) {
+  if (w == nullptr) return make_float4(v.x * s, v.y * s, v.z * s, v.w * s);
+  const float4 c = *reinterpret_cast<const float4*>(w + i);
+  return make_float4(v.x * s * c.x, v.y * s * c.y, v.z * s * c.z, v.w * s * c.w);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(QH_THREADS) qkv_halves_vec_kernel(const QkvHalvesArgs a) {
+  extern __shared__ __align__(16) float qh_smem[];
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int kv_heads = a.cache != nullptr ? a.nkv : 0;
+  const int q_cols = a.nh * a.kd, k_cols = kv_heads * a.kd, v_cols = kv_heads * a.vd;
+  const int cols = q_cols + k_cols + v_cols, heads = a.nh + 2 * kv_heads, half = a.rot_dims / 2;
+  float* x = qh_smem;                    // [cols]
+  float* turn = x + cols;                // [rot_dims]: cosines, then sines
+  float* head_ss = turn + a.rot_dims;    // [heads]
+  const float* src = static_cast<const float*>(a.qkv) + static_cast<long long>(t) * a.stride;
+  const int pos = a.positions[t];
+  for (int i = 4 * threadIdx.x; i < cols; i += 4 * QH_THREADS) {
+    float4 v = *reinterpret_cast<const float4*>(src + i);
+    if (a.bias != nullptr) {
+      const float4 b = *reinterpret_cast<const float4*>(a.bias + i);
+      v = make_float4(v.x + b.x, v.y + b.y, v.z + b.z, v.w + b.w);
+    }
+    *reinterpret_cast<float4*>(x + i) = v;
+  }
+  for (int i = threadIdx.x; i < half; i += QH_THREADS) {
+    float s, c;
+    sincosf(static_cast<float>(pos) * a.freqs[i], &s, &c);
+    turn[i] = c * a.rot_mult;
+    turn[half + i] = s * a.rot_mult;
+  }
+  __syncthreads();
+  auto begin_of = [&](int h) {
+    return h < a.nh ? h * a.kd : (h < a.nh + kv_heads ? q_cols + (h - a.nh) * a.kd : q_cols + k_cols + (h - a.nh - kv_heads) * a.vd);
+  };
+  const bool whole = a.norm_mode == NORM_WHOLE;
+  auto sum_of_squares = [&](int h) {
+    const int dim = h < a.nh + kv_heads ? a.kd : a.vd;
+    const float* row = x + begin_of(h);
+    float ss = 0.0f;
+    for (int i = 4 * lane; i < dim; i += 128) {
+      const float4 v = *reinterpret_cast<const float4*>(row + i);
+      ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+    }
+    return warp_sum(ss);
+  };
+  if (whole) {                           // one statistic over the projection's heads: every head's sum first
+    for (int h = warp; h < a.nh + kv_heads; h += QH_WARPS) {
+      const float ss = sum_of_squares(h);
+      if (lane == 0) head_ss[h] = ss;
+    }
+    __syncthreads();
+  }
+  int page = 0;
+  if (a.cache != nullptr) {
+    const int row = a.token_row[t], block = pos / a.page_size;
+    if (row < 0 || row >= a.num_rows || block >= a.max_blocks) {
+      if (threadIdx.x == 0) report(a.status, STATUS_ROW_OUT_OF_RANGE, row, t);
+      return;
+    }
+    page = a.block_table[static_cast<long long>(row) * a.max_blocks + block];
+    if (page <= 0 || page >= a.num_pages) {
+      if (threadIdx.x == 0) report(a.status, STATUS_PAGE_OUT_OF_RANGE, page, t);
+      return;
+    }
+  }
+  const long long page_elems = static_cast<long long>(a.nkv) * a.page_size * (a.kd + a.vd);
+  const float share = a.v_first != nullptr ? *a.v_share : 0.0f;
+  for (int h = warp; h < heads; h += QH_WARPS) {
+    const bool is_q = h < a.nh, is_v = h >= a.nh + kv_heads;
+    const int dim = is_v ? a.vd : a.kd, own = is_q ? h : (is_v ? h - a.nh - kv_heads : h - a.nh);
+    const float* row = x + begin_of(h);
+    float inv = 1.0f;
+    const float* w = nullptr;
+    if (is_v) {
+      if (a.value_unit_norm) inv = 1.0f / sqrtf(sum_of_squares(h) / static_cast<float>(dim) + a.eps);
+    } else if (a.norm_mode == NORM_PER_HEAD) {
+      inv = 1.0f / sqrtf(sum_of_squares(h) / static_cast<float>(dim) + a.eps);
+      w = is_q ? a.q_norm_w : a.k_norm_w;
+    } else if (whole) {
+      const int h0 = is_q ? 0 : a.nh, n = is_q ? a.nh : kv_heads;
+      float total = 0.0f;
+      for (int j = 0; j < n; ++j) total += head_ss[h0 + j];
+      inv = 1.0f / sqrtf(total / static_cast<float>(n * dim) + a.eps);
+      w = is_q ? a.q_norm_w : a.k_norm_w;
+      if (w != nullptr) w += own * dim;
+    }
+    T* dst;
+    if (is_q) {
+      dst = static_cast<T*>(a.q_out) + (static_cast<long long>(t) * a.nh + h) * a.kd;
+    } else {
+      const long long part = is_v ? static_cast<long long>(a.nkv) * a.page_size * a.kd : 0;
+      dst = static_cast<T*>(a.cache) + static_cast<long long>(page) * page_elems + part +
+            (static_cast<long long>(own) * a.page_size + pos % a.page_size) * dim;
+    }
+    auto put = [&](int i, float4 v) { store_four<T>(dst + (is_q ? i : kv_element_index(i, pos, dim, sizeof(T))), v); };
+    const int turned = is_v ? 0 : half;
+    for (int i = 4 * lane; i < dim - turned; i += 128) {        // four pairs, or four values that do not turn
+      if (i < turned) {
+        const float4 u = scaled4(*reinterpret_cast<const float4*>(row + i), inv, w, i);
+        const float4 v = scaled4(*reinterpret_cast<const float4*>(row + half + i), inv, w, half + i);
+        const float4 c = *reinterpret_cast<const float4*>(turn + i), s = *reinterpret_cast<const float4*>(turn + half + i);
+        put(i, make_float4(u.x * c.x - v.x * s.x, u.y * c.y - v.y * s.y, u.z * c.z - v.z * s.z, u.w * c.w - v.w * s.w));
+        put(half + i, make_float4(v.x * c.x + u.x * s.x, v.y * c.y + u.y * s.y, v.z * c.z + u.z * s.z, v.w * c.w + u.w * s.w));
+      } else {
+        const int at = i + turned;
+        float4 v = scaled4(*reinterpret_cast<const float4*>(row + at), inv, w, at);
+        if (is_v && a.v_first != nullptr) {
+          const float4 f = *reinterpret_cast<const float4*>(a.v_first + static_cast<long long>(t) * a.v_first_stride + own * a.vd + at);
+          const float keep = 1.0f - share;
+          v = make_float4(keep * v.x + share * f.x, keep * v.y + share * f.y, keep * v.z + share * f.z, keep * v.w + share * f.w);
+        }
+        put(at, v);
+      }
     }
   }
 }
@@ -320,9 +453,25 @@ ZB_API int zb_qkv_halves(void* q_out, const void* qkv, long long stride, const f
   a.num_pages = num_pages; a.num_rows = num_rows; a.nh = nh; a.nkv = nkv; a.kd = kd; a.vd = vd; a.status = status;
   const int kv_heads = cache != nullptr ? nkv : 0;
   const size_t smem = sizeof(float) * (static_cast<size_t>(nh) * kd + static_cast<size_t>(kv_heads) * (kd + vd) +
-                                       nh + 2 * kv_heads);
+                                       nh + 2 * kv_heads + a.rot_dims);
   if (smem > 200 * 1024) return ERR_UNSUPPORTED;
   auto s = static_cast<cudaStream_t>(stream);
+  auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  if (in_dtype == DTYPE_F32 && kd % 8 == 0 && vd % 8 == 0 && rot_dims % 8 == 0 && stride % 4 == 0 && v_first_stride % 4 == 0 &&
+      aligned(qkv) && aligned(bias) && aligned(q_norm_w) && aligned(k_norm_w) && aligned(v_first) && aligned(q_out) && aligned(cache)) {
+#define ZB_QHV(T)                                                                                               \
+  {                                                                                                             \
+    auto kernel = qkv_halves_vec_kernel<T>;                                                                     \
+    if (smem > 48 * 1024 && cuda_failed(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                                             static_cast<int>(smem))))                           \
+      return ERR_CUDA;                                                                                          \
+    kernel<<<tokens, QH_THREADS, smem, s>>>(a);                                                                 \
+  }
+    if (dtype == DTYPE_F32) ZB_QHV(float)
+    else ZB_QHV(__nv_bfloat16)
+#undef ZB_QHV
+    return launch_result();
+  }
 #define ZB_QH(IN, T)                                                                                            \
   {                                                                                                             \
     auto kernel = qkv_halves_kernel<IN, T>;                                                                     \

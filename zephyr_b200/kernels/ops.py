@@ -143,9 +143,11 @@ _SIGNATURES = {
     "zb_retention_max_channels": [],
     "zb_retention": [c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong,
                      c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
+    "zb_retention_step": [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_float, c_float, c_void_p, c_void_p, c_longlong,
+                          c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "zb_rotate_qk": [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
     "zb_gated_group_rms_norm": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                c_float, c_int, c_int, c_void_p],
+                                c_float, c_int, c_int, c_int, c_void_p],
     "zb_scaled_sum": [c_void_p, c_void_p, c_void_p, c_float, c_float, c_longlong, c_int, c_int, c_void_p],
     "zb_paged_decode_supported": [c_int, c_int, c_int, c_int],
     "zb_paged_decode": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int,
@@ -188,6 +190,8 @@ _SIGNATURES = {
                               c_longlong, c_longlong, c_longlong, c_int, c_void_p],
     "zb_gemm_small_act": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong, c_int, c_int,
                           c_void_p],
+    "zb_gemm_small_token_gate": [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_int,
+                                 c_longlong, c_longlong, c_longlong, c_void_p, c_void_p],
     "zb_gemm_nt_simt": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong,
                         c_int, c_int, c_void_p],
     "zb_fused_chain_stage_supported": [c_int, c_int, c_int, c_int, c_int],
@@ -815,21 +819,47 @@ def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Te
     return out
 
 
+def retention_step(projected: torch.Tensor, decay: torch.Tensor, freqs: torch.Tensor | None, rot_dims: int, k_scale: float,
+                   eps: float, heads: int, key_dim: int, value_dim: int, state: torch.Tensor, slots: torch.Tensor,
+                   row_q_start: torch.Tensor, row_q_len: torch.Tensor, positions: torch.Tensor, status: torch.Tensor,
+                   dtype: torch.dtype, write_state: bool = True) -> torch.Tensor:
+    """One token a request, in one kernel: ``projected`` float32 [T, q | k | v | gate] -> q and k rotated as ``rotate_qk`` does,
+    S <- decay S + k v^T, o = S^T q, each head's o divided by its root mean square, times silu(gate).  Returns
+    [T, heads * value_dim] in ``dtype``."""
+    _cuda(projected, decay, freqs, state, slots, row_q_start, row_q_len, positions, status)
+    _i32(slots, row_q_start, row_q_len, positions)
+    T, width = projected.shape
+    _require(projected.dtype == torch.float32 and projected.stride(1) == 1 and width >= 2 * heads * (key_dim + value_dim)
+             and positions.numel() == T and slots.numel() == T == row_q_len.numel(), "float32 rows of q, k, v and a gate, one a request")
+    _f32_vector(decay, heads, "the decays")
+    _require(rot_dims == 0 or freqs is not None, "a rotation needs frequencies")
+    _f32_vector(freqs, rot_dims // 2, "the frequencies")
+    _require(state.dim() == 2 and state.dtype == torch.float32 and state.stride(1) == 1
+             and state.shape[1] == heads * key_dim * value_dim, "state must be float32 [slots, heads * key_dim * value_dim]")
+    out = torch.empty((T, heads * value_dim), dtype=dtype, device=projected.device)
+    _check(library().zb_retention_step(
+        _ptr(out), _ptr(projected), projected.stride(0), _ptr(freqs), int(rot_dims), float(k_scale), float(eps), _ptr(decay),
+        _ptr(state), state.stride(0), _ptr(slots), _ptr(row_q_start), _ptr(row_q_len), _ptr(positions), T, heads, key_dim, value_dim,
+        state.shape[0], int(write_state), DTYPE_CODE[dtype], _ptr(status), _stream()), "retention_step")
+    return out
+
+
 def gated_group_rms_norm(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, group: int, eps: float,
-                         gate_first: bool) -> torch.Tensor:
+                         gate_first: bool, out_dtype: torch.dtype | None = None) -> torch.Tensor:
     """RMS norm of a float32 [T, W] over groups of ``group`` columns with a SiLU gate ([T, >= W], rows may
     be strided) multiplied in before the norm (``gate_first``) or after it; ``w`` float32, used
-    periodically (W values, or one group's).  The result has the gate's type."""
+    periodically (W values, or one group's).  The result has the gate's type, or ``out_dtype`` where the gate is float32."""
     _cuda(o, gate, w)
     _require(o.dim() == 2 and o.is_contiguous() and o.dtype == torch.float32, "o must be a contiguous float32 [T, W]")
     T, W = o.shape
     _require(gate.dim() == 2 and gate.stride(1) == 1 and gate.shape[0] == T and gate.shape[1] >= W
              and gate.dtype in DTYPE_CODE, "the gate must be [T, W] with unit inner stride")
     _require(w.dtype == torch.float32 and w.is_contiguous() and w.numel() in (W, group), "w: float32, W or group values")
-    out = torch.empty((T, W), dtype=gate.dtype, device=o.device)
+    _require(out_dtype in (None, gate.dtype) or gate.dtype == torch.float32, "only a float32 gate leaves another type")
+    out = torch.empty((T, W), dtype=out_dtype or gate.dtype, device=o.device)
     _check(library().zb_gated_group_rms_norm(_ptr(out), _ptr(o), _ptr(gate), gate.stride(0), _ptr(w), 0, w.numel(), T, W,
                                              int(group), float(eps), int(gate_first), DTYPE_CODE[gate.dtype],
-                                             _stream()), "gated_group_rms_norm")
+                                             DTYPE_CODE[out.dtype], _stream()), "gated_group_rms_norm")
     return out
 
 
@@ -1600,6 +1630,22 @@ def gemm_small(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None =
     _check(library().zb_gemm_small(_ptr(out), _ptr(x), _ptr(w), M, N, K, x.stride(0), w.stride(0), out.stride(0),
                                    DTYPE_CODE[out_dtype], (2 if act == "relu" else 1) if swiglu else 0, _stream()),
            "gemm_small")
+    return out
+
+
+def gemm_small_token_gate(x: torch.Tensor, w: torch.Tensor, table: torch.Tensor, offset: int, ids: torch.Tensor,
+                          status: torch.Tensor) -> torch.Tensor:
+    """``token_gate`` of the few-row product x w^T, in the product's epilogue: gelu_tanh(sum) times the values offset ..
+    offset + N of the tokens' rows of ``table``, [M, N] bfloat16."""
+    _cuda(x, w, table, ids, status)
+    _i32(ids)
+    _require(gemm_small_supported(x, w) and table.dtype == torch.bfloat16 and table.dim() == 2 and table.stride(1) == 1
+             and ids.numel() == x.shape[0], "few bfloat16 rows, one token id each")
+    (M, K), N = x.shape, w.shape[0]
+    out = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
+    _check(library().zb_gemm_small_token_gate(_ptr(out), _ptr(x), _ptr(w), _ptr(table), table.stride(0), int(offset), _ptr(ids),
+                                              table.shape[0], M, N, K, x.stride(0), w.stride(0), out.stride(0), _ptr(status),
+                                              _stream()), "gemm_small")
     return out
 
 

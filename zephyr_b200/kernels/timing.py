@@ -891,11 +891,23 @@ def retention(args) -> dict:
             runs["pieces"] = lambda i: ops.retention(*halves(i), decay, H, D, V, *where(i))
             pos = torch.arange(T, dtype=torch.int32, device=device)
             freqs = torch.rand(D // 2, device=device)
+            gate_w = torch.ones(V, device=device)
+            gates = [torch.randn((T, H * V), device=device) for _ in range(n)]
+            runs["unit norm and gate"] = lambda i: ops.gated_group_rms_norm(v[i % n], gates[i % n], gate_w, V, 1e-6, gate_first=False,
+                                                                            out_dtype=torch.bfloat16)
             runs["rotation"] = lambda i: ops.rotate_qk(qk[i % n], H, D, freqs, D, D ** -0.5, pos)
+        else:
+            pos = torch.full((T,), 4000, dtype=torch.int32, device=device)
+            freqs = torch.rand(D // 2, device=device)
+            projected = [torch.cat([qk[i], v[i], v[i]], dim=1) for i in range(n)]
+            runs["one kernel, rotation to gate"] = lambda i: ops.retention_step(
+                projected[i % n], decay, freqs, D, D ** -0.5, 1e-6, H, D, V, states[i % m], slots, starts, lens, pos, status, torch.bfloat16)
         for name, run in runs.items():
             us = _time(run, args.warmup, args.iters)
             row = {"us": round(us, 2)}
-            if name == "rotation":
+            if name == "unit norm and gate":
+                row["gbs"] = round(T * H * V * 10 / us / 1e3, 1)
+            elif name == "rotation":
                 row["gbs"] = round(T * 2 * H * D * 8 / us / 1e3, 1)
             elif what == "prompt":
                 row["tflops_of_the_recurrence"] = round(4 * T * H * D * V / us / 1e6, 2)
@@ -922,7 +934,7 @@ def plus_one_parts(args) -> dict:
     out = {"tokens": T, "hidden": W, "heads": H, "kv_heads": G, "head_dim": d, "window": window}
     seen = sum(min(p + 1, window + min(keep, max(0, p + 1 - window))) for p in range(T))
 
-    def attend(new_tokens: int, before: int, requests: int, vd: int, with_sinks: bool) -> float:
+    def attend(new_tokens: int, before: int, requests: int, vd: int, with_sinks: bool, heads: bool = False) -> float:
         rows = new_tokens * requests
         q = torch.randn((rows, H * d), device=device, dtype=bf)
         caches, table = _paged_inputs(requests, before + new_tokens, G, d, page, device)
@@ -938,7 +950,7 @@ def plus_one_parts(args) -> dict:
         tile_q0 = (torch.arange(per, dtype=torch.int32, device=device) * tile).repeat(requests)
         result = torch.empty((rows, H * vd), device=device, dtype=bf)
         extra = dict(keep_first=keep, sinks=sinks if with_sinks else None)
-        if vd != d:
+        if vd != d or heads:
             return _time(lambda i: ops.heads_attention(q, caches[i % len(caches)], table, tile_row, tile_q0, start, lens, ctx, H, G, d, vd,
                                                        window, d ** -0.5, status, result, single=single, max_context=before + new_tokens,
                                                        **extra), args.warmup, args.iters)
@@ -950,6 +962,10 @@ def plus_one_parts(args) -> dict:
             prompt = attend(T, 0, 1, vd, on)
             out[f"{name}, values of {vd}"] = {"prompt_us": round(prompt, 1), "prompt_tflops": round(seen * 2 * H * (d + vd) / prompt / 1e6, 1),
                                              "single_tokens_us": round(attend(1, args.context - 1, args.batch, vd, on), 1)}
+    out["single tokens of a kept window, us"] = {
+        f"{count} rows": {"keys shared among CTAs": round(attend(1, args.context - 1, count, d, True, heads=True), 1),
+                          "tiles of a group's heads": round(attend(1, args.context - 1, count, d, True), 1)}
+        for count in (1, 4, 8, 16, 32, 64)}
     blocks = -(-T // page)
     table = torch.arange(1, blocks + 1, dtype=torch.int32, device=device).view(1, -1)
     cache = torch.zeros((blocks + 1, 2, G, page, d), dtype=bf, device=device)

@@ -66,6 +66,8 @@ from .base import POSITION_ENCODINGS, Mixer, StepContext, lookup, register_mixer
 class Attention(Mixer):
     graph_safe = True
 
+    HEADS_SINGLE_ROWS = 32      # up to this many single tokens of a kept window share their keys among CTAs
+
     def __init__(self, spec: MixerSpec, weights: Mapping[str, torch.Tensor], dtype: torch.dtype,
                  device: torch.device | str):
         p = spec.params
@@ -218,6 +220,8 @@ class Attention(Mixer):
         plain_mask = not (self.chunk or self.pool or self.softcap > 0.0
                           or self.head_mix is not None or self.values_from_keys)
         self.heads_tile_tokens = 0
+        # A few single tokens of a kept window go there too, with a token's keys shared by as many CTAs as fill the SMs.
+        self.heads_single = plain_mask and ops.heads_attention_tile_tokens(self.nh, self.nkv, self.hd, self.vd, self.dtype) > 0
         if plain_mask and (self.score_mix is not None or not (equal and ops.paged_prefill_supported(self.nh, self.nkv, self.hd, self.dtype))):
             self.heads_tile_tokens = ops.heads_attention_tile_tokens(self.nh, self.nkv, self.hd, self.vd, self.dtype)
         self.fast_decode = equal and not self.windowed and ops.paged_decode_supported(self.nh, self.nkv, self.hd, self.dtype)
@@ -403,7 +407,12 @@ class Attention(Mixer):
             for which, by_group in (((self.prefill_tile_tokens, "multi"), False),
                                     ((self.tile_tokens, "single"), self.group <= 16)):
                 tile_row, tile_q0 = ctx.tiles[which]
-                if tile_row.numel() > 0:
+                if which[1] == "single" and self.heads_single and 0 < tile_row.numel() <= self.HEADS_SINGLE_ROWS:
+                    ops.heads_attention(q, cache, table, tile_row, tile_q0, ctx.row_q_start, ctx.row_q_len, ctx.row_ctx, self.nh,
+                                        self.nkv, self.hd, self.vd, self.window, self.scale, ctx.status, out,
+                                        keep_first=self.keep_first, distance_bias=self.distance_bias, sinks=self.sinks,
+                                        single=True, max_context=ctx.max_decode_context)
+                elif tile_row.numel() > 0:
                     ops.paged_prefill(q, cache, table, tile_row, tile_q0, ctx.row_q_start, ctx.row_q_len, ctx.row_ctx,
                                       *common, out=out, cross_values=mixed, by_group=by_group, **masks)
         else:

@@ -300,11 +300,10 @@ class Retention(Mixer):
         self.freqs, self.rot_dims, mult = halves() if halves is not None else (None, 0, 1.0)
         if mult != 1.0:
             raise ConfigError("retention's rotation takes no multiplier")
-        # One product with float32 sums out for everything that enters the recurrence, q | k | v (behind the unit
-        # norm of o a rounding of q or k counts in full where q . k is small); the gate comes out of a second
-        # product, in the model's type.
-        self.w_in = torch.cat([weights[p[n]] for n in ("q", "k", "v")], dim=0).contiguous()
-        self.w_g, self.w_o = weights[p["g"]], weights[p["o"]]
+        # One product with float32 sums out, q | k | v | gate (behind the unit norm of o a rounding of q or k counts
+        # in full where q . k is small).
+        self.w_in = torch.cat([weights[p[n]] for n in ("q", "k", "v", "g")], dim=0).contiguous()
+        self.w_o = weights[p["o"]]
         self.unit = torch.ones(self.vdim, dtype=torch.float32, device=self.w_o.device)
 
     @staticmethod
@@ -316,7 +315,7 @@ class Retention(Mixer):
                 p["o"]: WeightDecl((hidden, hv), ROLE_LINEAR)}
 
     def weights_read(self) -> list[torch.Tensor]:
-        return [self.w_in, self.w_g, self.w_o]
+        return [self.w_in, self.w_o]
 
     @staticmethod
     def cache_spec(spec: MixerSpec) -> StateCacheSpec:
@@ -325,18 +324,24 @@ class Retention(Mixer):
 
     def forward(self, x: torch.Tensor, ctx: StepContext, call: LayerCall,
                 out_dtype: torch.dtype | None = None) -> torch.Tensor:
-        hd = self.heads * self.dim
-        projected = ops.linear(x, self.w_in, out_dtype=torch.float32)      # q | k | v
+        hd, hv = self.heads * self.dim, self.heads * self.vdim
+        projected = ops.linear(x, self.w_in, out_dtype=torch.float32)      # q | k | v | gate
+        if ctx.num_decode_rows == ctx.num_rows == ctx.num_tokens:          # one token a request: one kernel
+            normed = ops.retention_step(projected, self.decay, self.freqs, self.rot_dims, self.dim ** -0.5, self.eps, self.heads, self.dim,
+                                        self.vdim, ctx.caches[call.cache], ctx.state_slots, ctx.row_q_start, ctx.row_q_len,
+                                        ctx.positions, ctx.status, self.dtype, write_state=call.writes_cache)
+            return ops.linear(normed, self.w_o, out_dtype=out_dtype)
         turned = ops.rotate_qk(projected, self.heads, self.dim, self.freqs, self.rot_dims, self.dim ** -0.5, ctx.positions)
-        q, k, v = turned[:, :hd], turned[:, hd:], projected[:, 2 * hd:]
+        q, k, v = turned[:, :hd], turned[:, hd:], projected[:, 2 * hd:2 * hd + hv]
         where = (ctx.caches[call.cache], ctx.state_slots, ctx.row_q_start, ctx.row_q_len, ctx.status)
-        # Runs of tokens in pieces on the tensor cores; single tokens, and everything in true 32-bit, token by token.
+        # Runs of tokens in pieces on the tensor cores; short ones, and everything in true 32-bit, token by token.
         if self.dtype == torch.bfloat16 and x.shape[0] >= self.PIECES_FROM * ctx.num_rows and self.dim <= ops.retention_max_channels():
             o = ops.retention(q, k, v, self.decay, self.heads, self.dim, self.vdim, *where, write_state=call.writes_cache)
         else:
             o = ops.decayed_state_scan("fixed", q, k, v, self.heads, self.dim, self.vdim, *where, decay=self.decay,
                                        write_state=call.writes_cache)
-        normed = ops.gated_group_rms_norm(o, ops.linear(x, self.w_g), self.unit, self.vdim, self.eps, gate_first=False)
+        normed = ops.gated_group_rms_norm(o, projected[:, 2 * hd + hv:], self.unit, self.vdim, self.eps, gate_first=False,
+                                          out_dtype=self.dtype)
         return ops.linear(normed, self.w_o, out_dtype=out_dtype)
 
 

@@ -2,8 +2,8 @@
 
 ``token_gate``: y = P (gelu(G x) * e), joined as x + N(y), where e is the layer's part (``dim`` values from ``offset`` on)
 of the token's row in a table that all such layers share, gelu is the tanh form and N an RMS norm with a scale.  The
-two products run in the model's type with float32 sums; the gate and its product with e are one float32 pass with one
-rounding.
+two products run in the model's type with float32 sums; the gate and its product with e are float32 with one rounding,
+in the first product's epilogue for few rows, one pass over its sums otherwise.
 """
 
 from __future__ import annotations
@@ -47,9 +47,12 @@ class TokenGate(SidePart):
         return [self.w_gate, self.w_proj, *self.norm.weights_read()]      # a step gathers a few rows of the table
 
     def forward(self, x: torch.Tensor, ctx: StepContext) -> DeferredSum:
-        gate = ops.linear(x, self.w_gate, out_dtype=torch.float32)
-        y = ops.linear(ops.token_gate(gate, self.table, self.offset, ctx.token_ids, ctx.status), self.w_proj)
-        return DeferredSum(y, self.norm, 1.0)
+        if x.shape[0] <= ops.SMALL_GEMM_ROWS and ops.gemm_small_supported(x, self.w_gate):
+            gated = ops.gemm_small_token_gate(x, self.w_gate, self.table, self.offset, ctx.token_ids, ctx.status)
+        else:
+            gate = ops.linear(x, self.w_gate, out_dtype=torch.float32)
+            gated = ops.token_gate(gate, self.table, self.offset, ctx.token_ids, ctx.status)
+        return DeferredSum(ops.linear(gated, self.w_proj), self.norm, 1.0)
 
 
 register_side("token_gate", TokenGate)

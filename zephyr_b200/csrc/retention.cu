@@ -29,7 +29,7 @@ namespace zb {
 
 constexpr int RC = 64;                  // tokens of a piece
 constexpr int RV = 64;                  // value columns of a tile
-constexpr int R_THREADS = 128;
+constexpr int R_THREADS = 256;
 constexpr int R_VST = RV + 8;           // a row of a value tile or a state tile in shared memory
 
 struct RetentionArgs {
@@ -107,12 +107,13 @@ __device__ __forceinline__ void load_split(__nv_bfloat16* hi, __nv_bfloat16* lo,
   }
 }
 
-// acc[8] (16 x 64) += A (16 x 16, hi and lo) * B (16 x 64), B stored [k][R_VST] in hi and lo tiles; `b` is this lane's
-// ldmatrix offset inside a 16 x 16 block.
-__device__ __forceinline__ void mma_rows_by_tile(float (&acc)[8][4], const unsigned (&ah)[4], const unsigned (&al)[4],
+// acc (16 x 16 N) += A (16 x 16, hi and lo) * B (16 x 16 N), B stored [k][R_VST] in hi and lo tiles, from this lane's
+// ldmatrix addresses inside the first 16 x 16 block on.
+template <int N>
+__device__ __forceinline__ void mma_rows_by_tile(float (&acc)[2 * N][4], const unsigned (&ah)[4], const unsigned (&al)[4],
                                                  const __nv_bfloat16* hi, const __nv_bfloat16* lo) {
 #pragma unroll
-  for (int n = 0; n < 4; ++n) {
+  for (int n = 0; n < N; ++n) {
     unsigned bh[4], bl[4];
     ldmatrix_x4_trans(bh, hi + n * 16);
     ldmatrix_x4_trans(bl, lo + n * 16);
@@ -162,7 +163,7 @@ __global__ void __launch_bounds__(R_THREADS) retention_local_kernel(const Retent
       unsigned ah[4], al[4];
       ldmatrix_x4_trans(ah, k_hi + ks * 16 * kst + mt * 16 + a_off);
       ldmatrix_x4_trans(al, k_lo + ks * 16 * kst + mt * 16 + a_off);
-      mma_rows_by_tile(acc, ah, al, v_hi + ks * 16 * R_VST + b_off, v_lo + ks * 16 * R_VST + b_off);
+      mma_rows_by_tile<4>(acc, ah, al, v_hi + ks * 16 * R_VST + b_off, v_lo + ks * 16 * R_VST + b_off);
     }
 #pragma unroll
     for (int i = 0; i < 8; ++i)
@@ -232,8 +233,9 @@ __global__ void __launch_bounds__(128) retention_carry_kernel(const RetentionArg
   if (a.write_state) store(state, now);
 }
 
-// The outputs of a piece's tokens for one head: the scores once, then value tile by value tile.
-__global__ void __launch_bounds__(R_THREADS) retention_output_kernel(const RetentionArgs a) {
+// The outputs of a piece's tokens for one head: the scores once, then value tile by value tile.  A warp owns 16 tokens
+// and half the columns of a tile (two warps form the same scores).
+__global__ void __launch_bounds__(R_THREADS, 2) retention_output_kernel(const RetentionArgs a) {
   extern __shared__ __align__(16) unsigned char r_smem[];
   __shared__ int found;
   __shared__ float power_s[RC + 1];
@@ -260,16 +262,17 @@ __global__ void __launch_bounds__(R_THREADS) retention_output_kernel(const Reten
   load_split(k_hi, k_lo, kst, a.k + t0 * a.k_stride + h * a.D, a.k_stride, RC, dk * 16, n, a.D, a.qk_vectors, one);
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
-  const int row0 = warp * 16;                                // this warp's tokens of the piece
+  const int wr = warp & 3, c_half = (warp >> 2) * (RV / 2);
+  const int row0 = wr * 16;                                  // this warp's tokens of the piece
   const bool works = row0 < n;
   const int q_off = (row0 + (lane & 7) + ((lane >> 3) & 1) * 8) * kst + (lane >> 4) * 8;
   const int k_off = ((lane & 7) + (lane >> 4) * 8) * kst + ((lane >> 3) & 1) * 8;
-  const int b_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * R_VST + (lane >> 4) * 8;
+  const int b_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * R_VST + (lane >> 4) * 8 + c_half;
   // Scores of the keys up to this warp's last token, decayed, as the hi and lo parts of the next product's operand.
   unsigned ph[4][4], pl[4][4];
 #pragma unroll
   for (int kg = 0; kg < 4; ++kg) {                           // 16 keys
-    if (!works || kg > warp) continue;
+    if (!works || kg > wr) continue;
     float s[2][4];
 #pragma unroll
     for (int i = 0; i < 2; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
@@ -308,28 +311,28 @@ __global__ void __launch_bounds__(R_THREADS) retention_output_kernel(const Reten
     load_split(s_hi, s_lo, R_VST, states + v0, a.V, dk * 16, RV, a.D, cols, a.state_vectors, one);
     __syncthreads();
     if (!works) continue;
-    float acc[8][4];
+    float acc[4][4];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
+    for (int i = 0; i < 4; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
     for (int ks = 0; ks < dk; ++ks) {
       unsigned ah[4], al[4];
       ldmatrix_x4(ah, q_hi + q_off + ks * 16);
       ldmatrix_x4(al, q_lo + q_off + ks * 16);
-      mma_rows_by_tile(acc, ah, al, s_hi + ks * 16 * R_VST + b_off, s_lo + ks * 16 * R_VST + b_off);
+      mma_rows_by_tile<2>(acc, ah, al, s_hi + ks * 16 * R_VST + b_off, s_lo + ks * 16 * R_VST + b_off);
     }
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
+    for (int i = 0; i < 4; ++i) {
       acc[i][0] *= lead0; acc[i][1] *= lead0;
       acc[i][2] *= lead1; acc[i][3] *= lead1;
     }
 #pragma unroll
     for (int kg = 0; kg < 4; ++kg)
-      if (kg <= warp) mma_rows_by_tile(acc, ph[kg], pl[kg], v_hi + kg * 16 * R_VST + b_off, v_lo + kg * 16 * R_VST + b_off);
+      if (kg <= wr) mma_rows_by_tile<2>(acc, ph[kg], pl[kg], v_hi + kg * 16 * R_VST + b_off, v_lo + kg * 16 * R_VST + b_off);
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
+    for (int i = 0; i < 4; ++i)
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
-        const int token = row0 + g + 8 * half, c = v0 + i * 8 + 2 * t;
+        const int token = row0 + g + 8 * half, c = v0 + c_half + i * 8 + 2 * t;
         if (token >= n || c >= a.V) continue;
         float* p = a.out + (t0 + token) * a.H * a.V + h * a.V + c;
         if (a.V % 2 == 0) {

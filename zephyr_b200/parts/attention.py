@@ -66,8 +66,6 @@ from .base import POSITION_ENCODINGS, Mixer, StepContext, lookup, register_mixer
 class Attention(Mixer):
     graph_safe = True
 
-    HEADS_SINGLE_ROWS = 32      # up to this many single tokens of a kept window share their keys among CTAs
-
     def __init__(self, spec: MixerSpec, weights: Mapping[str, torch.Tensor], dtype: torch.dtype,
                  device: torch.device | str):
         p = spec.params
@@ -220,7 +218,7 @@ class Attention(Mixer):
         plain_mask = not (self.chunk or self.pool or self.softcap > 0.0
                           or self.head_mix is not None or self.values_from_keys)
         self.heads_tile_tokens = 0
-        # A few single tokens of a kept window go there too, with a token's keys shared by as many CTAs as fill the SMs.
+        # Single tokens of a kept window go there too, with a token's keys shared by as many CTAs as fill the SMs.
         self.heads_single = plain_mask and ops.heads_attention_tile_tokens(self.nh, self.nkv, self.hd, self.vd, self.dtype) > 0
         if plain_mask and (self.score_mix is not None or not (equal and ops.paged_prefill_supported(self.nh, self.nkv, self.hd, self.dtype))):
             self.heads_tile_tokens = ops.heads_attention_tile_tokens(self.nh, self.nkv, self.hd, self.vd, self.dtype)
@@ -386,7 +384,8 @@ class Attention(Mixer):
         """Attention with kept first tokens, pooled blocks or mixed heads: every row, prompts and single
         tokens alike, on the mma.sync prompt kernel where it takes the shape (bfloat16, one width for keys
         and values that is a multiple of 32 up to 256; a single token's query rows are the heads of a group, so
-        its keys and values stream once a group), on the general kernel elsewhere.  With mixed heads
+        its keys and values stream once a group; where the kernel with all heads in one CTA takes the layer, single tokens
+        run there, a token's keys shared by several CTAs), on the general kernel elsewhere.  With mixed heads
         the kernel hands out every head's weights on every key/value head's values, unrounded, and a second
         kernel mixes them."""
         masks = {"chunk": self.chunk, "sinks": self.sinks, "keep_first": self.keep_first}
@@ -407,7 +406,7 @@ class Attention(Mixer):
             for which, by_group in (((self.prefill_tile_tokens, "multi"), False),
                                     ((self.tile_tokens, "single"), self.group <= 16)):
                 tile_row, tile_q0 = ctx.tiles[which]
-                if which[1] == "single" and self.heads_single and 0 < tile_row.numel() <= self.HEADS_SINGLE_ROWS:
+                if which[1] == "single" and self.heads_single and tile_row.numel() > 0:
                     ops.heads_attention(q, cache, table, tile_row, tile_q0, ctx.row_q_start, ctx.row_q_len, ctx.row_ctx, self.nh,
                                         self.nkv, self.hd, self.vd, self.window, self.scale, ctx.status, out,
                                         keep_first=self.keep_first, distance_bias=self.distance_bias, sinks=self.sinks,

@@ -280,7 +280,7 @@ class Retention(Mixer):
     graph_safe = True
     takes_out_dtype = True
 
-    PIECES_FROM = 8      # new tokens per request, on average, from which on a step runs in pieces
+    PIECES_FROM = 64      # new tokens per request, on average, from which on a step runs in pieces
 
     def __init__(self, spec: MixerSpec, weights: Mapping[str, torch.Tensor], dtype: torch.dtype,
                  device: torch.device | str):

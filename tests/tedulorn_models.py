@@ -58,7 +58,7 @@ CONFIGS = {
     # window of one token, one group, a decay of one and of nearly nothing, odd sizes of a layer's part of the table
     "B": model(131, 96, 1e-6, 7, [
         attention(4, 4, 32, 32, 36, 35, rot(10000.0, 32), 0.18, False, moe(7, 3, 1, 1, 48, 3.0, 64, 1.0)),
-        retention(2, 64, 64, rot(500000.0, 64), [1.0, 0.05], dense(72)),
+        retention(2, 64, 72, rot(500000.0, 64), [1.0, 0.05], dense(72)),
         attention(9, 3, 64, 64, 40, 0, rot(20.0, 10), 0.1, True, None),
         attention(6, 3, 32, 64, 1, 4, rot(100.0, 32), 0.3, True, moe(4, 1, 2, 1, 13, 0.5, 27, 0.7)),
         attention(3, 3, 16, 64, 50, 1, rot(100.0, 2), 0.35, True, dense(30))]),

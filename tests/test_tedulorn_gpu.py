@@ -115,8 +115,8 @@ def replay(folder, dtype, steps, page_size, max_requests=4, graphs=True):
 def assert_rows_match(rows, requests, folder, dtype, what, least=0.5, close_call=None, roundings=True):
     """Every compared row of logits within its bound (``replay_util.tolerance``) in float32; in bfloat16 no row beyond
     two bounds and at most one in ten beyond one.  A fault of a mask, a page or a routed token moves logits by tens to
-    hundreds of bounds.  ``roundings`` (bfloat16; the same tests run in float32 within one bound): or three times what rounding the parts' inputs and outputs alone does to the plain model on the
-    same rows, if that is more."""
+    hundreds of bounds.  ``roundings`` (bfloat16; the same tests run in float32 within one bound): or three times what rounding the parts'
+    inputs and outputs alone does to the plain model on the same rows, if that is more."""
     ratios, skipped, alone = {}, 0, {}
     for (rid, position), got in sorted(rows.items()):
         expected, margins = _plain(str(folder), tuple(requests[rid]))
